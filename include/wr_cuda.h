@@ -47,6 +47,7 @@ extern "C" {
 /* Element types (values of wr_dtype, src/core/internal.h:53-55). */
 #define WR_CUDA_F32 0
 #define WR_CUDA_F16 1
+#define WR_CUDA_BF16 2     /* weights and the matrix products of wr_cuda_model_create_mixed only */
 
 /* wr_cuda_kv_append flags. */
 #define WR_CUDA_APPEND_ROPE 1u  /* rotate K (and Q when given) before storing */
@@ -118,6 +119,20 @@ uint64_t wr_cuda_ctx_launch_count(wr_cuda_ctx *ctx);
  * WR_CUDA_ERR_LIMIT (session.c:755). */
 int  wr_cuda_kv_create(wr_cuda_ctx *ctx, uint32_t n_layers, uint32_t n_kv_heads,
                        uint32_t head_dim, uint32_t max_ctx, wr_cuda_kv **out);
+/* The same for a model whose layers keep different things (no reference
+ * counterpart: every layer of the reference keeps F16 rows of one head_dim,
+ * session.c:647-674).  Per layer: K/V pages of n_kv_heads heads with rows of
+ * k_dim and v_dim elements of `elem` (WR_CUDA_F32 or WR_CUDA_F16; n_kv_heads 0:
+ * none), and state_bytes of recurrent state (0: none).  Layers with F16 rows and
+ * k_dim = v_dim have the page layout of wr_cuda_kv_create and are accepted by
+ * every call below; other layers by wr_cuda_model_forward only. */
+#define WR_CUDA_MAX_LAYER_RUNS 1024
+typedef struct wr_cuda_cache_layer {
+    uint32_t n_kv_heads, k_dim, v_dim, elem;
+    uint64_t state_bytes;
+} wr_cuda_cache_layer;
+int  wr_cuda_kv_create_layout(wr_cuda_ctx *ctx, uint32_t n_layers, const wr_cuda_cache_layer *layers,
+                              uint32_t max_ctx, wr_cuda_kv **out);
 void wr_cuda_kv_destroy(wr_cuda_kv *kv);
 uint32_t wr_cuda_kv_max_ctx(const wr_cuda_kv *kv);
 
@@ -358,6 +373,94 @@ int wr_cuda_model_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t
                           const uint32_t *tokens, uint32_t out_from, float *hidden_out,
                           float *normed_out, float *const *logits_out, uint32_t *argmax_out,
                           float *attn_tap_out);
+
+/* ---- models whose layers differ ------------------------------------------- */
+
+/* A model put together from mixers: every layer names its own mixer (softmax
+ * attention, plain or differential; selective scan) and feed-forward with sizes
+ * of its own, a run list says in which order the layers are applied (a layer
+ * may run several times with the same weights; each run keeps a cache or state
+ * of its own).  It is a wr_cuda_model like the one above: created from host
+ * pointers, stepped by wr_cuda_model_forward, destroyed by
+ * wr_cuda_model_destroy; its sessions come from wr_cuda_model_kv_create.  (No
+ * reference counterpart: the reference's decode body knows one layer shape per
+ * architecture, src/core/session.c:405-568.)
+ *
+ * Tensors are host pointers with their element type (WR_CUDA_F32 or
+ * WR_CUDA_BF16); a projection is [out][in] as everywhere in this header.
+ * `compute` chooses the arithmetic: WR_CUDA_F32 keeps weights, activations and
+ * K/V rows in 32 bits; WR_CUDA_BF16 keeps weights in BF16, runs the matrix
+ * products of more than WR_CUDA_BATCH_MAX rows on BF16 activations with 32-bit
+ * accumulation, and keeps K/V rows in F16 (rounded to nearest).  In both the
+ * residual stream, norms, softmax and recurrences are 32-bit. */
+typedef struct wr_cuda_tensor {
+    const void *data;                 /* NULL: the layer does not have it */
+    uint32_t dtype, reserved;
+} wr_cuda_tensor;
+
+#define WR_CUDA_MIXER_ATTENTION 1
+#define WR_CUDA_MIXER_MAMBA1    2
+#define WR_CUDA_FFN_NONE        0
+#define WR_CUDA_FFN_POLYNORM    1
+#define WR_CUDA_POS_NONE        0
+#define WR_CUDA_POS_SINUSOIDAL  1     /* added to the embedding: sin, cos of p * base^(-2i/width) interleaved */
+
+typedef struct wr_cuda_mixed_layer {
+    uint32_t mixer, ffn;
+    wr_cuda_tensor norm1, norm2;      /* [width]; norm2 only with a feed-forward */
+    wr_cuda_tensor shift;             /* [width]: mixer input h + (h_before - h) * shift, or absent */
+
+    /* WR_CUDA_MIXER_ATTENTION.  n_maps = 2 is differential attention: every
+     * query head has two queries and every kv head two keys over one value, and
+     * the head's output is (a1 - lambda a2) over its own root mean square (eps
+     * diff_eps) times 1 - diff_init, lambda = exp(lq1.lk1) - exp(lq2.lk2) +
+     * diff_init.  q rows are [head][map][k_dim], k rows [kv head][map][k_dim]. */
+    uint32_t n_q_heads, n_kv_heads, n_maps, k_dim, v_dim;
+    uint32_t q_temp_every;            /* > 0: q times 1 + coef ln(floor((p+1)/every) + 1) */
+    float q_temp_coef, attn_scale, diff_init, diff_eps;
+    wr_cuda_tensor wq, wk, wv, wo, bq, bk, bv;      /* biases optional */
+    wr_cuda_tensor w_gate;            /* [n_q*v_dim][width]: heads times sigmoid(w_gate h), or absent */
+    wr_cuda_tensor lq1, lk1, lq2, lk2;              /* [k_dim], n_maps = 2 */
+
+    /* WR_CUDA_MIXER_MAMBA1: inner channels with `state` numbers each, a causal
+     * convolution of `taps` taps, step sizes through rank dt_rank. */
+    uint32_t inner, state, dt_rank, taps;
+    wr_cuda_tensor w_in, conv, conv_b, w_x, w_dt, dt_b, a_log, d, w_out;
+
+    /* WR_CUDA_FFN_POLYNORM: down(a N(z) + b N(z^2) + c N(z^3) + e), z = up h,
+     * N = over its own root mean square (eps ffn_eps); act = {a, b, c, e}. */
+    uint32_t ffn_dim;
+    float ffn_eps;
+    wr_cuda_tensor w_up, w_down, act;
+} wr_cuda_mixed_layer;
+
+typedef struct wr_cuda_mixed_desc {
+    uint32_t compute;                 /* WR_CUDA_F32 or WR_CUDA_BF16 */
+    uint32_t width, vocab, n_layers, n_runs;
+    uint32_t max_rows;                /* rows one forward pass may carry (prefill chunk) */
+    uint32_t norm_groups;             /* RMS norm over this many equal parts of the row */
+    uint32_t position;                /* WR_CUDA_POS_* */
+    float norm_eps, position_base;
+    const uint32_t *runs;             /* n_runs layer indices, in the order they are applied */
+    wr_cuda_tensor embed, head, final_norm;
+    const wr_cuda_mixed_layer *layers;
+} wr_cuda_mixed_desc;
+
+int  wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_desc *desc, wr_cuda_model **out);
+
+/* An empty session for a model of either kind, for up to max_ctx tokens.  With
+ * a mixed model wr_cuda_model_forward takes a step at the position the session
+ * stands at, at the one before its last step again (that step is then undone),
+ * or at 0 (the session starts over); any other position is WR_CUDA_ERR_STATE. */
+int  wr_cuda_model_kv_create(wr_cuda_ctx *ctx, wr_cuda_model *m, uint32_t max_ctx, wr_cuda_kv **out);
+
+/* wr_cuda_model_forward on a mixed model differs in three points: logits_out
+ * may name any number of rows (NULL entries are skipped, only the named rows
+ * reach the head), argmax_out still at most WR_CUDA_BATCH_MAX; attn_tap_out must
+ * be NULL; and hidden_tap, when set with the call below, receives the residual
+ * rows after every layer run of the following calls, [n_runs][n_rows][width]
+ * (host memory; NULL turns it off). */
+int  wr_cuda_model_set_hidden_tap(wr_cuda_model *m, float *hidden_tap);
 
 #ifdef __cplusplus
 }

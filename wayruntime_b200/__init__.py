@@ -10,12 +10,14 @@ from .binding import (  # noqa: F401
     Exchange,
     Context,
     DeviceModel,
+    MixedModel,
     KVCache,
     WrCudaError,
     MEM_DEVICE,
     MEM_HOST,
     F16,
     F32,
+    BF16,
     APPEND_ROPE,
     TRIPLE_PAD,
     device_check,
@@ -24,6 +26,6 @@ from .binding import (  # noqa: F401
 )
 
 __all__ = [
-    "Batch", "Context", "DeviceModel", "Exchange", "KVCache", "WrCudaError", "MEM_DEVICE", "MEM_HOST", "F16", "F32",
+    "Batch", "Context", "DeviceModel", "Exchange", "KVCache", "MixedModel", "WrCudaError", "MEM_DEVICE", "MEM_HOST", "F16", "F32", "BF16",
     "APPEND_ROPE", "TRIPLE_PAD", "device_check", "load_library", "status_name",
 ]

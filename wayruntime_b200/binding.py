@@ -17,7 +17,7 @@ _PKG = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_PKG, "lib", "libwr_cuda.so")
 
 MEM_HOST, MEM_DEVICE = 0, 1
-F32, F16 = 0, 1
+F32, F16, BF16 = 0, 1, 2
 APPEND_ROPE = 1
 TRIPLE_PAD = 4
 BATCH_MAX = 16
@@ -40,7 +40,8 @@ EXPORTS = [
     "wr_cuda_xchg_destroy",
     "wr_cuda_attn_exchange_combine", "wr_cuda_attn_decode_exchange",
     "wr_cuda_model_create", "wr_cuda_model_destroy", "wr_cuda_model_bytes", "wr_cuda_model_launches", "wr_cuda_model_last_enqueue_ns",
-    "wr_cuda_model_forward",
+    "wr_cuda_model_forward", "wr_cuda_kv_create_layout", "wr_cuda_model_create_mixed", "wr_cuda_model_kv_create",
+    "wr_cuda_model_set_hidden_tap",
 ]
 
 
@@ -68,6 +69,42 @@ class ModelDesc(C.Structure):
                [(n, C.c_float) for n in ("rms_eps", "rope_theta", "attn_scale", "reserved")] + \
                [("embed", C.c_void_p), ("lm_head", C.c_void_p), ("final_norm", C.c_void_p),
                 ("layers", C.POINTER(LayerDesc))]
+
+
+class CacheLayer(C.Structure):
+    """wr_cuda_cache_layer (include/wr_cuda.h)."""
+    _fields_ = [(n, C.c_uint32) for n in ("n_kv_heads", "k_dim", "v_dim", "elem")] + [("state_bytes", C.c_uint64)]
+
+
+class Tensor(C.Structure):
+    """wr_cuda_tensor (include/wr_cuda.h)."""
+    _fields_ = [("data", C.c_void_p), ("dtype", C.c_uint32), ("reserved", C.c_uint32)]
+
+
+MIXER_ATTENTION, MIXER_MAMBA1 = 1, 2
+FFN_NONE, FFN_POLYNORM = 0, 1
+POS_NONE, POS_SINUSOIDAL = 0, 1
+
+
+class MixedLayerDesc(C.Structure):
+    """wr_cuda_mixed_layer (include/wr_cuda.h)."""
+    TENSORS = ("norm1", "norm2", "shift", "wq", "wk", "wv", "wo", "bq", "bk", "bv", "w_gate", "lq1", "lk1", "lq2", "lk2",
+               "w_in", "conv", "conv_b", "w_x", "w_dt", "dt_b", "a_log", "d", "w_out", "w_up", "w_down", "act")
+    _fields_ = [("mixer", C.c_uint32), ("ffn", C.c_uint32)] + [(n, Tensor) for n in ("norm1", "norm2", "shift")] + \
+               [(n, C.c_uint32) for n in ("n_q_heads", "n_kv_heads", "n_maps", "k_dim", "v_dim", "q_temp_every")] + \
+               [(n, C.c_float) for n in ("q_temp_coef", "attn_scale", "diff_init", "diff_eps")] + \
+               [(n, Tensor) for n in ("wq", "wk", "wv", "wo", "bq", "bk", "bv", "w_gate", "lq1", "lk1", "lq2", "lk2")] + \
+               [(n, C.c_uint32) for n in ("inner", "state", "dt_rank", "taps")] + \
+               [(n, Tensor) for n in ("w_in", "conv", "conv_b", "w_x", "w_dt", "dt_b", "a_log", "d", "w_out")] + \
+               [("ffn_dim", C.c_uint32), ("ffn_eps", C.c_float)] + [(n, Tensor) for n in ("w_up", "w_down", "act")]
+
+
+class MixedDesc(C.Structure):
+    """wr_cuda_mixed_desc (include/wr_cuda.h)."""
+    _fields_ = [(n, C.c_uint32) for n in ("compute", "width", "vocab", "n_layers", "n_runs", "max_rows", "norm_groups",
+                                          "position")] + \
+               [("norm_eps", C.c_float), ("position_base", C.c_float), ("runs", C.POINTER(C.c_uint32))] + \
+               [(n, Tensor) for n in ("embed", "head", "final_norm")] + [("layers", C.POINTER(MixedLayerDesc))]
 
 
 _lib = None
@@ -125,6 +162,10 @@ def load_library():
         "wr_cuda_model_bytes": (C.c_uint64, [vp]),
         "wr_cuda_model_launches": (C.c_uint64, [vp]),
         "wr_cuda_model_last_enqueue_ns": (C.c_uint64, [vp]),
+        "wr_cuda_kv_create_layout": (i32, [vp, u32, C.POINTER(CacheLayer), u32, C.POINTER(vp)]),
+        "wr_cuda_model_create_mixed": (i32, [vp, C.POINTER(MixedDesc), C.POINTER(vp)]),
+        "wr_cuda_model_kv_create": (i32, [vp, vp, u32, C.POINTER(vp)]),
+        "wr_cuda_model_set_hidden_tap": (i32, [vp, vp]),
         "wr_cuda_model_forward": (i32, [vp, vp, i32, u32, C.POINTER(vp), C.POINTER(u32), C.POINTER(u32), u32,
                                         vp, vp, C.POINTER(vp), C.POINTER(u32), vp]),
     }
@@ -405,7 +446,7 @@ class DeviceModel:
     def __init__(self, ctx: "Context", weights: dict, *, n_layers, hidden, n_q_heads, n_kv_heads, head_dim,
                  vocab, ffn, rms_eps=1e-6, rope_theta=10000.0, n_rot_pairs=0, attn_scale=0.0, max_rows=256):
         self._ctx, self._lib = ctx, ctx._lib
-        self.vocab, self.hidden, self.n_layers = vocab, hidden, n_layers
+        self.vocab, self.hidden, self.n_layers, self.max_rows = vocab, hidden, n_layers, max_rows
         self.n_q, self.hd = n_q_heads, head_dim
 
         def ptr(name, optional=False):
@@ -451,18 +492,35 @@ class DeviceModel:
         """Host time the last forward pass spent enqueueing work, before waiting for the device."""
         return self._lib.wr_cuda_model_last_enqueue_ns(self._h) * 1e-6
 
+    def kv_create(self, max_ctx: int) -> "KVCache":
+        """An empty session of this model for up to max_ctx tokens."""
+        h = C.c_void_p()
+        _check(self._lib.wr_cuda_model_kv_create(self._ctx._h, self._h, max_ctx, C.byref(h)), "wr_cuda_model_kv_create")
+        return KVCache._of_handle(self._ctx, h, max_ctx)
+
     def forward(self, mode, kvs, positions, tokens, out_from=0, *, hidden=False, normed=False, logits=False,
                 argmax=False, attn_tap=False) -> dict:
-        """One forward pass; returns the requested results for rows [out_from, n) as numpy arrays."""
+        """One forward pass; returns the requested results for rows [out_from, n) as numpy arrays.
+        logits may be a list of places among those rows (the others are skipped): the result then has
+        one row per place, in the list's order."""
         n = len(tokens)
         n_out = n - out_from
         res = {}
         hid = np.empty((n_out, self.hidden), np.float32) if hidden else None
         nrm = np.empty((n_out, self.hidden), np.float32) if normed else None
-        lg = np.empty((n_out, self.vocab), np.float32) if logits else None
+        some = None if isinstance(logits, bool) else [int(i) for i in logits]
+        logits = bool(some) if some is not None else logits
+        lg = np.empty((len(some) if some is not None else n_out, self.vocab), np.float32) if logits else None
         am = (C.c_uint32 * max(n_out, 1))() if argmax else None
         tap = np.empty((self.n_layers, n, self.n_q * self.hd), np.float32) if attn_tap else None
-        lptrs = (C.c_void_p * max(n_out, 1))(*[lg[i].ctypes.data for i in range(n_out)]) if logits else None
+        lptrs = None
+        if logits:
+            lptrs = (C.c_void_p * max(n_out, 1))()
+            base, row = lg.ctypes.data, lg.strides[0]
+            for j, i in enumerate(some if some is not None else range(n_out)):
+                if not 0 <= i < n_out or lptrs[i]:
+                    raise ValueError("places out of range or named twice")
+                lptrs[i] = base + j * row
         _check(self._lib.wr_cuda_model_forward(
             self._ctx._h, self._h, mode, n, Context._handles(kvs), Context._u32s(positions),
             Context._u32s(tokens), out_from, hid.ctypes.data if hidden else None,
@@ -474,6 +532,50 @@ class DeviceModel:
         if argmax: res["argmax"] = np.array([am[i] for i in range(n_out)], np.uint32)
         if attn_tap: res["attn"] = tap
         return res
+
+
+class MixedModel(DeviceModel):
+    """wr_cuda_model of the mixed kind (wr_cuda_model_create_mixed).  `layers` is a list of dicts with the
+    scalar fields of wr_cuda_mixed_layer; `tensor(i, field)` returns layer i's array for a tensor field (or None),
+    and tensor(None, name) the model's embed, head and final_norm.  Arrays are float32, or uint16 holding
+    bfloat16 bits."""
+
+    def __init__(self, ctx: "Context", layers, runs, tensor, *, compute, width, vocab, norm_groups, norm_eps,
+                 position=POS_NONE, position_base=10000.0, max_rows=256):
+        self._ctx, self._lib = ctx, ctx._lib
+        self.vocab, self.hidden, self.n_layers, self.max_rows = vocab, width, len(runs), max_rows
+        self.n_q = self.hd = 0
+        keep = []
+
+        def ref(a):
+            if a is None:
+                return Tensor()
+            if a.dtype not in (np.float32, np.uint16):
+                raise ValueError("float32, or bfloat16 bits in uint16, expected")
+            a = np.ascontiguousarray(a)
+            keep.append(a)
+            return Tensor(a.ctypes.data, F32 if a.dtype == np.float32 else BF16, 0)
+
+        arr = (MixedLayerDesc * len(layers))()
+        for i, lay in enumerate(layers):
+            for k, v in lay.items():
+                setattr(arr[i], k, v)
+            for k in MixedLayerDesc.TENSORS:
+                setattr(arr[i], k, ref(tensor(i, k)))
+        d = MixedDesc(compute=compute, width=width, vocab=vocab, n_layers=len(layers), n_runs=len(runs),
+                      max_rows=max_rows, norm_groups=norm_groups, position=position, norm_eps=norm_eps,
+                      position_base=position_base, runs=(C.c_uint32 * len(runs))(*runs), embed=ref(tensor(None, "embed")),
+                      head=ref(tensor(None, "head")), final_norm=ref(tensor(None, "final_norm")), layers=arr)
+        h = C.c_void_p()
+        _check(self._lib.wr_cuda_model_create_mixed(ctx._h, C.byref(d), C.byref(h)), "wr_cuda_model_create_mixed")
+        self._h = h
+
+    def set_hidden_tap(self, out):
+        """Residual rows after every layer run of the following forward calls into `out`
+        (float32 [runs, rows, width]; None turns it off)."""
+        _check(self._lib.wr_cuda_model_set_hidden_tap(self._h, None if out is None else out.ctypes.data),
+               "wr_cuda_model_set_hidden_tap")
+        self._tap = out
 
 
 class Batch:
@@ -504,6 +606,13 @@ class KVCache:
         self._h = h
         self.n_layers, self.n_kv_heads, self.head_dim, self.max_ctx = (
             n_layers, n_kv_heads, head_dim, max_ctx)
+
+    @classmethod
+    def _of_handle(cls, ctx, handle, max_ctx):
+        kv = cls.__new__(cls)
+        kv._ctx, kv._lib, kv._h, kv.max_ctx = ctx, ctx._lib, handle, max_ctx
+        kv.n_layers = kv.n_kv_heads = kv.head_dim = None
+        return kv
 
     def close(self):
         if getattr(self, "_h", None) and getattr(self._ctx, "_h", None):

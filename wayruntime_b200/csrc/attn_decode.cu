@@ -150,7 +150,7 @@ int wr_decode_validate(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *kv,
     if (mem != WR_CUDA_MEM_HOST && mem != WR_CUDA_MEM_DEVICE) return WR_CUDA_ERR_INVAL;
     if (mem == WR_CUDA_MEM_DEVICE && (((uintptr_t)q | (uintptr_t)out) & 15u))
         return WR_CUDA_ERR_INVAL;                                         // rows move as 16-byte vectors
-    if (n_q == 0 || n_q % kv[0]->n_kv != 0) return WR_CUDA_ERR_INVAL;     // kernels.c:1429-1432
+    if (n_q == 0 || n_q % kv[0]->n_kv_at(layer) != 0) return WR_CUDA_ERR_INVAL;     // kernels.c:1429-1432
     for (uint32_t s = 0; s < n_sess; ++s) {
         if (seq_lens[s] == 0 && !emit_triples) return WR_CUDA_ERR_INVAL;  // kernels.c:1439
         if (seq_lens[s] > ctx->attn_max_seq) return WR_CUDA_ERR_LIMIT;    // kernels.c:1444
@@ -169,7 +169,7 @@ void wr_decode_plan(uint32_t n_sess, wr_cuda_kv *const *kv, uint32_t layer, cons
                     uint32_t n_q, uint32_t window, wr_decode::params &p, uint32_t &nt, uint32_t &items)
 {
     using namespace wr_decode;
-    const uint32_t n_kv = kv[0]->n_kv, hd = kv[0]->hd;
+    const uint32_t n_kv = kv[0]->n_kv_at(layer), hd = kv[0]->hd_at(layer);
     const uint32_t group = n_q / n_kv;
     nt = group <= 4 ? 1u : 2u;
     const uint32_t qsubs = (group + 4 * nt - 1) / (4 * nt);
@@ -219,7 +219,7 @@ int wr_decode_launch(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *kv, u
                      float scale_override, uint32_t window, int emit_triples, wr_decode_xchg *xchg,
                      bool early_tiles)
 {
-    const uint32_t n_kv = kv[0]->n_kv, hd = kv[0]->hd;
+    const uint32_t n_kv = kv[0]->n_kv_at(layer), hd = kv[0]->hd_at(layer);
     const uint32_t group = n_q / n_kv;
     const float scale = scale_for(hd, scale_override);
 
@@ -323,7 +323,7 @@ static int decode_common(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *k
     int rc = wr_decode_validate(ctx, n_sess, kv, layer, seq_lens, q, out, n_q, mem, emit_triples);
     if (rc != WR_CUDA_OK) return rc;
     WR_CUDA_TRY(cudaSetDevice(ctx->device));
-    const uint32_t hd = kv[0]->hd;
+    const uint32_t hd = kv[0]->hd_at(layer);
     const size_t q_bytes = (size_t)n_sess * n_q * hd * sizeof(float);
     const size_t out_row = emit_triples ? (WR_CUDA_TRIPLE_PAD + hd) : hd;
     const size_t out_bytes = (size_t)n_sess * n_q * out_row * sizeof(float);
@@ -370,7 +370,7 @@ extern "C" int wr_cuda_decode_step(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv
     rc = wr_decode_validate(ctx, n_sess, kv, layer, seq_lens, q, out, n_q_heads, mem, 0);
     if (rc != WR_CUDA_OK) return rc;
     WR_CUDA_TRY(cudaSetDevice(ctx->device));
-    const uint32_t hd = kv[0]->hd, n_kv = kv[0]->n_kv;
+    const uint32_t hd = kv[0]->hd_at(layer), n_kv = kv[0]->n_kv_at(layer);
     const size_t kv_bytes = (size_t)n_sess * n_kv * hd * sizeof(float);
     const size_t q_bytes = (size_t)n_sess * n_q_heads * hd * sizeof(float);
     const float *dk = k_rows, *dv = v_rows, *dq_in = nullptr;

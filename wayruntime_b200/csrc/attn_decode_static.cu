@@ -116,7 +116,7 @@ extern "C" int wr_cuda_attn_decode_static(wr_cuda_ctx *ctx, uint32_t n_sess, wr_
     if (rc != WR_CUDA_OK) return rc;
     if (!seq_lens || !q || !out) return WR_CUDA_ERR_INVAL;
     if ((((uintptr_t)q | (uintptr_t)out) & 15u)) return WR_CUDA_ERR_INVAL;
-    const uint32_t n_kv = kv[0]->n_kv, hd = kv[0]->hd;
+    const uint32_t n_kv = kv[0]->n_kv_at(layer), hd = kv[0]->hd_at(layer);
     if (hd != (uint32_t)kHd) return WR_CUDA_ERR_UNSUPPORTED;
     if (n_q_heads == 0 || n_q_heads % n_kv != 0) return WR_CUDA_ERR_INVAL;
     for (uint32_t s = 0; s < n_sess; ++s) {

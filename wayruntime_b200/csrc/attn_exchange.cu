@@ -291,7 +291,7 @@ extern "C" int wr_cuda_attn_decode_exchange(wr_cuda_ctx *ctx, wr_cuda_xchg *x, u
     std::lock_guard<std::mutex> g(ctx->lock);
     int rc = wr_decode_validate(ctx, n_sess, kv, layer, seq_lens, q, out, n_q_heads, WR_CUDA_MEM_DEVICE, 1);
     if (rc != WR_CUDA_OK) return rc;
-    if (kv[0]->hd != 128 || x->hd != 128) return WR_CUDA_ERR_UNSUPPORTED;      // the fused path is the head_dim-128 kernel's
+    if (kv[0]->hd_at(layer) != 128 || x->hd != 128) return WR_CUDA_ERR_UNSUPPORTED;      // the fused path is the head_dim-128 kernel's
     const uint32_t n_rows = n_sess * n_q_heads;
     if (n_rows == 0 || n_rows > x->max_rows) return WR_CUDA_ERR_INVAL;
     WR_CUDA_TRY(cudaSetDevice(ctx->device));

@@ -971,8 +971,8 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
     if (q_dtype != WR_CUDA_F32 && q_dtype != WR_CUDA_F16) return WR_CUDA_ERR_INVAL;
     if (mem != WR_CUDA_MEM_HOST && mem != WR_CUDA_MEM_DEVICE) return WR_CUDA_ERR_INVAL;
     if (n == 0) return WR_CUDA_OK;
-    if (n_q_heads == 0 || n_q_heads % kv->n_kv != 0) return WR_CUDA_ERR_INVAL;   // kernels.c:1429-1432
-    if (kv->hd != kHd) return WR_CUDA_ERR_UNSUPPORTED;       // tensor-core tiles are built for head_dim 128
+    if (kv->hd_at(layer) != kHd) return WR_CUDA_ERR_UNSUPPORTED;       // tensor-core tiles are built for head_dim 128
+    if (n_q_heads == 0 || n_q_heads % kv->n_kv_at(layer) != 0) return WR_CUDA_ERR_INVAL;   // kernels.c:1429-1432
     std::lock_guard<std::mutex> g(ctx->lock);
     if ((uint64_t)p0 + n > ctx->attn_max_seq) return WR_CUDA_ERR_LIMIT;           // kernels.c:1444
     if ((uint64_t)p0 + n > kv->max_ctx) return WR_CUDA_ERR_INVAL;                 // capacity, kernels.c:1449-1454
@@ -1045,7 +1045,7 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
     prefill_params p;
     p.pages = kv->d_pages + (size_t)layer * kv->n_pages;
     p.page_base = kv->contig[layer] ? (const char *)kv->pages[(size_t)layer * kv->n_pages] : nullptr;
-    p.page_bytes = wr_page_bytes(kv->n_kv, kHd);
+    p.page_bytes = wr_page_bytes(kv->n_kv_at(layer), kHd);
 #ifdef WR_PREFILL_TIMELINE
     if (!ctx->debug_buf) {
         WR_CUDA_TRY(cudaMalloc(&ctx->debug_buf, (kTlRoles * kTlEvents + 4 * kTlCtas) * sizeof(long long)));
@@ -1059,8 +1059,8 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
     p.n = n;
     p.p0 = p0;
     p.n_q = n_q_heads;
-    p.n_kv = kv->n_kv;
-    p.group = n_q_heads / kv->n_kv;
+    p.n_kv = kv->n_kv_at(layer);
+    p.group = n_q_heads / kv->n_kv_at(layer);
     p.window = window;
     p.n_qtiles = (n + kBM - 1) / kBM;
     p.n_tiles = prefill_tile_count(p.n_qtiles, p.n_kv, p.group);

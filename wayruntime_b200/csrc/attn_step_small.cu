@@ -268,7 +268,7 @@ __global__ void __launch_bounds__(kSmallThreads) attn_step_small_kernel(const st
 
 bool wr_step_small_covers(const wr_cuda_kv *kv, uint32_t n_q_heads, uint32_t position)
 {
-    return kv->hd == kHd && kv->n_kv > 0 && n_q_heads % kv->n_kv == 0 && n_q_heads / kv->n_kv <= kSmallMaxGroup &&
+    return kv->hd_at(0) == kHd && kv->n_kv_at(0) > 0 && n_q_heads % kv->n_kv_at(0) == 0 && n_q_heads / kv->n_kv_at(0) <= kSmallMaxGroup &&
            position + 1 <= kSmallMaxKeys;
 }
 
@@ -294,7 +294,7 @@ int wr_step_small_launch(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *k
     p.out = dout;
     p.q_norm = q_norm;
     p.k_norm = k_norm;
-    p.n_kv = kv[0]->n_kv;
+    p.n_kv = kv[0]->n_kv_at(0);
     p.n_q = n_q_heads;
     p.n_rot = (n_rot_pairs >= 1 && n_rot_pairs < half) ? n_rot_pairs : half;     // kernels.c:1381-1383
     p.eps = eps;

@@ -256,6 +256,123 @@ static int pool_take(wr_cuda_ctx *ctx, uint64_t page_bytes, size_t n, size_t *po
     return WR_CUDA_OK;
 }
 
+// Everything a session holds goes back to the pools it came from, cleared so that the next owner
+// starts from zeros.  Caller holds ctx->lock.
+static void kv_give_back(wr_cuda_kv *kv)
+{
+    wr_cuda_ctx *ctx = kv->ctx;
+    for (uint32_t L = 0; L < kv->n_layers && !kv->pages.empty(); ++L) {
+        const wr_kv_layer &lay = kv->layers[L];
+        void **first = kv->pages.data() + (size_t)L * kv->n_pages;
+        if (!lay.geom.n_kv || !first[0]) continue;
+        if (kv->contig[L]) {
+            (void)cudaMemsetAsync(first[0], 0, lay.page_bytes * kv->n_pages, ctx->stream);
+        } else {
+            for (uint32_t i = 0; i < kv->n_pages; ++i)
+                (void)cudaMemsetAsync(first[i], 0, lay.page_bytes, ctx->stream);
+        }
+        auto &fp = ctx->pools[lay.pool_index].free_pages;
+        for (uint32_t i = kv->n_pages; i-- > 0;) fp.push_back(first[i]);
+    }
+    if (kv->state[0]) {
+        auto &fp = ctx->pools[kv->state_pool].free_pages;
+        for (int i = 2; i-- > 0;) {
+            (void)cudaMemsetAsync(kv->state[i], 0, ctx->pools[kv->state_pool].page_bytes, ctx->stream);
+            fp.push_back(kv->state[i]);
+        }
+    }
+    (void)cudaStreamSynchronize(ctx->stream);
+    if (kv->d_pages) (void)cudaFree(kv->d_pages);
+    (void)cudaGetLastError();
+}
+
+extern "C" int wr_cuda_kv_create_layout(wr_cuda_ctx *ctx, uint32_t n_layers, const wr_cuda_cache_layer *layers,
+                                        uint32_t max_ctx, wr_cuda_kv **out)
+{
+    if (!ctx || !out) return WR_CUDA_ERR_INVAL;
+    *out = nullptr;
+    if (n_layers == 0 || !layers || max_ctx == 0) return WR_CUDA_ERR_INVAL;
+    if (n_layers > WR_CUDA_MAX_LAYER_RUNS) return WR_CUDA_ERR_LIMIT;
+    for (uint32_t L = 0; L < n_layers; ++L) {
+        const wr_cuda_cache_layer &l = layers[L];
+        if (l.n_kv_heads == 0) continue;
+        if (l.k_dim == 0 || l.v_dim == 0 || (l.elem != WR_CUDA_F32 && l.elem != WR_CUDA_F16)) return WR_CUDA_ERR_INVAL;
+        if (l.k_dim > WR_CUDA_HEAD_DIM_MAX || l.v_dim > WR_CUDA_HEAD_DIM_MAX) return WR_CUDA_ERR_LIMIT;
+    }
+    std::lock_guard<std::mutex> g(ctx->lock);
+    if (max_ctx > ctx->attn_max_seq) return WR_CUDA_ERR_LIMIT;  // session.c:755
+    WR_CUDA_TRY(cudaSetDevice(ctx->device));
+    wr_cuda_kv *kv = new (std::nothrow) wr_cuda_kv();
+    if (!kv) return WR_CUDA_ERR_NOMEM;
+    kv->ctx = ctx;
+    kv->n_layers = n_layers;
+    kv->max_ctx = max_ctx;
+    kv->n_pages = (max_ctx + kPageTokens - 1) / kPageTokens;
+    kv->layers.resize(n_layers);
+    const size_t total = (size_t)n_layers * kv->n_pages;
+    kv->pages.assign(total, nullptr);
+    // A layer whose pages came out of the pool back to back needs no table
+    // lookup on the device: page i sits at base + i * page_bytes.
+    kv->contig.assign(n_layers, 1);
+    int rc = WR_CUDA_OK;
+    for (uint32_t L = 0; L < n_layers; ++L) {
+        wr_kv_layer &lay = kv->layers[L];
+        lay.geom = {layers[L].n_kv_heads, layers[L].k_dim, layers[L].v_dim, layers[L].elem};
+        lay.page_bytes = wr_geom_page_bytes(lay.geom);
+        lay.state_off = kv->state_bytes;
+        lay.state_bytes = layers[L].state_bytes;
+        kv->state_bytes += (lay.state_bytes + 255u) & ~(uint64_t)255u;
+    }
+    // layers with pages of one size take them in one go (one slab at most)
+    for (uint32_t L = 0; L < n_layers && rc == WR_CUDA_OK; ++L) {
+        if (!kv->layers[L].geom.n_kv || kv->pages[(size_t)L * kv->n_pages]) continue;
+        std::vector<uint32_t> same;
+        for (uint32_t M = L; M < n_layers; ++M)
+            if (kv->layers[M].geom.n_kv && kv->layers[M].page_bytes == kv->layers[L].page_bytes) same.push_back(M);
+        std::vector<void *> got;
+        size_t pool = 0;
+        rc = pool_take(ctx, kv->layers[L].page_bytes, same.size() * kv->n_pages, &pool, got);
+        if (rc != WR_CUDA_OK) break;
+        for (size_t j = 0; j < same.size(); ++j) {
+            const uint32_t M = same[j];
+            kv->layers[M].pool_index = pool;
+            for (uint32_t i = 0; i < kv->n_pages; ++i) {
+                kv->pages[(size_t)M * kv->n_pages + i] = got[j * kv->n_pages + i];
+                if (i > 0 && (char *)got[j * kv->n_pages + i] !=
+                                 (char *)got[j * kv->n_pages + i - 1] + kv->layers[M].page_bytes)
+                    kv->contig[M] = 0;
+            }
+        }
+    }
+    if (rc == WR_CUDA_OK && kv->state_bytes) {
+        std::vector<void *> got;
+        rc = pool_take(ctx, kv->state_bytes, 2, &kv->state_pool, got);
+        if (rc == WR_CUDA_OK) {
+            kv->state[0] = got[0];
+            kv->state[1] = got[1];
+        }
+    }
+    if (rc == WR_CUDA_OK) {
+        cudaError_t e = cudaMalloc((void **)&kv->d_pages, total * sizeof(uint64_t));
+        if (e == cudaSuccess)
+            e = cudaMemcpyAsync(kv->d_pages, kv->pages.data(), total * sizeof(uint64_t),
+                                cudaMemcpyHostToDevice, ctx->stream);
+        if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+        if (e != cudaSuccess) {
+            (void)cudaGetLastError();
+            rc = e == cudaErrorMemoryAllocation ? WR_CUDA_ERR_NOMEM : WR_CUDA_ERR_INTERNAL;
+        }
+    }
+    if (rc != WR_CUDA_OK) {
+        kv_give_back(kv);
+        delete kv;
+        return rc;
+    }
+    ctx->live_kv++;
+    *out = kv;
+    return WR_CUDA_OK;
+}
+
 extern "C" int wr_cuda_kv_create(wr_cuda_ctx *ctx, uint32_t n_layers, uint32_t n_kv_heads,
                                  uint32_t head_dim, uint32_t max_ctx, wr_cuda_kv **out)
 {
@@ -264,49 +381,10 @@ extern "C" int wr_cuda_kv_create(wr_cuda_ctx *ctx, uint32_t n_layers, uint32_t n
     if (n_layers == 0 || n_kv_heads == 0 || head_dim == 0 || max_ctx == 0) return WR_CUDA_ERR_INVAL;
     if (head_dim & 1u) return WR_CUDA_ERR_INVAL;                // RoPE pairs (kernels.c:1366)
     if (head_dim > WR_CUDA_HEAD_DIM_MAX) return WR_CUDA_ERR_LIMIT;
-    if (n_layers > 64) return WR_CUDA_ERR_LIMIT;                // WR_MAX_LAYERS (internal.h:184)
-    std::lock_guard<std::mutex> g(ctx->lock);
-    if (max_ctx > ctx->attn_max_seq) return WR_CUDA_ERR_LIMIT;  // session.c:755
-    WR_CUDA_TRY(cudaSetDevice(ctx->device));
-    wr_cuda_kv *kv = new (std::nothrow) wr_cuda_kv();
-    if (!kv) return WR_CUDA_ERR_NOMEM;
-    kv->ctx = ctx;
-    kv->n_layers = n_layers;
-    kv->n_kv = n_kv_heads;
-    kv->hd = head_dim;
-    kv->max_ctx = max_ctx;
-    kv->n_pages = (max_ctx + kPageTokens - 1) / kPageTokens;
-    size_t total = (size_t)n_layers * kv->n_pages;
-    int rc = pool_take(ctx, wr_page_bytes(n_kv_heads, head_dim), total, &kv->pool_index, kv->pages);
-    if (rc != WR_CUDA_OK) {
-        delete kv;
-        return rc;
-    }
-    cudaError_t e = cudaMalloc((void **)&kv->d_pages, total * sizeof(uint64_t));
-    if (e == cudaSuccess)
-        e = cudaMemcpyAsync(kv->d_pages, kv->pages.data(), total * sizeof(uint64_t),
-                            cudaMemcpyHostToDevice, ctx->stream);
-    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
-    if (e != cudaSuccess) {
-        (void)cudaGetLastError();
-        auto &fp = ctx->pools[kv->pool_index].free_pages;
-        fp.insert(fp.end(), kv->pages.begin(), kv->pages.end());
-        if (kv->d_pages) (void)cudaFree(kv->d_pages);
-        delete kv;
-        return e == cudaErrorMemoryAllocation ? WR_CUDA_ERR_NOMEM : WR_CUDA_ERR_INTERNAL;
-    }
-    // A layer whose pages came out of the pool back to back needs no table
-    // lookup on the device: page i sits at base + i * page_bytes.
-    kv->contig.assign(n_layers, 1);
-    const uint64_t pb = wr_page_bytes(n_kv_heads, head_dim);
-    for (uint32_t L = 0; L < n_layers; ++L)
-        for (uint32_t i = 1; i < kv->n_pages; ++i)
-            if ((char *)kv->pages[(size_t)L * kv->n_pages + i] !=
-                (char *)kv->pages[(size_t)L * kv->n_pages + i - 1] + pb)
-                kv->contig[L] = 0;
-    ctx->live_kv++;
-    *out = kv;
-    return WR_CUDA_OK;
+    if (n_layers > WR_CUDA_MAX_LAYERS) return WR_CUDA_ERR_LIMIT;   // WR_MAX_LAYERS (internal.h:184)
+    const std::vector<wr_cuda_cache_layer> same(
+        n_layers, wr_cuda_cache_layer{n_kv_heads, head_dim, head_dim, WR_CUDA_F16, 0});
+    return wr_cuda_kv_create_layout(ctx, n_layers, same.data(), max_ctx, out);
 }
 
 extern "C" void wr_cuda_kv_destroy(wr_cuda_kv *kv)
@@ -316,14 +394,7 @@ extern "C" void wr_cuda_kv_destroy(wr_cuda_kv *kv)
     std::lock_guard<std::mutex> g(ctx->lock);
     (void)cudaSetDevice(ctx->device);
     (void)cudaStreamSynchronize(ctx->stream);
-    // Returned pages are cleared again so the next owner starts from zeros.
-    for (void *p : kv->pages)
-        (void)cudaMemsetAsync(p, 0, ctx->pools[kv->pool_index].page_bytes, ctx->stream);
-    auto &fp = ctx->pools[kv->pool_index].free_pages;
-    fp.insert(fp.end(), kv->pages.rbegin(), kv->pages.rend());
-    (void)cudaStreamSynchronize(ctx->stream);
-    if (kv->d_pages) (void)cudaFree(kv->d_pages);
-    (void)cudaGetLastError();
+    kv_give_back(kv);
     ctx->live_kv--;
     delete kv;
 }
@@ -337,7 +408,9 @@ int wr_kv_batch_check(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *kv, 
     for (uint32_t s = 0; s < n_sess; ++s) {
         if (!kv[s] || kv[s]->ctx != ctx) return WR_CUDA_ERR_INVAL;
         if (layer >= kv[s]->n_layers) return WR_CUDA_ERR_INVAL;
-        if (kv[s]->n_kv != kv[0]->n_kv || kv[s]->hd != kv[0]->hd) return WR_CUDA_ERR_INVAL;
+        if (kv[s]->hd_at(layer) == 0) return WR_CUDA_ERR_UNSUPPORTED;    // not the F16, K-as-long-as-V layout
+        if (kv[s]->n_kv_at(layer) != kv[0]->n_kv_at(layer) || kv[s]->hd_at(layer) != kv[0]->hd_at(layer))
+            return WR_CUDA_ERR_INVAL;
         for (uint32_t t = 0; t < s; ++t)
             if (kv[t] == kv[s]) return WR_CUDA_ERR_INVAL;          // distinct sessions (batch.c:133-137)
     }
@@ -384,14 +457,16 @@ static int kv_rows_xfer(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t layer, int wh
 {
     if (!ctx || !kv || kv->ctx != ctx || !buf) return WR_CUDA_ERR_INVAL;
     if (layer >= kv->n_layers || (which != 0 && which != 1)) return WR_CUDA_ERR_INVAL;
+    const uint32_t n_kv = kv->n_kv_at(layer), hd = kv->hd_at(layer);
+    if (hd == 0) return WR_CUDA_ERR_UNSUPPORTED;
     if (n == 0) return WR_CUDA_OK;
     if ((uint64_t)row0 + n > kv->max_ctx) return WR_CUDA_ERR_CTX_FULL;
     if (mem != WR_CUDA_MEM_HOST && mem != WR_CUDA_MEM_DEVICE) return WR_CUDA_ERR_INVAL;
     // device rows move as 16-byte vectors when head_dim allows it
-    if (mem == WR_CUDA_MEM_DEVICE && (kv->hd & 7u) == 0 && ((uintptr_t)buf & 15u)) return WR_CUDA_ERR_INVAL;
+    if (mem == WR_CUDA_MEM_DEVICE && (hd & 7u) == 0 && ((uintptr_t)buf & 15u)) return WR_CUDA_ERR_INVAL;
     std::lock_guard<std::mutex> g(ctx->lock);
     WR_CUDA_TRY(cudaSetDevice(ctx->device));
-    size_t bytes = (size_t)n * kv->n_kv * kv->hd * 2u;
+    size_t bytes = (size_t)n * n_kv * hd * 2u;
     uint16_t *dbuf = buf;
     if (mem == WR_CUDA_MEM_HOST) {
         int rc = wr_ctx_reserve_stage(ctx, bytes, 0);
@@ -400,10 +475,10 @@ static int kv_rows_xfer(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t layer, int wh
         if (to_cache)
             WR_CUDA_TRY(cudaMemcpyAsync(dbuf, buf, bytes, cudaMemcpyHostToDevice, ctx->stream));
     }
-    uint64_t work = (uint64_t)n * kv->n_kv * (wr_hd_pad(kv->hd) / 8u);
+    uint64_t work = (uint64_t)n * n_kv * (wr_hd_pad(hd) / 8u);
     uint32_t blocks = (uint32_t)std::min<uint64_t>((work + 255) / 256, (uint64_t)ctx->sm_count * 16);
     kv_rows_copy_kernel<<<blocks, 256, 0, ctx->stream>>>(
-        kv->d_pages + (size_t)layer * kv->n_pages, dbuf, row0, n, kv->n_kv, kv->hd, (uint32_t)which,
+        kv->d_pages + (size_t)layer * kv->n_pages, dbuf, row0, n, n_kv, hd, (uint32_t)which,
         to_cache);
     ctx->launches++;
     WR_CUDA_TRY(cudaGetLastError());
@@ -611,14 +686,14 @@ int wr_append_launch(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *const *kv, u
         p.b.pages[s] = kv[s]->d_pages + (size_t)layer * kv[s]->n_pages;
         p.b.seq_len[s] = positions[s];
     }
-    const uint32_t hd = kv[0]->hd, half = hd / 2u;
+    const uint32_t hd = kv[0]->hd_at(layer), half = hd / 2u;
     p.k_rows = dk;
     p.v_rows = dv;
     p.q_rows = dq;
     p.q_in = dq_in ? dq_in : dq;
     p.n_sess = n_sess;
     p.n_tokens = n_tokens;
-    p.n_kv = kv[0]->n_kv;
+    p.n_kv = kv[0]->n_kv_at(layer);
     p.n_q = n_q_heads;
     p.hd = hd;
     p.n_rot = (n_rot_pairs >= 1 && n_rot_pairs < half) ? n_rot_pairs : half;  // kernels.c:1381-1383
@@ -647,8 +722,8 @@ extern "C" int wr_cuda_kv_append(wr_cuda_ctx *ctx, uint32_t n_sess, wr_cuda_kv *
     std::lock_guard<std::mutex> g(ctx->lock);
     WR_CUDA_TRY(cudaSetDevice(ctx->device));
     const size_t rows = (size_t)n_sess * n_tokens;
-    const size_t kv_bytes = rows * kv[0]->n_kv * kv[0]->hd * sizeof(float);
-    const size_t q_bytes = q_rows ? rows * n_q_heads * kv[0]->hd * sizeof(float) : 0;
+    const size_t kv_bytes = rows * kv[0]->n_kv_at(layer) * kv[0]->hd_at(layer) * sizeof(float);
+    const size_t q_bytes = q_rows ? rows * n_q_heads * kv[0]->hd_at(layer) * sizeof(float) : 0;
     const float *dk = k_rows, *dv = v_rows;
     float *dq = q_rows;
     if (mem == WR_CUDA_MEM_HOST) {

@@ -1,0 +1,749 @@
+// mixers.cu — row kernels of the mixed layer stack (model_mixed.cu): embedding with positions, grouped RMS
+// norm with token shift, PolyNorm, causal convolution, selective scan, and what surrounds attention.
+//
+// All arithmetic is F32; activation rows that only feed a BF16 matrix product are stored in its type.  Rows are
+// wr_ld(n) values apart; the pad columns are written as zeros, so that a weight-streaming product may read whole
+// 16-byte vectors.  A row's result depends on its session alone: the same code serves a prompt's portion and a
+// decode step, whatever else is in the step.
+#include <cuda_bf16.h>
+
+#include <algorithm>
+
+#include "mixers.cuh"
+
+namespace {
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f32(__half v) { return __half2float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+template <> __device__ __forceinline__ __half from_f32<__half>(float v)
+{
+    return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f));
+}
+__device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float siluf(float x) { return x / (1.0f + expf(-x)); }
+
+// the session of a row and the row's place among the session's tokens of this step
+__device__ __forceinline__ uint32_t seq_of(const wr_rows &rw, uint32_t row) { return rw.decode ? row : 0u; }
+__device__ __forceinline__ uint32_t tok_of(const wr_rows &rw, uint32_t row) { return rw.decode ? 0u : row; }
+__device__ __forceinline__ uint32_t row0_of(const wr_rows &rw, uint32_t seq) { return rw.decode ? seq : 0u; }
+
+__device__ __forceinline__ float warp_sum(float v)
+{
+#pragma unroll
+    for (int o = 16; o >= 1; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+int finish_launch(wr_cuda_ctx *ctx)
+{
+    ctx->launches++;
+    WR_CUDA_TRY(cudaGetLastError());
+    return WR_CUDA_OK;
+}
+
+// ------------------------------------------------------------------ embedding
+
+template <typename TW>
+__global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint32_t *tokens, const TW *table,
+                                                    const double *turns, float *x, uint32_t width)
+{
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t row = blockIdx.x, ld = wr_ld(width);
+    const uint32_t pos = rw.seqs[seq_of(rw, row)].pos + tok_of(rw, row);
+    const TW *src = table + (size_t)tokens[row] * ld;
+    float *dst = x + (size_t)row * ld;
+    for (uint32_t i = threadIdx.x; i < ld; i += blockDim.x) {
+        float v = 0.f;
+        if (i < width) {
+            v = to_f32(src[i]);
+            if (turns) {
+                // the angle in turns, reduced before it leaves double: a position of 2^20 keeps its phase
+                const double a = turns[i >> 1] * (double)pos;
+                const float half_turns = 2.0f * (float)(a - rint(a));
+                v += (i & 1u) ? cospif(half_turns) : sinpif(half_turns);
+            }
+        }
+        dst[i] = v;
+    }
+}
+
+// ------------------------------------------------------- grouped norm, token shift
+
+constexpr uint32_t kNormThreads = 256, kNormWarps = kNormThreads / 32;
+
+// 1 / root mean square of every group of a row -> inv[groups]; part: kNormWarps-strided partial sums
+__device__ __forceinline__ void group_inv_rms(const float *x, uint32_t groups, uint32_t gs, uint32_t split, float eps,
+                                              float *part, float *inv)
+{
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t per = (gs + split - 1) / split;
+    for (uint32_t u = warp; u < groups * split; u += kNormWarps) {
+        const uint32_t g = u / split, lo = (u % split) * per, hi = min(lo + per, gs);
+        const float *xg = x + (size_t)g * gs;
+        float ss = 0.f;
+        for (uint32_t i = lo + lane; i < hi; i += 32) ss = fmaf(xg[i], xg[i], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) part[u] = ss;
+    }
+    __syncthreads();
+    for (uint32_t g = threadIdx.x; g < groups; g += kNormThreads) {
+        float ss = 0.f;
+        for (uint32_t s = 0; s < split; ++s) ss += part[g * split + s];
+        inv[g] = 1.0f / sqrtf(ss / (float)gs + eps);
+    }
+    __syncthreads();
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows rw, const wr_norm_args a, uint32_t split)
+{
+    extern __shared__ float sm_norm[];
+    float *inv = sm_norm, *inv_before = inv + a.groups, *part = inv_before + a.groups;
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t row = blockIdx.x, ld = wr_ld(a.width), gs = a.width / a.groups;
+    const float *x = a.x + (size_t)(a.gather ? a.gather[row] : row) * ld;
+    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld;
+    group_inv_rms(x, a.groups, gs, split, a.eps, part, inv);
+    if (!a.shift) {
+        for (uint32_t i = threadIdx.x; i < ld; i += kNormThreads)
+            out[i] = from_f32<TO>(i < a.width ? x[i] * inv[i / gs] * a.w[i] : 0.f);
+        return;
+    }
+    // the mixer reads h + (h' - h) * shift with h' the token before: this step's previous row (its norm is
+    // worked out again here), or the row the session's last step left
+    const wr_seq_dev s = rw.seqs[seq_of(rw, row)];
+    const uint32_t t = tok_of(rw, row);
+    const float *xb = x - ld;
+    if (t > 0) group_inv_rms(xb, a.groups, gs, split, a.eps, part, inv_before);
+    const float *kept = reinterpret_cast<const float *>(s.st_in + a.state_off);
+    float *keep = reinterpret_cast<float *>(s.st_out + a.state_off);
+    for (uint32_t i = threadIdx.x; i < ld; i += kNormThreads) {
+        float y = 0.f;
+        if (i < a.width) {
+            const float h = x[i] * inv[i / gs] * a.w[i];
+            float before = 0.f;
+            if (t > 0) before = xb[i] * inv_before[i / gs] * a.w[i];
+            else if (!s.fresh) before = kept[i];
+            y = h + (before - h) * a.shift[i];
+            if (t + 1 == s.n) keep[i] = h;
+        }
+        out[i] = from_f32<TO>(y);
+    }
+}
+
+// -------------------------------------------------------------------- PolyNorm
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256) polynorm_kernel(const wr_polynorm_args a)
+{
+    __shared__ float red[3][8];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t ld = wr_ld(a.ff), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const TI *z = static_cast<const TI *>(a.z) + (size_t)blockIdx.x * ld;
+    TO *out = static_cast<TO *>(a.out) + (size_t)blockIdx.x * ld;
+    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    for (uint32_t i = threadIdx.x; i < a.ff; i += 256) {
+        const float v = to_f32(z[i]), v2 = v * v, v3 = v2 * v;
+        s1 = fmaf(v, v, s1);
+        s2 = fmaf(v2, v2, s2);
+        s3 = fmaf(v3, v3, s3);
+    }
+    s1 = warp_sum(s1);
+    s2 = warp_sum(s2);
+    s3 = warp_sum(s3);
+    if (lane == 0) { red[0][warp] = s1; red[1][warp] = s2; red[2][warp] = s3; }
+    __syncthreads();
+    float k[3];
+#pragma unroll
+    for (int p = 0; p < 3; ++p) {
+        float t = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) t += red[p][w];
+        k[p] = 1.0f / sqrtf(t / (float)a.ff + a.eps);
+    }
+    const float ka = a.a * k[0], kb = a.b * k[1], kc = a.c * k[2];
+    for (uint32_t i = threadIdx.x; i < ld; i += 256) {
+        float y = 0.f;
+        if (i < a.ff) {
+            const float v = to_f32(z[i]);
+            y = fmaf(v, fmaf(v, fmaf(v, kc, kb), ka), a.e);
+        }
+        out[i] = from_f32<TO>(y);
+    }
+}
+
+// ----------------------------------------------------------------- convolution
+
+constexpr uint32_t kConvThreads = 128, kConvRows = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const wr_rows rw, const wr_conv_args a)
+{
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t c = blockIdx.x * kConvThreads + threadIdx.x, ld = wr_ld(a.inner), tail = a.taps - 1;
+    const uint32_t seq = blockIdx.z, row0 = row0_of(rw, seq);
+    const wr_seq_dev s = rw.seqs[seq];
+    if (c >= ld) return;
+    const T *x = static_cast<const T *>(a.x) + (size_t)row0 * a.x_ld + c;
+    T *out = static_cast<T *>(a.out) + (size_t)row0 * ld + c;
+    const uint32_t t0 = blockIdx.y * kConvRows, t1 = min(t0 + kConvRows, s.n);
+    if (c >= a.inner) {
+        for (uint32_t t = t0; t < t1; ++t) out[(size_t)t * ld] = from_f32<T>(0.f);
+        return;
+    }
+    const float *kept = reinterpret_cast<const float *>(s.st_in + a.state_off) + c;      // [taps-1][inner]
+    auto input = [&](int32_t t) -> float {                                               // token t of this step; < 0: before it
+        if (t >= 0) return to_f32(x[(size_t)t * a.x_ld]);
+        return s.fresh ? 0.f : kept[(size_t)((int32_t)tail + t) * a.inner];
+    };
+    const float bias = a.b[c];
+    for (uint32_t t = t0; t < t1; ++t) {
+        float acc = bias;
+        for (uint32_t j = 0; j < a.taps; ++j)
+            acc = fmaf(a.w[(size_t)j * ld + c], input((int32_t)(t + j) - (int32_t)tail), acc);
+        out[(size_t)t * ld] = from_f32<T>(siluf(acc));
+    }
+    if (t1 == s.n) {                                                                     // the block with the last token
+        float *keep = reinterpret_cast<float *>(s.st_out + a.state_off) + c;
+        for (uint32_t k = 0; k < tail; ++k)
+            keep[(size_t)k * a.inner] = input((int32_t)(s.n + k) - (int32_t)tail);
+    }
+}
+
+// -------------------------------------------------------------- selective scan
+//
+// A thread carries NS states of one channel through the step's tokens; the threads of a channel are
+// neighbouring lanes and add their parts of y with shuffles.  Token tiles (x, z, dt of the block's channels, B, C)
+// come in through a two-deep cp.async ring.  The state is F32 throughout.
+
+constexpr uint32_t kScanThreads = 128, kScanTile = 16;
+
+__device__ __forceinline__ float ex2(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+template <int BYTES> __device__ __forceinline__ void cp_async(void *dst, const void *src)
+{
+    asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
+}
+
+template <typename T, int NS>
+__global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, const wr_scan_args a, uint32_t tpc_log2)
+{
+    extern __shared__ __align__(16) uint8_t sm_scan[];
+    const uint32_t tpc = 1u << tpc_log2, cb = kScanThreads >> tpc_log2, ns = NS * tpc;      // channels, states held
+    float *bs = reinterpret_cast<float *>(sm_scan), *cs = bs + 2 * kScanTile * ns;          // [2][tile][ns]
+    float *dts = cs + 2 * kScanTile * ns;                                                   // [2][tile][cb]
+    T *xs = reinterpret_cast<T *>(dts + 2 * kScanTile * cb), *zs = xs + 2 * kScanTile * cb, *ys = zs + 2 * kScanTile * cb;
+    pdl_trigger();
+    const uint32_t seq = blockIdx.y, tid = threadIdx.x;
+    const uint32_t c_base = blockIdx.x * cb, cl = tid >> tpc_log2, part = tid & (tpc - 1), c = c_base + cl;
+    const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state);
+    for (uint32_t i = tid; i < 4 * kScanTile * ns; i += kScanThreads) bs[i] = 0.f;          // (B and C beyond `state`)
+    float A2[NS], S[NS];
+#pragma unroll
+    for (int j = 0; j < NS; ++j) {
+        const uint32_t n = part * NS + j;
+        A2[j] = (c < a.inner && n < a.state) ? a.a2[(size_t)c * lds + n] : 0.f;
+    }
+    const float D = c < a.inner ? a.d[c] : 0.f;
+    pdl_wait();
+    const wr_seq_dev s = rw.seqs[seq];
+    const uint32_t row0 = row0_of(rw, seq), n_tok = s.n;
+    const float *st_in = reinterpret_cast<const float *>(s.st_in + a.state_off);
+#pragma unroll
+    for (int j = 0; j < NS; ++j) {
+        const uint32_t n = part * NS + j;
+        S[j] = (!s.fresh && c < a.inner && n < a.state) ? st_in[(size_t)c * a.state + n] : 0.f;
+    }
+    __syncthreads();
+    const uint32_t xc4 = cb / 4, bc4 = (a.state + 3) / 4;            // 4-value pieces per token
+    auto request = [&](uint32_t tile) {
+        const uint32_t st = tile & 1, t0 = tile * kScanTile, nt = min(kScanTile, n_tok - t0);
+        for (uint32_t i = tid; i < nt * xc4; i += kScanThreads) {
+            const uint32_t t = i / xc4, q = i % xc4, ch = c_base + 4 * q;
+            if (ch >= ld) continue;
+            const size_t row = row0 + t0 + t;
+            const uint32_t at = (st * kScanTile + t) * cb + 4 * q;
+            cp_async<4 * sizeof(T)>(xs + at, static_cast<const T *>(a.x) + row * a.x_ld + ch);
+            cp_async<4 * sizeof(T)>(zs + at, static_cast<const T *>(a.z) + row * a.z_ld + ch);
+            cp_async<16>(dts + at, a.dt + row * ld + ch);
+        }
+        for (uint32_t i = tid; i < nt * bc4; i += kScanThreads) {
+            const uint32_t t = i / bc4, q = i % bc4;
+            const float *src = a.bc + (size_t)(row0 + t0 + t) * a.bc_ld + 4 * q;
+            cp_async<16>(bs + (st * kScanTile + t) * ns + 4 * q, src + a.b_off);
+            cp_async<16>(cs + (st * kScanTile + t) * ns + 4 * q, src + a.c_off);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const uint32_t tiles = (n_tok + kScanTile - 1) / kScanTile;
+    request(0);
+    for (uint32_t tile = 0; tile < tiles; ++tile) {
+        const uint32_t st = tile & 1, t0 = tile * kScanTile, nt = min(kScanTile, n_tok - t0);
+        if (tile + 1 < tiles) {
+            request(tile + 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        auto token = [&](uint32_t t) {
+            const uint32_t at = (st * kScanTile + t) * cb + cl;
+            const float dt = dts[at], x = to_f32(xs[at]), dx = dt * x;
+            const float *b = bs + (st * kScanTile + t) * ns + part * NS, *cc = cs + (st * kScanTile + t) * ns + part * NS;
+            float y = 0.f;
+#pragma unroll
+            for (int j = 0; j < NS; ++j) {
+                S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b[j]);
+                y = fmaf(S[j], cc[j], y);
+            }
+            for (uint32_t o = tpc >> 1; o >= 1; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+            if (part == (t & (tpc - 1))) {
+                y = fmaf(D, x, y);
+                ys[t * cb + cl] = from_f32<T>(y * siluf(to_f32(zs[at])));
+            }
+        };
+        if (nt == kScanTile) {
+#pragma unroll 4
+            for (uint32_t t = 0; t < kScanTile; ++t) token(t);
+        } else {
+            for (uint32_t t = 0; t < nt; ++t) token(t);
+        }
+        __syncthreads();
+        for (uint32_t i = tid; i < nt * cb; i += kScanThreads) {
+            const uint32_t t = i / cb, q = i % cb, ch = c_base + q;
+            if (ch < ld) {
+                T *o = static_cast<T *>(a.out) + (size_t)(row0 + t0 + t) * ld + ch;
+                *o = ch < a.inner ? ys[t * cb + q] : from_f32<T>(0.f);
+            }
+        }
+    }
+    float *st_out = reinterpret_cast<float *>(s.st_out + a.state_off);
+#pragma unroll
+    for (int j = 0; j < NS; ++j) {
+        const uint32_t n = part * NS + j;
+        if (c < a.inner && n < a.state) st_out[(size_t)c * a.state + n] = S[j];
+    }
+}
+
+template <typename T, int NS>
+int scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+{
+    uint32_t lg = 0;
+    while ((NS << lg) < (int)a.state) ++lg;
+    if (lg > 5) return WR_CUDA_ERR_LIMIT;
+    const uint32_t cb = kScanThreads >> lg, ns = NS << lg;
+    const size_t smem = (size_t)(4 * kScanTile * ns + 2 * kScanTile * cb) * 4 + (size_t)5 * kScanTile * cb * sizeof(T);
+    auto k = scan_kernel<T, NS>;
+    if (smem > 48 * 1024)
+        WR_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    WR_CUDA_TRY(wr_launch_pdl(k, dim3((wr_ld(a.inner) + cb - 1) / cb, rw.n_seq), dim3(kScanThreads), smem, ctx->stream, rw,
+                              a, lg));
+    return finish_launch(ctx);
+}
+
+// ------------------------------------------------------------- around attention
+
+// Queries out of the projection row (scale and temperature applied), K and V into the session's pages.
+template <typename TI, typename TQ>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const wr_rows rw, const wr_attn_prep_args a)
+{
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t row = blockIdx.x, tid = threadIdx.x;
+    const wr_seq_dev s = rw.seqs[seq_of(rw, row)];
+    const uint32_t pos = s.pos + tok_of(rw, row);
+    const wr_attn_geom g = a.g;
+    const TI *in = static_cast<const TI *>(a.qkv) + (size_t)row * a.ld;
+    float mul = a.scale;
+    if (a.temp_every) mul *= 1.0f + a.temp_coef * logf((float)((pos + 1u) / a.temp_every + 1u));
+    const uint32_t qs = g.q_stride(), nq = g.vq() * qs;
+    TQ *q = static_cast<TQ *>(a.q) + (size_t)row * nq;
+    for (uint32_t i = tid; i < nq; i += 256) {
+        const uint32_t vq = i / qs, e = i % qs, off = g.hd128 ? (vq % g.maps) * g.kd : 0u;     // the map's part of the row
+        float v = 0.f;
+        if (e >= off && e < off + g.kd) v = to_f32(in[vq * g.kd + e - off]) * mul;
+        q[i] = from_f32<TQ>(v);
+    }
+    char *page = reinterpret_cast<char *>(s.pages[(size_t)g.layer * s.n_pages + pos / kPageTokens]);
+    const uint32_t tok = pos % kPageTokens, kw = g.maps * g.kd;
+    auto put = [&](uint32_t head, uint32_t which, uint32_t d, float v) {
+        char *p = page + wr_geom_off(g.kv, head, which, tok, d);
+        if (g.kv.elem == WR_CUDA_F32) *reinterpret_cast<float *>(p) = v;
+        else *reinterpret_cast<__half *>(p) = from_f32<__half>(v);
+    };
+    for (uint32_t i = tid; i < g.n_kv * kw; i += 256) put(i / kw, 0, i % kw, to_f32(in[a.k_off + i]));
+    for (uint32_t i = tid; i < g.n_kv * g.vd; i += 256) put(i / g.vd, 1, i % g.vd, to_f32(in[a.v_off + i]));
+}
+
+// One warp per query head: combine the maps, norm over the head, gate.
+template <typename TG, typename TO>
+__global__ void __launch_bounds__(256) attn_finish_kernel(const wr_rows rw, const wr_attn_finish_args a)
+{
+    pdl_trigger();
+    pdl_wait();
+    const wr_attn_geom g = a.g;
+    const uint32_t row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, os = g.o_stride();
+    const uint32_t n_out = g.n_q * g.vd, ld = wr_ld(n_out);
+    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld;
+    for (uint32_t h = blockIdx.y * 8 + warp; h < g.n_q; h += gridDim.y * 8) {
+        const float *o1 = a.o + ((size_t)row * g.vq() + h * g.maps) * os, *o2 = o1 + os;
+        float k = 1.0f;
+        if (g.maps == 2) {
+            float ss = 0.f;
+            for (uint32_t i = lane; i < g.vd; i += 32) {
+                const float d = fmaf(-a.lambda, o2[i], o1[i]);
+                ss = fmaf(d, d, ss);
+            }
+            k = (1.0f - a.diff_init) / sqrtf(warp_sum(ss) / (float)g.vd + a.eps);
+        }
+        for (uint32_t i = lane; i < g.vd; i += 32) {
+            float v = g.maps == 2 ? fmaf(-a.lambda, o2[i], o1[i]) * k : o1[i];
+            if (a.gate)
+                v *= sigmoidf(to_f32(static_cast<const TG *>(a.gate)[(size_t)row * a.gate_ld + h * g.vd + i]));
+            out[h * g.vd + i] = from_f32<TO>(v);
+        }
+    }
+    if (blockIdx.y == 0 && threadIdx.x < ld - n_out) out[n_out + threadIdx.x] = from_f32<TO>(0.f);
+}
+
+// --------------------------------------------- attention over any cache layout
+
+__device__ __forceinline__ void load8(const char *p, uint32_t elem, float (&v)[8])
+{
+    if (elem == WR_CUDA_F32) {
+        const float4 a = *reinterpret_cast<const float4 *>(p), b = *reinterpret_cast<const float4 *>(p + 16);
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    } else {
+        const uint4 u = *reinterpret_cast<const uint4 *>(p);
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __half22float2(*reinterpret_cast<const __half2 *>(&w[i]));
+            v[2 * i] = f.x;
+            v[2 * i + 1] = f.y;
+        }
+    }
+}
+
+// Columns [d0, d0 + dims) of rows [key0, key0 + n_keys) of a head's K or V into shared memory (row stride `stride`).
+__device__ __forceinline__ void stage_rows(const uint64_t *table, const wr_kv_geom &g, uint32_t head, uint32_t which,
+                                           uint32_t key0, uint32_t n_keys, uint32_t d0, uint32_t dims, float *dst,
+                                           uint32_t stride)
+{
+    const uint32_t lo8 = d0 / 8u, n8 = (d0 + dims + 7u) / 8u - lo8;
+    for (uint32_t i = threadIdx.x; i < n_keys * n8; i += blockDim.x) {
+        const uint32_t k = i / n8, d = (lo8 + i % n8) * 8u, key = key0 + k;
+        const char *p = reinterpret_cast<const char *>(table[key / kPageTokens]) +
+                        wr_geom_off(g, head, which, key % kPageTokens, d);
+        float v[8];
+        load8(p, g.elem, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+            if (d + e >= d0 && d + e < d0 + dims) dst[k * stride + d + e - d0] = v[e];
+    }
+}
+
+constexpr uint32_t kAnyRows = 32, kAnyKeys = 32, kAnyThreads = 128;
+
+// Prompt rows: a block is 32 query rows of one query (head, map); four threads share a row.
+template <int VC>
+__global__ void __launch_bounds__(kAnyThreads) attn_rows_any_kernel(const wr_rows rw, const wr_attn_geom g,
+                                                                    const float *q, float *out)
+{
+    extern __shared__ float sm_any[];
+    const uint32_t ks = g.kd | 1u, vs = g.vd;
+    float *Q = sm_any, *K = Q + kAnyRows * ks, *V = K + kAnyKeys * ks, *P = V + kAnyKeys * vs;      // P: [rows][33]
+    pdl_trigger();
+    pdl_wait();
+    const wr_seq_dev s = rw.seqs[0];
+    const uint64_t *table = s.pages + (size_t)g.layer * s.n_pages;
+    const uint32_t t0 = blockIdx.x * kAnyRows, vq = blockIdx.y, head = vq / g.maps / (g.n_q / g.n_kv), map = vq % g.maps;
+    const uint32_t rows = min(kAnyRows, s.n - t0), r = threadIdx.x >> 2, sub = threadIdx.x & 3;
+    for (uint32_t i = threadIdx.x; i < kAnyRows * g.kd; i += kAnyThreads) {
+        const uint32_t rr = i / g.kd, d = i % g.kd;
+        Q[rr * ks + d] = rr < rows ? q[((size_t)(t0 + rr) * g.vq() + vq) * g.kd + d] : 0.f;
+    }
+    const uint32_t my_pos = s.pos + t0 + r, key_end = s.pos + t0 + rows;
+    float m = -INFINITY, l = 0.f, acc[VC];
+#pragma unroll
+    for (int i = 0; i < VC; ++i) acc[i] = 0.f;
+    for (uint32_t k0 = 0; k0 < key_end; k0 += kAnyKeys) {
+        const uint32_t nk = min(kAnyKeys, key_end - k0);
+        __syncthreads();
+        stage_rows(table, g.kv, head, 0, k0, nk, map * g.kd, g.kd, K, ks);
+        stage_rows(table, g.kv, head, 1, k0, nk, 0, g.vd, V, vs);
+        __syncthreads();
+        float sc[kAnyKeys / 4], mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < (int)kAnyKeys / 4; ++i) {
+            const uint32_t k = sub + 4 * i;
+            sc[i] = -INFINITY;
+            if (k < nk && k0 + k <= my_pos) {
+                float d = 0.f;
+                for (uint32_t e = 0; e < g.kd; ++e) d = fmaf(Q[r * ks + e], K[k * ks + e], d);
+                sc[i] = d;
+            }
+            mx = fmaxf(mx, sc[i]);
+        }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float m_new = fmaxf(m, mx);                        // (key 0 is visible to every row: finite from the start)
+        const float corr = expf(m - m_new);
+        float ps = 0.f;
+#pragma unroll
+        for (int i = 0; i < (int)kAnyKeys / 4; ++i) {
+            const float p = expf(sc[i] - m_new);
+            P[r * (kAnyKeys + 1) + sub + 4 * i] = p;
+            ps += p;
+        }
+        ps += __shfl_xor_sync(0xffffffffu, ps, 1);
+        ps += __shfl_xor_sync(0xffffffffu, ps, 2);
+        l = fmaf(l, corr, ps);
+        m = m_new;
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < VC; ++i) acc[i] *= corr;
+        for (uint32_t k = 0; k < nk; ++k) {
+            const float p = P[r * (kAnyKeys + 1) + k];
+#pragma unroll
+            for (int i = 0; i < VC; ++i) {
+                const uint32_t c = sub + 4 * i;
+                if (c < g.vd) acc[i] = fmaf(p, V[k * vs + c], acc[i]);
+            }
+        }
+    }
+    if (r < rows) {
+        const float inv = 1.0f / l;
+        float *o = out + ((size_t)(t0 + r) * g.vq() + vq) * g.vd;
+#pragma unroll
+        for (int i = 0; i < VC; ++i) {
+            const uint32_t c = sub + 4 * i;
+            if (c < g.vd) o[c] = acc[i] * inv;
+        }
+    }
+}
+
+// Decode: a block is one chunk of keys of one (session, kv head) for all of the head's queries.  Partial rows
+// (m, l, o[vd]) go to ws[session][vq][chunk]; attn_merge_any_kernel adds them up in chunk order.
+constexpr uint32_t kChunkKeys = 256;
+
+__host__ __device__ inline uint32_t any_ws_stride(uint32_t vd) { return vd + 2u; }
+
+__global__ void __launch_bounds__(kAnyThreads) attn_chunk_any_kernel(const wr_rows rw, const wr_attn_geom g,
+                                                                     const float *q, float *ws, uint32_t chunks)
+{
+    extern __shared__ float sm_any[];
+    const uint32_t nq = g.n_q / g.n_kv * g.maps, kw = g.maps * g.kd, ks = kw | 1u;
+    float *Q = sm_any, *K = Q + nq * g.kd, *S = K + kAnyKeys * ks, *M = S + nq * kChunkKeys, *L = M + nq;
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t chunk = blockIdx.x, head = blockIdx.y, seq = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const wr_seq_dev s = rw.seqs[seq];
+    const uint32_t len = s.pos + 1, lo = chunk * kChunkKeys;
+    if (lo >= len) return;
+    const uint32_t n = min(kChunkKeys, len - lo);
+    const uint64_t *table = s.pages + (size_t)g.layer * s.n_pages;
+    const float *qrow = q + ((size_t)seq * g.vq() + head * nq) * g.kd;
+    for (uint32_t i = threadIdx.x; i < nq * g.kd; i += kAnyThreads) Q[i] = qrow[i];
+    for (uint32_t k0 = 0; k0 < n; k0 += kAnyKeys) {
+        const uint32_t nk = min(kAnyKeys, n - k0);
+        __syncthreads();
+        stage_rows(table, g.kv, head, 0, lo + k0, nk, 0, kw, K, ks);
+        __syncthreads();
+        for (uint32_t i = threadIdx.x; i < nq * kAnyKeys; i += kAnyThreads) {
+            const uint32_t v = i / kAnyKeys, k = i % kAnyKeys;
+            if (k >= nk) continue;
+            const float *kr = K + k * ks + (v % g.maps) * g.kd, *qr = Q + v * g.kd;
+            float d = 0.f;
+            for (uint32_t e = 0; e < g.kd; ++e) d = fmaf(qr[e], kr[e], d);
+            S[v * kChunkKeys + k0 + k] = d;
+        }
+    }
+    __syncthreads();
+    for (uint32_t v = warp; v < nq; v += kAnyThreads / 32) {
+        float mx = -INFINITY, sum = 0.f;
+        for (uint32_t k = lane; k < n; k += 32) mx = fmaxf(mx, S[v * kChunkKeys + k]);
+#pragma unroll
+        for (int o = 16; o >= 1; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        for (uint32_t k = lane; k < n; k += 32) {
+            const float p = expf(S[v * kChunkKeys + k] - mx);
+            S[v * kChunkKeys + k] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        if (lane == 0) { M[v] = mx; L[v] = sum; }
+    }
+    __syncthreads();
+    const uint32_t stride = any_ws_stride(g.vd);
+    constexpr uint32_t B = 8;
+    for (uint32_t c = threadIdx.x; c < g.vd; c += kAnyThreads)
+        for (uint32_t v0 = 0; v0 < nq; v0 += B) {
+            float acc[B];
+#pragma unroll
+            for (uint32_t j = 0; j < B; ++j) acc[j] = 0.f;
+            for (uint32_t k = 0; k < n; ++k) {
+                const uint32_t key = lo + k;
+                const char *p = reinterpret_cast<const char *>(table[key / kPageTokens]) +
+                                wr_geom_off(g.kv, head, 1, key % kPageTokens, c);
+                const float x = g.kv.elem == WR_CUDA_F32 ? *reinterpret_cast<const float *>(p)
+                                                         : __half2float(*reinterpret_cast<const __half *>(p));
+#pragma unroll
+                for (uint32_t j = 0; j < B; ++j)
+                    if (v0 + j < nq) acc[j] = fmaf(S[(v0 + j) * kChunkKeys + k], x, acc[j]);
+            }
+#pragma unroll
+            for (uint32_t j = 0; j < B; ++j)
+                if (v0 + j < nq)
+                    ws[(((size_t)seq * g.vq() + head * nq + v0 + j) * chunks + chunk) * stride + 2 + c] = acc[j];
+        }
+    for (uint32_t v = threadIdx.x; v < nq; v += kAnyThreads) {
+        float *w = ws + (((size_t)seq * g.vq() + head * nq + v) * chunks + chunk) * stride;
+        w[0] = M[v];
+        w[1] = L[v];
+    }
+}
+
+__global__ void __launch_bounds__(128) attn_merge_any_kernel(const wr_rows rw, const wr_attn_geom g, const float *ws,
+                                                             float *out, uint32_t chunks)
+{
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t vq = blockIdx.x, seq = blockIdx.y;
+    const uint32_t n = (rw.seqs[seq].pos + 1 + kChunkKeys - 1) / kChunkKeys, stride = any_ws_stride(g.vd);
+    const float *w = ws + ((size_t)seq * g.vq() + vq) * chunks * stride;
+    float m = -INFINITY, l = 0.f;
+    for (uint32_t i = 0; i < n; ++i) m = fmaxf(m, w[(size_t)i * stride]);
+    for (uint32_t i = 0; i < n; ++i) l = fmaf(w[(size_t)i * stride + 1], expf(w[(size_t)i * stride] - m), l);
+    for (uint32_t c = threadIdx.x; c < g.vd; c += 128) {
+        float o = 0.f;
+        for (uint32_t i = 0; i < n; ++i) o = fmaf(w[(size_t)i * stride + 2 + c], expf(w[(size_t)i * stride] - m), o);
+        out[((size_t)seq * g.vq() + vq) * g.vd + c] = o / l;
+    }
+}
+
+template <typename K> int allow_smem(K k, size_t smem)
+{
+    if (smem > 227 * 1024) return WR_CUDA_ERR_LIMIT;
+    if (smem > 48 * 1024)
+        WR_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return WR_CUDA_OK;
+}
+
+template <int VC> int rows_any(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_geom &g, const float *q, float *out)
+{
+    const size_t smem = (size_t)(2 * kAnyRows * (g.kd | 1u) + kAnyKeys * g.vd + kAnyRows * (kAnyKeys + 1)) * 4;
+    int rc = allow_smem(attn_rows_any_kernel<VC>, smem);
+    if (rc != WR_CUDA_OK) return rc;
+    WR_CUDA_TRY(wr_launch_pdl(attn_rows_any_kernel<VC>, dim3((rw.n_rows + kAnyRows - 1) / kAnyRows, g.vq()),
+                              dim3(kAnyThreads), smem, ctx->stream, rw, g, q, out));
+    return finish_launch(ctx);
+}
+
+}  // namespace
+
+int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens, const void *table, int table_type,
+                    const double *turns, float *x, uint32_t width)
+{
+    if (table_type == WR_ACT_BF16)
+        embed_kernel<__nv_bfloat16><<<rw.n_rows, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width);
+    else
+        embed_kernel<float><<<rw.n_rows, 256, 0, ctx->stream>>>(rw, tokens, (const float *)table, turns, x, width);
+    return finish_launch(ctx);
+}
+
+int wr_group_norm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a)
+{
+    const uint32_t split = std::max(1u, kNormWarps / a.groups);
+    const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
+    if (smem > 48 * 1024) return WR_CUDA_ERR_LIMIT;
+    if (a.out_type == WR_ACT_BF16)
+        WR_CUDA_TRY(wr_launch_pdl(group_norm_kernel<__nv_bfloat16>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split));
+    else
+        WR_CUDA_TRY(wr_launch_pdl(group_norm_kernel<float>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split));
+    return finish_launch(ctx);
+}
+
+int wr_polynorm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_polynorm_args &a)
+{
+    if (a.z_type == WR_ACT_BF16)
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(rw.n_rows), dim3(256), 0, ctx->stream, a));
+    else
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float, float>, dim3(rw.n_rows), dim3(256), 0, ctx->stream, a));
+    return finish_launch(ctx);
+}
+
+int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args &a)
+{
+    const uint32_t n = rw.decode ? 1u : rw.n_rows;
+    const dim3 grid((wr_ld(a.inner) + kConvThreads - 1) / kConvThreads, (n + kConvRows - 1) / kConvRows, rw.n_seq);
+    if (a.type == WR_ACT_BF16)
+        WR_CUDA_TRY(wr_launch_pdl(conv_silu_kernel<__nv_bfloat16>, grid, dim3(kConvThreads), 0, ctx->stream, rw, a));
+    else
+        WR_CUDA_TRY(wr_launch_pdl(conv_silu_kernel<float>, grid, dim3(kConvThreads), 0, ctx->stream, rw, a));
+    return finish_launch(ctx);
+}
+
+int wr_scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+{
+    const bool bf = a.type == WR_ACT_BF16;
+    if (a.state <= 128) return bf ? scan_launch<__nv_bfloat16, 4>(ctx, rw, a) : scan_launch<float, 4>(ctx, rw, a);
+    return bf ? scan_launch<__nv_bfloat16, 16>(ctx, rw, a) : scan_launch<float, 16>(ctx, rw, a);
+}
+
+int wr_attn_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_prep_args &a)
+{
+    const dim3 grid(rw.n_rows), block(256);
+    const bool half_in = a.type == WR_ACT_F16, half_q = a.q_type == WR_ACT_F16;
+    if (half_in && half_q) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<__half, __half>, grid, block, 0, ctx->stream, rw, a));
+    else if (half_in) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<__half, float>, grid, block, 0, ctx->stream, rw, a));
+    else if (half_q) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<float, __half>, grid, block, 0, ctx->stream, rw, a));
+    else WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<float, float>, grid, block, 0, ctx->stream, rw, a));
+    return finish_launch(ctx);
+}
+
+int wr_attn_any_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_geom &g, const float *q, float *out,
+                       uint32_t max_len)
+{
+    if (!rw.decode) {
+        if (g.vd <= 64) return rows_any<16>(ctx, rw, g, q, out);
+        if (g.vd <= 128) return rows_any<32>(ctx, rw, g, q, out);
+        if (g.vd <= 256) return rows_any<64>(ctx, rw, g, q, out);
+        if (g.vd <= 512) return rows_any<128>(ctx, rw, g, q, out);
+        return WR_CUDA_ERR_LIMIT;
+    }
+    const uint32_t nq = g.n_q / g.n_kv * g.maps, chunks = (max_len + kChunkKeys - 1) / kChunkKeys;
+    int rc = wr_ctx_reserve_ws(ctx, (size_t)rw.n_seq * g.vq() * chunks * any_ws_stride(g.vd) * sizeof(float), 0);
+    if (rc != WR_CUDA_OK) return rc;
+    const size_t smem = (size_t)(nq * g.kd + kAnyKeys * ((g.maps * g.kd) | 1u) + nq * kChunkKeys + 2 * nq) * 4;
+    rc = allow_smem(attn_chunk_any_kernel, smem);
+    if (rc != WR_CUDA_OK) return rc;
+    WR_CUDA_TRY(wr_launch_pdl(attn_chunk_any_kernel, dim3(chunks, g.n_kv, rw.n_seq), dim3(kAnyThreads), smem, ctx->stream,
+                              rw, g, q, ctx->ws, chunks));
+    rc = finish_launch(ctx);
+    if (rc != WR_CUDA_OK) return rc;
+    WR_CUDA_TRY(wr_launch_pdl(attn_merge_any_kernel, dim3(g.vq(), rw.n_seq), dim3(128), 0, ctx->stream, rw, g,
+                              (const float *)ctx->ws, out, chunks));
+    return finish_launch(ctx);
+}
+
+int wr_attn_finish_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_finish_args &a)
+{
+    const dim3 grid(rw.n_rows, (a.g.n_q + 7) / 8), block(256);
+    if (a.out_type == WR_ACT_BF16)
+        WR_CUDA_TRY(wr_launch_pdl(attn_finish_kernel<__half, __nv_bfloat16>, grid, block, 0, ctx->stream, rw, a));
+    else
+        WR_CUDA_TRY(wr_launch_pdl(attn_finish_kernel<float, float>, grid, block, 0, ctx->stream, rw, a));
+    return finish_launch(ctx);
+}

@@ -47,6 +47,32 @@ __host__ __device__ inline uint32_t wr_elem_off(uint32_t tok, uint32_t d, uint32
     }
     return (tok * wr_hd_pad(hd) + d) * 2u;
 }
+// Geometry of one layer's pages.  Usually K and V rows are F16 and equally long (the layout above); a
+// layer may also keep K and V rows of different lengths, or F32 rows: its pages are then
+// [kv_head][64 tok][pad8(k_dim)] K rows followed by [64 tok][pad8(v_dim)] V rows, never swizzled.
+struct wr_kv_geom {
+    uint32_t n_kv, k_dim, v_dim, elem;                   // elem: WR_CUDA_F32 / WR_CUDA_F16
+};
+__host__ __device__ inline uint32_t wr_geom_esize(const wr_kv_geom &g) { return g.elem == WR_CUDA_F32 ? 4u : 2u; }
+__host__ __device__ inline bool wr_geom_uniform(const wr_kv_geom &g)
+{
+    return g.elem == WR_CUDA_F16 && g.k_dim == g.v_dim;
+}
+__host__ __device__ inline uint64_t wr_geom_head_bytes(const wr_kv_geom &g)
+{
+    return (uint64_t)kPageTokens * (wr_hd_pad(g.k_dim) + wr_hd_pad(g.v_dim)) * wr_geom_esize(g);
+}
+__host__ __device__ inline uint64_t wr_geom_page_bytes(const wr_kv_geom &g) { return g.n_kv * wr_geom_head_bytes(g); }
+// Byte offset of element d of token tok (within the page) of a head's K (which = 0) or V (which = 1) row.
+__host__ __device__ inline uint64_t wr_geom_off(const wr_kv_geom &g, uint32_t head, uint32_t which, uint32_t tok,
+                                                uint32_t d)
+{
+    const uint32_t es = wr_geom_esize(g), dim = which ? g.v_dim : g.k_dim;
+    uint64_t off = head * wr_geom_head_bytes(g);
+    if (which) off += (uint64_t)kPageTokens * wr_hd_pad(g.k_dim) * es;
+    if (wr_geom_uniform(g)) return off + wr_elem_off(tok, d, dim);
+    return off + ((uint64_t)tok * wr_hd_pad(dim) + d) * es;
+}
 // Byte offset of the (head, which) block inside a page; which: 0 = K, 1 = V.
 __host__ __device__ inline uint64_t wr_block_off(uint32_t head, uint32_t which, uint32_t hd)
 {
@@ -96,13 +122,44 @@ struct wr_cuda_ctx {
 };
 enum { WR_PDL_NONE = 0, WR_PDL_APPEND = 1, WR_PDL_DECODE_FULL = 2, WR_PDL_DECODE_PART = 3, WR_PDL_PREFILL_FULL = 4 };
 
+// What one layer of a session keeps: K/V pages, a recurrent state, both or neither.
+struct wr_kv_layer {
+    wr_kv_geom geom{};               // n_kv = 0: no pages
+    uint64_t page_bytes = 0;
+    size_t pool_index = 0;
+    uint64_t state_off = 0, state_bytes = 0;    // inside the session's state slot
+};
+
 struct wr_cuda_kv {
     wr_cuda_ctx *ctx = nullptr;
-    uint32_t n_layers = 0, n_kv = 0, hd = 0, max_ctx = 0, n_pages = 0;
-    std::vector<void *> pages;       // n_layers * n_pages page pointers (host copy)
+    uint32_t n_layers = 0, max_ctx = 0, n_pages = 0;
+    std::vector<wr_kv_layer> layers;
+    std::vector<void *> pages;       // n_layers * n_pages page pointers (host copy; null where a layer has none)
     uint64_t *d_pages = nullptr;     // same table on the device
     std::vector<uint8_t> contig;     // per layer: pages are consecutive in memory
-    size_t pool_index = 0;
+    // Recurrent state: two slots, each the state after some number of tokens (-1: nothing).  A step
+    // reads the slot that stands at its first position and writes the other one, so a step that
+    // fails — or whose tokens the host does not keep — leaves the state it started from intact.
+    uint64_t state_bytes = 0;
+    void *state[2] = {nullptr, nullptr};
+    int64_t state_len[2] = {-1, -1};
+    size_t state_pool = 0;
+
+    uint32_t n_kv_at(uint32_t layer) const { return layers[layer].geom.n_kv; }
+    // head_dim of a layer with the F16, K-as-long-as-V layout that the RoPE-append and hd kernels know; 0 otherwise
+    uint32_t hd_at(uint32_t layer) const
+    {
+        if (layer >= n_layers) return 0;
+        const wr_kv_geom &g = layers[layer].geom;
+        return g.n_kv && wr_geom_uniform(g) ? g.k_dim : 0u;
+    }
+    // the slot standing at `pos` tokens (pos > 0), or -1
+    int state_slot(uint32_t pos) const
+    {
+        for (int i = 0; i < 2; ++i)
+            if (state_len[i] == (int64_t)pos) return i;
+        return -1;
+    }
 };
 
 // Kernel-parameter block describing the sessions of one batched launch.
