@@ -648,6 +648,125 @@ def measure_whole_model():
     return out
 
 
+# ---- models whose layers differ (Tumadra), beside the dense stack at the same width, depth and widths of the parts
+
+MIXED_SIZES = {
+    # name: width, layers, ff, query heads, kv heads, inner, dt_rank, vocab
+    "w1024x28": (1024, 28, 3072, 8, 4, 2048, 64, 151936),
+    "w2048x12": (2048, 12, 6144, 16, 4, 4096, 128, 65536),
+    "w4096x4": (4096, 4, 12288, 32, 8, 8192, 256, 65536),
+}
+MIXED_PREFILL, MIXED_CTX = 2048, 1024
+
+
+class PooledWeights:
+    """Random weights of any shape cut from one small pool (the timing does not depend on the values)."""
+
+    def __init__(self, bf16):
+        from wayruntime_b200.checkpoint import f32_to_bf16
+        pool = np.random.default_rng(SEED).standard_normal((1 << 22) + 7).astype(np.float32) * 0.02
+        self.pool, self.bf16 = (f32_to_bf16(pool) if bf16 else pool), bf16
+
+    def get(self, name, shape):
+        if "norm" in name or name.endswith((".D", "shift")):
+            a = np.full(shape, 1.0 if "norm" in name else 0.5, np.float32)
+            from wayruntime_b200.checkpoint import f32_to_bf16
+            return f32_to_bf16(a) if self.bf16 else a
+        return np.resize(self.pool, shape)
+
+    f32 = get
+
+    def __contains__(self, name):
+        return True
+
+
+def mixed_config(size):
+    width, n, ff, heads, kv, inner, rank, vocab = MIXED_SIZES[size]
+    attn = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+            "mixer": {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
+                      "q_temp": {"coef": 0.1, "every": 1024}}}
+    scan = {"type": "mamba1", "mlp": {"kind": "dense", "ff": ff},
+            "mixer": {"inner": inner, "state": 16, "dt_rank": rank, "conv": 4}}
+    return {"architecture": "Tumadra", "width": width, "vocab": vocab, "norm": {"groups": 4, "eps": 1e-5},
+            "layers": [attn if i % 2 else scan for i in range(n)]}
+
+
+def dense_config(size):
+    width, n, ff, heads, kv, _inner, _rank, vocab = MIXED_SIZES[size]
+    return {"architectures": ["Qwen3ForCausalLM"], "hidden_size": width, "intermediate_size": ff, "num_hidden_layers": n,
+            "num_attention_heads": heads, "num_key_value_heads": kv, "head_dim": 128, "vocab_size": vocab,
+            "tie_word_embeddings": True, "rope_theta": 1e6, "rms_norm_eps": 1e-6}
+
+
+def measure_mixed(args):
+    """Prefill and decode throughput of a mixed model (BF16) and of the dense F32 stack at equal size, each through
+    its forward call: prefill of MIXED_PREFILL tokens, decode of 1 and 16 sessions at MIXED_CTX tokens, arg-max on the
+    device, CUDA events on the context's stream around the calls (host enqueueing included)."""
+    import torch
+    import wayruntime_b200 as wr
+    from wayruntime_b200 import models
+    out = {"only": "mixed", "prefill_tokens": MIXED_PREFILL, "decode_context": MIXED_CTX, "data": "synthetic",
+           "weights": "random, repeated from one pool", "sizes": {}}
+    rng = np.random.default_rng(SEED)
+    for size in (args.mixed_size.split(",") if args.mixed_size else MIXED_SIZES):
+        row = out["sizes"][size] = {}
+        for kind, cfg, dtype, rows in (("tumadra_bf16", mixed_config(size), "bfloat16", MIXED_PREFILL),
+                                       ("dense_f32", dense_config(size), "float32", 256)):
+            if args.mixed_kind and kind != args.mixed_kind:
+                continue
+            ctx = wr.Context(0)
+            stream = torch.cuda.ExternalStream(ctx.stream, device=0)
+            m = models.build(ctx, cfg, PooledWeights(dtype == "bfloat16"), dtype, rows)
+            vocab = m.vocab
+            toks = [int(t) for t in rng.integers(0, vocab, MIXED_PREFILL)]
+
+            def timed(fn, reps):
+                ev = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+                ms = []
+                for _ in range(reps):
+                    ev[0].record(stream)
+                    fn()
+                    ev[1].record(stream)
+                    ev[1].synchronize()
+                    ms.append(ev[0].elapsed_time(ev[1]))
+                return float(np.median(ms))
+
+            kv = m.kv_create(MIXED_PREFILL + 8)
+
+            def prefill():
+                for lo in range(0, MIXED_PREFILL, rows):
+                    part = toks[lo:lo + rows]
+                    last = lo + len(part) == MIXED_PREFILL
+                    m.forward(m.FWD_PREFILL, [kv], [lo], part, out_from=len(part) - 1, argmax=last)
+            reps = max(3, min(args.steps, 20))
+            timed(prefill, 2)
+            ms = timed(prefill, reps)
+            kv.close()
+            res = row[kind] = {"device_weight_bytes": m.device_bytes, "prefill_ms": r4(ms),
+                               "prefill_tok_s": r4(MIXED_PREFILL / ms * 1e3)}
+            for n in (1, 16):
+                kvs = [m.kv_create(MIXED_CTX + 256) for _ in range(n)]
+                for kv in kvs:
+                    for lo in range(0, MIXED_CTX, rows):
+                        part = toks[lo:min(lo + rows, MIXED_CTX)]
+                        m.forward(m.FWD_PREFILL, [kv], [lo], part, out_from=len(part))
+                pos = [MIXED_CTX]
+
+                def decode():
+                    m.forward(m.FWD_DECODE, kvs, [pos[0]] * n, toks[:n], argmax=True)
+                    pos[0] += 1
+                timed(decode, 5)
+                l0 = m.launches
+                ms = timed(decode, 50)
+                res[f"decode_{n}"] = {"ms": r4(ms), "tok_s": r4(n / ms * 1e3), "enqueue_ms": r4(m.last_enqueue_ms),
+                                      "launches": (m.launches - l0) // 50}
+                for kv in kvs:
+                    kv.close()
+            m.close()
+            ctx.close()
+    print(json.dumps(out))
+
+
 def wr_batch(kvs):
     import wayruntime_b200 as wr
     return wr.Batch(kvs)
@@ -1015,13 +1134,18 @@ def main():
                     help="launch every step from Python instead of replaying a CUDA graph")
     ap.add_argument("--no-whole-model", action="store_true",
                     help="skip the config-1 whole-model section (about a minute of host time)")
-    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode"],
-                    help="'prefill' / 'decode': run only that kernel's measurement (for profiling)")
+    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "mixed"],
+                    help="'prefill' / 'decode': run only that kernel's measurement (for profiling); 'mixed': Tumadra "
+                         "models beside the dense stack at equal size, nothing else")
+    ap.add_argument("--mixed-size", default="", help="with --only mixed: sizes, with commas between them")
+    ap.add_argument("--mixed-kind", default="", choices=["", "tumadra_bf16", "dense_f32"], help="with --only mixed: one model only")
     args = ap.parse_args()
     if args.impl == "reference":
         if args.steps > 20:
             args.steps = 20            # bounded sample: each step is a full 16-session pass
         run_reference_arm(args)
+    elif args.only == "mixed":
+        measure_mixed(args)
     else:
         run_gpu_arm(args)
 
