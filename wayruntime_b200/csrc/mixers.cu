@@ -26,6 +26,67 @@ template <> __device__ __forceinline__ __half from_f32<__half>(float v)
 __device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float siluf(float x) { return x / (1.0f + expf(-x)); }
 
+// four / eight consecutive values (addresses aligned to the vector)
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16 *p)
+{
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ float4 load4(const __half *p)
+{
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const float2 a = __half22float2(*reinterpret_cast<const __half2 *>(&u.x)), b = __half22float2(*reinterpret_cast<const __half2 *>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16 *p, float4 v)
+{
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+template <typename T> __device__ __forceinline__ void load8v(const T *p, float (&v)[8])
+{
+    const float4 a = load4(p), b = load4(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8v(const __nv_bfloat16 *p, float (&v)[8])
+{
+    const uint4 u = *reinterpret_cast<const uint4 *>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+template <typename T> __device__ __forceinline__ void store8v(T *p, const float (&v)[8])
+{
+    store4(p, make_float4(v[0], v[1], v[2], v[3]));
+    store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+__device__ __forceinline__ void store8v(__nv_bfloat16 *p, const float (&v)[8])
+{
+    uint32_t w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        w[i] = *reinterpret_cast<const uint32_t *>(&h);
+    }
+    *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+}
+__device__ __forceinline__ void store8v(__half *p, const float (&v)[8])
+{
+    uint32_t w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __half2 h = __halves2half2(from_f32<__half>(v[2 * i]), from_f32<__half>(v[2 * i + 1]));
+        w[i] = *reinterpret_cast<const uint32_t *>(&h);
+    }
+    *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+}
+
 // the session of a row and the row's place among the session's tokens of this step
 __device__ __forceinline__ uint32_t seq_of(const wr_rows &rw, uint32_t row) { return rw.decode ? row : 0u; }
 __device__ __forceinline__ uint32_t tok_of(const wr_rows &rw, uint32_t row) { return rw.decode ? 0u : row; }
@@ -137,23 +198,117 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows 
     }
 }
 
+// The same for rows that cut evenly into NW warps' parts of at most 128 * NV values, none across a group border:
+// each warp keeps its part (and the previous row's) in registers between the sum and the scaling.
+template <typename TO, int NW, int NV>
+__global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows rw, const wr_norm_args a)
+{
+    __shared__ float part[2][NW];
+    pdl_trigger();
+    const uint32_t row = blockIdx.x, ld = wr_ld(a.width), unit = a.width / NW, per_group = NW / a.groups;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, at = warp * unit + 4 * lane;
+    float4 w[NV], sh[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const bool in = 4 * lane + 128 * i < unit;
+        w[i] = in ? load4(a.w + at + 128 * i) : make_float4(0, 0, 0, 0);
+        if (a.shift) sh[i] = in ? load4(a.shift + at + 128 * i) : make_float4(0, 0, 0, 0);
+    }
+    pdl_wait();
+    const float *x = a.x + (size_t)(a.gather ? a.gather[row] : row) * ld + at, *xb = x - ld;
+    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld + at;
+    uint32_t t = 0, n = 0, fresh = 0;
+    const float *kept = nullptr;
+    float *keep = nullptr;
+    if (a.shift) {
+        const wr_seq_dev &s = rw.seqs[seq_of(rw, row)];
+        t = tok_of(rw, row);
+        n = s.n;
+        fresh = s.fresh;
+        kept = reinterpret_cast<const float *>(s.st_in + a.state_off) + at;
+        keep = reinterpret_cast<float *>(s.st_out + a.state_off) + at;
+    }
+    float4 v[NV], b[NV];
+    float ss = 0.f, sb = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        v[i] = b[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (4 * lane + 128 * i < unit) {
+            v[i] = load4(x + 128 * i);
+            if (a.shift) {
+                if (t > 0) b[i] = load4(xb + 128 * i);
+                else if (!fresh) b[i] = load4(kept + 128 * i);
+            }
+        }
+        ss = fmaf(v[i].w, v[i].w, fmaf(v[i].z, v[i].z, fmaf(v[i].y, v[i].y, fmaf(v[i].x, v[i].x, ss))));
+        sb = fmaf(b[i].w, b[i].w, fmaf(b[i].z, b[i].z, fmaf(b[i].y, b[i].y, fmaf(b[i].x, b[i].x, sb))));
+    }
+    ss = warp_sum(ss);
+    sb = warp_sum(sb);
+    if (lane == 0) { part[0][warp] = ss; part[1][warp] = sb; }
+    __syncthreads();
+    const uint32_t g0 = warp / per_group * per_group;
+    const float gs = (float)(a.width / a.groups);
+    ss = sb = 0.f;
+    for (uint32_t i = 0; i < per_group; ++i) {
+        ss += part[0][g0 + i];
+        sb += part[1][g0 + i];
+    }
+    const float inv = 1.0f / sqrtf(ss / gs + a.eps), inv_b = 1.0f / sqrtf(sb / gs + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (4 * lane + 128 * i >= unit) continue;
+        float4 h = make_float4(v[i].x * inv * w[i].x, v[i].y * inv * w[i].y, v[i].z * inv * w[i].z, v[i].w * inv * w[i].w);
+        if (a.shift) {
+            float4 p = b[i];                                     // (the row a step left is kept normed)
+            if (t > 0) p = make_float4(p.x * inv_b * w[i].x, p.y * inv_b * w[i].y, p.z * inv_b * w[i].z, p.w * inv_b * w[i].w);
+            if (t + 1 == n) store4(keep + 128 * i, h);
+            h = make_float4(h.x + (p.x - h.x) * sh[i].x, h.y + (p.y - h.y) * sh[i].y, h.z + (p.z - h.z) * sh[i].z,
+                            h.w + (p.w - h.w) * sh[i].w);
+        }
+        store4(out + 128 * i, h);
+    }
+    if (warp == NW - 1 && lane < ld - a.width)                   // pad columns
+        static_cast<TO *>(a.out)[(size_t)row * ld + a.width + lane] = from_f32<TO>(0.f);
+}
+
+template <typename TO, int NW> bool group_norm_reg(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a, cudaError_t &e)
+{
+    if (NW % a.groups || a.width % (4 * NW)) return false;
+    const uint32_t vecs = (a.width / NW + 127) / 128;
+    const dim3 grid(rw.n_rows), block(NW * 32);
+    if (vecs <= 2) e = wr_launch_pdl(group_norm_reg_kernel<TO, NW, 2>, grid, block, 0, ctx->stream, rw, a);
+    else if (vecs <= 4) e = wr_launch_pdl(group_norm_reg_kernel<TO, NW, 4>, grid, block, 0, ctx->stream, rw, a);
+    else if (vecs <= 8) e = wr_launch_pdl(group_norm_reg_kernel<TO, NW, 8>, grid, block, 0, ctx->stream, rw, a);
+    else return false;
+    return true;
+}
+
 // -------------------------------------------------------------------- PolyNorm
 
-template <typename TI, typename TO>
-__global__ void __launch_bounds__(256) polynorm_kernel(const wr_polynorm_args a)
+constexpr uint32_t kPolyThreads = 512, kPolyWarps = kPolyThreads / 32;
+
+template <typename T>
+__global__ void __launch_bounds__(kPolyThreads) polynorm_kernel(const wr_polynorm_args a)
 {
-    __shared__ float red[3][8];
+    __shared__ float red[3][kPolyWarps];
     pdl_trigger();
     pdl_wait();
     const uint32_t ld = wr_ld(a.ff), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const TI *z = static_cast<const TI *>(a.z) + (size_t)blockIdx.x * ld;
-    TO *out = static_cast<TO *>(a.out) + (size_t)blockIdx.x * ld;
+    const T *z = static_cast<const T *>(a.z) + (size_t)blockIdx.x * ld;
+    T *out = static_cast<T *>(a.out) + (size_t)blockIdx.x * ld;
     float s1 = 0.f, s2 = 0.f, s3 = 0.f;
-    for (uint32_t i = threadIdx.x; i < a.ff; i += 256) {
-        const float v = to_f32(z[i]), v2 = v * v, v3 = v2 * v;
-        s1 = fmaf(v, v, s1);
-        s2 = fmaf(v2, v2, s2);
-        s3 = fmaf(v3, v3, s3);
+    for (uint32_t i = 8 * threadIdx.x; i < a.ff; i += 8 * kPolyThreads) {
+        float v[8];
+        load8v(z + i, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            if (i + e >= a.ff) v[e] = 0.f;
+            const float v2 = v[e] * v[e], v3 = v2 * v[e];
+            s1 = fmaf(v[e], v[e], s1);
+            s2 = fmaf(v2, v2, s2);
+            s3 = fmaf(v3, v3, s3);
+        }
     }
     s1 = warp_sum(s1);
     s2 = warp_sum(s2);
@@ -165,57 +320,83 @@ __global__ void __launch_bounds__(256) polynorm_kernel(const wr_polynorm_args a)
     for (int p = 0; p < 3; ++p) {
         float t = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) t += red[p][w];
+        for (uint32_t w = 0; w < kPolyWarps; ++w) t += red[p][w];
         k[p] = 1.0f / sqrtf(t / (float)a.ff + a.eps);
     }
     const float ka = a.a * k[0], kb = a.b * k[1], kc = a.c * k[2];
-    for (uint32_t i = threadIdx.x; i < ld; i += 256) {
-        float y = 0.f;
-        if (i < a.ff) {
-            const float v = to_f32(z[i]);
-            y = fmaf(v, fmaf(v, fmaf(v, kc, kb), ka), a.e);
-        }
-        out[i] = from_f32<TO>(y);
+    for (uint32_t i = 8 * threadIdx.x; i < ld; i += 8 * kPolyThreads) {
+        float v[8];
+        load8v(z + i, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = i + e < a.ff ? fmaf(v[e], fmaf(v[e], fmaf(v[e], kc, kb), ka), a.e) : 0.f;
+        store8v(out + i, v);
     }
 }
 
 // ----------------------------------------------------------------- convolution
 
-constexpr uint32_t kConvThreads = 128, kConvRows = 8;
+constexpr uint32_t kConvThreads = 128, kConvRows = 16;
 
-template <typename T>
+// A thread takes four channels through kConvRows tokens; with TAPS > 0 the last inputs stay in registers, with
+// TAPS = 0 (any number) each is fetched again.
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const wr_rows rw, const wr_conv_args a)
 {
     pdl_trigger();
+    const uint32_t ld = wr_ld(a.inner), c = 4 * (blockIdx.x * kConvThreads + threadIdx.x), taps = TAPS ? TAPS : a.taps, tail = taps - 1;
+    if (c >= ld) {
+        pdl_wait();
+        return;
+    }
+    constexpr int R = TAPS ? TAPS : 1;
+    float4 w[R];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = load4(a.w + (size_t)j * ld + c);
+    const float4 bias = load4(a.b + c);
     pdl_wait();
-    const uint32_t c = blockIdx.x * kConvThreads + threadIdx.x, ld = wr_ld(a.inner), tail = a.taps - 1;
     const uint32_t seq = blockIdx.z, row0 = row0_of(rw, seq);
     const wr_seq_dev s = rw.seqs[seq];
-    if (c >= ld) return;
     const T *x = static_cast<const T *>(a.x) + (size_t)row0 * a.x_ld + c;
     T *out = static_cast<T *>(a.out) + (size_t)row0 * ld + c;
     const uint32_t t0 = blockIdx.y * kConvRows, t1 = min(t0 + kConvRows, s.n);
-    if (c >= a.inner) {
-        for (uint32_t t = t0; t < t1; ++t) out[(size_t)t * ld] = from_f32<T>(0.f);
-        return;
-    }
-    const float *kept = reinterpret_cast<const float *>(s.st_in + a.state_off) + c;      // [taps-1][inner]
-    auto input = [&](int32_t t) -> float {                                               // token t of this step; < 0: before it
-        if (t >= 0) return to_f32(x[(size_t)t * a.x_ld]);
-        return s.fresh ? 0.f : kept[(size_t)((int32_t)tail + t) * a.inner];
+    const float *kept = reinterpret_cast<const float *>(s.st_in + a.state_off) + c;      // [taps-1][ld]
+    auto input = [&](int32_t t) -> float4 {                                              // token t of this step; < 0: before it
+        if (t >= 0) return load4(x + (size_t)t * a.x_ld);
+        return s.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(kept + (size_t)((int32_t)tail + t) * ld);
     };
-    const float bias = a.b[c];
+    auto step = [](float4 &acc, const float4 wj, const float4 v) {
+        acc = make_float4(fmaf(wj.x, v.x, acc.x), fmaf(wj.y, v.y, acc.y), fmaf(wj.z, v.z, acc.z), fmaf(wj.w, v.w, acc.w));
+    };
+    float4 win[R];
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) win[j] = input((int32_t)t0 + j - TAPS);
     for (uint32_t t = t0; t < t1; ++t) {
-        float acc = bias;
-        for (uint32_t j = 0; j < a.taps; ++j)
-            acc = fmaf(a.w[(size_t)j * ld + c], input((int32_t)(t + j) - (int32_t)tail), acc);
-        out[(size_t)t * ld] = from_f32<T>(siluf(acc));
+        float4 acc = bias;
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+            win[TAPS - 1] = load4(x + (size_t)t * a.x_ld);
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) step(acc, w[j], win[j]);
+        } else {
+            for (uint32_t j = 0; j < taps; ++j)
+                step(acc, load4(a.w + (size_t)j * ld + c), input((int32_t)(t + j) - (int32_t)tail));
+        }
+        store4(out + (size_t)t * ld, make_float4(siluf(acc.x), siluf(acc.y), siluf(acc.z), siluf(acc.w)));
     }
     if (t1 == s.n) {                                                                     // the block with the last token
         float *keep = reinterpret_cast<float *>(s.st_out + a.state_off) + c;
         for (uint32_t k = 0; k < tail; ++k)
-            keep[(size_t)k * a.inner] = input((int32_t)(s.n + k) - (int32_t)tail);
+            store4(keep + (size_t)k * ld, input((int32_t)(s.n + k) - (int32_t)tail));
     }
+}
+
+template <typename T> cudaError_t conv_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args &a)
+{
+    const uint32_t n = rw.decode ? 1u : rw.n_rows;
+    const dim3 grid((wr_ld(a.inner) / 4 + kConvThreads - 1) / kConvThreads, (n + kConvRows - 1) / kConvRows, rw.n_seq), block(kConvThreads);
+    if (a.taps == 4) return wr_launch_pdl(conv_silu_kernel<T, 4>, grid, block, 0, ctx->stream, rw, a);
+    return wr_launch_pdl(conv_silu_kernel<T, 0>, grid, block, 0, ctx->stream, rw, a);
 }
 
 // -------------------------------------------------------------- selective scan
@@ -224,7 +405,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const wr_rows r
 // neighbouring lanes and add their parts of y with shuffles.  Token tiles (x, z, dt of the block's channels, B, C)
 // come in through a two-deep cp.async ring.  The state is F32 throughout.
 
-constexpr uint32_t kScanThreads = 128, kScanTile = 16;
+constexpr uint32_t kScanThreads = 128;
 
 __device__ __forceinline__ float ex2(float x)
 {
@@ -237,19 +418,24 @@ template <int BYTES> __device__ __forceinline__ void cp_async(void *dst, const v
     asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
 }
 
-template <typename T, int NS>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, const wr_scan_args a, uint32_t tpc_log2)
+// NS: states a thread carries; LG: log2 of the threads that share a channel.  Four tokens go through the state
+// at a time; their partial sums are then exchanged so that each of the channel's threads finishes its own tokens.
+template <typename T, int NS, int LG>
+__global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, const wr_scan_args a)
 {
+    constexpr uint32_t TPC = 1u << LG, CB = kScanThreads >> LG, HELD = NS * TPC;            // channels per block, states held
+    constexpr uint32_t TILE = HELD > 128 ? 16 : 32;                                         // tokens per stage
+    constexpr int U = 4, KEEP = LG >= 2 ? 1 : U >> LG;                                      // tokens at a time; left per thread
     extern __shared__ __align__(16) uint8_t sm_scan[];
-    const uint32_t tpc = 1u << tpc_log2, cb = kScanThreads >> tpc_log2, ns = NS * tpc;      // channels, states held
-    float *bs = reinterpret_cast<float *>(sm_scan), *cs = bs + 2 * kScanTile * ns;          // [2][tile][ns]
-    float *dts = cs + 2 * kScanTile * ns;                                                   // [2][tile][cb]
-    T *xs = reinterpret_cast<T *>(dts + 2 * kScanTile * cb), *zs = xs + 2 * kScanTile * cb, *ys = zs + 2 * kScanTile * cb;
+    float *bs = reinterpret_cast<float *>(sm_scan), *cs = bs + 2 * TILE * HELD;             // [2][TILE][HELD]
+    float *dts = cs + 2 * TILE * HELD;                                                      // [2][TILE][CB]
+    T *xs = reinterpret_cast<T *>(dts + 2 * TILE * CB), *zs = xs + 2 * TILE * CB, *ys = zs + 2 * TILE * CB;
     pdl_trigger();
     const uint32_t seq = blockIdx.y, tid = threadIdx.x;
-    const uint32_t c_base = blockIdx.x * cb, cl = tid >> tpc_log2, part = tid & (tpc - 1), c = c_base + cl;
-    const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state);
-    for (uint32_t i = tid; i < 4 * kScanTile * ns; i += kScanThreads) bs[i] = 0.f;          // (B and C beyond `state`)
+    const uint32_t c_base = blockIdx.x * CB, cl = tid >> LG, part = tid & (TPC - 1), c = c_base + cl;
+    const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state), bc4 = (a.state + 3) / 4;      // 4-value pieces per token
+    if (HELD > 4 * bc4)
+        for (uint32_t i = tid; i < 4 * TILE * HELD; i += kScanThreads) bs[i] = 0.f;         // (B and C beyond `state`)
     float A2[NS], S[NS];
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
@@ -267,14 +453,13 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
         S[j] = (!s.fresh && c < a.inner && n < a.state) ? st_in[(size_t)c * a.state + n] : 0.f;
     }
     __syncthreads();
-    const uint32_t xc4 = cb / 4, bc4 = (a.state + 3) / 4;            // 4-value pieces per token
     auto request = [&](uint32_t tile) {
-        const uint32_t st = tile & 1, t0 = tile * kScanTile, nt = min(kScanTile, n_tok - t0);
-        for (uint32_t i = tid; i < nt * xc4; i += kScanThreads) {
-            const uint32_t t = i / xc4, q = i % xc4, ch = c_base + 4 * q;
+        const uint32_t st = tile & 1, t0 = tile * TILE, nt = min(TILE, n_tok - t0);
+        for (uint32_t i = tid; i < nt * (CB / 4); i += kScanThreads) {
+            const uint32_t t = i / (CB / 4), q = i % (CB / 4), ch = c_base + 4 * q;
             if (ch >= ld) continue;
             const size_t row = row0 + t0 + t;
-            const uint32_t at = (st * kScanTile + t) * cb + 4 * q;
+            const uint32_t at = (st * TILE + t) * CB + 4 * q;
             cp_async<4 * sizeof(T)>(xs + at, static_cast<const T *>(a.x) + row * a.x_ld + ch);
             cp_async<4 * sizeof(T)>(zs + at, static_cast<const T *>(a.z) + row * a.z_ld + ch);
             cp_async<16>(dts + at, a.dt + row * ld + ch);
@@ -282,15 +467,15 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
         for (uint32_t i = tid; i < nt * bc4; i += kScanThreads) {
             const uint32_t t = i / bc4, q = i % bc4;
             const float *src = a.bc + (size_t)(row0 + t0 + t) * a.bc_ld + 4 * q;
-            cp_async<16>(bs + (st * kScanTile + t) * ns + 4 * q, src + a.b_off);
-            cp_async<16>(cs + (st * kScanTile + t) * ns + 4 * q, src + a.c_off);
+            cp_async<16>(bs + (st * TILE + t) * HELD + 4 * q, src + a.b_off);
+            cp_async<16>(cs + (st * TILE + t) * HELD + 4 * q, src + a.c_off);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    const uint32_t tiles = (n_tok + kScanTile - 1) / kScanTile;
+    const uint32_t tiles = (n_tok + TILE - 1) / TILE;
     request(0);
     for (uint32_t tile = 0; tile < tiles; ++tile) {
-        const uint32_t st = tile & 1, t0 = tile * kScanTile, nt = min(kScanTile, n_tok - t0);
+        const uint32_t st = tile & 1, t0 = tile * TILE, nt = min(TILE, n_tok - t0);
         if (tile + 1 < tiles) {
             request(tile + 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -298,34 +483,72 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        auto token = [&](uint32_t t) {
-            const uint32_t at = (st * kScanTile + t) * cb + cl;
-            const float dt = dts[at], x = to_f32(xs[at]), dx = dt * x;
-            const float *b = bs + (st * kScanTile + t) * ns + part * NS, *cc = cs + (st * kScanTile + t) * ns + part * NS;
-            float y = 0.f;
+#pragma unroll 1
+        for (uint32_t tb = 0; tb < nt; tb += U) {
+            float y[U];
+            auto token = [&](int u) {
+                const uint32_t t = st * TILE + tb + u;
+                const float dt = dts[t * CB + cl], dx = dt * to_f32(xs[t * CB + cl]);
+                const float *b = bs + t * HELD + part * NS, *cc = cs + t * HELD + part * NS;
+                y[u] = 0.f;
 #pragma unroll
-            for (int j = 0; j < NS; ++j) {
-                S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b[j]);
-                y = fmaf(S[j], cc[j], y);
+                for (int j = 0; j < NS; j += 4) {
+                    const float4 b4 = load4(b + j), c4 = load4(cc + j);
+                    S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b4.x);
+                    S[j + 1] = fmaf(ex2(dt * A2[j + 1]), S[j + 1], dx * b4.y);
+                    S[j + 2] = fmaf(ex2(dt * A2[j + 2]), S[j + 2], dx * b4.z);
+                    S[j + 3] = fmaf(ex2(dt * A2[j + 3]), S[j + 3], dx * b4.w);
+                    y[u] = fmaf(S[j], c4.x, y[u]);
+                    y[u] = fmaf(S[j + 1], c4.y, y[u]);
+                    y[u] = fmaf(S[j + 2], c4.z, y[u]);
+                    y[u] = fmaf(S[j + 3], c4.w, y[u]);
+                }
+            };
+            if (tb + U <= nt) {
+#pragma unroll
+                for (int u = 0; u < U; ++u) token(u);
+            } else {
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    y[u] = 0.f;
+                    if (tb + u < nt) token(u);
+                }
             }
-            for (uint32_t o = tpc >> 1; o >= 1; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (part == (t & (tpc - 1))) {
-                y = fmaf(D, x, y);
-                ys[t * cb + cl] = from_f32<T>(y * siluf(to_f32(zs[at])));
+            uint32_t first = 0, width = U;                       // this thread keeps tokens [first, first + width)
+#pragma unroll
+            for (uint32_t o = 1; o < TPC; o <<= 1) {
+                if (width > 1) {
+                    const uint32_t half = width / 2;
+                    const bool upper = (part & o) != 0;
+#pragma unroll
+                    for (int i = 0; i < U / 2; ++i) {
+                        if (i < (int)half) {
+                            const float send = upper ? y[i] : y[i + half], own = upper ? y[i + half] : y[i];
+                            y[i] = own + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                    }
+                    if (upper) first += half;
+                    width = half;
+                } else {
+                    y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+                }
             }
-        };
-        if (nt == kScanTile) {
-#pragma unroll 4
-            for (uint32_t t = 0; t < kScanTile; ++t) token(t);
-        } else {
-            for (uint32_t t = 0; t < nt; ++t) token(t);
+#pragma unroll
+            for (int i = 0; i < KEEP; ++i) {
+                const uint32_t t = tb + first + i, at = (st * TILE + t) * CB + cl;
+                if (t < nt && part < 4) {
+                    const float v = fmaf(D, to_f32(xs[at]), y[i]) * siluf(to_f32(zs[at]));
+                    ys[t * CB + cl] = from_f32<T>(c < a.inner ? v : 0.f);
+                }
+            }
         }
         __syncthreads();
-        for (uint32_t i = tid; i < nt * cb; i += kScanThreads) {
-            const uint32_t t = i / cb, q = i % cb, ch = c_base + q;
+        for (uint32_t i = tid; i < nt * (CB / 4); i += kScanThreads) {
+            const uint32_t t = i / (CB / 4), q = i % (CB / 4), ch = c_base + 4 * q;
             if (ch < ld) {
                 T *o = static_cast<T *>(a.out) + (size_t)(row0 + t0 + t) * ld + ch;
-                *o = ch < a.inner ? ys[t * cb + q] : from_f32<T>(0.f);
+                if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2 *>(o) = *reinterpret_cast<const uint2 *>(ys + t * CB + 4 * q);
+                else *reinterpret_cast<float4 *>(o) = *reinterpret_cast<const float4 *>(ys + t * CB + 4 * q);
             }
         }
     }
@@ -337,54 +560,92 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
     }
 }
 
-template <typename T, int NS>
-int scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+template <typename T, int NS, int LG> int scan_one(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
-    uint32_t lg = 0;
-    while ((NS << lg) < (int)a.state) ++lg;
-    if (lg > 5) return WR_CUDA_ERR_LIMIT;
-    const uint32_t cb = kScanThreads >> lg, ns = NS << lg;
-    const size_t smem = (size_t)(4 * kScanTile * ns + 2 * kScanTile * cb) * 4 + (size_t)5 * kScanTile * cb * sizeof(T);
-    auto k = scan_kernel<T, NS>;
+    constexpr uint32_t CB = kScanThreads >> LG, HELD = NS << LG, TILE = HELD > 128 ? 16 : 32;
+    constexpr size_t smem = (size_t)(4 * TILE * HELD + 2 * TILE * CB) * 4 + (size_t)5 * TILE * CB * sizeof(T);
+    auto k = scan_kernel<T, NS, LG>;
     if (smem > 48 * 1024)
         WR_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    WR_CUDA_TRY(wr_launch_pdl(k, dim3((wr_ld(a.inner) + cb - 1) / cb, rw.n_seq), dim3(kScanThreads), smem, ctx->stream, rw,
-                              a, lg));
+    WR_CUDA_TRY(wr_launch_pdl(k, dim3((wr_ld(a.inner) + CB - 1) / CB, rw.n_seq), dim3(kScanThreads), smem, ctx->stream, rw, a));
     return finish_launch(ctx);
+}
+
+template <typename T> int scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+{
+    if (a.state <= 4) return scan_one<T, 4, 0>(ctx, rw, a);
+    if (a.state <= 8) return scan_one<T, 4, 1>(ctx, rw, a);
+    if (a.state <= 16) return scan_one<T, 4, 2>(ctx, rw, a);
+    if (a.state <= 32) return scan_one<T, 4, 3>(ctx, rw, a);
+    if (a.state <= 64) return scan_one<T, 4, 4>(ctx, rw, a);
+    if (a.state <= 128) return scan_one<T, 4, 5>(ctx, rw, a);
+    if (a.state <= 256) return scan_one<T, 8, 5>(ctx, rw, a);
+    if (a.state <= 512) return scan_one<T, 16, 5>(ctx, rw, a);
+    return WR_CUDA_ERR_LIMIT;
 }
 
 // ------------------------------------------------------------- around attention
 
-// Queries out of the projection row (scale and temperature applied), K and V into the session's pages.
-template <typename TI, typename TQ>
+// Queries out of the projection row (scale and temperature applied), K and V into the session's pages.  The row's
+// queries, keys and values are one list of pieces of W values; the blocks of grid.y share it.
+template <typename TI, typename TQ, int W>
 __global__ void __launch_bounds__(256) attn_prep_kernel(const wr_rows rw, const wr_attn_prep_args a)
 {
     pdl_trigger();
     pdl_wait();
-    const uint32_t row = blockIdx.x, tid = threadIdx.x;
+    const uint32_t row = blockIdx.x;
     const wr_seq_dev s = rw.seqs[seq_of(rw, row)];
     const uint32_t pos = s.pos + tok_of(rw, row);
     const wr_attn_geom g = a.g;
     const TI *in = static_cast<const TI *>(a.qkv) + (size_t)row * a.ld;
     float mul = a.scale;
     if (a.temp_every) mul *= 1.0f + a.temp_coef * logf((float)((pos + 1u) / a.temp_every + 1u));
-    const uint32_t qs = g.q_stride(), nq = g.vq() * qs;
-    TQ *q = static_cast<TQ *>(a.q) + (size_t)row * nq;
-    for (uint32_t i = tid; i < nq; i += 256) {
-        const uint32_t vq = i / qs, e = i % qs, off = g.hd128 ? (vq % g.maps) * g.kd : 0u;     // the map's part of the row
-        float v = 0.f;
-        if (e >= off && e < off + g.kd) v = to_f32(in[vq * g.kd + e - off]) * mul;
-        q[i] = from_f32<TQ>(v);
-    }
+    const uint32_t qs = g.q_stride(), kw = g.maps * g.kd;
+    const uint32_t nq = g.vq() * qs / W, nk = g.n_kv * kw / W, nv = g.n_kv * g.vd / W;
+    TQ *q = static_cast<TQ *>(a.q) + (size_t)row * g.vq() * qs;
     char *page = reinterpret_cast<char *>(s.pages[(size_t)g.layer * s.n_pages + pos / kPageTokens]);
-    const uint32_t tok = pos % kPageTokens, kw = g.maps * g.kd;
-    auto put = [&](uint32_t head, uint32_t which, uint32_t d, float v) {
-        char *p = page + wr_geom_off(g.kv, head, which, tok, d);
-        if (g.kv.elem == WR_CUDA_F32) *reinterpret_cast<float *>(p) = v;
-        else *reinterpret_cast<__half *>(p) = from_f32<__half>(v);
-    };
-    for (uint32_t i = tid; i < g.n_kv * kw; i += 256) put(i / kw, 0, i % kw, to_f32(in[a.k_off + i]));
-    for (uint32_t i = tid; i < g.n_kv * g.vd; i += 256) put(i / g.vd, 1, i % g.vd, to_f32(in[a.v_off + i]));
+    const uint32_t tok = pos % kPageTokens;
+    for (uint32_t i = blockIdx.y * 256 + threadIdx.x; i < nq + nk + nv; i += gridDim.y * 256) {
+        float v[W];
+        auto fetch = [&](const TI *p) {
+            if constexpr (W == 8) load8v(p, v);
+            else v[0] = to_f32(*p);
+        };
+        if (i < nq) {
+            const uint32_t at = i * W, vq = at / qs, e = at % qs, off = g.hd128 ? (vq % g.maps) * g.kd : 0u;   // the map's part of the row
+            if (e >= off && e < off + g.kd) {
+                fetch(in + vq * g.kd + e - off);
+#pragma unroll
+                for (int j = 0; j < W; ++j) v[j] *= mul;
+            } else {
+#pragma unroll
+                for (int j = 0; j < W; ++j) v[j] = 0.f;
+            }
+            if constexpr (W == 8) store8v(q + at, v);
+            else q[at] = from_f32<TQ>(v[0]);
+            continue;
+        }
+        const uint32_t which = i < nq + nk ? 0u : 1u, at = (i - nq - which * nk) * W, dim = which ? g.vd : kw;
+        fetch(in + (which ? a.v_off : a.k_off) + at);
+        char *p = page + wr_geom_off(g.kv, at / dim, which, tok, at % dim);
+        if constexpr (W == 8) {
+            if (g.kv.elem == WR_CUDA_F32) store8v(reinterpret_cast<float *>(p), v);
+            else store8v(reinterpret_cast<__half *>(p), v);
+        } else {
+            if (g.kv.elem == WR_CUDA_F32) *reinterpret_cast<float *>(p) = v[0];
+            else *reinterpret_cast<__half *>(p) = from_f32<__half>(v[0]);
+        }
+    }
+}
+
+template <typename TI, typename TQ> cudaError_t prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_prep_args &a)
+{
+    const wr_attn_geom &g = a.g;
+    const uint32_t w = g.kd % 8 == 0 && g.vd % 8 == 0 ? 8 : 1;
+    const uint32_t items = (g.vq() * g.q_stride() + g.n_kv * (g.maps * g.kd + g.vd)) / w;
+    const dim3 grid(rw.n_rows, rw.n_rows <= WR_CUDA_BATCH_MAX ? (items + 255) / 256 : (items + 1023) / 1024), block(256);
+    if (w == 8) return wr_launch_pdl(attn_prep_kernel<TI, TQ, 8>, grid, block, 0, ctx->stream, rw, a);
+    return wr_launch_pdl(attn_prep_kernel<TI, TQ, 1>, grid, block, 0, ctx->stream, rw, a);
 }
 
 // One warp per query head: combine the maps, norm over the head, gate.
@@ -399,6 +660,31 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const wr_rows rw, cons
     TO *out = static_cast<TO *>(a.out) + (size_t)row * ld;
     for (uint32_t h = blockIdx.y * 8 + warp; h < g.n_q; h += gridDim.y * 8) {
         const float *o1 = a.o + ((size_t)row * g.vq() + h * g.maps) * os, *o2 = o1 + os;
+        if (g.vd <= 128 && g.vd % 4 == 0) {                      // a lane's four values stay in registers
+            const uint32_t i = 4 * lane;
+            float4 d = make_float4(0.f, 0.f, 0.f, 0.f), gt = d;
+            if (i < g.vd) {
+                d = load4(o1 + i);
+                if (a.gate) gt = load4(static_cast<const TG *>(a.gate) + (size_t)row * a.gate_ld + h * g.vd + i);
+                if (g.maps == 2) {
+                    const float4 e = load4(o2 + i);
+                    d = make_float4(fmaf(-a.lambda, e.x, d.x), fmaf(-a.lambda, e.y, d.y), fmaf(-a.lambda, e.z, d.z),
+                                    fmaf(-a.lambda, e.w, d.w));
+                }
+            }
+            float k = 1.0f;
+            if (g.maps == 2) {
+                const float ss = fmaf(d.w, d.w, fmaf(d.z, d.z, fmaf(d.y, d.y, d.x * d.x)));
+                k = (1.0f - a.diff_init) / sqrtf(warp_sum(ss) / (float)g.vd + a.eps);
+            }
+            if (i < g.vd) {
+                d = make_float4(d.x * k, d.y * k, d.z * k, d.w * k);
+                if (a.gate)
+                    d = make_float4(d.x * sigmoidf(gt.x), d.y * sigmoidf(gt.y), d.z * sigmoidf(gt.z), d.w * sigmoidf(gt.w));
+                store4(out + h * g.vd + i, d);
+            }
+            continue;
+        }
         float k = 1.0f;
         if (g.maps == 2) {
             float ss = 0.f;
@@ -665,51 +951,49 @@ int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens,
 
 int wr_group_norm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a)
 {
-    const uint32_t split = std::max(1u, kNormWarps / a.groups);
-    const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
-    if (smem > 48 * 1024) return WR_CUDA_ERR_LIMIT;
-    if (a.out_type == WR_ACT_BF16)
-        WR_CUDA_TRY(wr_launch_pdl(group_norm_kernel<__nv_bfloat16>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split));
-    else
-        WR_CUDA_TRY(wr_launch_pdl(group_norm_kernel<float>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split));
+    const bool bf = a.out_type == WR_ACT_BF16;
+    // few rows: more warps on each (which kernel serves a row is a matter of the step's kind, not of its row count)
+    cudaError_t e = cudaSuccess;
+    const bool done = rw.n_rows <= WR_CUDA_BATCH_MAX
+                          ? (bf ? group_norm_reg<__nv_bfloat16, 16>(ctx, rw, a, e) : group_norm_reg<float, 16>(ctx, rw, a, e))
+                          : (bf ? group_norm_reg<__nv_bfloat16, 8>(ctx, rw, a, e) : group_norm_reg<float, 8>(ctx, rw, a, e));
+    if (!done) {
+        const uint32_t split = std::max(1u, kNormWarps / a.groups);
+        const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
+        if (smem > 48 * 1024) return WR_CUDA_ERR_LIMIT;
+        const dim3 grid(rw.n_rows), block(kNormThreads);
+        e = bf ? wr_launch_pdl(group_norm_kernel<__nv_bfloat16>, grid, block, smem, ctx->stream, rw, a, split)
+               : wr_launch_pdl(group_norm_kernel<float>, grid, block, smem, ctx->stream, rw, a, split);
+    }
+    WR_CUDA_TRY(e);
     return finish_launch(ctx);
 }
 
 int wr_polynorm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_polynorm_args &a)
 {
     if (a.z_type == WR_ACT_BF16)
-        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(rw.n_rows), dim3(256), 0, ctx->stream, a));
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<__nv_bfloat16>, dim3(rw.n_rows), dim3(kPolyThreads), 0, ctx->stream, a));
     else
-        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float, float>, dim3(rw.n_rows), dim3(256), 0, ctx->stream, a));
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float>, dim3(rw.n_rows), dim3(kPolyThreads), 0, ctx->stream, a));
     return finish_launch(ctx);
 }
 
 int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args &a)
 {
-    const uint32_t n = rw.decode ? 1u : rw.n_rows;
-    const dim3 grid((wr_ld(a.inner) + kConvThreads - 1) / kConvThreads, (n + kConvRows - 1) / kConvRows, rw.n_seq);
-    if (a.type == WR_ACT_BF16)
-        WR_CUDA_TRY(wr_launch_pdl(conv_silu_kernel<__nv_bfloat16>, grid, dim3(kConvThreads), 0, ctx->stream, rw, a));
-    else
-        WR_CUDA_TRY(wr_launch_pdl(conv_silu_kernel<float>, grid, dim3(kConvThreads), 0, ctx->stream, rw, a));
+    WR_CUDA_TRY(a.type == WR_ACT_BF16 ? conv_launch<__nv_bfloat16>(ctx, rw, a) : conv_launch<float>(ctx, rw, a));
     return finish_launch(ctx);
 }
 
 int wr_scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
-    const bool bf = a.type == WR_ACT_BF16;
-    if (a.state <= 128) return bf ? scan_launch<__nv_bfloat16, 4>(ctx, rw, a) : scan_launch<float, 4>(ctx, rw, a);
-    return bf ? scan_launch<__nv_bfloat16, 16>(ctx, rw, a) : scan_launch<float, 16>(ctx, rw, a);
+    return a.type == WR_ACT_BF16 ? scan_launch<__nv_bfloat16>(ctx, rw, a) : scan_launch<float>(ctx, rw, a);
 }
 
 int wr_attn_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_prep_args &a)
 {
-    const dim3 grid(rw.n_rows), block(256);
     const bool half_in = a.type == WR_ACT_F16, half_q = a.q_type == WR_ACT_F16;
-    if (half_in && half_q) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<__half, __half>, grid, block, 0, ctx->stream, rw, a));
-    else if (half_in) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<__half, float>, grid, block, 0, ctx->stream, rw, a));
-    else if (half_q) WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<float, __half>, grid, block, 0, ctx->stream, rw, a));
-    else WR_CUDA_TRY(wr_launch_pdl(attn_prep_kernel<float, float>, grid, block, 0, ctx->stream, rw, a));
+    WR_CUDA_TRY(half_in ? (half_q ? prep_launch<__half, __half>(ctx, rw, a) : prep_launch<__half, float>(ctx, rw, a))
+                        : (half_q ? prep_launch<float, __half>(ctx, rw, a) : prep_launch<float, float>(ctx, rw, a)));
     return finish_launch(ctx);
 }
 

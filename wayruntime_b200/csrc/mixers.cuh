@@ -52,7 +52,7 @@ struct wr_conv_args {
     const void *x; int type;         // [rows][x_ld], channels first
     uint32_t x_ld, inner, taps;
     const float *w, *b;              // [taps][wr_ld(inner)] (tap-major), [inner]
-    uint64_t state_off;              // [taps-1][inner] F32
+    uint64_t state_off;              // [taps-1][wr_ld(inner)] F32
     void *out;                       // [rows][wr_ld(inner)] of `type`
 };
 int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args &a);

@@ -278,7 +278,7 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
         set_off(o.a2, a);
         set_off(o.d, pk.vec(l.d, l.inner));
         o.conv_off = o.cache.state_bytes;
-        o.scan_off = o.conv_off + up256((size_t)(l.taps - 1) * l.inner * 4);
+        o.scan_off = o.conv_off + up256((size_t)(l.taps - 1) * ldi * 4);
         o.cache.state_bytes = o.scan_off + up256((size_t)l.inner * l.state * 4);
     }
     if (l.ffn == WR_CUDA_FFN_POLYNORM) {
@@ -519,6 +519,17 @@ struct Step {
             ++m->launches;
             return wr_gemm_launch(ctx, mat.x_map, mat.map, a);
         }
+        ++m->launches;
+        if (x->compute == WR_CUDA_BF16) {
+            wr_skinny_args a{};
+            a.x = static_cast<const float *>(in); a.x_ld = in_ld; a.x_k = wr_ld(mat.k);
+            a.rows = rw.n_rows; a.n = mat.n; a.k = mat.k;
+            a.out = static_cast<float *>(out); a.out_ld = out_ld;
+            a.bias = bias;
+            a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
+            a.add = add; a.add_ld = out_ld;
+            return wr_skinny_launch(ctx, mat.map, a);
+        }
         GemvParams p{};
         p.seg[0] = {mat.w, static_cast<float *>(out), mat.n, out_ld};
         p.n_seg = 1;
@@ -529,9 +540,8 @@ struct Step {
         p.add = add; p.add_stride = out_ld;
         p.bias = bias;
         p.act = softplus ? WR_GEMV_ACT_SOFTPLUS : WR_GEMV_ACT_NONE;
-        ++m->launches;
         ctx->launches++;
-        return wr_gemv_launch(ctx, p, mat.n, x->compute);
+        return wr_gemv_launch(ctx, p, mat.n, WR_CUDA_F32);
     }
 
     int norm(const float *w, const float *shift, uint64_t state_off)
