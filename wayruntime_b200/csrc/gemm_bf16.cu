@@ -273,6 +273,11 @@ int wr_gemm_map_rows(CUtensorMap *map, const void *x, uint32_t rows, uint32_t k,
     return map_2d(map, x, rows, k, ld, kBM);
 }
 
+int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld)
+{
+    return map_2d(map, split_rows, 2 * WR_CUDA_BATCH_MAX, k, ld, 2 * WR_CUDA_BATCH_MAX);
+}
+
 int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_gemm_args &a)
 {
     if (a.m == 0 || a.n == 0 || a.k == 0 || (a.out_ld & 7u) || (a.out_bf16_ld & 7u) || (a.add_ld & 7u))

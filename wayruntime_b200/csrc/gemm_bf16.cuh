@@ -28,16 +28,19 @@ int wr_gemm_map_rows(CUtensorMap *map, const void *x, uint32_t rows, uint32_t k,
 // Enqueue out[m][n] = act(x . w^T + bias) + add on the context's stream.
 int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_gemm_args &args);
 
-// The same product for at most WR_CUDA_BATCH_MAX rows of F32 activations, weights streamed once: every row's bits
-// are the same whatever the other rows are and however many.  out F32.
+// The same product for at most WR_CUDA_BATCH_MAX rows, weights streamed once.  The activation rows are "split": an
+// F32 value is kept as two BF16 numbers, its rounding in row r and what is left in row WR_CUDA_BATCH_MAX + r of one
+// buffer, so the product sees about 16 bits of it.  A row's bits do not depend on the other rows.  out F32.
 struct wr_skinny_args {
-    const float *x;        // [rows][x_ld], columns up to x_k (a multiple of 8, at least k) hold finite values
-    uint32_t x_ld, x_k, rows, n, k;
+    uint32_t rows, n, k;
     float *out;            // [rows][out_ld]
     uint32_t out_ld;
+    void *out_split;       // the result (before the residual) as split rows too, or null
+    uint32_t out_split_ld;
     const float *bias;     // [n] or null
     uint32_t act;          // WR_GEMM_ACT_*
     const float *add;      // [rows][add_ld] or null (may alias out)
     uint32_t add_ld;
 };
-int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &w, const wr_skinny_args &args);
+int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld);
+int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_skinny_args &args);

@@ -1,13 +1,12 @@
 // gemm_skinny.cu — out[r][n] = act(w[n] . x[r] + bias) + add for up to 16 rows: a decode step's projections.
 //
 // HBM-bound: the weights are all the traffic.  The operands are swapped — 128 weight rows are the tensor core's M,
-// the activation rows its N — and each F32 activation enters as two BF16 numbers (its rounding and the remainder,
-// 16 + 16 columns), so that the product keeps about 16 bits of the activations instead of 8.  A CTA owns 128
-// weight rows and a slice of K; the CTAs of a cluster share the rows and add their slices through distributed
-// shared memory in rank order.  Warp 0 streams weights with TMA — they depend on nothing, so it starts before the
-// kernel ahead has finished —, warps 2-5 turn activations into the swizzled operand and later finish the rows,
-// warp 1 issues tcgen05.mma.  All 32 columns are always computed, the absent rows as zeros: a row's result does
-// not depend on how many rows share the step.
+// the activation rows its N, each F32 activation as two BF16 numbers in two columns (split rows, see
+// gemm_bf16.cuh).  A CTA owns 128 weight rows and a slice of K; the CTAs of a cluster share the rows and add their
+// slices through distributed shared memory in rank order.  Warp 0 streams both operands with TMA — the weights
+// depend on nothing, so their first stages are requested before the kernel ahead has finished —, warp 1 issues
+// tcgen05.mma, warps 2-5 finish the rows.  All columns are always computed: a row's result does not depend on how
+// many rows share the step.
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -17,12 +16,13 @@
 
 namespace {
 
-constexpr uint32_t kM = 128, kN = 32, kBK = 64, kRows = WR_CUDA_BATCH_MAX;
-constexpr uint32_t kThreads = 192, kStages = 4;
+constexpr uint32_t kRows = WR_CUDA_BATCH_MAX, kM = 128, kN = 2 * kRows, kBK = 64;
+constexpr uint32_t kThreads = 192, kStages = 5;
 constexpr uint32_t kABytes = kM * kBK * 2, kBBytes = kN * kBK * 2, kStageBytes = kABytes + kBBytes;
 constexpr uint32_t kRedFloats = kRows * kM;              // one rank's sums
+constexpr uint32_t kMaxSplit = 8;
 constexpr uint32_t kTmemCols = 32;
-constexpr uint32_t kAhead = 4;                           // activation blocks held in registers
+static_assert((kMaxSplit - 1) * kRedFloats * 4 <= kStages * kStageBytes, "the other ranks' sums fit where the stages were");
 
 struct SkinnyParams {
     wr_skinny_args a;
@@ -33,16 +33,6 @@ struct SkinnyParams {
 
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
-// a pair as BF16 (hi) and what is left of it (lo)
-__device__ __forceinline__ void split_bf16(float x, float y, uint32_t &hi, uint32_t &lo)
-{
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const float2 f = __bfloat1622float2(h);
-    const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
-    hi = *reinterpret_cast<const uint32_t *>(&h);
-    lo = *reinterpret_cast<const uint32_t *>(&l);
-}
-
 __device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
 __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 __device__ __forceinline__ void store_rank0(float *p, float v)
@@ -52,20 +42,21 @@ __device__ __forceinline__ void store_rank0(float *p, float v)
     asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
 }
 
-__global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_constant__ CUtensorMap w_map, const SkinnyParams p)
+__global__ void __launch_bounds__(kThreads)
+gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, const SkinnyParams p)
 {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t full[kStages], empty[kStages], acc_full;
     __shared__ uint32_t tmem_slot;
     uint8_t *stages = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023u) & ~(uintptr_t)1023u);
-    float *red = reinterpret_cast<float *>(stages + kStages * kStageBytes);      // [rank - 1][row][128]
+    float *red = reinterpret_cast<float *>(stages);      // [rank - 1][row][128], once the products are done
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = blockIdx.x % p.split, n0 = (blockIdx.x / p.split) * kM;
     const uint32_t kb0 = p.k_blocks * rank / p.split, kb1 = p.k_blocks * (rank + 1) / p.split, nkb = kb1 - kb0;
     pdl_trigger();
     if (threadIdx.x == 0) {
         for (uint32_t i = 0; i < kStages; ++i) {
-            mbar_init(&full[i], 5);                      // the weights' arrival and one per activation warp
+            mbar_init(&full[i], 1);
             mbar_init(&empty[i], 1);
         }
         mbar_init(&acc_full, 1);
@@ -75,24 +66,35 @@ __global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_cons
     tc5::fence_before();
     __syncthreads();
     tc5::fence_after();
-    if (p.split > 1) cluster_arrive();                   // (waited for before the first remote store)
     const uint32_t tmem = tmem_slot;
     float s[kRows];
 
     if (warp == 0) {
         if (lane == 0) {
+            auto weights = [&](uint32_t it) {
+                const uint32_t st = it % kStages;
+                uint8_t *a = stages + st * kStageBytes;
+                mbar_expect_tx(&full[st], kStageBytes);
+                tc5::tma_load_2d(a, &w_map, (int)((kb0 + it) * kBK), (int)n0, &full[st]);
+                tc5::tma_load_2d(a + kABytes / 2, &w_map, (int)((kb0 + it) * kBK), (int)(n0 + kM / 2), &full[st]);
+            };
+            auto rows = [&](uint32_t it) {
+                const uint32_t st = it % kStages;
+                tc5::tma_load_2d(stages + st * kStageBytes + kABytes, &x_map, (int)((kb0 + it) * kBK), 0, &full[st]);
+            };
             bool ok = true;
             uint32_t it = 0;
+            const uint32_t first = nkb < kStages ? nkb : kStages;
+            for (; it < first; ++it) weights(it);
+            pdl_wait();
+            for (uint32_t i = 0; i < first; ++i) rows(i);
             for (; it < nkb; ++it) {
-                const uint32_t st = it % kStages;
-                if (it >= kStages && !mbar_wait(&empty[st], (it / kStages - 1) & 1, p.wait_limit)) {
+                if (!mbar_wait(&empty[it % kStages], (it / kStages - 1) & 1, p.wait_limit)) {
                     ok = false;
                     break;
                 }
-                uint8_t *a = stages + st * kStageBytes;
-                mbar_expect_tx(&full[st], kABytes);
-                tc5::tma_load_2d(a, &w_map, (int)((kb0 + it) * kBK), (int)n0, &full[st]);
-                tc5::tma_load_2d(a + kABytes / 2, &w_map, (int)((kb0 + it) * kBK), (int)(n0 + kM / 2), &full[st]);
+                weights(it);
+                rows(it);
             }
             if (!ok) atomicCAS(p.err, 0, 51);
             const uint32_t last = it < kStages ? it : kStages;
@@ -122,47 +124,8 @@ __global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_cons
         if (!ok && lane == 0) atomicCAS(p.err, 0, 52);
         __syncwarp();
     } else {
-        const uint32_t tid = threadIdx.x - 64, r = tid >> 3, c = tid & 7;
-        const bool present = r < p.a.rows;
-        const float *x = p.a.x + (size_t)(present ? r : 0) * p.a.x_ld;
         pdl_wait();
-        float4 buf[kAhead][2];
-        auto load = [&](uint32_t it, float4 (&b)[2]) {
-            const uint32_t k = (kb0 + it) * kBK + c * 8;
-            b[0] = b[1] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (present && it < nkb && k < p.a.x_k) {
-                b[0] = *reinterpret_cast<const float4 *>(x + k);
-                b[1] = *reinterpret_cast<const float4 *>(x + k + 4);
-            }
-        };
-#pragma unroll
-        for (uint32_t j = 0; j < kAhead; ++j) load(j, buf[j]);
-        bool ok = true;
-        for (uint32_t base = 0; base < nkb && ok; base += kAhead) {
-#pragma unroll
-            for (uint32_t j = 0; j < kAhead; ++j) {
-                const uint32_t it = base + j, st = it % kStages;
-                if (it < nkb && ok) {
-                    if (it >= kStages) ok = mbar_wait(&empty[st], (it / kStages - 1) & 1, p.wait_limit);
-                    if (ok) {
-                        uint4 hi, lo;
-                        split_bf16(buf[j][0].x, buf[j][0].y, hi.x, lo.x);
-                        split_bf16(buf[j][0].z, buf[j][0].w, hi.y, lo.y);
-                        split_bf16(buf[j][1].x, buf[j][1].y, hi.z, lo.z);
-                        split_bf16(buf[j][1].z, buf[j][1].w, hi.w, lo.w);
-                        uint8_t *b = stages + st * kStageBytes + kABytes + r * 128 + ((c ^ (r & 7)) << 4);
-                        *reinterpret_cast<uint4 *>(b) = hi;
-                        *reinterpret_cast<uint4 *>(b + kRows * 128) = lo;
-                        fence_proxy_async();
-                    }
-                    __syncwarp();
-                    if (ok && lane == 0) mbar_arrive(&full[st]);
-                    load(it + kAhead, buf[j]);
-                }
-            }
-        }
-        if (ok) ok = mbar_wait(&acc_full, 0, p.wait_limit);
-        if (!ok && lane == 0) atomicCAS(p.err, 0, 53);
+        if (!mbar_wait(&acc_full, 0, p.wait_limit) && lane == 0) atomicCAS(p.err, 0, 53);
         __syncwarp();
         tc5::fence_after();
         float v[kN];
@@ -173,10 +136,12 @@ __global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_cons
     }
     const uint32_t m = (warp & 3) * 32 + lane;           // (finishing warps)
     if (p.split > 1) {
+        cluster_arrive();                                // every rank's products are done: its stages are free
         cluster_wait();
         if (warp >= 2 && rank > 0) {
 #pragma unroll
-            for (uint32_t i = 0; i < kRows; ++i) store_rank0(red + (rank - 1) * kRedFloats + i * kM + m, s[i]);
+            for (uint32_t i = 0; i < kRows; ++i)
+                if (i < p.a.rows) store_rank0(red + (rank - 1) * kRedFloats + i * kM + m, s[i]);
         }
         cluster_arrive();
         cluster_wait();
@@ -190,6 +155,12 @@ __global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_cons
                 for (uint32_t q = 1; q < p.split; ++q) y += red[(q - 1) * kRedFloats + i * kM + m];
                 y += bias;
                 if (p.a.act == WR_GEMM_ACT_SOFTPLUS) y = softplus(y);
+                if (p.a.out_split) {
+                    __nv_bfloat16 *o = static_cast<__nv_bfloat16 *>(p.a.out_split) + (size_t)i * p.a.out_split_ld + n0 + m;
+                    const __nv_bfloat16 hi = __float2bfloat16_rn(y);
+                    o[0] = hi;
+                    o[(size_t)kRows * p.a.out_split_ld] = __float2bfloat16_rn(y - __bfloat162float(hi));
+                }
                 if (p.a.add) y += p.a.add[(size_t)i * p.a.add_ld + n0 + m];
                 p.a.out[(size_t)i * p.a.out_ld + n0 + m] = y;
             }
@@ -203,23 +174,21 @@ __global__ void __launch_bounds__(kThreads) gemm_skinny_kernel(const __grid_cons
 
 }  // namespace
 
-int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &w, const wr_skinny_args &a)
+int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_skinny_args &a)
 {
-    if (a.rows == 0 || a.rows > kRows || a.n == 0 || a.k == 0 || (a.x_ld & 3u) || (a.x_k & 7u) || a.x_k < a.k || a.x_ld < a.x_k)
-        return WR_CUDA_ERR_INVAL;
+    if (a.rows == 0 || a.rows > kRows || a.n == 0 || a.k == 0) return WR_CUDA_ERR_INVAL;
     SkinnyParams p;
     p.a = a;
     p.k_blocks = (a.k + kBK - 1) / kBK;
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
     const uint32_t tiles = (a.n + kM - 1) / kM;
-    // enough CTAs to draw the full bandwidth, while a slice still has a few blocks of K
+    // two CTAs per SM where a slice still has a few blocks of K
     p.split = 1;
-    while (p.split < 8 && tiles * p.split < 128 && p.k_blocks >= 8 * p.split) p.split *= 2;
-    const size_t smem = kStages * kStageBytes + (p.split - 1) * kRedFloats * 4 + 1024;
+    while (p.split < kMaxSplit && tiles * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
+    constexpr size_t smem = kStages * kStageBytes + 1024;
     if (!(ctx->attr_flags & 128u)) {
-        WR_CUDA_TRY(cudaFuncSetAttribute(gemm_skinny_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)(kStages * kStageBytes + 7 * kRedFloats * 4 + 1024)));
+        WR_CUDA_TRY(cudaFuncSetAttribute(gemm_skinny_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         ctx->attr_flags |= 128u;
     }
     cudaLaunchConfig_t cfg = {};
@@ -236,7 +205,7 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &w, const wr_skinny_arg
     attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = p.split > 1 ? 2 : 1;
-    WR_CUDA_TRY(cudaLaunchKernelEx(&cfg, gemm_skinny_kernel, w, p));
+    WR_CUDA_TRY(cudaLaunchKernelEx(&cfg, gemm_skinny_kernel, x, w, p));
     ctx->launches++;
     WR_CUDA_TRY(cudaGetLastError());
     return WR_CUDA_OK;

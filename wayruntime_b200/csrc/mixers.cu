@@ -87,6 +87,42 @@ __device__ __forceinline__ void store8v(__half *p, const float (&v)[8])
     *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
 }
 
+// Where a kernel leaves its rows: plain ones of type T, or (Split) F32 values as two BF16 numbers, the second
+// WR_CUDA_BATCH_MAX rows behind the first.
+struct Split {};
+template <typename T> struct Out {
+    T *p;
+    __device__ __forceinline__ Out(void *base, uint32_t row, uint32_t ld) : p(static_cast<T *>(base) + (size_t)row * ld) {}
+    __device__ __forceinline__ void put(uint32_t i, float v) const { p[i] = from_f32<T>(v); }
+    __device__ __forceinline__ void put4(uint32_t i, float4 v) const { store4(p + i, v); }
+    __device__ __forceinline__ void put8(uint32_t i, const float (&v)[8]) const { store8v(p + i, v); }
+};
+template <> struct Out<Split> {
+    __nv_bfloat16 *p;
+    size_t lo;
+    __device__ __forceinline__ Out(void *base, uint32_t row, uint32_t ld)
+        : p(static_cast<__nv_bfloat16 *>(base) + (size_t)row * ld), lo((size_t)WR_CUDA_BATCH_MAX * ld) {}
+    static __device__ __forceinline__ float rest(float v) { return v - __bfloat162float(__float2bfloat16_rn(v)); }
+    __device__ __forceinline__ void put(uint32_t i, float v) const
+    {
+        p[i] = __float2bfloat16_rn(v);
+        p[lo + i] = __float2bfloat16_rn(rest(v));
+    }
+    __device__ __forceinline__ void put4(uint32_t i, float4 v) const
+    {
+        store4(p + i, v);
+        store4(p + lo + i, make_float4(rest(v.x), rest(v.y), rest(v.z), rest(v.w)));
+    }
+    __device__ __forceinline__ void put8(uint32_t i, const float (&v)[8]) const
+    {
+        float r[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) r[e] = rest(v[e]);
+        store8v(p + i, v);
+        store8v(p + lo + i, r);
+    }
+};
+
 // the session of a row and the row's place among the session's tokens of this step
 __device__ __forceinline__ uint32_t seq_of(const wr_rows &rw, uint32_t row) { return rw.decode ? row : 0u; }
 __device__ __forceinline__ uint32_t tok_of(const wr_rows &rw, uint32_t row) { return rw.decode ? 0u : row; }
@@ -114,11 +150,11 @@ __global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint
 {
     pdl_trigger();
     pdl_wait();
-    const uint32_t row = blockIdx.x, ld = wr_ld(width);
+    const uint32_t row = blockIdx.y, ld = wr_ld(width);
     const uint32_t pos = rw.seqs[seq_of(rw, row)].pos + tok_of(rw, row);
     const TW *src = table + (size_t)tokens[row] * ld;
     float *dst = x + (size_t)row * ld;
-    for (uint32_t i = threadIdx.x; i < ld; i += blockDim.x) {
+    for (uint32_t i = blockIdx.x * 256 + threadIdx.x; i < ld; i += gridDim.x * 256) {
         float v = 0.f;
         if (i < width) {
             v = to_f32(src[i]);
@@ -169,11 +205,11 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows 
     pdl_wait();
     const uint32_t row = blockIdx.x, ld = wr_ld(a.width), gs = a.width / a.groups;
     const float *x = a.x + (size_t)(a.gather ? a.gather[row] : row) * ld;
-    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld;
+    const Out<TO> out(a.out, row, ld);
     group_inv_rms(x, a.groups, gs, split, a.eps, part, inv);
     if (!a.shift) {
         for (uint32_t i = threadIdx.x; i < ld; i += kNormThreads)
-            out[i] = from_f32<TO>(i < a.width ? x[i] * inv[i / gs] * a.w[i] : 0.f);
+            out.put(i, i < a.width ? x[i] * inv[i / gs] * a.w[i] : 0.f);
         return;
     }
     // the mixer reads h + (h' - h) * shift with h' the token before: this step's previous row (its norm is
@@ -194,7 +230,7 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows 
             y = h + (before - h) * a.shift[i];
             if (t + 1 == s.n) keep[i] = h;
         }
-        out[i] = from_f32<TO>(y);
+        out.put(i, y);
     }
 }
 
@@ -216,7 +252,7 @@ __global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows r
     }
     pdl_wait();
     const float *x = a.x + (size_t)(a.gather ? a.gather[row] : row) * ld + at, *xb = x - ld;
-    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld + at;
+    const Out<TO> out(a.out, row, ld);
     uint32_t t = 0, n = 0, fresh = 0;
     const float *kept = nullptr;
     float *keep = nullptr;
@@ -266,10 +302,9 @@ __global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows r
             h = make_float4(h.x + (p.x - h.x) * sh[i].x, h.y + (p.y - h.y) * sh[i].y, h.z + (p.z - h.z) * sh[i].z,
                             h.w + (p.w - h.w) * sh[i].w);
         }
-        store4(out + 128 * i, h);
+        out.put4(at + 128 * i, h);
     }
-    if (warp == NW - 1 && lane < ld - a.width)                   // pad columns
-        static_cast<TO *>(a.out)[(size_t)row * ld + a.width + lane] = from_f32<TO>(0.f);
+    if (warp == NW - 1 && lane < ld - a.width) out.put(a.width + lane, 0.f);                 // pad columns
 }
 
 template <typename TO, int NW> bool group_norm_reg(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a, cudaError_t &e)
@@ -284,11 +319,21 @@ template <typename TO, int NW> bool group_norm_reg(wr_cuda_ctx *ctx, const wr_ro
     return true;
 }
 
+template <typename TO> cudaError_t norm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a)
+{
+    // few rows: more warps on each (which kernel serves a row is a matter of the step's kind, not of its row count)
+    cudaError_t e = cudaSuccess;
+    if (rw.n_rows <= WR_CUDA_BATCH_MAX ? group_norm_reg<TO, 16>(ctx, rw, a, e) : group_norm_reg<TO, 8>(ctx, rw, a, e)) return e;
+    const uint32_t split = std::max(1u, kNormWarps / a.groups);
+    const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
+    return wr_launch_pdl(group_norm_kernel<TO>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split);
+}
+
 // -------------------------------------------------------------------- PolyNorm
 
 constexpr uint32_t kPolyThreads = 512, kPolyWarps = kPolyThreads / 32;
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(kPolyThreads) polynorm_kernel(const wr_polynorm_args a)
 {
     __shared__ float red[3][kPolyWarps];
@@ -296,7 +341,7 @@ __global__ void __launch_bounds__(kPolyThreads) polynorm_kernel(const wr_polynor
     pdl_wait();
     const uint32_t ld = wr_ld(a.ff), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const T *z = static_cast<const T *>(a.z) + (size_t)blockIdx.x * ld;
-    T *out = static_cast<T *>(a.out) + (size_t)blockIdx.x * ld;
+    const Out<TO> out(a.out, blockIdx.x, ld);
     float s1 = 0.f, s2 = 0.f, s3 = 0.f;
     for (uint32_t i = 8 * threadIdx.x; i < a.ff; i += 8 * kPolyThreads) {
         float v[8];
@@ -329,7 +374,7 @@ __global__ void __launch_bounds__(kPolyThreads) polynorm_kernel(const wr_polynor
         load8v(z + i, v);
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[e] = i + e < a.ff ? fmaf(v[e], fmaf(v[e], fmaf(v[e], kc, kb), ka), a.e) : 0.f;
-        store8v(out + i, v);
+        out.put8(i, v);
     }
 }
 
@@ -382,7 +427,9 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const wr_rows r
             for (uint32_t j = 0; j < taps; ++j)
                 step(acc, load4(a.w + (size_t)j * ld + c), input((int32_t)(t + j) - (int32_t)tail));
         }
-        store4(out + (size_t)t * ld, make_float4(siluf(acc.x), siluf(acc.y), siluf(acc.z), siluf(acc.w)));
+        acc = make_float4(siluf(acc.x), siluf(acc.y), siluf(acc.z), siluf(acc.w));
+        store4(out + (size_t)t * ld, acc);
+        if (a.out_split) Out<Split>(a.out_split, row0 + t, ld).put4(c, acc);
     }
     if (t1 == s.n) {                                                                     // the block with the last token
         float *keep = reinterpret_cast<float *>(s.st_out + a.state_off) + c;
@@ -418,24 +465,42 @@ template <int BYTES> __device__ __forceinline__ void cp_async(void *dst, const v
     asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
 }
 
-// NS: states a thread carries; LG: log2 of the threads that share a channel.  Four tokens go through the state
-// at a time; their partial sums are then exchanged so that each of the channel's threads finishes its own tokens.
-template <typename T, int NS, int LG>
+template <int NS> __device__ __forceinline__ void load_states(const float *p, float (&v)[NS])
+{
+    if constexpr (NS == 1) {
+        v[0] = *p;
+    } else if constexpr (NS == 2) {
+        const float2 f = *reinterpret_cast<const float2 *>(p);
+        v[0] = f.x;
+        v[1] = f.y;
+    } else {
+#pragma unroll
+        for (int j = 0; j < NS; j += 4) {
+            const float4 f = load4(p + j);
+            v[j] = f.x; v[j + 1] = f.y; v[j + 2] = f.z; v[j + 3] = f.w;
+        }
+    }
+}
+
+// NS: states a thread carries; LG: log2 of the threads that share a channel.  U tokens go through the state at a
+// time; their partial sums are then exchanged so that each of the channel's threads finishes tokens of its own.
+template <typename T, typename TO, int NS, int LG>
 __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, const wr_scan_args a)
 {
     constexpr uint32_t TPC = 1u << LG, CB = kScanThreads >> LG, HELD = NS * TPC;            // channels per block, states held
+    constexpr uint32_t BST = (HELD + 3) & ~3u;                                              // a token's B (or C) in shared memory
     constexpr uint32_t TILE = HELD > 128 ? 16 : 32;                                         // tokens per stage
-    constexpr int U = 4, KEEP = LG >= 2 ? 1 : U >> LG;                                      // tokens at a time; left per thread
+    constexpr int LU = LG < 2 ? 2 : LG > 4 ? 4 : LG, U = NS > 4 ? 4 : 1 << LU, KEEP = U > (int)TPC ? U / (int)TPC : 1;
     extern __shared__ __align__(16) uint8_t sm_scan[];
-    float *bs = reinterpret_cast<float *>(sm_scan), *cs = bs + 2 * TILE * HELD;             // [2][TILE][HELD]
-    float *dts = cs + 2 * TILE * HELD;                                                      // [2][TILE][CB]
-    T *xs = reinterpret_cast<T *>(dts + 2 * TILE * CB), *zs = xs + 2 * TILE * CB, *ys = zs + 2 * TILE * CB;
+    float *bs = reinterpret_cast<float *>(sm_scan), *cs = bs + 2 * TILE * BST;              // [2][TILE][BST]
+    float *dts = cs + 2 * TILE * BST, *ys = dts + 2 * TILE * CB;                            // [2][TILE][CB], [TILE][CB]
+    T *xs = reinterpret_cast<T *>(ys + TILE * CB), *zs = xs + 2 * TILE * CB;
     pdl_trigger();
     const uint32_t seq = blockIdx.y, tid = threadIdx.x;
     const uint32_t c_base = blockIdx.x * CB, cl = tid >> LG, part = tid & (TPC - 1), c = c_base + cl;
     const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state), bc4 = (a.state + 3) / 4;      // 4-value pieces per token
-    if (HELD > 4 * bc4)
-        for (uint32_t i = tid; i < 4 * TILE * HELD; i += kScanThreads) bs[i] = 0.f;         // (B and C beyond `state`)
+    if (BST > 4 * bc4)
+        for (uint32_t i = tid; i < 4 * TILE * BST; i += kScanThreads) bs[i] = 0.f;          // (B and C beyond `state`)
     float A2[NS], S[NS];
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
@@ -467,8 +532,8 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
         for (uint32_t i = tid; i < nt * bc4; i += kScanThreads) {
             const uint32_t t = i / bc4, q = i % bc4;
             const float *src = a.bc + (size_t)(row0 + t0 + t) * a.bc_ld + 4 * q;
-            cp_async<16>(bs + (st * TILE + t) * HELD + 4 * q, src + a.b_off);
-            cp_async<16>(cs + (st * TILE + t) * HELD + 4 * q, src + a.c_off);
+            cp_async<16>(bs + (st * TILE + t) * BST + 4 * q, src + a.b_off);
+            cp_async<16>(cs + (st * TILE + t) * BST + 4 * q, src + a.c_off);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -489,19 +554,14 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
             auto token = [&](int u) {
                 const uint32_t t = st * TILE + tb + u;
                 const float dt = dts[t * CB + cl], dx = dt * to_f32(xs[t * CB + cl]);
-                const float *b = bs + t * HELD + part * NS, *cc = cs + t * HELD + part * NS;
+                float b[NS], cc[NS];
+                load_states<NS>(bs + t * BST + part * NS, b);
+                load_states<NS>(cs + t * BST + part * NS, cc);
                 y[u] = 0.f;
 #pragma unroll
-                for (int j = 0; j < NS; j += 4) {
-                    const float4 b4 = load4(b + j), c4 = load4(cc + j);
-                    S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b4.x);
-                    S[j + 1] = fmaf(ex2(dt * A2[j + 1]), S[j + 1], dx * b4.y);
-                    S[j + 2] = fmaf(ex2(dt * A2[j + 2]), S[j + 2], dx * b4.z);
-                    S[j + 3] = fmaf(ex2(dt * A2[j + 3]), S[j + 3], dx * b4.w);
-                    y[u] = fmaf(S[j], c4.x, y[u]);
-                    y[u] = fmaf(S[j + 1], c4.y, y[u]);
-                    y[u] = fmaf(S[j + 2], c4.z, y[u]);
-                    y[u] = fmaf(S[j + 3], c4.w, y[u]);
+                for (int j = 0; j < NS; ++j) {
+                    S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b[j]);
+                    y[u] = fmaf(S[j], cc[j], y[u]);
                 }
             };
             if (tb + U <= nt) {
@@ -536,20 +596,16 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
 #pragma unroll
             for (int i = 0; i < KEEP; ++i) {
                 const uint32_t t = tb + first + i, at = (st * TILE + t) * CB + cl;
-                if (t < nt && part < 4) {
+                if (t < nt && part < (uint32_t)U) {
                     const float v = fmaf(D, to_f32(xs[at]), y[i]) * siluf(to_f32(zs[at]));
-                    ys[t * CB + cl] = from_f32<T>(c < a.inner ? v : 0.f);
+                    ys[t * CB + cl] = c < a.inner ? v : 0.f;
                 }
             }
         }
         __syncthreads();
         for (uint32_t i = tid; i < nt * (CB / 4); i += kScanThreads) {
             const uint32_t t = i / (CB / 4), q = i % (CB / 4), ch = c_base + 4 * q;
-            if (ch < ld) {
-                T *o = static_cast<T *>(a.out) + (size_t)(row0 + t0 + t) * ld + ch;
-                if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2 *>(o) = *reinterpret_cast<const uint2 *>(ys + t * CB + 4 * q);
-                else *reinterpret_cast<float4 *>(o) = *reinterpret_cast<const float4 *>(ys + t * CB + 4 * q);
-            }
+            if (ch < ld) Out<TO>(a.out, row0 + t0 + t, ld).put4(ch, load4(ys + t * CB + 4 * q));
         }
     }
     float *st_out = reinterpret_cast<float *>(s.st_out + a.state_off);
@@ -560,27 +616,32 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
     }
 }
 
-template <typename T, int NS, int LG> int scan_one(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+template <typename T, typename TO, int NS, int LG> int scan_one(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
-    constexpr uint32_t CB = kScanThreads >> LG, HELD = NS << LG, TILE = HELD > 128 ? 16 : 32;
-    constexpr size_t smem = (size_t)(4 * TILE * HELD + 2 * TILE * CB) * 4 + (size_t)5 * TILE * CB * sizeof(T);
-    auto k = scan_kernel<T, NS, LG>;
+    constexpr uint32_t CB = kScanThreads >> LG, HELD = NS << LG, BST = (HELD + 3) & ~3u, TILE = HELD > 128 ? 16 : 32;
+    constexpr size_t smem = (size_t)(4 * TILE * BST + 3 * TILE * CB) * 4 + (size_t)4 * TILE * CB * sizeof(T);
+    auto k = scan_kernel<T, TO, NS, LG>;
     if (smem > 48 * 1024)
         WR_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     WR_CUDA_TRY(wr_launch_pdl(k, dim3((wr_ld(a.inner) + CB - 1) / CB, rw.n_seq), dim3(kScanThreads), smem, ctx->stream, rw, a));
     return finish_launch(ctx);
 }
 
-template <typename T> int scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+// One state per thread while that is what it takes to fill the device, two above; a choice by the model's sizes
+// alone, so that a session's sums are added in one order whatever the step looks like.
+template <typename T, typename TO> int scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
-    if (a.state <= 4) return scan_one<T, 4, 0>(ctx, rw, a);
-    if (a.state <= 8) return scan_one<T, 4, 1>(ctx, rw, a);
-    if (a.state <= 16) return scan_one<T, 4, 2>(ctx, rw, a);
-    if (a.state <= 32) return scan_one<T, 4, 3>(ctx, rw, a);
-    if (a.state <= 64) return scan_one<T, 4, 4>(ctx, rw, a);
-    if (a.state <= 128) return scan_one<T, 4, 5>(ctx, rw, a);
-    if (a.state <= 256) return scan_one<T, 8, 5>(ctx, rw, a);
-    if (a.state <= 512) return scan_one<T, 16, 5>(ctx, rw, a);
+    const bool few = (uint64_t)a.inner * a.state < 131072;
+    if (a.state <= 1) return scan_one<T, TO, 1, 0>(ctx, rw, a);
+    if (a.state <= 2) return scan_one<T, TO, 1, 1>(ctx, rw, a);
+    if (a.state <= 4) return scan_one<T, TO, 1, 2>(ctx, rw, a);
+    if (a.state <= 8) return scan_one<T, TO, 1, 3>(ctx, rw, a);
+    if (a.state <= 16) return few ? scan_one<T, TO, 1, 4>(ctx, rw, a) : scan_one<T, TO, 2, 3>(ctx, rw, a);
+    if (a.state <= 32) return few ? scan_one<T, TO, 1, 5>(ctx, rw, a) : scan_one<T, TO, 2, 4>(ctx, rw, a);
+    if (a.state <= 64) return scan_one<T, TO, 2, 5>(ctx, rw, a);
+    if (a.state <= 128) return scan_one<T, TO, 4, 5>(ctx, rw, a);
+    if (a.state <= 256) return scan_one<T, TO, 8, 5>(ctx, rw, a);
+    if (a.state <= 512) return scan_one<T, TO, 16, 5>(ctx, rw, a);
     return WR_CUDA_ERR_LIMIT;
 }
 
@@ -657,7 +718,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const wr_rows rw, cons
     const wr_attn_geom g = a.g;
     const uint32_t row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, os = g.o_stride();
     const uint32_t n_out = g.n_q * g.vd, ld = wr_ld(n_out);
-    TO *out = static_cast<TO *>(a.out) + (size_t)row * ld;
+    const Out<TO> out(a.out, row, ld);
     for (uint32_t h = blockIdx.y * 8 + warp; h < g.n_q; h += gridDim.y * 8) {
         const float *o1 = a.o + ((size_t)row * g.vq() + h * g.maps) * os, *o2 = o1 + os;
         if (g.vd <= 128 && g.vd % 4 == 0) {                      // a lane's four values stay in registers
@@ -681,7 +742,7 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const wr_rows rw, cons
                 d = make_float4(d.x * k, d.y * k, d.z * k, d.w * k);
                 if (a.gate)
                     d = make_float4(d.x * sigmoidf(gt.x), d.y * sigmoidf(gt.y), d.z * sigmoidf(gt.z), d.w * sigmoidf(gt.w));
-                store4(out + h * g.vd + i, d);
+                out.put4(h * g.vd + i, d);
             }
             continue;
         }
@@ -698,10 +759,10 @@ __global__ void __launch_bounds__(256) attn_finish_kernel(const wr_rows rw, cons
             float v = g.maps == 2 ? fmaf(-a.lambda, o2[i], o1[i]) * k : o1[i];
             if (a.gate)
                 v *= sigmoidf(to_f32(static_cast<const TG *>(a.gate)[(size_t)row * a.gate_ld + h * g.vd + i]));
-            out[h * g.vd + i] = from_f32<TO>(v);
+            out.put(h * g.vd + i, v);
         }
     }
-    if (blockIdx.y == 0 && threadIdx.x < ld - n_out) out[n_out + threadIdx.x] = from_f32<TO>(0.f);
+    if (blockIdx.y == 0 && threadIdx.x < ld - n_out) out.put(n_out + threadIdx.x, 0.f);
 }
 
 // --------------------------------------------- attention over any cache layout
@@ -942,39 +1003,33 @@ template <int VC> int rows_any(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_att
 int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens, const void *table, int table_type,
                     const double *turns, float *x, uint32_t width)
 {
+    const dim3 grid((wr_ld(width) + 255) / 256, rw.n_rows);
     if (table_type == WR_ACT_BF16)
-        embed_kernel<__nv_bfloat16><<<rw.n_rows, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width);
+        embed_kernel<__nv_bfloat16><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width);
     else
-        embed_kernel<float><<<rw.n_rows, 256, 0, ctx->stream>>>(rw, tokens, (const float *)table, turns, x, width);
+        embed_kernel<float><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const float *)table, turns, x, width);
     return finish_launch(ctx);
 }
 
 int wr_group_norm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_norm_args &a)
 {
-    const bool bf = a.out_type == WR_ACT_BF16;
-    // few rows: more warps on each (which kernel serves a row is a matter of the step's kind, not of its row count)
     cudaError_t e = cudaSuccess;
-    const bool done = rw.n_rows <= WR_CUDA_BATCH_MAX
-                          ? (bf ? group_norm_reg<__nv_bfloat16, 16>(ctx, rw, a, e) : group_norm_reg<float, 16>(ctx, rw, a, e))
-                          : (bf ? group_norm_reg<__nv_bfloat16, 8>(ctx, rw, a, e) : group_norm_reg<float, 8>(ctx, rw, a, e));
-    if (!done) {
-        const uint32_t split = std::max(1u, kNormWarps / a.groups);
-        const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
-        if (smem > 48 * 1024) return WR_CUDA_ERR_LIMIT;
-        const dim3 grid(rw.n_rows), block(kNormThreads);
-        e = bf ? wr_launch_pdl(group_norm_kernel<__nv_bfloat16>, grid, block, smem, ctx->stream, rw, a, split)
-               : wr_launch_pdl(group_norm_kernel<float>, grid, block, smem, ctx->stream, rw, a, split);
-    }
+    if (a.out_type == WR_ACT_BF16) e = norm_launch<__nv_bfloat16>(ctx, rw, a);
+    else if (a.out_type == WR_ACT_SPLIT) e = norm_launch<Split>(ctx, rw, a);
+    else e = norm_launch<float>(ctx, rw, a);
     WR_CUDA_TRY(e);
     return finish_launch(ctx);
 }
 
 int wr_polynorm_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_polynorm_args &a)
 {
+    const dim3 grid(rw.n_rows), block(kPolyThreads);
     if (a.z_type == WR_ACT_BF16)
-        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<__nv_bfloat16>, dim3(rw.n_rows), dim3(kPolyThreads), 0, ctx->stream, a));
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, ctx->stream, a));
+    else if (a.out_type == WR_ACT_SPLIT)
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float, Split>, grid, block, 0, ctx->stream, a));
     else
-        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float>, dim3(rw.n_rows), dim3(kPolyThreads), 0, ctx->stream, a));
+        WR_CUDA_TRY(wr_launch_pdl(polynorm_kernel<float, float>, grid, block, 0, ctx->stream, a));
     return finish_launch(ctx);
 }
 
@@ -986,7 +1041,8 @@ int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args 
 
 int wr_scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
-    return a.type == WR_ACT_BF16 ? scan_launch<__nv_bfloat16>(ctx, rw, a) : scan_launch<float>(ctx, rw, a);
+    if (a.type == WR_ACT_BF16) return scan_launch<__nv_bfloat16, __nv_bfloat16>(ctx, rw, a);
+    return a.out_type == WR_ACT_SPLIT ? scan_launch<float, Split>(ctx, rw, a) : scan_launch<float, float>(ctx, rw, a);
 }
 
 int wr_attn_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_prep_args &a)
@@ -1027,6 +1083,8 @@ int wr_attn_finish_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_fin
     const dim3 grid(rw.n_rows, (a.g.n_q + 7) / 8), block(256);
     if (a.out_type == WR_ACT_BF16)
         WR_CUDA_TRY(wr_launch_pdl(attn_finish_kernel<__half, __nv_bfloat16>, grid, block, 0, ctx->stream, rw, a));
+    else if (a.out_type == WR_ACT_SPLIT)
+        WR_CUDA_TRY(wr_launch_pdl(attn_finish_kernel<float, Split>, grid, block, 0, ctx->stream, rw, a));
     else
         WR_CUDA_TRY(wr_launch_pdl(attn_finish_kernel<float, float>, grid, block, 0, ctx->stream, rw, a));
     return finish_launch(ctx);

@@ -20,7 +20,7 @@ struct wr_rows {
 };
 
 // element types of activation rows
-enum { WR_ACT_F32 = 0, WR_ACT_BF16 = 1, WR_ACT_F16 = 2 };
+enum { WR_ACT_F32 = 0, WR_ACT_BF16 = 1, WR_ACT_F16 = 2, WR_ACT_SPLIT = 3 };    // SPLIT: see gemm_bf16.cuh
 
 __host__ __device__ inline uint32_t wr_ld(uint32_t n) { return (n + 7u) & ~7u; }   // row stride of n values
 
@@ -54,6 +54,7 @@ struct wr_conv_args {
     const float *w, *b;              // [taps][wr_ld(inner)] (tap-major), [inner]
     uint64_t state_off;              // [taps-1][wr_ld(inner)] F32
     void *out;                       // [rows][wr_ld(inner)] of `type`
+    void *out_split;                 // the same as split rows too, or null (F32 only)
 };
 int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args &a);
 
@@ -67,7 +68,7 @@ struct wr_scan_args {
     const float *d;                  // [inner]
     uint32_t inner, state;
     uint64_t state_off;              // [inner][state] F32
-    void *out;                       // [rows][wr_ld(inner)] of `type`
+    void *out; int out_type;         // [rows][wr_ld(inner)]
 };
 int wr_scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a);
 

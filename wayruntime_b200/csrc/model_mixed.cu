@@ -1,10 +1,10 @@
 // model_mixed.cu — the layer stack of models whose layers differ (wr_cuda_model_create_mixed).
 //
 // The stack is a run list over layers; each layer is norm -> (token shift) -> mixer -> residual, then
-// norm -> feed-forward -> residual.  Steps of up to WR_CUDA_BATCH_MAX rows (every decode step, and short
-// portions of a prompt) go through the weight-streaming products of gemv.cu with F32 activations; longer
-// portions of a BF16 model go through the tensor-core product of gemm_bf16.cu with BF16 activations; an F32
-// model always uses the former.  The residual stream, norms, softmax and recurrences are F32 in both.
+// norm -> feed-forward -> residual.  An F32 model's projections are the products of gemv.cu.  A BF16 model's are
+// tensor-core products: steps of up to WR_CUDA_BATCH_MAX rows (every decode step, and short portions of a prompt)
+// keep F32 activations and take the weight-streaming one (gemm_skinny.cu), longer portions keep BF16 activations
+// and take gemm_bf16.cu.  The residual stream, norms, softmax and recurrences are F32 in all of them.
 //
 // A session (wr_cuda_kv) holds K/V pages for the attention runs and two slots of recurrent state; a step reads
 // the slot that stands at its first position and writes the other, so nothing a failed step does is kept.
@@ -33,7 +33,7 @@ struct Mat {                             // [n][k], rows wr_ld(k) apart, in the 
     const void *w = nullptr;
     uint32_t n = 0, k = 0;
     CUtensorMap map{};                   // BF16 models
-    CUtensorMap x_map{};                 // its input rows
+    CUtensorMap x_map{}, xs_map{};       // its input rows: BF16, and split
 };
 
 struct Layer {
@@ -79,6 +79,7 @@ struct wr_mixed {
     Mat head;
     // row scratch
     float *resid = nullptr, *dbc = nullptr, *dt = nullptr, *attn = nullptr, *logits = nullptr, *normed = nullptr;
+    float *conv_f32 = nullptr;           // few rows of a BF16 model: the convolution for the scan (mid has it split)
     void *xin = nullptr, *proj = nullptr, *mid = nullptr, *scan_out = nullptr, *q = nullptr, *dbc16 = nullptr, *head_in = nullptr;
     uint32_t *tokens = nullptr, *gather = nullptr, *best = nullptr, *part_i = nullptr;
     float *part_v = nullptr;
@@ -303,6 +304,7 @@ int fix_mat(Mat &m, const wr_mixed &x, const void *input, uint32_t input_rows, u
     if (x.compute != WR_CUDA_BF16) return WR_CUDA_OK;
     int rc = wr_gemm_map_weight(&m.map, m.w, m.n, m.k, wr_ld(m.k));
     if (rc == WR_CUDA_OK) rc = wr_gemm_map_rows(&m.x_map, input, input_rows, m.k, input_ld);
+    if (rc == WR_CUDA_OK) rc = wr_skinny_map_rows(&m.xs_map, input, m.k, input_ld);
     return rc;
 }
 
@@ -410,7 +412,8 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
     struct { void **p; size_t bytes; } want[] = {
         {(void **)&x->resid, R * x->ldw * 4}, {&x->xin, act(x->ldw)}, {&x->proj, act(proj)},
         {&x->mid, act(mid)}, {&x->scan_out, act(scan)}, {&x->q, std::max(R * q, few * q_few * 4)}, {(void **)&x->attn, R * att * 4},
-        {(void **)&x->dbc, R * dbc * 4}, {&x->dbc16, bf ? R * dbc * 2 : 0}, {(void **)&x->dt, R * scan * 4},
+        {(void **)&x->dbc, R * dbc * 4}, {&x->dbc16, bf ? std::max(R, 2 * few) * dbc * 2 : 0},
+        {(void **)&x->conv_f32, bf ? few * scan * 4 : 0}, {(void **)&x->dt, R * scan * 4},
         {&x->head_in, (size_t)kHeadRows * x->ldw * 4}, {(void **)&x->normed, (size_t)kHeadRows * x->ldw * 4},
         {(void **)&x->logits, (size_t)kHeadRows * ldv * 4}, {(void **)&x->tokens, R * 4}, {(void **)&x->gather, R * 4},
         {(void **)&x->best, few * 4}, {(void **)&x->part_v, few * WR_ARGMAX_PARTS * 4},
@@ -501,9 +504,11 @@ struct Step {
     bool wide;                           // BF16 tensor-core products (else weight-streaming ones on F32 rows)
     std::unique_lock<std::mutex> *lock;
 
-    int act() const { return wide ? WR_ACT_BF16 : WR_ACT_F32; }
+    bool split() const { return !wide && x->compute == WR_CUDA_BF16; }
+    int act() const { return wide ? WR_ACT_BF16 : WR_ACT_F32; }                              // a product's output rows
+    int in_act() const { return split() ? (int)WR_ACT_SPLIT : act(); }                       // a product's input rows
 
-    // out = act(mat . in + bias) + add; `in` is the buffer the matrix's row map was made for
+    // out = act(mat . in + bias) + add; `in` is the buffer the matrix's row maps were made for
     int product(const Mat &mat, const void *in, uint32_t in_ld, void *out, uint32_t out_ld, int out_type,
                 const float *bias = nullptr, bool softplus = false, const float *add = nullptr, void *copy16 = nullptr)
     {
@@ -522,13 +527,13 @@ struct Step {
         ++m->launches;
         if (x->compute == WR_CUDA_BF16) {
             wr_skinny_args a{};
-            a.x = static_cast<const float *>(in); a.x_ld = in_ld; a.x_k = wr_ld(mat.k);
             a.rows = rw.n_rows; a.n = mat.n; a.k = mat.k;
             a.out = static_cast<float *>(out); a.out_ld = out_ld;
+            a.out_split = copy16; a.out_split_ld = copy16 ? out_ld : 0;
             a.bias = bias;
             a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
             a.add = add; a.add_ld = out_ld;
-            return wr_skinny_launch(ctx, mat.map, a);
+            return wr_skinny_launch(ctx, mat.xs_map, mat.map, a);
         }
         GemvParams p{};
         p.seg[0] = {mat.w, static_cast<float *>(out), mat.n, out_ld};
@@ -549,7 +554,7 @@ struct Step {
         wr_norm_args a{};
         a.x = x->resid; a.w = w; a.shift = shift; a.state_off = state_off;
         a.width = x->width; a.groups = x->groups; a.eps = x->eps;
-        a.out = x->xin; a.out_type = act();
+        a.out = x->xin; a.out_type = in_act();
         ++m->launches;
         return wr_group_norm_launch(ctx, rw, a);
     }
@@ -588,7 +593,7 @@ struct Step {
         f.lambda = l.lambda; f.diff_init = l.diff_init; f.eps = l.diff_eps;
         f.gate = l.gated ? static_cast<const char *>(x->proj) + (size_t)l.g_off * (wide ? 2 : 4) : nullptr;
         f.gate_type = pt; f.gate_ld = l.proj_ld;
-        f.out = x->mid; f.out_type = act();
+        f.out = x->mid; f.out_type = in_act();
         ++m->launches;
         TRY(wr_attn_finish_launch(ctx, rw, f));
         return product(l.o, x->mid, wr_ld(l.o.k), x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
@@ -601,17 +606,19 @@ struct Step {
         wr_conv_args c{};
         c.x = x->proj; c.type = act(); c.x_ld = 2 * ldi; c.inner = l.inner; c.taps = l.taps;
         c.w = l.conv; c.b = l.conv_b; c.state_off = state_off + l.conv_off;
-        c.out = x->mid;
+        c.out = split() ? static_cast<void *>(x->conv_f32) : x->mid;
+        c.out_split = split() ? x->mid : nullptr;
         TRY(wr_conv_silu_launch(ctx, rw, c));
-        TRY(product(l.x, x->mid, ldi, x->dbc, l.dbc_ld, WR_ACT_F32, nullptr, false, nullptr, wide ? x->dbc16 : nullptr));
+        TRY(product(l.x, x->mid, ldi, x->dbc, l.dbc_ld, WR_ACT_F32, nullptr, false, nullptr,
+                    x->compute == WR_CUDA_BF16 ? x->dbc16 : nullptr));
         TRY(product(l.dt, x->dbc, l.dbc_ld, x->dt, ldi, WR_ACT_F32, l.dt_b, true));
         wr_scan_args s{};
-        s.x = x->mid; s.x_ld = ldi;
+        s.x = c.out; s.x_ld = ldi;
         s.z = static_cast<const char *>(x->proj) + (size_t)ldi * es; s.z_ld = 2 * ldi;
         s.type = act();
         s.dt = x->dt; s.bc = x->dbc; s.bc_ld = l.dbc_ld; s.b_off = l.b_off; s.c_off = l.c_off;
         s.a2 = l.a2; s.d = l.d; s.inner = l.inner; s.state = l.state; s.state_off = state_off + l.scan_off;
-        s.out = x->scan_out;
+        s.out = x->scan_out; s.out_type = in_act();
         TRY(wr_scan_launch(ctx, rw, s));
         m->launches += 2;
         return product(l.out, x->scan_out, ldi, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
@@ -622,7 +629,7 @@ struct Step {
         TRY(norm(l.norm2, nullptr, 0));
         TRY(product(l.up, x->xin, x->ldw, x->proj, wr_ld(l.ff), act()));
         wr_polynorm_args p{};
-        p.z = x->proj; p.z_type = act(); p.out = x->mid; p.out_type = act(); p.ff = l.ff;
+        p.z = x->proj; p.z_type = act(); p.out = x->mid; p.out_type = in_act(); p.ff = l.ff;
         p.a = l.act[0]; p.b = l.act[1]; p.c = l.act[2]; p.e = l.act[3]; p.eps = l.ffn_eps;
         ++m->launches;
         TRY(wr_polynorm_launch(ctx, rw, p));
@@ -726,7 +733,7 @@ int wr_mixed_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t n_ro
             wr_norm_args a{};
             a.x = x->resid; a.gather = x->gather + done; a.w = x->final_norm;
             a.width = x->width; a.groups = x->groups; a.eps = x->eps;
-            a.out = x->head_in; a.out_type = head.act();
+            a.out = x->head_in; a.out_type = head.in_act();
             if (logits_out || argmax_out) {
                 TRY(wr_group_norm_launch(ctx, head.rw, a));
                 TRY(head.product(x->head, x->head_in, x->ldw, x->logits, ldv, WR_ACT_F32));
