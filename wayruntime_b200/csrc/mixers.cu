@@ -8,6 +8,7 @@
 #include <cuda_bf16.h>
 
 #include <algorithm>
+#include <type_traits>
 
 #include "mixers.cuh"
 
@@ -154,18 +155,18 @@ __global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint
     const uint32_t pos = rw.seqs[seq_of(rw, row)].pos + tok_of(rw, row);
     const TW *src = table + (size_t)tokens[row] * ld;
     float *dst = x + (size_t)row * ld;
-    for (uint32_t i = blockIdx.x * 256 + threadIdx.x; i < ld; i += gridDim.x * 256) {
-        float v = 0.f;
-        if (i < width) {
-            v = to_f32(src[i]);
-            if (turns) {
-                // the angle in turns, reduced before it leaves double: a position of 2^20 keeps its phase
-                const double a = turns[i >> 1] * (double)pos;
-                const float half_turns = 2.0f * (float)(a - rint(a));
-                v += (i & 1u) ? cospif(half_turns) : sinpif(half_turns);
-            }
+    // a pair of columns shares its angle; ld is even
+    for (uint32_t i = 2 * (blockIdx.x * 256 + threadIdx.x); i < ld; i += 2 * gridDim.x * 256) {
+        float v0 = i < width ? to_f32(src[i]) : 0.f, v1 = i + 1 < width ? to_f32(src[i + 1]) : 0.f;
+        if (turns && i < width) {
+            // the angle in turns, reduced before it leaves double: a position of 2^20 keeps its phase
+            const double a = turns[i >> 1] * (double)pos;
+            float sn, cs;
+            sincospif(2.0f * (float)(a - rint(a)), &sn, &cs);
+            v0 += sn;
+            if (i + 1 < width) v1 += cs;
         }
-        dst[i] = v;
+        *reinterpret_cast<float2 *>(dst + i) = make_float2(v0, v1);
     }
 }
 
@@ -415,21 +416,31 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const wr_rows r
     float4 win[R];
 #pragma unroll
     for (int j = 1; j < TAPS; ++j) win[j] = input((int32_t)t0 + j - TAPS);
-    for (uint32_t t = t0; t < t1; ++t) {
-        float4 acc = bias;
+    for (uint32_t t = t0; t < t1; t += 4) {
+        float4 next[4];
         if constexpr (TAPS > 0) {
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
-            win[TAPS - 1] = load4(x + (size_t)t * a.x_ld);
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) step(acc, w[j], win[j]);
-        } else {
-            for (uint32_t j = 0; j < taps; ++j)
-                step(acc, load4(a.w + (size_t)j * ld + c), input((int32_t)(t + j) - (int32_t)tail));
+            for (int i = 0; i < 4; ++i)
+                if (t + i < t1) next[i] = load4(x + (size_t)(t + i) * a.x_ld);
         }
-        acc = make_float4(siluf(acc.x), siluf(acc.y), siluf(acc.z), siluf(acc.w));
-        store4(out + (size_t)t * ld, acc);
-        if (a.out_split) Out<Split>(a.out_split, row0 + t, ld).put4(c, acc);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            if (t + i >= t1) break;
+            float4 acc = bias;
+            if constexpr (TAPS > 0) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+                win[TAPS - 1] = next[i];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) step(acc, w[j], win[j]);
+            } else {
+                for (uint32_t j = 0; j < taps; ++j)
+                    step(acc, load4(a.w + (size_t)j * ld + c), input((int32_t)(t + i + j) - (int32_t)tail));
+            }
+            acc = make_float4(siluf(acc.x), siluf(acc.y), siluf(acc.z), siluf(acc.w));
+            store4(out + (size_t)(t + i) * ld, acc);
+            if (a.out_split) Out<Split>(a.out_split, row0 + t + i, ld).put4(c, acc);
+        }
     }
     if (t1 == s.n) {                                                                     // the block with the last token
         float *keep = reinterpret_cast<float *>(s.st_out + a.state_off) + c;
@@ -551,27 +562,46 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
 #pragma unroll 1
         for (uint32_t tb = 0; tb < nt; tb += U) {
             float y[U];
-            auto token = [&](int u) {
-                const uint32_t t = st * TILE + tb + u;
-                const float dt = dts[t * CB + cl], dx = dt * to_f32(xs[t * CB + cl]);
-                float b[NS], cc[NS];
-                load_states<NS>(bs + t * BST + part * NS, b);
-                load_states<NS>(cs + t * BST + part * NS, cc);
-                y[u] = 0.f;
+            // NT tokens from u0 on: everything they need first, then the decays, then the state's chain
+            auto tokens = [&](int u0, auto n_tokens) {
+                constexpr int NT = decltype(n_tokens)::value;
+                float dx[NT], b[NT][NS], cc[NT][NS], e[NT][NS];
 #pragma unroll
-                for (int j = 0; j < NS; ++j) {
-                    S[j] = fmaf(ex2(dt * A2[j]), S[j], dx * b[j]);
-                    y[u] = fmaf(S[j], cc[j], y[u]);
+                for (int i = 0; i < NT; ++i) {
+                    const uint32_t t = st * TILE + tb + u0 + i;
+                    const float dt = dts[t * CB + cl];
+                    dx[i] = dt * to_f32(xs[t * CB + cl]);
+                    load_states<NS>(bs + t * BST + part * NS, b[i]);
+                    load_states<NS>(cs + t * BST + part * NS, cc[i]);
+#pragma unroll
+                    for (int j = 0; j < NS; ++j) e[i][j] = dt * A2[j];
+                }
+#pragma unroll
+                for (int i = 0; i < NT; ++i)
+#pragma unroll
+                    for (int j = 0; j < NS; ++j) {
+                        e[i][j] = ex2(e[i][j]);
+                        b[i][j] *= dx[i];
+                    }
+#pragma unroll
+                for (int i = 0; i < NT; ++i) {
+                    y[u0 + i] = 0.f;
+#pragma unroll
+                    for (int j = 0; j < NS; ++j) {
+                        S[j] = fmaf(e[i][j], S[j], b[i][j]);
+                        y[u0 + i] = fmaf(S[j], cc[i][j], y[u0 + i]);
+                    }
                 }
             };
             if (tb + U <= nt) {
+                constexpr int NT = NS > 4 ? 1 : NS > 2 ? 4 : U < 8 ? U : 8;
 #pragma unroll
-                for (int u = 0; u < U; ++u) token(u);
+                for (int u = 0; u < U; u += NT) tokens(u, std::integral_constant<int, NT>());
             } else {
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
                     y[u] = 0.f;
-                    if (tb + u < nt) token(u);
+                    if (tb + u < nt) tokens(u, std::integral_constant<int, 1>());
                 }
             }
             uint32_t first = 0, width = U;                       // this thread keeps tokens [first, first + width)
@@ -1003,7 +1033,7 @@ template <int VC> int rows_any(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_att
 int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens, const void *table, int table_type,
                     const double *turns, float *x, uint32_t width)
 {
-    const dim3 grid((wr_ld(width) + 255) / 256, rw.n_rows);
+    const dim3 grid((wr_ld(width) + 511) / 512, rw.n_rows);
     if (table_type == WR_ACT_BF16)
         embed_kernel<__nv_bfloat16><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width);
     else
