@@ -24,8 +24,30 @@ template <> __device__ __forceinline__ __half from_f32<__half>(float v)
 {
     return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f));
 }
-__device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float siluf(float x) { return x / (1.0f + expf(-x)); }
+// (a few units in the last place: the exponential and the quotient are the short sequences)
+__device__ __forceinline__ float sigmoidf(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float siluf(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+
+// two F32 values in one 64-bit register: one issue slot for two elements
+__device__ __forceinline__ uint64_t pack2(float a, float b)
+{
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c)
+{
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b)
+{
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 
 // four / eight consecutive values (addresses aligned to the vector)
 __device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
@@ -476,22 +498,78 @@ template <int BYTES> __device__ __forceinline__ void cp_async(void *dst, const v
     asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
 }
 
-template <int NS> __device__ __forceinline__ void load_states(const float *p, float (&v)[NS])
-{
-    if constexpr (NS == 1) {
-        v[0] = *p;
-    } else if constexpr (NS == 2) {
-        const float2 f = *reinterpret_cast<const float2 *>(p);
-        v[0] = f.x;
-        v[1] = f.y;
-    } else {
+// The states of a thread: NS values, two to a register pair where there are two.
+template <int NS> struct States {
+    static constexpr int P = NS / 2;
+    uint64_t v[P];
+    __device__ __forceinline__ void load(const float *p)
+    {
+        if constexpr (NS == 2) {
+            v[0] = *reinterpret_cast<const uint64_t *>(p);
+        } else {
 #pragma unroll
-        for (int j = 0; j < NS; j += 4) {
-            const float4 f = load4(p + j);
-            v[j] = f.x; v[j + 1] = f.y; v[j + 2] = f.z; v[j + 3] = f.w;
+            for (int j = 0; j < P; j += 2) {
+                const ulonglong2 u = *reinterpret_cast<const ulonglong2 *>(p + 2 * j);
+                v[j] = u.x;
+                v[j + 1] = u.y;
+            }
         }
     }
-}
+    __device__ __forceinline__ void scale(float f)
+    {
+        const uint64_t ff = pack2(f, f);
+#pragma unroll
+        for (int j = 0; j < P; ++j) v[j] = mul2(v[j], ff);
+    }
+    // 2^(f * a)
+    __device__ __forceinline__ void decay(float f, const States &a)
+    {
+        const uint64_t ff = pack2(f, f);
+#pragma unroll
+        for (int j = 0; j < P; ++j) {
+            float x, y;
+            unpack2(mul2(a.v[j], ff), x, y);
+            v[j] = pack2(ex2(x), ex2(y));
+        }
+    }
+    // this = e * this + b
+    __device__ __forceinline__ void advance(const States &e, const States &b)
+    {
+#pragma unroll
+        for (int j = 0; j < P; ++j) v[j] = fma2(e.v[j], v[j], b.v[j]);
+    }
+    __device__ __forceinline__ float dot(const States &c) const
+    {
+        uint64_t t = mul2(v[0], c.v[0]);
+#pragma unroll
+        for (int j = 1; j < P; ++j) t = fma2(v[j], c.v[j], t);
+        float x, y;
+        unpack2(t, x, y);
+        return x + y;
+    }
+    __device__ __forceinline__ void set(int j, float f)
+    {
+        float x, y;
+        unpack2(v[j / 2], x, y);
+        v[j / 2] = j % 2 ? pack2(x, f) : pack2(f, y);
+    }
+    __device__ __forceinline__ float get(int j) const
+    {
+        float x, y;
+        unpack2(v[j / 2], x, y);
+        return j % 2 ? y : x;
+    }
+};
+template <> struct States<1> {
+    float v;
+    __device__ __forceinline__ void load(const float *p) { v = *p; }
+    __device__ __forceinline__ void scale(float f) { v *= f; }
+    __device__ __forceinline__ void decay(float f, const States &a) { v = ex2(f * a.v); }
+    __device__ __forceinline__ void advance(const States &e, const States &b) { v = fmaf(e.v, v, b.v); }
+    __device__ __forceinline__ float dot(const States &c) const { return v * c.v; }
+    __device__ __forceinline__ void set(int, float f) { v = f; }
+    __device__ __forceinline__ float get(int) const { return v; }
+};
 
 // NS: states a thread carries; LG: log2 of the threads that share a channel.  U tokens go through the state at a
 // time; their partial sums are then exchanged so that each of the channel's threads finishes tokens of its own.
@@ -512,11 +590,11 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
     const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state), bc4 = (a.state + 3) / 4;      // 4-value pieces per token
     if (BST > 4 * bc4)
         for (uint32_t i = tid; i < 4 * TILE * BST; i += kScanThreads) bs[i] = 0.f;          // (B and C beyond `state`)
-    float A2[NS], S[NS];
+    States<NS> A2, S;
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
         const uint32_t n = part * NS + j;
-        A2[j] = (c < a.inner && n < a.state) ? a.a2[(size_t)c * lds + n] : 0.f;
+        A2.set(j, (c < a.inner && n < a.state) ? a.a2[(size_t)c * lds + n] : 0.f);
     }
     const float D = c < a.inner ? a.d[c] : 0.f;
     pdl_wait();
@@ -526,7 +604,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
         const uint32_t n = part * NS + j;
-        S[j] = (!s.fresh && c < a.inner && n < a.state) ? st_in[(size_t)c * a.state + n] : 0.f;
+        S.set(j, (!s.fresh && c < a.inner && n < a.state) ? st_in[(size_t)c * a.state + n] : 0.f);
     }
     __syncthreads();
     auto request = [&](uint32_t tile) {
@@ -559,51 +637,27 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-#pragma unroll 1
-        for (uint32_t tb = 0; tb < nt; tb += U) {
-            float y[U];
-            // NT tokens from u0 on: everything they need first, then the decays, then the state's chain
-            auto tokens = [&](int u0, auto n_tokens) {
-                constexpr int NT = decltype(n_tokens)::value;
-                float dx[NT], b[NT][NS], cc[NT][NS], e[NT][NS];
+        // What NT tokens bring, worked out one group ahead of the state's chain: decays, dt x B, C
+        constexpr int NT = U / 2;
+        struct Group { States<NS> e[NT], b[NT], c[NT]; };
+        auto fetch = [&](Group &g, uint32_t t0, auto n_tokens) {
 #pragma unroll
-                for (int i = 0; i < NT; ++i) {
-                    const uint32_t t = st * TILE + tb + u0 + i;
-                    const float dt = dts[t * CB + cl];
-                    dx[i] = dt * to_f32(xs[t * CB + cl]);
-                    load_states<NS>(bs + t * BST + part * NS, b[i]);
-                    load_states<NS>(cs + t * BST + part * NS, cc[i]);
-#pragma unroll
-                    for (int j = 0; j < NS; ++j) e[i][j] = dt * A2[j];
-                }
-#pragma unroll
-                for (int i = 0; i < NT; ++i)
-#pragma unroll
-                    for (int j = 0; j < NS; ++j) {
-                        e[i][j] = ex2(e[i][j]);
-                        b[i][j] *= dx[i];
-                    }
-#pragma unroll
-                for (int i = 0; i < NT; ++i) {
-                    y[u0 + i] = 0.f;
-#pragma unroll
-                    for (int j = 0; j < NS; ++j) {
-                        S[j] = fmaf(e[i][j], S[j], b[i][j]);
-                        y[u0 + i] = fmaf(S[j], cc[i][j], y[u0 + i]);
-                    }
-                }
-            };
-            if (tb + U <= nt) {
-                constexpr int NT = NS > 4 ? 1 : NS > 2 ? 4 : U < 8 ? U : 8;
-#pragma unroll
-                for (int u = 0; u < U; u += NT) tokens(u, std::integral_constant<int, NT>());
-            } else {
-#pragma unroll
-                for (int u = 0; u < U; ++u) {
-                    y[u] = 0.f;
-                    if (tb + u < nt) tokens(u, std::integral_constant<int, 1>());
-                }
+            for (int i = 0; i < decltype(n_tokens)::value; ++i) {
+                const uint32_t t = st * TILE + t0 + i;
+                const float dt = dts[t * CB + cl], dx = dt * to_f32(xs[t * CB + cl]);
+                g.b[i].load(bs + t * BST + part * NS);
+                g.c[i].load(cs + t * BST + part * NS);
+                g.e[i].decay(dt, A2);
+                g.b[i].scale(dx);
             }
+        };
+        float y[U];
+        auto chain = [&](const Group &g, int i, int u) {
+            S.advance(g.e[i], g.b[i]);
+            y[u] = S.dot(g.c[i]);
+        };
+        // the channel's threads exchange their parts of U tokens' sums and finish some tokens each
+        auto finish = [&](uint32_t tb) {
             uint32_t first = 0, width = U;                       // this thread keeps tokens [first, first + width)
 #pragma unroll
             for (uint32_t o = 1; o < TPC; o <<= 1) {
@@ -631,6 +685,34 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
                     ys[t * CB + cl] = c < a.inner ? v : 0.f;
                 }
             }
+        };
+        Group ga, gb;
+        if (nt == TILE) {
+            using All = std::integral_constant<int, NT>;
+            fetch(ga, 0, All());
+#pragma unroll 1
+            for (uint32_t tb = 0; tb < TILE; tb += U) {
+                fetch(gb, tb + NT, All());
+#pragma unroll
+                for (int i = 0; i < NT; ++i) chain(ga, i, i);
+                if (tb + U < TILE) fetch(ga, tb + U, All());
+#pragma unroll
+                for (int i = 0; i < NT; ++i) chain(gb, i, NT + i);
+                finish(tb);
+            }
+        } else {
+#pragma unroll 1
+            for (uint32_t tb = 0; tb < nt; tb += U) {
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    y[u] = 0.f;
+                    if (tb + u < nt) {
+                        fetch(ga, tb + u, std::integral_constant<int, 1>());
+                        chain(ga, 0, u);
+                    }
+                }
+                finish(tb);
+            }
         }
         __syncthreads();
         for (uint32_t i = tid; i < nt * (CB / 4); i += kScanThreads) {
@@ -642,7 +724,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
         const uint32_t n = part * NS + j;
-        if (c < a.inner && n < a.state) st_out[(size_t)c * a.state + n] = S[j];
+        if (c < a.inner && n < a.state) st_out[(size_t)c * a.state + n] = S.get(j);
     }
 }
 
