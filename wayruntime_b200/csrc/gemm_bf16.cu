@@ -2,8 +2,8 @@
 //
 // Persistent CTAs (one per SM) walk output tiles of 128 rows x BN columns, m fastest so that the
 // tiles in flight share weight rows in L2.  Warp 0 feeds a ring of shared-memory stages with TMA
-// (64 K-values of both operands per stage, 128-byte swizzle; what lies beyond K, m or n arrives as
-// zeros), warp 1 issues tcgen05.mma into one of two TMEM accumulators, warps 2-5 read the other one
+// (64 K-values of both operands per stage: activations through a tensor map, weights as linear copies
+// of blocks stored in the operand's layout; what lies beyond K arrives as zeros), warp 1 issues tcgen05.mma into one of two TMEM accumulators, warps 2-5 read the other one
 // back and write the finished rows (bias, softplus, residual; F32, BF16 or saturated F16), so that a
 // tile's output overlaps the next tile's products.  Every wait is bounded by the context's wait
 // limit; a warp that gives up records an error word and all of them leave.
@@ -18,7 +18,6 @@ namespace {
 
 constexpr uint32_t kBM = 128, kBK = 64;
 constexpr uint32_t kThreads = 192;
-constexpr uint32_t kBoxRows = 64;                        // rows of one weight box
 constexpr uint32_t kABytes = kBM * kBK * 2;
 constexpr uint32_t kStageBudget = 196608;
 
@@ -31,6 +30,7 @@ template <uint32_t BN> struct Tile {
 
 struct GemmParams {
     wr_gemm_args a;
+    wr_weight w;
     uint32_t m_tiles, tiles, k_blocks;
     long long wait_limit;
     int *err;
@@ -51,7 +51,7 @@ __device__ __forceinline__ uint32_t pack_f16(float a, float b)
 
 template <uint32_t BN>
 __global__ void __launch_bounds__(kThreads, 1)
-gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, const GemmParams p)
+gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
 {
     using T = Tile<BN>;
     extern __shared__ uint8_t smem_raw[];
@@ -91,12 +91,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constan
                         break;
                     }
                     uint8_t *a = stages + st * (kABytes + T::kBBytes), *b = a + kABytes;
-                    mbar_expect_tx(&full[st], kABytes + T::kBBytes);
+                    const uint32_t nb0 = n0 / kWBlock, nb = min(BN / kWBlock, wr_weight_blocks(p.w.n) - nb0);
+                    mbar_expect_tx(&full[st], kABytes + nb * kWBlockBytes);
                     tc5::tma_load_2d(a, &x_map, (int)(kb * kBK), (int)m0, &full[st]);
-#pragma unroll
-                    for (uint32_t i = 0; i < BN / kBoxRows; ++i)
-                        tc5::tma_load_2d(b + i * kBoxRows * kBK * 2, &w_map, (int)(kb * kBK), (int)(n0 + i * kBoxRows),
-                                         &full[st]);
+                    const char *w = static_cast<const char *>(p.w.blocks) + ((size_t)nb0 * p.k_blocks + kb) * kWBlockBytes;
+                    for (uint32_t i = 0; i < nb; ++i)
+                        bulk_g2s(b + i * kWBlockBytes, w + (size_t)i * p.k_blocks * kWBlockBytes, kWBlockBytes, &full[st]);
                 }
             }
             if (!ok) atomicCAS(p.err, 0, 41);
@@ -147,7 +147,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constan
                 break;
             }
             tc5::fence_after();
-            const uint32_t n_pad = (p.a.n + 7u) & ~7u;
+            const uint32_t n_pad = (p.w.n + 7u) & ~7u;
 #pragma unroll 1
             for (uint32_t c0 = 0; c0 < BN && n0 + c0 < n_pad; c0 += 32) {
                 float v[32];
@@ -240,7 +240,7 @@ int map_2d(CUtensorMap *map, const void *base, uint32_t rows, uint32_t k, uint32
 }
 
 template <uint32_t BN>
-int launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_gemm_args &a)
+int launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_gemm_args &a)
 {
     constexpr uint32_t flag = BN == 256 ? 16u : BN == 128 ? 32u : 64u;
     if (!(ctx->attr_flags & flag)) {
@@ -250,13 +250,14 @@ int launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const w
     }
     GemmParams p;
     p.a = a;
+    p.w = w;
     p.m_tiles = (a.m + kBM - 1) / kBM;
-    p.tiles = p.m_tiles * ((a.n + BN - 1) / BN);
-    p.k_blocks = (a.k + kBK - 1) / kBK;
+    p.tiles = p.m_tiles * ((w.n + BN - 1) / BN);
+    p.k_blocks = wr_weight_blocks(w.k);
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
     const uint32_t grid = std::min<uint32_t>(p.tiles, (uint32_t)ctx->sm_count);
-    WR_CUDA_TRY(wr_launch_pdl(gemm_bf16_kernel<BN>, dim3(grid), dim3(kThreads), Tile<BN>::kSmem, ctx->stream, x, w, p));
+    WR_CUDA_TRY(wr_launch_pdl(gemm_bf16_kernel<BN>, dim3(grid), dim3(kThreads), Tile<BN>::kSmem, ctx->stream, x, p));
     ctx->launches++;
     WR_CUDA_TRY(cudaGetLastError());
     return WR_CUDA_OK;
@@ -264,10 +265,6 @@ int launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const w
 
 }  // namespace
 
-int wr_gemm_map_weight(CUtensorMap *map, const void *w, uint32_t n, uint32_t k, uint32_t ld)
-{
-    return map_2d(map, w, n, k, ld, kBoxRows);
-}
 int wr_gemm_map_rows(CUtensorMap *map, const void *x, uint32_t rows, uint32_t k, uint32_t ld)
 {
     return map_2d(map, x, rows, k, ld, kBM);
@@ -278,16 +275,16 @@ int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uin
     return map_2d(map, split_rows, 2 * WR_CUDA_BATCH_MAX, k, ld, 2 * WR_CUDA_BATCH_MAX);
 }
 
-int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_gemm_args &a)
+int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_gemm_args &a)
 {
-    if (a.m == 0 || a.n == 0 || a.k == 0 || (a.out_ld & 7u) || (a.out_bf16_ld & 7u) || (a.add_ld & 7u))
+    if (a.m == 0 || w.n == 0 || w.k == 0 || (a.out_ld & 7u) || (a.out_bf16_ld & 7u) || (a.add_ld & 7u))
         return WR_CUDA_ERR_INVAL;
     // the tile width that finishes first: rounds over the device times the width's share of the work
     const uint32_t m_tiles = (a.m + kBM - 1) / kBM;
     uint32_t best = 0;
     uint64_t best_cost = ~0ull;
     for (uint32_t bn : {256u, 128u, 64u}) {
-        const uint64_t tiles = (uint64_t)m_tiles * ((a.n + bn - 1) / bn);
+        const uint64_t tiles = (uint64_t)m_tiles * ((w.n + bn - 1) / bn);
         const uint64_t cost = ((tiles + ctx->sm_count - 1) / ctx->sm_count) * (bn + 48u);
         if (cost < best_cost) {
             best_cost = cost;

@@ -9,30 +9,48 @@ enum { WR_GEMM_OUT_F32 = 0, WR_GEMM_OUT_BF16 = 1, WR_GEMM_OUT_F16 = 2 };
 enum { WR_GEMM_ACT_NONE = 0, WR_GEMM_ACT_SOFTPLUS = 1 };
 
 struct wr_gemm_args {
-    uint32_t m, n, k;
-    void *out;             // [m][out_ld] of out_type; out_ld a multiple of 8, at least n
+    uint32_t m;
+    void *out;             // [m][out_ld] of out_type; out_ld a multiple of 8, at least w.n
     uint32_t out_ld, out_type;
     void *out_bf16;        // a second copy of the result in BF16 (before the residual), or null
     uint32_t out_bf16_ld;
-    const float *bias;     // [n rounded up to 8] or null
+    const float *bias;     // [w.n rounded up to 8] or null
     uint32_t act;          // WR_GEMM_ACT_* after the bias
     const float *add;      // [m][add_ld] residual added last (may alias an F32 out), or null
     uint32_t add_ld;
 };
 
-// Tensor maps of the operands: a weight [n][k] with rows ld elements apart, and activation rows [rows][k].
-// ld a multiple of 8, base 16-byte aligned.  WR_CUDA_ERR_INTERNAL when the driver refuses the map.
-int wr_gemm_map_weight(CUtensorMap *map, const void *w, uint32_t n, uint32_t k, uint32_t ld);
+// A BF16 weight [n][k] as the tensor core reads it: blocks of 64 rows x 64 K-values, each the 8 KB image of a
+// 128-byte-swizzled operand (row r at r * 128, its 16-byte piece c at c ^ (r & 7)), K-blocks of a row block one
+// after the other.  A block is one linear bulk copy, and a CTA's walk along K is one contiguous read.  Rows and
+// K-values beyond n and k are zeros.
+constexpr uint32_t kWBlock = 64, kWBlockBytes = kWBlock * kWBlock * 2;
+struct wr_weight {
+    const void *blocks;
+    uint32_t n, k;
+};
+__host__ __device__ inline uint32_t wr_weight_blocks(uint32_t n) { return (n + kWBlock - 1) / kWBlock; }
+inline size_t wr_weight_bytes(uint32_t n, uint32_t k) { return (size_t)wr_weight_blocks(n) * wr_weight_blocks(k) * kWBlockBytes; }
+// byte offset of element (r, i)
+inline size_t wr_weight_off(uint32_t k, uint32_t r, uint32_t i)
+{
+    const size_t block = (size_t)(r / kWBlock) * wr_weight_blocks(k) + i / kWBlock;
+    const uint32_t rr = r % kWBlock, ii = i % kWBlock;
+    return block * kWBlockBytes + rr * 128u + (((ii >> 3) ^ (rr & 7u)) << 4) + (ii & 7u) * 2u;
+}
+
+// Tensor map of activation rows [rows][k], ld elements apart (a multiple of 8; base 16-byte aligned).
+// WR_CUDA_ERR_INTERNAL when the driver refuses the map.
 int wr_gemm_map_rows(CUtensorMap *map, const void *x, uint32_t rows, uint32_t k, uint32_t ld);
 
 // Enqueue out[m][n] = act(x . w^T + bias) + add on the context's stream.
-int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_gemm_args &args);
+int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_gemm_args &args);
 
 // The same product for at most WR_CUDA_BATCH_MAX rows, weights streamed once.  The activation rows are "split": an
 // F32 value is kept as two BF16 numbers, its rounding in row r and what is left in row WR_CUDA_BATCH_MAX + r of one
 // buffer, so the product sees about 16 bits of it.  A row's bits do not depend on the other rows.  out F32.
 struct wr_skinny_args {
-    uint32_t rows, n, k;
+    uint32_t rows;
     float *out;            // [rows][out_ld]
     uint32_t out_ld;
     void *out_split;       // the result (before the residual) as split rows too, or null
@@ -43,4 +61,4 @@ struct wr_skinny_args {
     uint32_t add_ld;
 };
 int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld);
-int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_skinny_args &args);
+int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_skinny_args &args);

@@ -26,6 +26,7 @@ static_assert((kMaxSplit - 1) * kRedFloats * 4 <= kStages * kStageBytes, "the ot
 
 struct SkinnyParams {
     wr_skinny_args a;
+    wr_weight w;
     uint32_t k_blocks, split;
     long long wait_limit;
     int *err;
@@ -43,7 +44,7 @@ __device__ __forceinline__ void store_rank0(float *p, float v)
 }
 
 __global__ void __launch_bounds__(kThreads)
-gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, const SkinnyParams p)
+gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams p)
 {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t full[kStages], empty[kStages], acc_full;
@@ -71,12 +72,18 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_const
 
     if (warp == 0) {
         if (lane == 0) {
+            asm volatile("prefetch.tensormap [%0];" ::"l"(&x_map) : "memory");
+            // the row tile's one or two blocks of weights
+            const uint32_t nb = min(kM / kWBlock, wr_weight_blocks(p.w.n) - n0 / kWBlock);
+            const char *w = static_cast<const char *>(p.w.blocks) + ((size_t)(n0 / kWBlock) * p.k_blocks + kb0) * kWBlockBytes;
+            const uint64_t policy = l2_policy_evict_first();         // streamed once
             auto weights = [&](uint32_t it) {
                 const uint32_t st = it % kStages;
                 uint8_t *a = stages + st * kStageBytes;
-                mbar_expect_tx(&full[st], kStageBytes);
-                tc5::tma_load_2d(a, &w_map, (int)((kb0 + it) * kBK), (int)n0, &full[st]);
-                tc5::tma_load_2d(a + kABytes / 2, &w_map, (int)((kb0 + it) * kBK), (int)(n0 + kM / 2), &full[st]);
+                mbar_expect_tx(&full[st], nb * kWBlockBytes + kBBytes);
+                for (uint32_t i = 0; i < nb; ++i)
+                    bulk_g2s_hint(a + i * kWBlockBytes, w + ((size_t)i * p.k_blocks + it) * kWBlockBytes, kWBlockBytes, &full[st],
+                                  policy);
             };
             auto rows = [&](uint32_t it) {
                 const uint32_t st = it % kStages;
@@ -146,7 +153,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_const
         cluster_arrive();
         cluster_wait();
     }
-    if (warp >= 2 && rank == 0 && n0 + m < p.a.n) {
+    if (warp >= 2 && rank == 0 && n0 + m < p.w.n) {
         const float bias = p.a.bias ? p.a.bias[n0 + m] : 0.f;
 #pragma unroll
         for (uint32_t i = 0; i < kRows; ++i) {
@@ -174,15 +181,16 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_const
 
 }  // namespace
 
-int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &w, const wr_skinny_args &a)
+int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_skinny_args &a)
 {
-    if (a.rows == 0 || a.rows > kRows || a.n == 0 || a.k == 0) return WR_CUDA_ERR_INVAL;
+    if (a.rows == 0 || a.rows > kRows || w.n == 0 || w.k == 0) return WR_CUDA_ERR_INVAL;
     SkinnyParams p;
     p.a = a;
-    p.k_blocks = (a.k + kBK - 1) / kBK;
+    p.w = w;
+    p.k_blocks = wr_weight_blocks(w.k);
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
-    const uint32_t tiles = (a.n + kM - 1) / kM;
+    const uint32_t tiles = (w.n + kM - 1) / kM;
     // two CTAs per SM where a slice still has a few blocks of K
     p.split = 1;
     while (p.split < kMaxSplit && tiles * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
@@ -205,7 +213,7 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const CUtensorMap &
     attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = p.split > 1 ? 2 : 1;
-    WR_CUDA_TRY(cudaLaunchKernelEx(&cfg, gemm_skinny_kernel, x, w, p));
+    WR_CUDA_TRY(cudaLaunchKernelEx(&cfg, gemm_skinny_kernel, x, p));
     ctx->launches++;
     WR_CUDA_TRY(cudaGetLastError());
     return WR_CUDA_OK;

@@ -728,6 +728,82 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const wr_rows rw, co
     }
 }
 
+// One token per session (a decode step): four states per thread straight from memory, nothing staged.
+constexpr uint32_t kStepThreads = 256;
+
+template <typename TO, int LG>
+__global__ void __launch_bounds__(kStepThreads) scan_step_kernel(const wr_rows rw, const wr_scan_args a)
+{
+    constexpr uint32_t TPC = 1u << LG;
+    pdl_trigger();
+    const uint32_t seq = blockIdx.y, part = threadIdx.x & (TPC - 1), c = (blockIdx.x * kStepThreads + threadIdx.x) >> LG;
+    const uint32_t ld = wr_ld(a.inner), lds = wr_ld(a.state);
+    const bool in = c < a.inner;
+    float4 a2 = make_float4(0.f, 0.f, 0.f, 0.f);
+    const uint32_t n0 = 4 * part;
+    if (in && n0 < lds) a2 = load4(a.a2 + (size_t)c * lds + n0);
+    const float D = in ? a.d[c] : 0.f;
+    pdl_wait();
+    const wr_seq_dev s = rw.seqs[seq];
+    float y = 0.f, x = 0.f, z = 0.f;
+    if (in) {
+        const float *from = reinterpret_cast<const float *>(s.st_in + a.state_off) + (size_t)c * a.state + n0;
+        float *to = reinterpret_cast<float *>(s.st_out + a.state_off) + (size_t)c * a.state + n0;
+        const float *bc = a.bc + (size_t)seq * a.bc_ld + n0;
+        x = static_cast<const float *>(a.x)[(size_t)seq * a.x_ld + c];
+        z = static_cast<const float *>(a.z)[(size_t)seq * a.z_ld + c];
+        const float dt = a.dt[(size_t)seq * ld + c], dx = dt * x;
+        const uint32_t left = n0 < a.state ? a.state - n0 : 0u;
+        float S[4] = {0.f, 0.f, 0.f, 0.f};
+        if (!s.fresh) {
+            if (left >= 4 && a.state % 4 == 0) {
+                const float4 v = load4(from);
+                S[0] = v.x; S[1] = v.y; S[2] = v.z; S[3] = v.w;
+            } else {
+#pragma unroll
+                for (uint32_t j = 0; j < 4; ++j)
+                    if (j < left) S[j] = from[j];
+            }
+        }
+        float4 b = make_float4(0.f, 0.f, 0.f, 0.f), cc = b;
+        if (left) {
+            b = load4(bc + a.b_off);
+            cc = load4(bc + a.c_off);
+        }
+        S[0] = fmaf(ex2(dt * a2.x), S[0], dx * b.x);
+        S[1] = fmaf(ex2(dt * a2.y), S[1], dx * b.y);
+        S[2] = fmaf(ex2(dt * a2.z), S[2], dx * b.z);
+        S[3] = fmaf(ex2(dt * a2.w), S[3], dx * b.w);
+        y = fmaf(S[3], cc.w, fmaf(S[2], cc.z, fmaf(S[1], cc.y, S[0] * cc.x)));
+        if (left >= 4 && a.state % 4 == 0) {
+            store4(to, make_float4(S[0], S[1], S[2], S[3]));
+        } else {
+#pragma unroll
+            for (uint32_t j = 0; j < 4; ++j)
+                if (j < left) to[j] = S[j];
+        }
+    }
+#pragma unroll
+    for (uint32_t o = TPC >> 1; o >= 1; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (part == 0 && c < ld) Out<TO>(a.out, seq, ld).put(c, in ? fmaf(D, x, y) * siluf(z) : 0.f);
+}
+
+template <typename TO, int LG> int scan_step_one(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+{
+    const dim3 grid(((wr_ld(a.inner) << LG) + kStepThreads - 1) / kStepThreads, rw.n_seq);
+    WR_CUDA_TRY(wr_launch_pdl(scan_step_kernel<TO, LG>, grid, dim3(kStepThreads), 0, ctx->stream, rw, a));
+    return finish_launch(ctx);
+}
+template <typename TO> int scan_step(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
+{
+    if (a.state <= 4) return scan_step_one<TO, 0>(ctx, rw, a);
+    if (a.state <= 8) return scan_step_one<TO, 1>(ctx, rw, a);
+    if (a.state <= 16) return scan_step_one<TO, 2>(ctx, rw, a);
+    if (a.state <= 32) return scan_step_one<TO, 3>(ctx, rw, a);
+    if (a.state <= 64) return scan_step_one<TO, 4>(ctx, rw, a);
+    return scan_step_one<TO, 5>(ctx, rw, a);                     // (128 states at most)
+}
+
 template <typename T, typename TO, int NS, int LG> int scan_one(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
     constexpr uint32_t CB = kScanThreads >> LG, HELD = NS << LG, BST = (HELD + 3) & ~3u, TILE = HELD > 128 ? 16 : 32;
@@ -1153,6 +1229,8 @@ int wr_conv_silu_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_conv_args 
 
 int wr_scan_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_scan_args &a)
 {
+    if (rw.decode && a.type == WR_ACT_F32 && a.state <= 128)
+        return a.out_type == WR_ACT_SPLIT ? scan_step<Split>(ctx, rw, a) : scan_step<float>(ctx, rw, a);
     if (a.type == WR_ACT_BF16) return scan_launch<__nv_bfloat16, __nv_bfloat16>(ctx, rw, a);
     return a.out_type == WR_ACT_SPLIT ? scan_launch<float, Split>(ctx, rw, a) : scan_launch<float, float>(ctx, rw, a);
 }

@@ -29,11 +29,10 @@ constexpr double kLog2e = 1.4426950408889634;
 
 size_t up256(size_t n) { return (n + 255u) & ~(size_t)255u; }
 
-struct Mat {                             // [n][k], rows wr_ld(k) apart, in the model's weight type
+struct Mat {                             // [n][k]: F32 rows wr_ld(k) apart, or BF16 blocks (wr_weight)
     const void *w = nullptr;
     uint32_t n = 0, k = 0;
-    CUtensorMap map{};                   // BF16 models
-    CUtensorMap x_map{}, xs_map{};       // its input rows: BF16, and split
+    CUtensorMap x_map{}, xs_map{};       // BF16 models: its input rows, and its input as split rows
 };
 
 struct Layer {
@@ -140,8 +139,8 @@ struct Packer {
         for (size_t i = 0; i < n; ++i) f(o)[i] = elem(t, i);
         return o;
     }
-    // [rows][k] out of parts, rows wr_ld(k) apart, in `type`; zeros elsewhere
-    size_t mat(std::initializer_list<Part> parts, uint32_t rows, uint32_t k, int type)
+    // [rows][k] out of parts, zeros elsewhere: rows wr_ld(k) apart in `type` ...
+    size_t rows_of(std::initializer_list<Part> parts, uint32_t rows, uint32_t k, int type)
     {
         const size_t ld = wr_ld(k), es = type == WR_CUDA_BF16 ? 2 : 4;
         const size_t o = place(((size_t)rows * ld) * es);
@@ -149,15 +148,34 @@ struct Packer {
             for (uint32_t r = 0; r < p.n; ++r) {
                 uint8_t *dst = buf.data() + o + (size_t)(p.at + r) * ld * es;
                 const size_t src = (size_t)(p.row0 + r) * k;
-                if (type == WR_CUDA_BF16 && p.t->dtype == WR_CUDA_BF16) {
-                    memcpy(dst, static_cast<const uint16_t *>(p.t->data) + src, (size_t)k * 2);
-                } else if (type == WR_CUDA_BF16) {
-                    for (uint32_t i = 0; i < k; ++i) reinterpret_cast<uint16_t *>(dst)[i] = f32_to_bf16(elem(*p.t, src + i));
-                } else {
-                    for (uint32_t i = 0; i < k; ++i) reinterpret_cast<float *>(dst)[i] = elem(*p.t, src + i);
+                for (uint32_t i = 0; i < k; ++i) {
+                    if (type == WR_CUDA_BF16) reinterpret_cast<uint16_t *>(dst)[i] = bits(*p.t, src + i);
+                    else reinterpret_cast<float *>(dst)[i] = elem(*p.t, src + i);
                 }
             }
         return o;
+    }
+    // ... or, for the products of a BF16 model, in blocks (wr_weight)
+    size_t mat(std::initializer_list<Part> parts, uint32_t rows, uint32_t k, int type)
+    {
+        if (type != WR_CUDA_BF16) return rows_of(parts, rows, k, type);
+        const size_t o = place(wr_weight_bytes(rows, k));
+        for (const Part &p : parts)
+            for (uint32_t r = 0; r < p.n; ++r) {
+                const size_t src = (size_t)(p.row0 + r) * k;
+                for (uint32_t i = 0; i < k; i += 8) {            // pieces of eight stay together
+                    uint16_t *dst = reinterpret_cast<uint16_t *>(buf.data() + o + wr_weight_off(k, p.at + r, i));
+                    const uint32_t n = std::min(8u, k - i);
+                    if (p.t->dtype == WR_CUDA_BF16) memcpy(dst, static_cast<const uint16_t *>(p.t->data) + src + i, n * 2);
+                    else
+                        for (uint32_t e = 0; e < n; ++e) dst[e] = f32_to_bf16(elem(*p.t, src + i + e));
+                }
+            }
+        return o;
+    }
+    static uint16_t bits(const wr_cuda_tensor &t, size_t i)
+    {
+        return t.dtype == WR_CUDA_BF16 ? static_cast<const uint16_t *>(t.data)[i] : f32_to_bf16(elem(t, i));
     }
 };
 
@@ -302,8 +320,7 @@ int fix_mat(Mat &m, const wr_mixed &x, const void *input, uint32_t input_rows, u
     if (!m.w) return WR_CUDA_OK;
     fix(m.w, x.weights);
     if (x.compute != WR_CUDA_BF16) return WR_CUDA_OK;
-    int rc = wr_gemm_map_weight(&m.map, m.w, m.n, m.k, wr_ld(m.k));
-    if (rc == WR_CUDA_OK) rc = wr_gemm_map_rows(&m.x_map, input, input_rows, m.k, input_ld);
+    int rc = wr_gemm_map_rows(&m.x_map, input, input_rows, m.k, input_ld);
     if (rc == WR_CUDA_OK) rc = wr_skinny_map_rows(&m.xs_map, input, m.k, input_ld);
     return rc;
 }
@@ -362,7 +379,7 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
     x->runs.assign(d->runs, d->runs + d->n_runs);
 
     Packer pk;
-    set_off(x->embed, pk.mat({{&d->embed, 0, d->vocab, 0}}, d->vocab, d->width, type));
+    set_off(x->embed, pk.rows_of({{&d->embed, 0, d->vocab, 0}}, d->vocab, d->width, type));
     x->head.n = d->vocab;
     x->head.k = d->width;
     set_off(x->head.w, pk.mat({{&d->head, 0, d->vocab, 0}}, d->vocab, d->width, type));
@@ -514,7 +531,7 @@ struct Step {
     {
         if (wide) {
             wr_gemm_args a{};
-            a.m = rw.n_rows; a.n = mat.n; a.k = mat.k;
+            a.m = rw.n_rows;
             a.out = out; a.out_ld = out_ld;
             a.out_type = out_type == WR_ACT_F32 ? WR_GEMM_OUT_F32 : out_type == WR_ACT_BF16 ? WR_GEMM_OUT_BF16 : WR_GEMM_OUT_F16;
             a.out_bf16 = copy16; a.out_bf16_ld = copy16 ? out_ld : 0;
@@ -522,18 +539,18 @@ struct Step {
             a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
             a.add = add; a.add_ld = add ? out_ld : 0;
             ++m->launches;
-            return wr_gemm_launch(ctx, mat.x_map, mat.map, a);
+            return wr_gemm_launch(ctx, mat.x_map, {mat.w, mat.n, mat.k}, a);
         }
         ++m->launches;
         if (x->compute == WR_CUDA_BF16) {
             wr_skinny_args a{};
-            a.rows = rw.n_rows; a.n = mat.n; a.k = mat.k;
+            a.rows = rw.n_rows;
             a.out = static_cast<float *>(out); a.out_ld = out_ld;
             a.out_split = copy16; a.out_split_ld = copy16 ? out_ld : 0;
             a.bias = bias;
             a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
             a.add = add; a.add_ld = out_ld;
-            return wr_skinny_launch(ctx, mat.xs_map, mat.map, a);
+            return wr_skinny_launch(ctx, mat.xs_map, {mat.w, mat.n, mat.k}, a);
         }
         GemvParams p{};
         p.seg[0] = {mat.w, static_cast<float *>(out), mat.n, out_ld};
