@@ -3,7 +3,7 @@
 // HBM-bound: the weights are all the traffic.  The operands are swapped — 128 weight rows are the tensor core's M,
 // the activation rows its N, each F32 activation as two BF16 numbers in two columns (split rows, see
 // gemm_bf16.cuh).  A CTA owns 128 weight rows and a slice of K; the CTAs of a cluster share the rows and add their
-// slices through distributed shared memory in rank order.  Warp 0 streams both operands with TMA — the weights
+// slices up, in rank order, out of each other's shared memory.  Warp 0 streams both operands with TMA — the weights
 // depend on nothing, so their first stages are requested before the kernel ahead has finished —, warp 1 issues
 // tcgen05.mma, warps 2-5 finish the rows.  All columns are always computed: a row's result does not depend on how
 // many rows share the step.
@@ -19,10 +19,9 @@ namespace {
 constexpr uint32_t kRows = WR_CUDA_BATCH_MAX, kM = 128, kN = 2 * kRows, kBK = 64;
 constexpr uint32_t kThreads = 192, kStages = 5;
 constexpr uint32_t kABytes = kM * kBK * 2, kBBytes = kN * kBK * 2, kStageBytes = kABytes + kBBytes;
-constexpr uint32_t kRedFloats = kRows * kM;              // one rank's sums
 constexpr uint32_t kMaxSplit = 8;
 constexpr uint32_t kTmemCols = 32;
-static_assert((kMaxSplit - 1) * kRedFloats * 4 <= kStages * kStageBytes, "the other ranks' sums fit where the stages were");
+static_assert(kRows * kM * 4 <= kStages * kStageBytes, "a CTA's sums fit where its stages were");
 
 struct SkinnyParams {
     wr_skinny_args a;
@@ -36,11 +35,29 @@ __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log
 
 __device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
 __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ void store_rank0(float *p, float v)
+__device__ __forceinline__ float load_rank(const float *p, uint32_t rank)
 {
     uint32_t remote;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(remote) : "r"(smem_u32(p)));
-    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(smem_u32(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote) : "memory");
+    return v;
+}
+
+// bias, activation, copies and residual of one finished sum: activation row i, weight row n
+__device__ __forceinline__ void put(const SkinnyParams &p, uint32_t i, uint32_t n, float y)
+{
+    if (n >= p.w.n) return;
+    if (p.a.bias) y += p.a.bias[n];
+    if (p.a.act == WR_GEMM_ACT_SOFTPLUS) y = softplus(y);
+    if (p.a.out_split) {
+        __nv_bfloat16 *o = static_cast<__nv_bfloat16 *>(p.a.out_split) + (size_t)i * p.a.out_split_ld + n;
+        const __nv_bfloat16 hi = __float2bfloat16_rn(y);
+        o[0] = hi;
+        o[(size_t)kRows * p.a.out_split_ld] = __float2bfloat16_rn(y - __bfloat162float(hi));
+    }
+    if (p.a.add) y += p.a.add[(size_t)i * p.a.add_ld + n];
+    p.a.out[(size_t)i * p.a.out_ld + n] = y;
 }
 
 __global__ void __launch_bounds__(kThreads)
@@ -50,7 +67,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
     __shared__ __align__(8) uint64_t full[kStages], empty[kStages], acc_full;
     __shared__ uint32_t tmem_slot;
     uint8_t *stages = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023u) & ~(uintptr_t)1023u);
-    float *red = reinterpret_cast<float *>(stages);      // [rank - 1][row][128], once the products are done
+    float *red = reinterpret_cast<float *>(stages);      // [row][128], once the products are done
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = blockIdx.x % p.split, n0 = (blockIdx.x / p.split) * kM;
     const uint32_t kb0 = p.k_blocks * rank / p.split, kb1 = p.k_blocks * (rank + 1) / p.split, nkb = kb1 - kb0;
@@ -142,36 +159,37 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
         for (uint32_t i = 0; i < kRows; ++i) s[i] = v[i] + v[kRows + i];
     }
     const uint32_t m = (warp & 3) * 32 + lane;           // (finishing warps)
-    if (p.split > 1) {
-        cluster_arrive();                                // every rank's products are done: its stages are free
-        cluster_wait();
-        if (warp >= 2 && rank > 0) {
+    if (p.split == 1) {
+        if (warp >= 2) {
 #pragma unroll
             for (uint32_t i = 0; i < kRows; ++i)
-                if (i < p.a.rows) store_rank0(red + (rank - 1) * kRedFloats + i * kM + m, s[i]);
+                if (i < p.a.rows) put(p, i, n0 + m, s[i]);
+        }
+    } else {
+        // every rank lays its sums out in its own shared memory (its products are done with it) and finishes its
+        // share of the weight rows from all of them
+        if (warp >= 2) {
+#pragma unroll
+            for (uint32_t i = 0; i < kRows; ++i)
+                if (i < p.a.rows) red[i * kM + m] = s[i];
         }
         cluster_arrive();
         cluster_wait();
-    }
-    if (warp >= 2 && rank == 0 && n0 + m < p.w.n) {
-        const float bias = p.a.bias ? p.a.bias[n0 + m] : 0.f;
+        if (warp >= 2) {
+            const uint32_t share = kM / p.split;
+            for (uint32_t j = threadIdx.x - 64; j < p.a.rows * share; j += kThreads - 64) {
+                const uint32_t i = j / share, mm = rank * share + j % share;
+                float v[kMaxSplit];
 #pragma unroll
-        for (uint32_t i = 0; i < kRows; ++i) {
-            if (i < p.a.rows) {
-                float y = s[i];
-                for (uint32_t q = 1; q < p.split; ++q) y += red[(q - 1) * kRedFloats + i * kM + m];
-                y += bias;
-                if (p.a.act == WR_GEMM_ACT_SOFTPLUS) y = softplus(y);
-                if (p.a.out_split) {
-                    __nv_bfloat16 *o = static_cast<__nv_bfloat16 *>(p.a.out_split) + (size_t)i * p.a.out_split_ld + n0 + m;
-                    const __nv_bfloat16 hi = __float2bfloat16_rn(y);
-                    o[0] = hi;
-                    o[(size_t)kRows * p.a.out_split_ld] = __float2bfloat16_rn(y - __bfloat162float(hi));
-                }
-                if (p.a.add) y += p.a.add[(size_t)i * p.a.add_ld + n0 + m];
-                p.a.out[(size_t)i * p.a.out_ld + n0 + m] = y;
+                for (uint32_t q = 0; q < kMaxSplit; ++q) v[q] = q < p.split ? load_rank(red + i * kM + mm, q) : 0.f;
+                float y = v[0];
+#pragma unroll
+                for (uint32_t q = 1; q < kMaxSplit; ++q) y += v[q];      // (+0 beyond the last rank)
+                put(p, i, n0 + mm, y);
             }
         }
+        cluster_arrive();                                // nobody leaves while its sums are being read
+        cluster_wait();
     }
     tc5::fence_before();
     __syncthreads();
