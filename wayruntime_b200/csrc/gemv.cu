@@ -1,9 +1,7 @@
-// gemv.cu — y[r][n] = sum_k W[n][k] x[r][k] for a few activation rows: weights stream from HBM once.
+// gemv.cu — y[r][n] = sum_k W[n][k] x[r][k] in F32 for a few activation rows: weights stream from HBM once.
 //
-// Serves every projection of the F32 layer stack (src/core/kernels.c:978-1090: GGML-layout
-// W[out][in]) and the rows of a decode step of the mixed stack, whose weights may be BF16.
-// Activations and sums are F32 with either weight type.
-#include <cuda_bf16.h>
+// Serves every projection of the F32 layer stack (src/core/kernels.c:978-1090: GGML-layout W[out][in]) and those
+// of the mixed stack's F32 models.
 #include <math.h>
 
 #include "gemv.cuh"
@@ -70,7 +68,7 @@ __device__ __forceinline__ bool reduce_writer(int lane)
 // y[r][n] = sum_k W[n][k] * x[r][k], optionally with RMSNorm fused on x, and a
 // residual add or SiLU(gate)*up on the way out.  Two kernels, one arithmetic:
 // K is cut into four quarters; inside a quarter lane l takes the 16-byte
-// weight vectors (4 F32 or 8 BF16 values) l, l+32, ... in ascending order with fused multiply-adds, starting
+// vectors l, l+32, ... in ascending order with fused multiply-adds, starting
 // from zero; lane l then adds its four quarter sums in order; the 32 lane sums
 // are added by the xor butterfly (offsets 16, 8, 4, 2, 1).  The fused norm
 // multiplies x by the norm weight first and the finished sum by
@@ -91,7 +89,7 @@ __device__ __forceinline__ bool reduce_writer(int lane)
 
 struct KQuarters {
     uint32_t vec, per;     // 16-byte vectors in K; vectors per quarter
-    __device__ __forceinline__ KQuarters(uint32_t k, uint32_t vn) : vec(k / vn), per((k / vn + 3) / 4) {}
+    __device__ __forceinline__ explicit KQuarters(uint32_t k) : vec(k / 4), per((k / 4 + 3) / 4) {}
     __device__ __forceinline__ uint32_t lo(uint32_t q) const { return q * per < vec ? q * per : vec; }
     __device__ __forceinline__ uint32_t hi(uint32_t q) const { return (q + 1) * per < vec ? (q + 1) * per : vec; }
 };
@@ -133,43 +131,16 @@ __device__ __forceinline__ float finish(const GemvParams &p, uint32_t s, uint32_
     return y;
 }
 
-// One 16-byte vector of weights and what it does: N values, their dot product with N activations.
-template <typename W> struct WVec;
-template <> struct WVec<float> {
-    static constexpr int N = 4;
-    float4 v;
-    __device__ __forceinline__ void load(const float *p) { v = ldg_stream(p); }
-    __device__ __forceinline__ float dot(const float4 (&x)[1], float acc) const { return dot4(v, x[0], acc); }
-};
-template <> struct WVec<__nv_bfloat16> {
-    static constexpr int N = 8;
-    uint4 v;
-    __device__ __forceinline__ void load(const __nv_bfloat16 *p)
-    {
-        const float4 f = ldg_stream(reinterpret_cast<const float *>(p));
-        v = make_uint4(__float_as_uint(f.x), __float_as_uint(f.y), __float_as_uint(f.z), __float_as_uint(f.w));
-    }
-    static __device__ __forceinline__ float4 four(uint32_t a, uint32_t b)
-    {
-        return make_float4(__uint_as_float(a << 16), __uint_as_float(a & 0xffff0000u), __uint_as_float(b << 16),
-                           __uint_as_float(b & 0xffff0000u));
-    }
-    __device__ __forceinline__ float dot(const float4 (&x)[2], float acc) const
-    {
-        return dot4(four(v.z, v.w), x[1], dot4(four(v.x, v.y), x[0], acc));
-    }
-};
-
 // weight rows of a CTA / warp: plain, or swiglu (first half gate rows, second half the same rows of up)
-template <typename W, int NR>
+template <int NR>
 __device__ __forceinline__ void weight_rows(const GemvParams &p, const GemvSeg &seg, uint32_t n0,
-                                            const W *(&wrow)[NR])
+                                            const float *(&wrow)[NR])
 {
     constexpr int H = (NR >= 2) ? NR / 2 : 1;
 #pragma unroll
     for (int c = 0; c < NR; ++c) {
         uint32_t n = p.swiglu ? n0 + (c % H) : n0 + c;
-        const W *base = static_cast<const W *>(p.swiglu ? ((c < H) ? p.seg[0].w : p.seg[1].w) : seg.w);
+        const float *base = p.swiglu ? ((c < H) ? p.seg[0].w : p.seg[1].w) : seg.w;
         if (n >= seg.n) n = seg.n - 1;               // clamped rows are computed and dropped
         wrow[c] = base + (size_t)n * p.k;
     }
@@ -177,7 +148,7 @@ __device__ __forceinline__ void weight_rows(const GemvParams &p, const GemvSeg &
 
 constexpr int kPrefetchRegs = 16;        // 16-byte weight vectors a lane holds before the dependency wait
 
-template <typename W, int RG, int C>
+template <int RG, int C>
 __global__ void __launch_bounds__(kGemvThreads) gemv_splitk_kernel(const GemvParams p)
 {
     __shared__ float part[kGemvWarps][C * RG + RG][32];      // per quarter (= warp): every lane's partial sums
@@ -193,16 +164,15 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_splitk_kernel(const GemvPar
     const GemvSeg seg = p.seg[s];
     constexpr int H = (C >= 2) ? C / 2 : 1;
     const uint32_t n0 = cta * (p.swiglu ? H : C);
-    constexpr int VN = WVec<W>::N, XV = VN / 4;              // values per weight vector; float4s of x beside it
-    const W *wrow[C];
-    weight_rows<W, C>(p, seg, n0, wrow);
+    const float *wrow[C];
+    weight_rows<C>(p, seg, n0, wrow);
     const float *xrow[RG];
 #pragma unroll
     for (int r = 0; r < RG; ++r) {
         const uint32_t row = (r0 + r < p.rows) ? r0 + r : p.rows - 1;    // clamped rows are dropped at the end
         xrow[r] = p.x + (size_t)row * p.x_stride;
     }
-    const KQuarters kq(p.k, VN);
+    const KQuarters kq(p.k);
     const uint32_t v_lo = kq.lo(warp), v_hi = kq.hi(warp);
 
     float acc[C][RG], ss[RG];
@@ -216,35 +186,28 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_splitk_kernel(const GemvPar
     // (all of it for K up to 512 * PV) are requested before the dependency wait, so their trip from
     // HBM overlaps that kernel's tail; the activations are read after it.
     constexpr int PV = kPrefetchRegs / C;
-    WVec<W> wbuf[PV][C];
+    float4 wbuf[PV][C];
 #pragma unroll
     for (int i = 0; i < PV; ++i) {
         const uint32_t v = v_lo + lane + 32u * i;
         if (v < v_hi) {
 #pragma unroll
-            for (int c = 0; c < C; ++c) wbuf[i][c].load(wrow[c] + VN * v);
+            for (int c = 0; c < C; ++c) wbuf[i][c] = ldg_stream(wrow[c] + 4 * v);
         }
     }
     pdl_wait();
-    auto step = [&](uint32_t v, const WVec<W> (&w)[C]) {
-        float4 nw[XV];
-        if (p.norm_w) {
-#pragma unroll
-            for (int h = 0; h < XV; ++h) nw[h] = *reinterpret_cast<const float4 *>(p.norm_w + VN * v + 4 * h);
-        }
+    auto step = [&](uint32_t v, const float4 (&w)[C]) {
+        float4 nw = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (p.norm_w) nw = *reinterpret_cast<const float4 *>(p.norm_w + 4 * v);
 #pragma unroll
         for (int r = 0; r < RG; ++r) {
-            float4 xv[XV];
-#pragma unroll
-            for (int h = 0; h < XV; ++h) {
-                xv[h] = *reinterpret_cast<const float4 *>(xrow[r] + VN * v + 4 * h);
-                if (p.norm_w) {
-                    ss[r] = sumsq4(ss[r], xv[h]);
-                    xv[h] = mul4(xv[h], nw[h]);
-                }
+            float4 xv = *reinterpret_cast<const float4 *>(xrow[r] + 4 * v);
+            if (p.norm_w) {
+                ss[r] = sumsq4(ss[r], xv);
+                xv = mul4(xv, nw);
             }
 #pragma unroll
-            for (int c = 0; c < C; ++c) acc[c][r] = w[c].dot(xv, acc[c][r]);
+            for (int c = 0; c < C; ++c) acc[c][r] = dot4(w[c], xv, acc[c][r]);
         }
     };
 #pragma unroll
@@ -254,9 +217,9 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_splitk_kernel(const GemvPar
     }
 #pragma unroll 2
     for (uint32_t v = v_lo + lane + 32u * PV; v < v_hi; v += 32) {
-        WVec<W> w[C];
+        float4 w[C];
 #pragma unroll
-        for (int c = 0; c < C; ++c) w[c].load(wrow[c] + VN * v);
+        for (int c = 0; c < C; ++c) w[c] = ldg_stream(wrow[c] + 4 * v);
         step(v, w);
     }
     constexpr int M = C * RG;
@@ -295,11 +258,10 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_splitk_kernel(const GemvPar
 }
 
 // RG: activation rows per CTA (row group); NW: weight rows per warp.
-template <typename W, int RG, int NW>
+template <int RG, int NW>
 __global__ void __launch_bounds__(kGemvThreads) gemv_rows_kernel(const GemvParams p)
 {
-    constexpr int VN = WVec<W>::N, XV = VN / 4;
-    constexpr int kPieceVec = kChunk / VN;           // weight vectors' worth of x staged per row and pass
+    constexpr int kPieceVec = kChunk / 4;            // 16-byte vectors of x staged per row and pass
     __shared__ __align__(16) float xs[RG][kChunk];
     __shared__ float inv_rms[RG];
     pdl_trigger();
@@ -313,9 +275,9 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_rows_kernel(const GemvParam
     const GemvSeg seg = p.seg[s];
     constexpr int H = (NW >= 2) ? NW / 2 : 1;
     const uint32_t n0 = (cta * kGemvWarps + warp) * (p.swiglu ? H : NW);
-    const W *wrow[NW];
-    weight_rows<W, NW>(p, seg, n0, wrow);
-    const KQuarters kq(p.k, VN);
+    const float *wrow[NW];
+    weight_rows<NW>(p, seg, n0, wrow);
+    const KQuarters kq(p.k);
     pdl_wait();
 
     if (p.norm_w) {                                  // sum of squares in the shared order
@@ -326,11 +288,8 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_rows_kernel(const GemvParam
 #pragma unroll 1
                 for (uint32_t q = 0; q < 4; ++q) {
                     float ss = 0.f;
-                    for (uint32_t v = kq.lo(q) + lane; v < kq.hi(q); v += 32) {
-#pragma unroll
-                        for (int h = 0; h < XV; ++h)
-                            ss = sumsq4(ss, *reinterpret_cast<const float4 *>(xr + VN * v + 4 * h));
-                    }
+                    for (uint32_t v = kq.lo(q) + lane; v < kq.hi(q); v += 32)
+                        ss = sumsq4(ss, *reinterpret_cast<const float4 *>(xr + 4 * v));
                     t = (q == 0) ? ss : __fadd_rn(t, ss);
                 }
             }
@@ -356,29 +315,26 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_rows_kernel(const GemvParam
         for (uint32_t c0 = v_lo; c0 < v_hi; c0 += kPieceVec) {
             const uint32_t nvec = (v_hi - c0 < (uint32_t)kPieceVec) ? v_hi - c0 : (uint32_t)kPieceVec;
             __syncthreads();                         // the previous piece has been consumed
-            const uint32_t nx = nvec * XV, x0 = c0 * XV;     // float4s of x
-            for (uint32_t i = tid; i < RG * nx; i += kGemvThreads) {
-                const uint32_t r = i / nx, vv = i % nx;
+            for (uint32_t i = tid; i < RG * nvec; i += kGemvThreads) {
+                const uint32_t r = i / nvec, vv = i % nvec;
                 float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (r0 + r < p.rows) {
-                    v = *reinterpret_cast<const float4 *>(p.x + (size_t)(r0 + r) * p.x_stride + 4 * (x0 + vv));
-                    if (p.norm_w) v = mul4(v, *reinterpret_cast<const float4 *>(p.norm_w + 4 * (x0 + vv)));
+                    v = *reinterpret_cast<const float4 *>(p.x + (size_t)(r0 + r) * p.x_stride + 4 * (c0 + vv));
+                    if (p.norm_w) v = mul4(v, *reinterpret_cast<const float4 *>(p.norm_w + 4 * (c0 + vv)));
                 }
                 *reinterpret_cast<float4 *>(&xs[r][4 * vv]) = v;
             }
             __syncthreads();
 #pragma unroll 2
             for (uint32_t vv = lane; vv < nvec; vv += 32) {
-                WVec<W> w[NW];
+                float4 w[NW];
 #pragma unroll
-                for (int c = 0; c < NW; ++c) w[c].load(wrow[c] + VN * (c0 + vv));
+                for (int c = 0; c < NW; ++c) w[c] = ldg_stream(wrow[c] + 4 * (c0 + vv));
 #pragma unroll
                 for (int r = 0; r < RG; ++r) {
-                    float4 xv[XV];
+                    const float4 xv = *reinterpret_cast<const float4 *>(&xs[r][4 * vv]);
 #pragma unroll
-                    for (int h = 0; h < XV; ++h) xv[h] = *reinterpret_cast<const float4 *>(&xs[r][VN * vv + 4 * h]);
-#pragma unroll
-                    for (int c = 0; c < NW; ++c) acc[c][r] = w[c].dot(xv, acc[c][r]);
+                    for (int c = 0; c < NW; ++c) acc[c][r] = dot4(w[c], xv, acc[c][r]);
                 }
             }
         }
@@ -434,37 +390,37 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_rows_kernel(const GemvParam
     }
 }
 
-template <typename W, int RG, int NW>
+template <int RG, int NW>
 void launch_gemv_t(const GemvParams &p, uint32_t ctas, cudaStream_t st)
 {
     dim3 grid(ctas, (p.rows + RG - 1) / RG);
-    (void)wr_launch_pdl(gemv_rows_kernel<W, RG, NW>, grid, dim3(kGemvThreads), 0, st, p);
+    (void)wr_launch_pdl(gemv_rows_kernel<RG, NW>, grid, dim3(kGemvThreads), 0, st, p);
 }
 
-template <typename W, int RG, int C>
+template <int RG, int C>
 void launch_splitk_t(const GemvParams &p, uint32_t ctas, cudaStream_t st)
 {
     dim3 grid(ctas, (p.rows + RG - 1) / RG);
-    (void)wr_launch_pdl(gemv_splitk_kernel<W, RG, C>, grid, dim3(kGemvThreads), 0, st, p);
+    (void)wr_launch_pdl(gemv_splitk_kernel<RG, C>, grid, dim3(kGemvThreads), 0, st, p);
 }
 
-template <typename W, int C>
+template <int C>
 void launch_splitk(const GemvParams &p, uint32_t ctas, cudaStream_t st)
 {
-    if (p.rows == 1) launch_splitk_t<W, 1, C>(p, ctas, st);
-    else if (p.rows == 2) launch_splitk_t<W, 2, C>(p, ctas, st);
-    else launch_splitk_t<W, 4, C>(p, ctas, st);
+    if (p.rows == 1) launch_splitk_t<1, C>(p, ctas, st);
+    else if (p.rows == 2) launch_splitk_t<2, C>(p, ctas, st);
+    else launch_splitk_t<4, C>(p, ctas, st);
 }
 
-template <typename W, int NW>
+template <int NW>
 void launch_gemv_rg(const GemvParams &p, uint32_t ctas, cudaStream_t st)
 {
     const uint32_t r = p.rows;
-    if (r == 1) launch_gemv_t<W, 1, NW>(p, ctas, st);
-    else if (r == 2) launch_gemv_t<W, 2, NW>(p, ctas, st);
-    else if (r <= 4) launch_gemv_t<W, 4, NW>(p, ctas, st);
-    else if (r <= 8) launch_gemv_t<W, 8, NW>(p, ctas, st);
-    else launch_gemv_t<W, 16, NW>(p, ctas, st);
+    if (r == 1) launch_gemv_t<1, NW>(p, ctas, st);
+    else if (r == 2) launch_gemv_t<2, NW>(p, ctas, st);
+    else if (r <= 4) launch_gemv_t<4, NW>(p, ctas, st);
+    else if (r <= 8) launch_gemv_t<8, NW>(p, ctas, st);
+    else launch_gemv_t<16, NW>(p, ctas, st);
 }
 
 // Weight rows per warp from the total output width: narrow outputs take one row
@@ -479,8 +435,9 @@ int weight_rows_per_warp(uint32_t n_total)
 
 constexpr uint32_t kSplitKRowsMax = 4;
 
-template <typename W>
-int launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t n_total_for_width)
+}  // namespace
+
+int wr_gemv_launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t n_total_for_width)
 {
     if (p.rows <= kSplitKRowsMax) {
         // weight rows per CTA: 2 for narrow outputs (more CTAs), 4 otherwise
@@ -495,8 +452,8 @@ int launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t n_total_for_width)
                 p.cta_end[s] = ctas;
             }
         }
-        if (c == 4) launch_splitk<W, 4>(p, ctas, ctx->stream);
-        else launch_splitk<W, 2>(p, ctas, ctx->stream);
+        if (c == 4) launch_splitk<4>(p, ctas, ctx->stream);
+        else launch_splitk<2>(p, ctas, ctx->stream);
         WR_CUDA_TRY(cudaGetLastError());
         return WR_CUDA_OK;
     }
@@ -512,16 +469,9 @@ int launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t n_total_for_width)
         }
     }
     cudaStream_t st = ctx->stream;
-    if (nw == 4) launch_gemv_rg<W, 4>(p, ctas, st);
-    else if (nw == 2) launch_gemv_rg<W, 2>(p, ctas, st);
-    else launch_gemv_rg<W, 1>(p, ctas, st);
+    if (nw == 4) launch_gemv_rg<4>(p, ctas, st);
+    else if (nw == 2) launch_gemv_rg<2>(p, ctas, st);
+    else launch_gemv_rg<1>(p, ctas, st);
     WR_CUDA_TRY(cudaGetLastError());
     return WR_CUDA_OK;
-}
-
-}  // namespace
-
-int wr_gemv_launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t width, int w_type)
-{
-    return w_type == WR_CUDA_BF16 ? launch<__nv_bfloat16>(ctx, p, width) : launch<float>(ctx, p, width);
 }

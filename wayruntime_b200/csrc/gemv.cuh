@@ -4,7 +4,7 @@
 #include "wr_internal.cuh"
 
 struct GemvSeg {
-    const void *w;         // [n][k] row-major (GGML layout of a [k -> n] weight)
+    const float *w;        // [n][k] row-major (GGML layout of a [k -> n] weight)
     float *out;            // [rows][out_stride]
     uint32_t n, out_stride;
 };
@@ -26,6 +26,6 @@ struct GemvParams {
     uint32_t act;          // WR_GEMV_ACT_* on the result (after the bias)
 };
 
-// Enqueue y[r][n] = sum_k W[n][k] x[r][k] with W in `w_type` (WR_CUDA_F32: k a multiple of 4;
-// WR_CUDA_BF16: of 8) on the context's stream.  `width` is the output width the tiling is chosen by.
-int wr_gemv_launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t width, int w_type);
+// Enqueue y[r][n] = sum_k W[n][k] x[r][k] on the context's stream (k a multiple of 4).  `width` is the output width
+// the tiling is chosen by.
+int wr_gemv_launch(wr_cuda_ctx *ctx, GemvParams &p, uint32_t width);

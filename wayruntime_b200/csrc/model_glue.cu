@@ -17,7 +17,7 @@
 // share the call (same lanes, same order), which keeps batched logits
 // byte-equal to serial ones as the reference promises (src/core/batch.c:1-40).
 //
-// Kernels: a row-block GEMV (each warp owns 1-4 weight rows, the activation
+// Kernels: a row-block GEMV (gemv.cu: each warp owns 1-4 weight rows, the activation
 // rows sit in shared memory, the weights stream from HBM exactly once per group
 // of up to 16 activation rows) with optional fused RMSNorm on the input, fused
 // residual add or SiLU*up on the output; per-head RMSNorm; embedding gather;
@@ -166,7 +166,7 @@ namespace {
 int gemv(wr_cuda_model *m, GemvParams &p, uint32_t n_total_for_width)
 {
     ++m->launches;
-    return wr_gemv_launch(m->ctx, p, n_total_for_width, WR_CUDA_F32);
+    return wr_gemv_launch(m->ctx, p, n_total_for_width);
 }
 
 size_t up256(size_t n) { return (n + 255u) & ~(size_t)255u; }

@@ -553,7 +553,7 @@ struct Step {
             return wr_skinny_launch(ctx, mat.xs_map, {mat.w, mat.n, mat.k}, a);
         }
         GemvParams p{};
-        p.seg[0] = {mat.w, static_cast<float *>(out), mat.n, out_ld};
+        p.seg[0] = {static_cast<const float *>(mat.w), static_cast<float *>(out), mat.n, out_ld};
         p.n_seg = 1;
         p.x = static_cast<const float *>(in);
         p.x_stride = in_ld;
@@ -563,7 +563,7 @@ struct Step {
         p.bias = bias;
         p.act = softplus ? WR_GEMV_ACT_SOFTPLUS : WR_GEMV_ACT_NONE;
         ctx->launches++;
-        return wr_gemv_launch(ctx, p, mat.n, WR_CUDA_F32);
+        return wr_gemv_launch(ctx, p, mat.n);
     }
 
     int norm(const float *w, const float *shift, uint64_t state_off)
