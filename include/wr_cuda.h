@@ -123,8 +123,9 @@ int  wr_cuda_kv_create(wr_cuda_ctx *ctx, uint32_t n_layers, uint32_t n_kv_heads,
  * counterpart: every layer of the reference keeps F16 rows of one head_dim,
  * session.c:647-674).  Per layer: K/V pages of n_kv_heads heads with rows of
  * k_dim and v_dim elements of `elem` (WR_CUDA_F32 or WR_CUDA_F16; n_kv_heads 0:
- * none), and state_bytes of recurrent state (0: none).  Layers with F16 rows and
- * k_dim = v_dim have the page layout of wr_cuda_kv_create and are accepted by
+ * none), and state_bytes of recurrent state (0: none).  v_dim 0: one row per token
+ * and head that serves as key and value (a multiple of 64 elements when F16).
+ * Layers with F16 rows and k_dim = v_dim have the page layout of wr_cuda_kv_create and are accepted by
  * every call below; other layers by wr_cuda_model_forward only. */
 #define WR_CUDA_MAX_LAYER_RUNS 1024
 typedef struct wr_cuda_cache_layer {
@@ -377,8 +378,8 @@ int wr_cuda_model_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t
 /* ---- models whose layers differ ------------------------------------------- */
 
 /* A model put together from mixers: every layer names its own mixer (softmax
- * attention, plain or differential; selective scan) and feed-forward with sizes
- * of its own, a run list says in which order the layers are applied (a layer
+ * attention, plain or differential; attention over a latent; selective scan) and
+ * feed-forward (dense or a mixture of experts) with sizes of its own, a run list says in which order the layers are applied (a layer
  * may run several times with the same weights; each run keeps a cache or state
  * of its own).  It is a wr_cuda_model like the one above: created from host
  * pointers, stepped by wr_cuda_model_forward, destroyed by
@@ -400,14 +401,20 @@ typedef struct wr_cuda_tensor {
 
 #define WR_CUDA_MIXER_ATTENTION 1
 #define WR_CUDA_MIXER_MAMBA1    2
+#define WR_CUDA_MIXER_LATENT    3
 #define WR_CUDA_FFN_NONE        0
 #define WR_CUDA_FFN_POLYNORM    1
+#define WR_CUDA_FFN_SWIGLU      2     /* w_down(silu(w_gate_up h) * (w_up h)) */
+#define WR_CUDA_FFN_MOE         3     /* a mixture of experts (below) */
+#define WR_CUDA_NORM_RMS        0
+#define WR_CUDA_NORM_LAYER      1     /* the mean is taken off first */
 #define WR_CUDA_POS_NONE        0
 #define WR_CUDA_POS_SINUSOIDAL  1     /* added to the embedding: sin, cos of p * base^(-2i/width) interleaved */
 
 typedef struct wr_cuda_mixed_layer {
     uint32_t mixer, ffn;
-    wr_cuda_tensor norm1, norm2;      /* [width]; norm2 only with a feed-forward */
+    uint32_t parallel, reserved0;     /* 1: the feed-forward reads norm1's output too and there is no norm2 */
+    wr_cuda_tensor norm1, norm2;      /* [width]; norm2 only with a feed-forward of its own input */
     wr_cuda_tensor shift;             /* [width]: mixer input h + (h_before - h) * shift, or absent */
 
     /* WR_CUDA_MIXER_ATTENTION.  n_maps = 2 is differential attention: every
@@ -432,6 +439,30 @@ typedef struct wr_cuda_mixed_layer {
     uint32_t ffn_dim;
     float ffn_eps;
     wr_cuda_tensor w_up, w_down, act;
+
+    /* WR_CUDA_MIXER_LATENT: n_q_heads heads whose keys and values are linear in a
+     * row of kv_rank numbers that all heads share, the only thing kept per token
+     * besides one key part of rot_dim numbers with rotary positions (pairs i and
+     * i + rot_dim/2, angle p * rope_base^(-2i/rot_dim)).  q = w_uq norm(w_dq h), per
+     * head [k_dim | rot_dim rotated]; w_dkv h = [kv_rank, RMS-normed | rot_dim];
+     * score = attn_scale (q . w_uk c + q_rot . k_rot), value = w_uv c.  kv_from = 1 +
+     * j: the layer has no w_dkv and reads the rows that the latest run of layer j
+     * before it has left; 0: its own. */
+    uint32_t rot_dim, q_rank, kv_rank, kv_from;
+    double rope_base;
+    float latent_eps;
+    uint32_t reserved1;
+    wr_cuda_tensor w_dq, dq_norm, w_uq, w_dkv, dkv_norm, w_uk, w_uv;       /* and wo */
+
+    /* WR_CUDA_FFN_SWIGLU: w_gate_up [ffn_dim][width], w_up, w_down.
+     * WR_CUDA_FFN_MOE: of n_experts the top_k with the largest logits (router h +
+     * router_b), weighted by the softmax over theirs; an expert of ffn_dim is
+     * down(g sigmoid(moe_alpha g) (u + 1)), g = min(gate h, moe_limit), u = up h
+     * within +-moe_limit.  experts: {gate, up, down} of every expert. */
+    uint32_t n_experts, top_k;
+    float moe_alpha, moe_limit;
+    wr_cuda_tensor w_gate_up, router, router_b;
+    const wr_cuda_tensor *experts;
 } wr_cuda_mixed_layer;
 
 typedef struct wr_cuda_mixed_desc {
@@ -441,6 +472,9 @@ typedef struct wr_cuda_mixed_desc {
     uint32_t norm_groups;             /* RMS norm over this many equal parts of the row */
     uint32_t position;                /* WR_CUDA_POS_* */
     float norm_eps, position_base;
+    uint32_t norm;                    /* WR_CUDA_NORM_*, of norm1, norm2 and final_norm */
+    float embed_scale, residual_mult; /* factor on embedding rows; on what a sublayer adds to the residual */
+    uint32_t reserved;
     const uint32_t *runs;             /* n_runs layer indices, in the order they are applied */
     wr_cuda_tensor embed, head, final_norm;
     const wr_cuda_mixed_layer *layers;

@@ -81,29 +81,37 @@ class Tensor(C.Structure):
     _fields_ = [("data", C.c_void_p), ("dtype", C.c_uint32), ("reserved", C.c_uint32)]
 
 
-MIXER_ATTENTION, MIXER_MAMBA1 = 1, 2
-FFN_NONE, FFN_POLYNORM = 0, 1
+MIXER_ATTENTION, MIXER_MAMBA1, MIXER_LATENT = 1, 2, 3
+FFN_NONE, FFN_POLYNORM, FFN_SWIGLU, FFN_MOE = 0, 1, 2, 3
+NORM_RMS, NORM_LAYER = 0, 1
 POS_NONE, POS_SINUSOIDAL = 0, 1
 
 
 class MixedLayerDesc(C.Structure):
     """wr_cuda_mixed_layer (include/wr_cuda.h)."""
     TENSORS = ("norm1", "norm2", "shift", "wq", "wk", "wv", "wo", "bq", "bk", "bv", "w_gate", "lq1", "lk1", "lq2", "lk2",
-               "w_in", "conv", "conv_b", "w_x", "w_dt", "dt_b", "a_log", "d", "w_out", "w_up", "w_down", "act")
-    _fields_ = [("mixer", C.c_uint32), ("ffn", C.c_uint32)] + [(n, Tensor) for n in ("norm1", "norm2", "shift")] + \
+               "w_in", "conv", "conv_b", "w_x", "w_dt", "dt_b", "a_log", "d", "w_out", "w_up", "w_down", "act",
+               "w_dq", "dq_norm", "w_uq", "w_dkv", "dkv_norm", "w_uk", "w_uv", "w_gate_up", "router", "router_b")
+    _fields_ = [(n, C.c_uint32) for n in ("mixer", "ffn", "parallel", "reserved0")] + [(n, Tensor) for n in ("norm1", "norm2", "shift")] + \
                [(n, C.c_uint32) for n in ("n_q_heads", "n_kv_heads", "n_maps", "k_dim", "v_dim", "q_temp_every")] + \
                [(n, C.c_float) for n in ("q_temp_coef", "attn_scale", "diff_init", "diff_eps")] + \
                [(n, Tensor) for n in ("wq", "wk", "wv", "wo", "bq", "bk", "bv", "w_gate", "lq1", "lk1", "lq2", "lk2")] + \
                [(n, C.c_uint32) for n in ("inner", "state", "dt_rank", "taps")] + \
                [(n, Tensor) for n in ("w_in", "conv", "conv_b", "w_x", "w_dt", "dt_b", "a_log", "d", "w_out")] + \
-               [("ffn_dim", C.c_uint32), ("ffn_eps", C.c_float)] + [(n, Tensor) for n in ("w_up", "w_down", "act")]
+               [("ffn_dim", C.c_uint32), ("ffn_eps", C.c_float)] + [(n, Tensor) for n in ("w_up", "w_down", "act")] + \
+               [(n, C.c_uint32) for n in ("rot_dim", "q_rank", "kv_rank", "kv_from")] + \
+               [("rope_base", C.c_double), ("latent_eps", C.c_float), ("reserved1", C.c_uint32)] + \
+               [(n, Tensor) for n in ("w_dq", "dq_norm", "w_uq", "w_dkv", "dkv_norm", "w_uk", "w_uv")] + \
+               [("n_experts", C.c_uint32), ("top_k", C.c_uint32), ("moe_alpha", C.c_float), ("moe_limit", C.c_float)] + \
+               [(n, Tensor) for n in ("w_gate_up", "router", "router_b")] + [("experts", C.POINTER(Tensor))]
 
 
 class MixedDesc(C.Structure):
     """wr_cuda_mixed_desc (include/wr_cuda.h)."""
     _fields_ = [(n, C.c_uint32) for n in ("compute", "width", "vocab", "n_layers", "n_runs", "max_rows", "norm_groups",
                                           "position")] + \
-               [("norm_eps", C.c_float), ("position_base", C.c_float), ("runs", C.POINTER(C.c_uint32))] + \
+               [("norm_eps", C.c_float), ("position_base", C.c_float), ("norm", C.c_uint32), ("embed_scale", C.c_float),
+                ("residual_mult", C.c_float), ("reserved", C.c_uint32), ("runs", C.POINTER(C.c_uint32))] + \
                [(n, Tensor) for n in ("embed", "head", "final_norm")] + [("layers", C.POINTER(MixedLayerDesc))]
 
 
@@ -536,12 +544,13 @@ class DeviceModel:
 
 class MixedModel(DeviceModel):
     """wr_cuda_model of the mixed kind (wr_cuda_model_create_mixed).  `layers` is a list of dicts with the
-    scalar fields of wr_cuda_mixed_layer; `tensor(i, field)` returns layer i's array for a tensor field (or None),
-    and tensor(None, name) the model's embed, head and final_norm.  Arrays are float32, or uint16 holding
+    scalar fields of wr_cuda_mixed_layer; `tensor(i, field)` returns layer i's array for a tensor field (or None;
+    for "experts" the gate, up and down arrays of every expert, one after the other), and tensor(None, name) the
+    model's embed, head and final_norm.  Arrays are float32, or uint16 holding
     bfloat16 bits."""
 
     def __init__(self, ctx: "Context", layers, runs, tensor, *, compute, width, vocab, norm_groups, norm_eps,
-                 position=POS_NONE, position_base=10000.0, max_rows=256):
+                 position=POS_NONE, position_base=10000.0, norm=NORM_RMS, embed_scale=1.0, residual_mult=1.0, max_rows=256):
         self._ctx, self._lib = ctx, ctx._lib
         self.vocab, self.hidden, self.n_layers, self.max_rows = vocab, width, len(runs), max_rows
         self.n_q = self.hd = 0
@@ -562,9 +571,12 @@ class MixedModel(DeviceModel):
                 setattr(arr[i], k, v)
             for k in MixedLayerDesc.TENSORS:
                 setattr(arr[i], k, ref(tensor(i, k)))
+            if lay.get("n_experts"):
+                parts = [ref(a) for a in tensor(i, "experts")]
+                arr[i].experts = (Tensor * len(parts))(*parts)
         d = MixedDesc(compute=compute, width=width, vocab=vocab, n_layers=len(layers), n_runs=len(runs),
                       max_rows=max_rows, norm_groups=norm_groups, position=position, norm_eps=norm_eps,
-                      position_base=position_base, runs=(C.c_uint32 * len(runs))(*runs), embed=ref(tensor(None, "embed")),
+                      position_base=position_base, norm=norm, embed_scale=embed_scale, residual_mult=residual_mult, runs=(C.c_uint32 * len(runs))(*runs), embed=ref(tensor(None, "embed")),
                       head=ref(tensor(None, "head")), final_norm=ref(tensor(None, "final_norm")), layers=arr)
         h = C.c_void_p()
         _check(self._lib.wr_cuda_model_create_mixed(ctx._h, C.byref(d), C.byref(h)), "wr_cuda_model_create_mixed")

@@ -5,7 +5,8 @@
 // (64 K-values of both operands per stage: activations through a tensor map, weights as linear copies
 // of blocks stored in the operand's layout; what lies beyond K arrives as zeros), warp 1 issues tcgen05.mma into one of two TMEM accumulators, warps 2-5 read the other one
 // back and write the finished rows (bias, softplus, residual; F32, BF16 or saturated F16), so that a
-// tile's output overlaps the next tile's products.  Every wait is bounded by the context's wait
+// tile's output overlaps the next tile's products.  Columns may be gate / up pairs, of which the activation leaves
+// (wr_pair_args), and row tiles may have weights of their own (wr_group_args).  Every wait is bounded by the context's wait
 // limit; a warp that gives up records an error word and all of them leave.
 #include <cuda_bf16.h>
 
@@ -31,7 +32,7 @@ template <uint32_t BN> struct Tile {
 struct GemmParams {
     wr_gemm_args a;
     wr_weight w;
-    uint32_t m_tiles, tiles, k_blocks;
+    uint32_t m_tiles, n_tiles, k_blocks;
     long long wait_limit;
     int *err;
 };
@@ -77,13 +78,16 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
     tc5::fence_after();
     const uint32_t tmem = tmem_slot;
     pdl_wait();
+    const uint32_t m_tiles = p.a.group.list ? *p.a.group.count : p.m_tiles, tiles = m_tiles * p.n_tiles;
 
     if (warp == 0) {
         if (lane == 0) {
             uint32_t it = 0;
             bool ok = true;
-            for (uint32_t tile = blockIdx.x; tile < p.tiles && ok; tile += gridDim.x) {
-                const uint32_t m0 = (tile % p.m_tiles) * kBM, n0 = (tile / p.m_tiles) * BN;
+            for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
+                const uint32_t m0 = (tile % m_tiles) * kBM, n0 = (tile / m_tiles) * BN;
+                const char *blocks = static_cast<const char *>(p.w.blocks);
+                if (p.a.group.list) blocks += p.a.group.list[tile % m_tiles] * p.a.group.stride;
                 for (uint32_t kb = 0; kb < p.k_blocks; ++kb, ++it) {
                     const uint32_t st = it % T::kStages;
                     if (it >= T::kStages && !mbar_wait(&empty[st], (it / T::kStages - 1) & 1, p.wait_limit)) {
@@ -94,7 +98,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
                     const uint32_t nb0 = n0 / kWBlock, nb = min(BN / kWBlock, wr_weight_blocks(p.w.n) - nb0);
                     mbar_expect_tx(&full[st], kABytes + nb * kWBlockBytes);
                     tc5::tma_load_2d(a, &x_map, (int)(kb * kBK), (int)m0, &full[st]);
-                    const char *w = static_cast<const char *>(p.w.blocks) + ((size_t)nb0 * p.k_blocks + kb) * kWBlockBytes;
+                    const char *w = blocks + ((size_t)nb0 * p.k_blocks + kb) * kWBlockBytes;
                     for (uint32_t i = 0; i < nb; ++i)
                         bulk_g2s(b + i * kWBlockBytes, w + (size_t)i * p.k_blocks * kWBlockBytes, kWBlockBytes, &full[st]);
                 }
@@ -111,7 +115,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
         constexpr uint32_t idesc = tc5::idesc_bf16(kBM, BN);
         uint32_t it = 0, n_tile = 0;
         bool ok = true;
-        for (uint32_t tile = blockIdx.x; tile < p.tiles && ok; tile += gridDim.x, ++n_tile) {
+        for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++n_tile) {
             const uint32_t acc = n_tile & 1;
             if (n_tile >= 2 && !mbar_wait(&acc_empty[acc], (n_tile / 2 - 1) & 1, p.wait_limit)) {
                 ok = false;
@@ -139,8 +143,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
         const uint32_t quarter = warp & 3;                       // TMEM lanes this warp may read
         uint32_t n_tile = 0;
         bool ok = true;
-        for (uint32_t tile = blockIdx.x; tile < p.tiles && ok; tile += gridDim.x, ++n_tile) {
-            const uint32_t m0 = (tile % p.m_tiles) * kBM, n0 = (tile / p.m_tiles) * BN;
+        for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++n_tile) {
+            const uint32_t m0 = (tile % m_tiles) * kBM, n0 = (tile / m_tiles) * BN;
             const uint32_t acc = n_tile & 1, row = m0 + quarter * 32 + lane;
             if (!mbar_wait(&acc_full[acc], (n_tile / 2) & 1, p.wait_limit)) {
                 ok = false;
@@ -157,7 +161,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
 #pragma unroll
                     for (uint32_t g = 0; g < 4; ++g) {
                         const uint32_t col = n0 + c0 + 8 * g;
-                        if (col < n_pad) {
+                        if (col >= p.a.pair.from) {
+                            if ((g & 1u) || col >= n_pad) continue;
+                            float y[8];
+#pragma unroll
+                            for (int e = 0; e < 8; ++e)
+                                y[e] = wr_pair_act(p.a.pair.act, p.a.pair.alpha, p.a.pair.limit, v[8 * g + e],
+                                                   v[8 * ((g + 1) & 3u) + e]);
+                            *reinterpret_cast<uint4 *>((__nv_bfloat16 *)p.a.pair.out + (size_t)row * p.a.pair.ld +
+                                                       (col - p.a.pair.from) / 2) =
+                                make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]), pack_bf16(y[4], y[5]),
+                                           pack_bf16(y[6], y[7]));
+                        } else if (col < n_pad) {
                             float *u = v + 8 * g;
                             if (p.a.bias) {
                                 const float4 b0 = *reinterpret_cast<const float4 *>(p.a.bias + col);
@@ -173,6 +188,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
                                 *reinterpret_cast<uint4 *>((__nv_bfloat16 *)p.a.out_bf16 + (size_t)row * p.a.out_bf16_ld + col) =
                                     make_uint4(pack_bf16(u[0], u[1]), pack_bf16(u[2], u[3]), pack_bf16(u[4], u[5]),
                                                pack_bf16(u[6], u[7]));
+                            if (p.a.mul != 1.f) {
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) u[e] *= p.a.mul;
+                            }
                             if (p.a.add) {
                                 const float *r = p.a.add + (size_t)row * p.a.add_ld + col;
                                 const float4 r0 = *reinterpret_cast<const float4 *>(r);
@@ -252,11 +271,11 @@ int launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_
     p.a = a;
     p.w = w;
     p.m_tiles = (a.m + kBM - 1) / kBM;
-    p.tiles = p.m_tiles * ((w.n + BN - 1) / BN);
+    p.n_tiles = (w.n + BN - 1) / BN;
     p.k_blocks = wr_weight_blocks(w.k);
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
-    const uint32_t grid = std::min<uint32_t>(p.tiles, (uint32_t)ctx->sm_count);
+    const uint32_t grid = std::min<uint32_t>((a.group.list ? a.group.max : p.m_tiles) * p.n_tiles, (uint32_t)ctx->sm_count);
     WR_CUDA_TRY(wr_launch_pdl(gemm_bf16_kernel<BN>, dim3(grid), dim3(kThreads), Tile<BN>::kSmem, ctx->stream, x, p));
     ctx->launches++;
     WR_CUDA_TRY(cudaGetLastError());
@@ -270,17 +289,18 @@ int wr_gemm_map_rows(CUtensorMap *map, const void *x, uint32_t rows, uint32_t k,
     return map_2d(map, x, rows, k, ld, kBM);
 }
 
-int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld)
+int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld, uint32_t groups)
 {
-    return map_2d(map, split_rows, 2 * WR_CUDA_BATCH_MAX, k, ld, 2 * WR_CUDA_BATCH_MAX);
+    return map_2d(map, split_rows, groups * 2 * WR_CUDA_BATCH_MAX, k, ld, 2 * WR_CUDA_BATCH_MAX);
 }
 
 int wr_gemm_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_gemm_args &a)
 {
-    if (a.m == 0 || w.n == 0 || w.k == 0 || (a.out_ld & 7u) || (a.out_bf16_ld & 7u) || (a.add_ld & 7u))
+    if (a.m == 0 || w.n == 0 || w.k == 0 || (a.out_ld & 7u) || (a.out_bf16_ld & 7u) || (a.add_ld & 7u) ||
+        (a.pair.from != ~0u && ((a.pair.from & 15u) || (a.pair.ld & 7u))))
         return WR_CUDA_ERR_INVAL;
     // the tile width that finishes first: rounds over the device times the width's share of the work
-    const uint32_t m_tiles = (a.m + kBM - 1) / kBM;
+    const uint32_t m_tiles = a.group.list ? a.group.max : (a.m + kBM - 1) / kBM;
     uint32_t best = 0;
     uint64_t best_cost = ~0ull;
     for (uint32_t bn : {256u, 128u, 64u}) {

@@ -8,6 +8,27 @@
 enum { WR_GEMM_OUT_F32 = 0, WR_GEMM_OUT_BF16 = 1, WR_GEMM_OUT_F16 = 2 };
 enum { WR_GEMM_ACT_NONE = 0, WR_GEMM_ACT_SOFTPLUS = 1 };
 
+// Gate and up products of a gated feed-forward in one: weight rows from `from` on come in groups of sixteen, eight
+// gate rows and then the eight up rows that belong to them, and what leaves is act(gate, up), eight values a group.
+enum { WR_PAIR_SILU = 0, WR_PAIR_LIMITED = 1 };
+struct wr_pair_args {
+    uint32_t from = ~0u;   // a multiple of 16; ~0: there are none
+    uint32_t act = WR_PAIR_SILU;
+    float alpha = 1.f, limit = 0.f;      // WR_PAIR_LIMITED: g sigmoid(alpha g) (u + 1), g <= limit, |u| <= limit
+    void *out = nullptr;   // rows of BF16 values (many rows), or split rows (few)
+    uint32_t ld = 0;
+};
+// One product per group of rows, each with a weight of its own (experts), `stride` bytes apart.  `list` names the
+// weight of every 128-row tile of the activations (many rows), or of every group (few rows: group g's results are
+// rows 16 g .. of out, split rows 32 g .. of pair.out, and its input the split rows x_rows * g ..).
+struct wr_group_args {
+    const uint32_t *list = nullptr;      // device memory, as is:
+    const uint32_t *count = nullptr;     // how many entries the list has
+    uint32_t max = 0;                    // at most this many
+    uint32_t x_rows = 0;
+    size_t stride = 0;
+};
+
 struct wr_gemm_args {
     uint32_t m;
     void *out;             // [m][out_ld] of out_type; out_ld a multiple of 8, at least w.n
@@ -18,6 +39,9 @@ struct wr_gemm_args {
     uint32_t act;          // WR_GEMM_ACT_* after the bias
     const float *add;      // [m][add_ld] residual added last (may alias an F32 out), or null
     uint32_t add_ld;
+    float mul = 1.f;       // on the result before the residual
+    wr_pair_args pair;
+    wr_group_args group;   // m: rows the buffers hold
 };
 
 // A BF16 weight [n][k] as the tensor core reads it: blocks of 64 rows x 64 K-values, each the 8 KB image of a
@@ -32,7 +56,7 @@ struct wr_weight {
 __host__ __device__ inline uint32_t wr_weight_blocks(uint32_t n) { return (n + kWBlock - 1) / kWBlock; }
 inline size_t wr_weight_bytes(uint32_t n, uint32_t k) { return (size_t)wr_weight_blocks(n) * wr_weight_blocks(k) * kWBlockBytes; }
 // byte offset of element (r, i)
-inline size_t wr_weight_off(uint32_t k, uint32_t r, uint32_t i)
+__host__ __device__ inline size_t wr_weight_off(uint32_t k, uint32_t r, uint32_t i)
 {
     const size_t block = (size_t)(r / kWBlock) * wr_weight_blocks(k) + i / kWBlock;
     const uint32_t rr = r % kWBlock, ii = i % kWBlock;
@@ -59,6 +83,20 @@ struct wr_skinny_args {
     uint32_t act;          // WR_GEMM_ACT_*
     const float *add;      // [rows][add_ld] or null (may alias out)
     uint32_t add_ld;
+    float mul = 1.f;       // on the result before the residual
+    wr_pair_args pair;
+    wr_group_args group;
 };
-int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld);
+int wr_skinny_map_rows(CUtensorMap *map, const void *split_rows, uint32_t k, uint32_t ld, uint32_t groups = 1);
 int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w, const wr_skinny_args &args);
+
+#ifdef __CUDACC__
+// act(gate, up) of wr_pair_args (the exponential and the quotient are the short sequences)
+__device__ __forceinline__ float wr_pair_act(uint32_t act, float alpha, float limit, float g, float u)
+{
+    if (act == WR_PAIR_SILU) return __fdividef(g, 1.0f + __expf(-g)) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
+#endif

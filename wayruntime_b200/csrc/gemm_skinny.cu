@@ -44,20 +44,34 @@ __device__ __forceinline__ float load_rank(const float *p, uint32_t rank)
     return v;
 }
 
+// row i as split rows: the value's rounding, and what is left kRows rows behind it
+__device__ __forceinline__ void put_split(void *out, uint32_t ld, uint32_t i, uint32_t n, float y)
+{
+    __nv_bfloat16 *o = static_cast<__nv_bfloat16 *>(out) + (size_t)i * ld + n;
+    const __nv_bfloat16 hi = __float2bfloat16_rn(y);
+    o[0] = hi;
+    o[(size_t)kRows * ld] = __float2bfloat16_rn(y - __bfloat162float(hi));
+}
+
+// a gate row and the up row that belongs to it
+__device__ __forceinline__ void put_pair(const SkinnyParams &p, uint32_t group, uint32_t i, uint32_t n, float g, float u)
+{
+    if (n >= p.w.n) return;
+    const uint32_t c = n - p.a.pair.from;
+    put_split(p.a.pair.out, p.a.pair.ld, 2 * kRows * group + i, c / 16 * 8 + (c & 7u),
+              wr_pair_act(p.a.pair.act, p.a.pair.alpha, p.a.pair.limit, g, u));
+}
+
 // bias, activation, copies and residual of one finished sum: activation row i, weight row n
-__device__ __forceinline__ void put(const SkinnyParams &p, uint32_t i, uint32_t n, float y)
+__device__ __forceinline__ void put(const SkinnyParams &p, uint32_t group, uint32_t i, uint32_t n, float y)
 {
     if (n >= p.w.n) return;
     if (p.a.bias) y += p.a.bias[n];
     if (p.a.act == WR_GEMM_ACT_SOFTPLUS) y = softplus(y);
-    if (p.a.out_split) {
-        __nv_bfloat16 *o = static_cast<__nv_bfloat16 *>(p.a.out_split) + (size_t)i * p.a.out_split_ld + n;
-        const __nv_bfloat16 hi = __float2bfloat16_rn(y);
-        o[0] = hi;
-        o[(size_t)kRows * p.a.out_split_ld] = __float2bfloat16_rn(y - __bfloat162float(hi));
-    }
+    if (p.a.out_split) put_split(p.a.out_split, p.a.out_split_ld, i, n, y);
+    y *= p.a.mul;
     if (p.a.add) y += p.a.add[(size_t)i * p.a.add_ld + n];
-    p.a.out[(size_t)i * p.a.out_ld + n] = y;
+    p.a.out[((size_t)kRows * group + i) * p.a.out_ld + n] = y;
 }
 
 __global__ void __launch_bounds__(kThreads)
@@ -71,7 +85,14 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = blockIdx.x % p.split, n0 = (blockIdx.x / p.split) * kM;
     const uint32_t kb0 = p.k_blocks * rank / p.split, kb1 = p.k_blocks * (rank + 1) / p.split, nkb = kb1 - kb0;
+    const uint32_t group = blockIdx.y;
+    const char *blocks = static_cast<const char *>(p.w.blocks);
     pdl_trigger();
+    if (p.a.group.list) {                                // (the same answer in every CTA of a cluster)
+        pdl_wait();
+        if (group >= *p.a.group.count) return;
+        blocks += p.a.group.list[group] * p.a.group.stride;
+    }
     if (threadIdx.x == 0) {
         for (uint32_t i = 0; i < kStages; ++i) {
             mbar_init(&full[i], 1);
@@ -92,7 +113,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
             asm volatile("prefetch.tensormap [%0];" ::"l"(&x_map) : "memory");
             // the row tile's one or two blocks of weights
             const uint32_t nb = min(kM / kWBlock, wr_weight_blocks(p.w.n) - n0 / kWBlock);
-            const char *w = static_cast<const char *>(p.w.blocks) + ((size_t)(n0 / kWBlock) * p.k_blocks + kb0) * kWBlockBytes;
+            const char *w = blocks + ((size_t)(n0 / kWBlock) * p.k_blocks + kb0) * kWBlockBytes;
             const uint64_t policy = l2_policy_evict_first();         // streamed once
             auto weights = [&](uint32_t it) {
                 const uint32_t st = it % kStages;
@@ -104,7 +125,8 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
             };
             auto rows = [&](uint32_t it) {
                 const uint32_t st = it % kStages;
-                tc5::tma_load_2d(stages + st * kStageBytes + kABytes, &x_map, (int)((kb0 + it) * kBK), 0, &full[st]);
+                tc5::tma_load_2d(stages + st * kStageBytes + kABytes, &x_map, (int)((kb0 + it) * kBK), (int)(p.a.group.x_rows * group),
+                                 &full[st]);
             };
             bool ok = true;
             uint32_t it = 0;
@@ -163,7 +185,11 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
         if (warp >= 2) {
 #pragma unroll
             for (uint32_t i = 0; i < kRows; ++i)
-                if (i < p.a.rows) put(p, i, n0 + m, s[i]);
+                if (i < p.a.rows) {
+                    const float up = __shfl_xor_sync(0xffffffffu, s[i], 8);
+                    if (n0 + m < p.a.pair.from) put(p, group, i, n0 + m, s[i]);
+                    else if (!(m & 8u)) put_pair(p, group, i, n0 + m, s[i], up);
+                }
         }
     } else {
         // every rank lays its sums out in its own shared memory (its products are done with it) and finishes its
@@ -179,13 +205,17 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap x_map, const SkinnyParams
             const uint32_t share = kM / p.split;
             for (uint32_t j = threadIdx.x - 64; j < p.a.rows * share; j += kThreads - 64) {
                 const uint32_t i = j / share, mm = rank * share + j % share;
-                float v[kMaxSplit];
+                auto sum = [&](uint32_t at) {
+                    float v[kMaxSplit];
 #pragma unroll
-                for (uint32_t q = 0; q < kMaxSplit; ++q) v[q] = q < p.split ? load_rank(red + i * kM + mm, q) : 0.f;
-                float y = v[0];
+                    for (uint32_t q = 0; q < kMaxSplit; ++q) v[q] = q < p.split ? load_rank(red + i * kM + at, q) : 0.f;
+                    float y = v[0];
 #pragma unroll
-                for (uint32_t q = 1; q < kMaxSplit; ++q) y += v[q];      // (+0 beyond the last rank)
-                put(p, i, n0 + mm, y);
+                    for (uint32_t q = 1; q < kMaxSplit; ++q) y += v[q];  // (+0 beyond the last rank)
+                    return y;
+                };
+                if (n0 + mm < p.a.pair.from) put(p, group, i, n0 + mm, sum(mm));
+                else if (!(mm & 8u)) put_pair(p, group, i, n0 + mm, sum(mm), sum(mm + 8));
             }
         }
         cluster_arrive();                                // nobody leaves while its sums are being read
@@ -208,7 +238,8 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w,
     p.k_blocks = wr_weight_blocks(w.k);
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
-    const uint32_t tiles = (w.n + kM - 1) / kM;
+    if (a.pair.from != ~0u && (a.pair.from & 15u)) return WR_CUDA_ERR_INVAL;
+    const uint32_t tiles = (w.n + kM - 1) / kM, groups = a.group.list ? a.group.max : 1u;
     // two CTAs per SM where a slice still has a few blocks of K
     p.split = 1;
     while (p.split < kMaxSplit && tiles * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
@@ -218,7 +249,7 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w,
         ctx->attr_flags |= 128u;
     }
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(tiles * p.split);
+    cfg.gridDim = dim3(tiles * p.split, groups);
     cfg.blockDim = dim3(kThreads);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = ctx->stream;

@@ -24,6 +24,7 @@ struct GemvParams {
     uint32_t swiglu;       // seg[0] = gate, seg[1] = up: seg[0].out <- SiLU(gate) * up
     const float *bias;     // added to segment 0's result, or null
     uint32_t act;          // WR_GEMV_ACT_* on the result (after the bias)
+    float mul = 1.f;       // on the result before the residual
 };
 
 // Enqueue y[r][n] = sum_k W[n][k] x[r][k] on the context's stream (k a multiple of 4).  `width` is the output width

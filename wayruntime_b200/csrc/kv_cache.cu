@@ -296,7 +296,8 @@ extern "C" int wr_cuda_kv_create_layout(wr_cuda_ctx *ctx, uint32_t n_layers, con
     for (uint32_t L = 0; L < n_layers; ++L) {
         const wr_cuda_cache_layer &l = layers[L];
         if (l.n_kv_heads == 0) continue;
-        if (l.k_dim == 0 || l.v_dim == 0 || (l.elem != WR_CUDA_F32 && l.elem != WR_CUDA_F16)) return WR_CUDA_ERR_INVAL;
+        if (l.v_dim == 0 && l.elem == WR_CUDA_F16 && l.k_dim % 64) return WR_CUDA_ERR_INVAL;
+        if (l.k_dim == 0 || (l.elem != WR_CUDA_F32 && l.elem != WR_CUDA_F16)) return WR_CUDA_ERR_INVAL;
         if (l.k_dim > WR_CUDA_HEAD_DIM_MAX || l.v_dim > WR_CUDA_HEAD_DIM_MAX) return WR_CUDA_ERR_LIMIT;
     }
     std::lock_guard<std::mutex> g(ctx->lock);

@@ -10,166 +10,15 @@
 #include <algorithm>
 #include <type_traits>
 
-#include "mixers.cuh"
+#include "rows_dev.cuh"
 
 namespace {
-
-__device__ __forceinline__ float to_f32(float v) { return v; }
-__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ float to_f32(__half v) { return __half2float(v); }
-template <typename T> __device__ __forceinline__ T from_f32(float v);
-template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-template <> __device__ __forceinline__ __half from_f32<__half>(float v)
-{
-    return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f));
-}
-// (a few units in the last place: the exponential and the quotient are the short sequences)
-__device__ __forceinline__ float sigmoidf(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
-__device__ __forceinline__ float siluf(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
-
-// two F32 values in one 64-bit register: one issue slot for two elements
-__device__ __forceinline__ uint64_t pack2(float a, float b)
-{
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float &a, float &b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c)
-{
-    uint64_t d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b)
-{
-    uint64_t d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-
-// four / eight consecutive values (addresses aligned to the vector)
-__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
-__device__ __forceinline__ float4 load4(const __nv_bfloat16 *p)
-{
-    const uint2 u = *reinterpret_cast<const uint2 *>(p);
-    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
-                       __uint_as_float(u.y & 0xffff0000u));
-}
-__device__ __forceinline__ float4 load4(const __half *p)
-{
-    const uint2 u = *reinterpret_cast<const uint2 *>(p);
-    const float2 a = __half22float2(*reinterpret_cast<const __half2 *>(&u.x)), b = __half22float2(*reinterpret_cast<const __half2 *>(&u.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16 *p, float4 v)
-{
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
-}
-template <typename T> __device__ __forceinline__ void load8v(const T *p, float (&v)[8])
-{
-    const float4 a = load4(p), b = load4(p + 4);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-__device__ __forceinline__ void load8v(const __nv_bfloat16 *p, float (&v)[8])
-{
-    const uint4 u = *reinterpret_cast<const uint4 *>(p);
-    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        v[2 * i] = __uint_as_float(w[i] << 16);
-        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-    }
-}
-template <typename T> __device__ __forceinline__ void store8v(T *p, const float (&v)[8])
-{
-    store4(p, make_float4(v[0], v[1], v[2], v[3]));
-    store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
-}
-__device__ __forceinline__ void store8v(__nv_bfloat16 *p, const float (&v)[8])
-{
-    uint32_t w[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-        w[i] = *reinterpret_cast<const uint32_t *>(&h);
-    }
-    *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-}
-__device__ __forceinline__ void store8v(__half *p, const float (&v)[8])
-{
-    uint32_t w[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const __half2 h = __halves2half2(from_f32<__half>(v[2 * i]), from_f32<__half>(v[2 * i + 1]));
-        w[i] = *reinterpret_cast<const uint32_t *>(&h);
-    }
-    *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-}
-
-// Where a kernel leaves its rows: plain ones of type T, or (Split) F32 values as two BF16 numbers, the second
-// WR_CUDA_BATCH_MAX rows behind the first.
-struct Split {};
-template <typename T> struct Out {
-    T *p;
-    __device__ __forceinline__ Out(void *base, uint32_t row, uint32_t ld) : p(static_cast<T *>(base) + (size_t)row * ld) {}
-    __device__ __forceinline__ void put(uint32_t i, float v) const { p[i] = from_f32<T>(v); }
-    __device__ __forceinline__ void put4(uint32_t i, float4 v) const { store4(p + i, v); }
-    __device__ __forceinline__ void put8(uint32_t i, const float (&v)[8]) const { store8v(p + i, v); }
-};
-template <> struct Out<Split> {
-    __nv_bfloat16 *p;
-    size_t lo;
-    __device__ __forceinline__ Out(void *base, uint32_t row, uint32_t ld)
-        : p(static_cast<__nv_bfloat16 *>(base) + (size_t)row * ld), lo((size_t)WR_CUDA_BATCH_MAX * ld) {}
-    static __device__ __forceinline__ float rest(float v) { return v - __bfloat162float(__float2bfloat16_rn(v)); }
-    __device__ __forceinline__ void put(uint32_t i, float v) const
-    {
-        p[i] = __float2bfloat16_rn(v);
-        p[lo + i] = __float2bfloat16_rn(rest(v));
-    }
-    __device__ __forceinline__ void put4(uint32_t i, float4 v) const
-    {
-        store4(p + i, v);
-        store4(p + lo + i, make_float4(rest(v.x), rest(v.y), rest(v.z), rest(v.w)));
-    }
-    __device__ __forceinline__ void put8(uint32_t i, const float (&v)[8]) const
-    {
-        float r[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) r[e] = rest(v[e]);
-        store8v(p + i, v);
-        store8v(p + lo + i, r);
-    }
-};
-
-// the session of a row and the row's place among the session's tokens of this step
-__device__ __forceinline__ uint32_t seq_of(const wr_rows &rw, uint32_t row) { return rw.decode ? row : 0u; }
-__device__ __forceinline__ uint32_t tok_of(const wr_rows &rw, uint32_t row) { return rw.decode ? 0u : row; }
-__device__ __forceinline__ uint32_t row0_of(const wr_rows &rw, uint32_t seq) { return rw.decode ? seq : 0u; }
-
-__device__ __forceinline__ float warp_sum(float v)
-{
-#pragma unroll
-    for (int o = 16; o >= 1; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-
-int finish_launch(wr_cuda_ctx *ctx)
-{
-    ctx->launches++;
-    WR_CUDA_TRY(cudaGetLastError());
-    return WR_CUDA_OK;
-}
 
 // ------------------------------------------------------------------ embedding
 
 template <typename TW>
 __global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint32_t *tokens, const TW *table,
-                                                    const double *turns, float *x, uint32_t width)
+                                                    const double *turns, float *x, uint32_t width, float scale)
 {
     pdl_trigger();
     pdl_wait();
@@ -179,7 +28,7 @@ __global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint
     float *dst = x + (size_t)row * ld;
     // a pair of columns shares its angle; ld is even
     for (uint32_t i = 2 * (blockIdx.x * 256 + threadIdx.x); i < ld; i += 2 * gridDim.x * 256) {
-        float v0 = i < width ? to_f32(src[i]) : 0.f, v1 = i + 1 < width ? to_f32(src[i + 1]) : 0.f;
+        float v0 = i < width ? to_f32(src[i]) * scale : 0.f, v1 = i + 1 < width ? to_f32(src[i + 1]) * scale : 0.f;
         if (turns && i < width) {
             // the angle in turns, reduced before it leaves double: a position of 2^20 keeps its phase
             const double a = turns[i >> 1] * (double)pos;
@@ -196,17 +45,36 @@ __global__ void __launch_bounds__(256) embed_kernel(const wr_rows rw, const uint
 
 constexpr uint32_t kNormThreads = 256, kNormWarps = kNormThreads / 32;
 
-// 1 / root mean square of every group of a row -> inv[groups]; part: kNormWarps-strided partial sums
+// 1 / root mean square of every group of a row -> inv[groups], of its deviations from the group's mean -> mean[groups]
+// with `centre` (mean: zeros without); part: groups * split partial sums
 __device__ __forceinline__ void group_inv_rms(const float *x, uint32_t groups, uint32_t gs, uint32_t split, float eps,
-                                              float *part, float *inv)
+                                              bool centre, float *part, float *mean, float *inv)
 {
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t per = (gs + split - 1) / split;
+    if (centre) {
+        for (uint32_t u = warp; u < groups * split; u += kNormWarps) {
+            const uint32_t g = u / split, lo = (u % split) * per, hi = min(lo + per, gs);
+            const float *xg = x + (size_t)g * gs;
+            float s = 0.f;
+            for (uint32_t i = lo + lane; i < hi; i += 32) s += xg[i];
+            s = warp_sum(s);
+            if (lane == 0) part[u] = s;
+        }
+        __syncthreads();
+    }
+    for (uint32_t g = threadIdx.x; g < groups; g += kNormThreads) {
+        float s = 0.f;
+        for (uint32_t i = 0; centre && i < split; ++i) s += part[g * split + i];
+        mean[g] = s / (float)gs;
+    }
+    __syncthreads();
     for (uint32_t u = warp; u < groups * split; u += kNormWarps) {
         const uint32_t g = u / split, lo = (u % split) * per, hi = min(lo + per, gs);
         const float *xg = x + (size_t)g * gs;
         float ss = 0.f;
-        for (uint32_t i = lo + lane; i < hi; i += 32) ss = fmaf(xg[i], xg[i], ss);
+        const float m = mean[g];
+        for (uint32_t i = lo + lane; i < hi; i += 32) ss = fmaf(xg[i] - m, xg[i] - m, ss);
         ss = warp_sum(ss);
         if (lane == 0) part[u] = ss;
     }
@@ -223,16 +91,17 @@ template <typename TO>
 __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows rw, const wr_norm_args a, uint32_t split)
 {
     extern __shared__ float sm_norm[];
-    float *inv = sm_norm, *inv_before = inv + a.groups, *part = inv_before + a.groups;
+    float *inv = sm_norm, *inv_before = inv + a.groups, *mean = inv_before + a.groups, *mean_before = mean + a.groups,
+          *part = mean_before + a.groups;
     pdl_trigger();
     pdl_wait();
     const uint32_t row = blockIdx.x, ld = wr_ld(a.width), gs = a.width / a.groups;
     const float *x = a.x + (size_t)(a.gather ? a.gather[row] : row) * ld;
     const Out<TO> out(a.out, row, ld);
-    group_inv_rms(x, a.groups, gs, split, a.eps, part, inv);
+    group_inv_rms(x, a.groups, gs, split, a.eps, a.centre, part, mean, inv);
     if (!a.shift) {
         for (uint32_t i = threadIdx.x; i < ld; i += kNormThreads)
-            out.put(i, i < a.width ? x[i] * inv[i / gs] * a.w[i] : 0.f);
+            out.put(i, i < a.width ? (x[i] - mean[i / gs]) * inv[i / gs] * a.w[i] : 0.f);
         return;
     }
     // the mixer reads h + (h' - h) * shift with h' the token before: this step's previous row (its norm is
@@ -240,15 +109,15 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows 
     const wr_seq_dev s = rw.seqs[seq_of(rw, row)];
     const uint32_t t = tok_of(rw, row);
     const float *xb = x - ld;
-    if (t > 0) group_inv_rms(xb, a.groups, gs, split, a.eps, part, inv_before);
+    if (t > 0) group_inv_rms(xb, a.groups, gs, split, a.eps, a.centre, part, mean_before, inv_before);
     const float *kept = reinterpret_cast<const float *>(s.st_in + a.state_off);
     float *keep = reinterpret_cast<float *>(s.st_out + a.state_off);
     for (uint32_t i = threadIdx.x; i < ld; i += kNormThreads) {
         float y = 0.f;
         if (i < a.width) {
-            const float h = x[i] * inv[i / gs] * a.w[i];
+            const float h = (x[i] - mean[i / gs]) * inv[i / gs] * a.w[i];
             float before = 0.f;
-            if (t > 0) before = xb[i] * inv_before[i / gs] * a.w[i];
+            if (t > 0) before = (xb[i] - mean_before[i / gs]) * inv_before[i / gs] * a.w[i];
             else if (!s.fresh) before = kept[i];
             y = h + (before - h) * a.shift[i];
             if (t + 1 == s.n) keep[i] = h;
@@ -262,7 +131,7 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(const wr_rows 
 template <typename TO, int NW, int NV>
 __global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows rw, const wr_norm_args a)
 {
-    __shared__ float part[2][NW];
+    __shared__ float part[4][NW];
     pdl_trigger();
     const uint32_t row = blockIdx.x, ld = wr_ld(a.width), unit = a.width / NW, per_group = NW / a.groups;
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, at = warp * unit + 4 * lane;
@@ -299,6 +168,36 @@ __global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows r
                 else if (!fresh) b[i] = load4(kept + 128 * i);
             }
         }
+    }
+    const uint32_t g0 = warp / per_group * per_group;
+    const float gs = (float)(a.width / a.groups);
+    if (a.centre) {                                              // the group's mean comes off first (not off a kept row)
+        float s = 0.f, q = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+            q += (b[i].x + b[i].y) + (b[i].z + b[i].w);
+        }
+        s = warp_sum(s);
+        q = warp_sum(q);
+        if (lane == 0) { part[2][warp] = s; part[3][warp] = q; }
+        __syncthreads();
+        s = q = 0.f;
+        for (uint32_t i = 0; i < per_group; ++i) {
+            s += part[2][g0 + i];
+            q += part[3][g0 + i];
+        }
+        s /= gs;
+        q = t > 0 ? q / gs : 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (4 * lane + 128 * i < unit) {
+                v[i] = make_float4(v[i].x - s, v[i].y - s, v[i].z - s, v[i].w - s);
+                b[i] = make_float4(b[i].x - q, b[i].y - q, b[i].z - q, b[i].w - q);
+            }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
         ss = fmaf(v[i].w, v[i].w, fmaf(v[i].z, v[i].z, fmaf(v[i].y, v[i].y, fmaf(v[i].x, v[i].x, ss))));
         sb = fmaf(b[i].w, b[i].w, fmaf(b[i].z, b[i].z, fmaf(b[i].y, b[i].y, fmaf(b[i].x, b[i].x, sb))));
     }
@@ -306,8 +205,6 @@ __global__ void __launch_bounds__(NW * 32) group_norm_reg_kernel(const wr_rows r
     sb = warp_sum(sb);
     if (lane == 0) { part[0][warp] = ss; part[1][warp] = sb; }
     __syncthreads();
-    const uint32_t g0 = warp / per_group * per_group;
-    const float gs = (float)(a.width / a.groups);
     ss = sb = 0.f;
     for (uint32_t i = 0; i < per_group; ++i) {
         ss += part[0][g0 + i];
@@ -348,7 +245,7 @@ template <typename TO> cudaError_t norm_launch(wr_cuda_ctx *ctx, const wr_rows &
     cudaError_t e = cudaSuccess;
     if (rw.n_rows <= WR_CUDA_BATCH_MAX ? group_norm_reg<TO, 16>(ctx, rw, a, e) : group_norm_reg<TO, 8>(ctx, rw, a, e)) return e;
     const uint32_t split = std::max(1u, kNormWarps / a.groups);
-    const size_t smem = (size_t)(2 * a.groups + a.groups * split) * 4;
+    const size_t smem = (size_t)(4 * a.groups + a.groups * split) * 4;
     return wr_launch_pdl(group_norm_kernel<TO>, dim3(rw.n_rows), dim3(kNormThreads), smem, ctx->stream, rw, a, split);
 }
 
@@ -998,8 +895,9 @@ __global__ void __launch_bounds__(kAnyThreads) attn_rows_any_kernel(const wr_row
                                                                     const float *q, float *out)
 {
     extern __shared__ float sm_any[];
-    const uint32_t ks = g.kd | 1u, vs = g.vd;
-    float *Q = sm_any, *K = Q + kAnyRows * ks, *V = K + kAnyKeys * ks, *P = V + kAnyKeys * vs;      // P: [rows][33]
+    const uint32_t ks = g.kd | 1u, vs = g.shared ? ks : g.vd;
+    // P: [rows][33]; where the key's first columns are the value, one copy of the row serves both
+    float *Q = sm_any, *K = Q + kAnyRows * ks, *P = K + kAnyKeys * ks, *V = g.shared ? K : P + kAnyRows * (kAnyKeys + 1);
     pdl_trigger();
     pdl_wait();
     const wr_seq_dev s = rw.seqs[0];
@@ -1018,7 +916,7 @@ __global__ void __launch_bounds__(kAnyThreads) attn_rows_any_kernel(const wr_row
         const uint32_t nk = min(kAnyKeys, key_end - k0);
         __syncthreads();
         stage_rows(table, g.kv, head, 0, k0, nk, map * g.kd, g.kd, K, ks);
-        stage_rows(table, g.kv, head, 1, k0, nk, 0, g.vd, V, vs);
+        if (!g.shared) stage_rows(table, g.kv, head, 1, k0, nk, 0, g.vd, V, vs);
         __syncthreads();
         float sc[kAnyKeys / 4], mx = -INFINITY;
 #pragma unroll
@@ -1071,26 +969,29 @@ __global__ void __launch_bounds__(kAnyThreads) attn_rows_any_kernel(const wr_row
 }
 
 // Decode: a block is one chunk of keys of one (session, kv head) for all of the head's queries.  Partial rows
-// (m, l, o[vd]) go to ws[session][vq][chunk]; attn_merge_any_kernel adds them up in chunk order.
+// (m, l, o[vd]) go to ws[session][vq][chunk]; attn_merge_any_kernel adds them up in chunk order.  A head with many
+// queries is served by `parts` blocks of `per` queries each.
 constexpr uint32_t kChunkKeys = 256;
 
 __host__ __device__ inline uint32_t any_ws_stride(uint32_t vd) { return vd + 2u; }
 
 __global__ void __launch_bounds__(kAnyThreads) attn_chunk_any_kernel(const wr_rows rw, const wr_attn_geom g,
-                                                                     const float *q, float *ws, uint32_t chunks)
+                                                                     const float *q, float *ws, uint32_t chunks,
+                                                                     uint32_t parts, uint32_t per)
 {
     extern __shared__ float sm_any[];
-    const uint32_t nq = g.n_q / g.n_kv * g.maps, kw = g.maps * g.kd, ks = kw | 1u;
+    const uint32_t group = g.n_q / g.n_kv * g.maps, kw = g.maps * g.kd, ks = kw | 1u;
+    const uint32_t head = blockIdx.y / parts, v_lo = blockIdx.y % parts * per, nq = min(per, group - v_lo);
     float *Q = sm_any, *K = Q + nq * g.kd, *S = K + kAnyKeys * ks, *M = S + nq * kChunkKeys, *L = M + nq;
     pdl_trigger();
     pdl_wait();
-    const uint32_t chunk = blockIdx.x, head = blockIdx.y, seq = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t chunk = blockIdx.x, seq = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const wr_seq_dev s = rw.seqs[seq];
     const uint32_t len = s.pos + 1, lo = chunk * kChunkKeys;
     if (lo >= len) return;
     const uint32_t n = min(kChunkKeys, len - lo);
     const uint64_t *table = s.pages + (size_t)g.layer * s.n_pages;
-    const float *qrow = q + ((size_t)seq * g.vq() + head * nq) * g.kd;
+    const float *qrow = q + ((size_t)seq * g.vq() + head * group + v_lo) * g.kd;
     for (uint32_t i = threadIdx.x; i < nq * g.kd; i += kAnyThreads) Q[i] = qrow[i];
     for (uint32_t k0 = 0; k0 < n; k0 += kAnyKeys) {
         const uint32_t nk = min(kAnyKeys, n - k0);
@@ -1100,7 +1001,7 @@ __global__ void __launch_bounds__(kAnyThreads) attn_chunk_any_kernel(const wr_ro
         for (uint32_t i = threadIdx.x; i < nq * kAnyKeys; i += kAnyThreads) {
             const uint32_t v = i / kAnyKeys, k = i % kAnyKeys;
             if (k >= nk) continue;
-            const float *kr = K + k * ks + (v % g.maps) * g.kd, *qr = Q + v * g.kd;
+            const float *kr = K + k * ks + ((v_lo + v) % g.maps) * g.kd, *qr = Q + v * g.kd;
             float d = 0.f;
             for (uint32_t e = 0; e < g.kd; ++e) d = fmaf(qr[e], kr[e], d);
             S[v * kChunkKeys + k0 + k] = d;
@@ -1131,7 +1032,7 @@ __global__ void __launch_bounds__(kAnyThreads) attn_chunk_any_kernel(const wr_ro
             for (uint32_t k = 0; k < n; ++k) {
                 const uint32_t key = lo + k;
                 const char *p = reinterpret_cast<const char *>(table[key / kPageTokens]) +
-                                wr_geom_off(g.kv, head, 1, key % kPageTokens, c);
+                                wr_geom_off(g.kv, head, g.shared ? 0u : 1u, key % kPageTokens, c);
                 const float x = g.kv.elem == WR_CUDA_F32 ? *reinterpret_cast<const float *>(p)
                                                          : __half2float(*reinterpret_cast<const __half *>(p));
 #pragma unroll
@@ -1141,10 +1042,10 @@ __global__ void __launch_bounds__(kAnyThreads) attn_chunk_any_kernel(const wr_ro
 #pragma unroll
             for (uint32_t j = 0; j < B; ++j)
                 if (v0 + j < nq)
-                    ws[(((size_t)seq * g.vq() + head * nq + v0 + j) * chunks + chunk) * stride + 2 + c] = acc[j];
+                    ws[(((size_t)seq * g.vq() + head * group + v_lo + v0 + j) * chunks + chunk) * stride + 2 + c] = acc[j];
         }
     for (uint32_t v = threadIdx.x; v < nq; v += kAnyThreads) {
-        float *w = ws + (((size_t)seq * g.vq() + head * nq + v) * chunks + chunk) * stride;
+        float *w = ws + (((size_t)seq * g.vq() + head * group + v_lo + v) * chunks + chunk) * stride;
         w[0] = M[v];
         w[1] = L[v];
     }
@@ -1168,17 +1069,9 @@ __global__ void __launch_bounds__(128) attn_merge_any_kernel(const wr_rows rw, c
     }
 }
 
-template <typename K> int allow_smem(K k, size_t smem)
-{
-    if (smem > 227 * 1024) return WR_CUDA_ERR_LIMIT;
-    if (smem > 48 * 1024)
-        WR_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return WR_CUDA_OK;
-}
-
 template <int VC> int rows_any(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_geom &g, const float *q, float *out)
 {
-    const size_t smem = (size_t)(2 * kAnyRows * (g.kd | 1u) + kAnyKeys * g.vd + kAnyRows * (kAnyKeys + 1)) * 4;
+    const size_t smem = (size_t)(2 * kAnyRows * (g.kd | 1u) + (g.shared ? 0u : kAnyKeys * g.vd) + kAnyRows * (kAnyKeys + 1)) * 4;
     int rc = allow_smem(attn_rows_any_kernel<VC>, smem);
     if (rc != WR_CUDA_OK) return rc;
     WR_CUDA_TRY(wr_launch_pdl(attn_rows_any_kernel<VC>, dim3((rw.n_rows + kAnyRows - 1) / kAnyRows, g.vq()),
@@ -1189,13 +1082,13 @@ template <int VC> int rows_any(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_att
 }  // namespace
 
 int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens, const void *table, int table_type,
-                    const double *turns, float *x, uint32_t width)
+                    const double *turns, float *x, uint32_t width, float scale)
 {
     const dim3 grid((wr_ld(width) + 511) / 512, rw.n_rows);
     if (table_type == WR_ACT_BF16)
-        embed_kernel<__nv_bfloat16><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width);
+        embed_kernel<__nv_bfloat16><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const __nv_bfloat16 *)table, turns, x, width, scale);
     else
-        embed_kernel<float><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const float *)table, turns, x, width);
+        embed_kernel<float><<<grid, 256, 0, ctx->stream>>>(rw, tokens, (const float *)table, turns, x, width, scale);
     return finish_launch(ctx);
 }
 
@@ -1253,14 +1146,21 @@ int wr_attn_any_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_geom &
         if (g.vd <= 512) return rows_any<128>(ctx, rw, g, q, out);
         return WR_CUDA_ERR_LIMIT;
     }
-    const uint32_t nq = g.n_q / g.n_kv * g.maps, chunks = (max_len + kChunkKeys - 1) / kChunkKeys;
+    const uint32_t group = g.n_q / g.n_kv * g.maps, chunks = (max_len + kChunkKeys - 1) / kChunkKeys;
     int rc = wr_ctx_reserve_ws(ctx, (size_t)rw.n_seq * g.vq() * chunks * any_ws_stride(g.vd) * sizeof(float), 0);
     if (rc != WR_CUDA_OK) return rc;
-    const size_t smem = (size_t)(nq * g.kd + kAnyKeys * ((g.maps * g.kd) | 1u) + nq * kChunkKeys + 2 * nq) * 4;
+    auto bytes = [&](uint32_t nq) {
+        return (size_t)(nq * g.kd + kAnyKeys * ((g.maps * g.kd) | 1u) + nq * kChunkKeys + 2 * nq) * 4;
+    };
+    uint32_t parts = 1;
+    while (parts < group && bytes((group + parts - 1) / parts) > 200 * 1024) ++parts;
+    const uint32_t per = (group + parts - 1) / parts;
+    parts = (group + per - 1) / per;
+    const size_t smem = bytes(per);
     rc = allow_smem(attn_chunk_any_kernel, smem);
     if (rc != WR_CUDA_OK) return rc;
-    WR_CUDA_TRY(wr_launch_pdl(attn_chunk_any_kernel, dim3(chunks, g.n_kv, rw.n_seq), dim3(kAnyThreads), smem, ctx->stream,
-                              rw, g, q, ctx->ws, chunks));
+    WR_CUDA_TRY(wr_launch_pdl(attn_chunk_any_kernel, dim3(chunks, g.n_kv * parts, rw.n_seq), dim3(kAnyThreads), smem,
+                              ctx->stream, rw, g, q, ctx->ws, chunks, parts, per));
     rc = finish_launch(ctx);
     if (rc != WR_CUDA_OK) return rc;
     WR_CUDA_TRY(wr_launch_pdl(attn_merge_any_kernel, dim3(g.vq(), rw.n_seq), dim3(128), 0, ctx->stream, rw, g,

@@ -24,9 +24,9 @@ enum { WR_ACT_F32 = 0, WR_ACT_BF16 = 1, WR_ACT_F16 = 2, WR_ACT_SPLIT = 3 };    /
 
 __host__ __device__ inline uint32_t wr_ld(uint32_t n) { return (n + 7u) & ~7u; }   // row stride of n values
 
-// x[r] = table[token[r]] (+ sinusoidal position vector; turns[i] = frequency of pair i in turns per token)
+// x[r] = scale * table[token[r]] (+ sinusoidal position vector; turns[i] = frequency of pair i in turns per token)
 int wr_embed_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const uint32_t *tokens, const void *table, int table_type,
-                    const double *turns, float *x, uint32_t width);
+                    const double *turns, float *x, uint32_t width, float scale);
 
 struct wr_norm_args {
     const float *x;                  // [rows][wr_ld(width)]
@@ -35,6 +35,7 @@ struct wr_norm_args {
     uint64_t state_off;              // where the previous token's row is kept in the state (with shift)
     uint32_t width, groups;
     float eps;
+    bool centre;                     // layer norm: the group's mean comes off first
     void *out;                       // [rows][wr_ld(width)] of out_type
     int out_type;
 };
@@ -76,6 +77,7 @@ struct wr_attn_geom {
     uint32_t n_q, n_kv, maps, kd, vd;    // query heads, kv heads, maps per head, query/key size per map, value size
     uint32_t layer;                      // page-table layer
     wr_kv_geom kv;                       // the cache's layout (k_dim >= maps*kd, v_dim >= vd)
+    bool shared;                         // a key's first vd numbers are its value (v_dim 0 in the cache)
     bool hd128;                          // served by the head_dim-128 kernels: queries zero-padded to 128
     __host__ __device__ uint32_t vq() const { return n_q * maps; }               // queries per row
     __host__ __device__ uint32_t q_stride() const { return hd128 ? 128u : kd; }
@@ -105,3 +107,106 @@ struct wr_attn_finish_args {
     void *out; int out_type;         // [rows][wr_ld(n_q*vd)]
 };
 int wr_attn_finish_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_finish_args &a);
+
+// ---- attention over a latent (latent.cu)
+
+// Where the parts of a latent layer's rows lie: the cached row is [latent, padded to 64 | rotated key part, padded to
+// 64], a head's query [unrotated, padded to 16 | rotated, padded to 16].
+struct wr_latent_geom {
+    uint32_t heads, dim, rot, vdim, q_rank, kv_rank;
+    __host__ __device__ uint32_t dim_pad() const { return (dim + 15u) & ~15u; }
+    __host__ __device__ uint32_t rot_pad() const { return (rot + 15u) & ~15u; }
+    __host__ __device__ uint32_t vdim_pad() const { return (vdim + 15u) & ~15u; }
+    __host__ __device__ uint32_t q_head() const { return dim_pad() + rot_pad(); }
+    __host__ __device__ uint32_t rank_pad() const { return (kv_rank + 63u) & ~63u; }
+    __host__ __device__ uint32_t row() const { return rank_pad() + ((rot + 63u) & ~63u); }
+};
+
+// The projection's rows, normed and rotated: the query latent for the next product, and (own) the session's row.
+struct wr_latent_prep_args {
+    wr_latent_geom g;
+    const float *in;                 // [rows][ld]: query latent at 0, latent at c_off, rotated key part at r_off
+    uint32_t ld, c_off, r_off;
+    const float *q_norm, *c_norm;
+    float eps;
+    const double *turns;             // [rot/2] frequencies in turns per token
+    void *cq; int cq_type;           // [rows][wr_ld(q_rank)]
+    bool own;
+    uint32_t layer;                  // page-table layer
+    wr_kv_geom kv;
+};
+int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_prep_args &a);
+
+// Queries moved into the latent: out[row][head] = scale [w_uk^T q | rotated q], padded as the cached row.  w_uk: rows of
+// dim_pad() per head, F32 rows wr_ld(kv_rank) apart or F16 in blocks (wr_weight).
+struct wr_latent_query_args {
+    wr_latent_geom g;
+    const float *q;                  // [rows][heads][q_head()]
+    const void *w_uk; int w_type;    // WR_ACT_F32 / WR_ACT_F16
+    const double *turns;
+    float scale;
+    float *out;                      // [rows][heads][row()]
+};
+int wr_latent_query_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_query_args &a);
+
+// Latent attention rows back into values: out[row][head * vdim + v] = w_uv o; w_uv as w_uk, vdim_pad() rows per head.
+struct wr_latent_value_args {
+    wr_latent_geom g;
+    const float *o;                  // [rows][heads][kv_rank]
+    const void *w_uv; int w_type;
+    void *out; int out_type;         // [rows][out_ld]; the columns up to wr_ld(heads * vdim) are written
+    uint32_t out_ld;
+};
+int wr_latent_value_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_value_args &a);
+
+// ---- mixture of experts (moe.cu)
+
+// The chosen experts of every row and their weights, and the rows grouped by expert.  Many rows: expert e's (row, slot)
+// pairs take consecutive places from a multiple of `tile` on; list names the expert of each tile of places.  Few
+// rows: list names the experts somebody chose, and a pair's place is its expert's number in the list.
+struct wr_route_args {
+    const float *logits;             // [rows][ld]
+    uint32_t ld;
+    const float *bias;               // [experts]
+    uint32_t experts, top, tile;     // tile 0: few rows
+    float *weight;                   // [rows][top]
+    uint32_t *expert, *place;        // [rows][top]
+    uint32_t *row_of;                // [places]: the row at a place, ~0 where there is none (many rows)
+    uint32_t *list, *count;
+};
+inline uint32_t wr_route_tiles(uint32_t rows, uint32_t experts, uint32_t top, uint32_t tile)
+{
+    const uint32_t pairs = rows * top, used = experts < pairs ? experts : pairs;
+    return tile ? pairs / tile + used : used;
+}
+int wr_route_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_route_args &a);
+
+// out[place] = x[row_of[place]] (BF16 rows of ld values)
+int wr_moe_gather_launch(wr_cuda_ctx *ctx, const void *x, void *out, uint32_t ld, const uint32_t *row_of,
+                         const uint32_t *count, uint32_t max_tiles, uint32_t tile);
+
+// resid[row] += mul * sum over slots of weight * y[place], slots in order
+struct wr_combine_args {
+    const void *y; int type;         // [places][ld]; few rows: F32, place's row r at 16 place + r
+    uint32_t ld, width, top;
+    bool few;
+    const float *weight;
+    const uint32_t *place;
+    float mul;
+    float *resid;                    // [rows][ld]
+};
+int wr_moe_combine_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_combine_args &a);
+
+// F32 experts: out[place] = act(gate x, up x) (up != null) or gate x, tiles of kMoeTileF32 places; x rows through row_of
+// or (null) places themselves.
+constexpr uint32_t kMoeTileF32 = 32;
+struct wr_moe_f32_args {
+    const float *x, *gate, *up;      // weights of expert 0; those of expert e at e * stride floats
+    size_t stride;
+    uint32_t x_ld, n, k, out_ld;     // rows of weights wr_ld(k) apart
+    float alpha, limit;
+    const uint32_t *row_of, *list, *count;
+    uint32_t max_tiles;
+    float *out;
+};
+int wr_moe_f32_launch(wr_cuda_ctx *ctx, const wr_moe_f32_args &a);

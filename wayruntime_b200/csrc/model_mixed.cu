@@ -1,7 +1,7 @@
 // model_mixed.cu — the layer stack of models whose layers differ (wr_cuda_model_create_mixed).
 //
 // The stack is a run list over layers; each layer is norm -> (token shift) -> mixer -> residual, then
-// norm -> feed-forward -> residual.  An F32 model's projections are the products of gemv.cu.  A BF16 model's are
+// norm -> feed-forward -> residual, or (parallel) norm -> mixer + feed-forward -> residual.  An F32 model's projections are the products of gemv.cu.  A BF16 model's are
 // tensor-core products: steps of up to WR_CUDA_BATCH_MAX rows (every decode step, and short portions of a prompt)
 // keep F32 activations and take the weight-streaming one (gemm_skinny.cu), longer portions keep BF16 activations
 // and take gemm_bf16.cu.  The residual stream, norms, softmax and recurrences are F32 in all of them.
@@ -29,10 +29,13 @@ constexpr double kLog2e = 1.4426950408889634;
 
 size_t up256(size_t n) { return (n + 255u) & ~(size_t)255u; }
 
+constexpr uint32_t kMoeTile = 128;       // rows of a tile of gemm_bf16.cu
+
 struct Mat {                             // [n][k]: F32 rows wr_ld(k) apart, or BF16 blocks (wr_weight)
     const void *w = nullptr;
     uint32_t n = 0, k = 0;
     CUtensorMap x_map{}, xs_map{};       // BF16 models: its input rows, and its input as split rows
+    wr_pair_args pair;                   // BF16 models: gate and up rows side by side (where they lie, act)
 };
 
 struct Layer {
@@ -55,6 +58,26 @@ struct Layer {
     uint32_t ff = 0;
     Mat up, down;
     float act[4] = {0, 0, 0, 0}, ffn_eps = 0.f;
+    // gated feed-forward: gate and up rows are part of `first` and its down columns part of `o` where a latent
+    // layer's sublayers read one norm (fused); else products of their own.  F32: gate and `up` by themselves.
+    bool parallel = false, fused = false;
+    Mat gate;
+    uint32_t ff_at = 0;                  // where the feed-forward's values lie in a row of `o`'s input (fused)
+    // attention over a latent: `first` = [query latent | latent | rotated key part | router | gate and up]
+    wr_latent_geom lat{};
+    Mat first, uq;
+    const void *uk = nullptr, *uv = nullptr;
+    const float *q_norm = nullptr, *c_norm = nullptr;
+    const double *turns = nullptr;
+    uint32_t rot_off = 0, logit_off = 0, kv_from = 0;
+    float latent_eps = 0.f;
+    // mixture of experts: gate and up of all experts, down of all experts
+    uint32_t experts = 0, top = 0;
+    float alpha = 0.f, limit = 0.f;
+    Mat router, e_up, e_down;            // (n, k of one expert)
+    size_t up_stride = 0, down_stride = 0;                       // bytes; F32: gate, then up_at floats behind it up
+    size_t up_at = 0;
+    const float *router_b = nullptr;
     wr_cuda_cache_layer cache{};
 };
 
@@ -63,9 +86,10 @@ struct Layer {
 struct wr_mixed {
     int compute = WR_CUDA_F32;
     uint32_t width = 0, ldw = 0, max_rows = 0, groups = 1;
-    float eps = 0.f;
+    float eps = 0.f, embed_scale = 1.f, residual_mult = 1.f;
+    bool centre = false;                 // layer norm
     std::vector<Layer> layers;
-    std::vector<uint32_t> runs;
+    std::vector<uint32_t> runs, rows_of; // rows_of: the run whose cache a run reads
     std::vector<uint64_t> state_off;     // per run, inside a session's slot
     std::vector<wr_cuda_cache_layer> cache;
     uint64_t state_bytes = 0;
@@ -80,6 +104,13 @@ struct wr_mixed {
     float *resid = nullptr, *dbc = nullptr, *dt = nullptr, *attn = nullptr, *logits = nullptr, *normed = nullptr;
     float *conv_f32 = nullptr;           // few rows of a BF16 model: the convolution for the scan (mid has it split)
     void *xin = nullptr, *proj = nullptr, *mid = nullptr, *scan_out = nullptr, *q = nullptr, *dbc16 = nullptr, *head_in = nullptr;
+    // latent attention: first product's rows, query latent, queries in the latent, attended latents
+    float *lat = nullptr, *qa = nullptr, *olat = nullptr;
+    void *cq = nullptr;
+    // experts: choice, places, gathered inputs, activations, results
+    float *e_weight = nullptr;
+    uint32_t *e_expert = nullptr, *e_place = nullptr, *e_row_of = nullptr, *e_list = nullptr, *e_count = nullptr;
+    void *e_in = nullptr, *e_act = nullptr, *e_out = nullptr;
     uint32_t *tokens = nullptr, *gather = nullptr, *best = nullptr, *part_i = nullptr;
     float *part_v = nullptr;
     wr_seq_dev *seqs = nullptr;
@@ -105,17 +136,38 @@ uint16_t f32_to_bf16(float f)
     if ((u & 0x7fffffffu) > 0x7f800000u) return (uint16_t)((u >> 16) | 0x40u);
     return (uint16_t)((u + 0x7fffu + ((u >> 16) & 1u)) >> 16);
 }
+uint16_t f32_to_f16(float f)
+{
+    const __half h = __float2half_rn(std::min(std::max(f, -65504.f), 65504.f));
+    uint16_t u;
+    memcpy(&u, &h, 2);
+    return u;
+}
 float elem(const wr_cuda_tensor &t, size_t i)
 {
     return t.dtype == WR_CUDA_BF16 ? bf16_to_f32(static_cast<const uint16_t *>(t.data)[i])
                                    : static_cast<const float *>(t.data)[i];
 }
 
-// Rows [0, n) of a tensor at row `at` of a stacked weight.
+// Rows [row0, row0 + n) of a tensor at row `at` of a stacked weight, columns from `col` on.  Rows may come in groups that
+// lie `stride` apart, the rows of a group from `first` on at `second`.
 struct Part {
     const wr_cuda_tensor *t;
     uint32_t row0, n, at;
+    uint32_t col = 0, k = 0;             // k: the tensor's row length where it is not the stacked weight's
+    uint32_t group = ~0u, stride = 0, first = ~0u, second = 0;
+    uint32_t dst(uint32_t r) const
+    {
+        const uint32_t w = r % group;
+        return at + r / group * stride + (w < first ? w : second + w - first);
+    }
+    Part &in_groups(uint32_t g, uint32_t s, uint32_t f = ~0u, uint32_t f_at = 0)
+    {
+        group = g; stride = s; first = f; second = f_at;
+        return *this;
+    }
 };
+typedef std::vector<Part> Parts;
 
 // Weights are laid out in host memory first (sizes are known once everything is placed), then copied in one go.
 struct Packer {
@@ -140,33 +192,37 @@ struct Packer {
         return o;
     }
     // [rows][k] out of parts, zeros elsewhere: rows wr_ld(k) apart in `type` ...
-    size_t rows_of(std::initializer_list<Part> parts, uint32_t rows, uint32_t k, int type)
+    size_t rows_of(const Parts &parts, uint32_t rows, uint32_t k, int type)
     {
         const size_t ld = wr_ld(k), es = type == WR_CUDA_BF16 ? 2 : 4;
         const size_t o = place(((size_t)rows * ld) * es);
         for (const Part &p : parts)
             for (uint32_t r = 0; r < p.n; ++r) {
-                uint8_t *dst = buf.data() + o + (size_t)(p.at + r) * ld * es;
-                const size_t src = (size_t)(p.row0 + r) * k;
-                for (uint32_t i = 0; i < k; ++i) {
+                uint8_t *dst = buf.data() + o + ((size_t)p.dst(r) * ld + p.col) * es;
+                const uint32_t pk = p.k ? p.k : k;
+                const size_t src = (size_t)(p.row0 + r) * pk;
+                for (uint32_t i = 0; i < pk; ++i) {
                     if (type == WR_CUDA_BF16) reinterpret_cast<uint16_t *>(dst)[i] = bits(*p.t, src + i);
                     else reinterpret_cast<float *>(dst)[i] = elem(*p.t, src + i);
                 }
             }
         return o;
     }
-    // ... or, for the products of a BF16 model, in blocks (wr_weight)
-    size_t mat(std::initializer_list<Part> parts, uint32_t rows, uint32_t k, int type)
+    // ... or, for the products of a BF16 model, in blocks (wr_weight) of BF16 or F16 values
+    size_t mat(const Parts &parts, uint32_t rows, uint32_t k, int type)
     {
-        if (type != WR_CUDA_BF16) return rows_of(parts, rows, k, type);
+        if (type == WR_CUDA_F32) return rows_of(parts, rows, k, type);
         const size_t o = place(wr_weight_bytes(rows, k));
         for (const Part &p : parts)
             for (uint32_t r = 0; r < p.n; ++r) {
-                const size_t src = (size_t)(p.row0 + r) * k;
-                for (uint32_t i = 0; i < k; i += 8) {            // pieces of eight stay together
-                    uint16_t *dst = reinterpret_cast<uint16_t *>(buf.data() + o + wr_weight_off(k, p.at + r, i));
-                    const uint32_t n = std::min(8u, k - i);
-                    if (p.t->dtype == WR_CUDA_BF16) memcpy(dst, static_cast<const uint16_t *>(p.t->data) + src + i, n * 2);
+                const uint32_t pk = p.k ? p.k : k;
+                const size_t src = (size_t)(p.row0 + r) * pk;
+                for (uint32_t i = 0; i < pk; i += 8) {           // pieces of eight stay together (col: a multiple of 8)
+                    uint16_t *dst = reinterpret_cast<uint16_t *>(buf.data() + o + wr_weight_off(k, p.dst(r), p.col + i));
+                    const uint32_t n = std::min(8u, pk - i);
+                    if (type == WR_CUDA_F16)
+                        for (uint32_t e = 0; e < n; ++e) dst[e] = f32_to_f16(elem(*p.t, src + i + e));
+                    else if (p.t->dtype == WR_CUDA_BF16) memcpy(dst, static_cast<const uint16_t *>(p.t->data) + src + i, n * 2);
                     else
                         for (uint32_t e = 0; e < n; ++e) dst[e] = f32_to_bf16(elem(*p.t, src + i + e));
                 }
@@ -186,7 +242,8 @@ int check_layer(const wr_cuda_mixed_layer &l)
 {
     for (const wr_cuda_tensor *t : {&l.norm1, &l.norm2, &l.shift, &l.wq, &l.wk, &l.wv, &l.wo, &l.bq, &l.bk, &l.bv, &l.w_gate,
                                     &l.lq1, &l.lk1, &l.lq2, &l.lk2, &l.w_in, &l.conv, &l.conv_b, &l.w_x, &l.w_dt, &l.dt_b,
-                                    &l.a_log, &l.d, &l.w_out, &l.w_up, &l.w_down, &l.act})
+                                    &l.a_log, &l.d, &l.w_out, &l.w_up, &l.w_down, &l.act, &l.w_dq, &l.dq_norm, &l.w_uq, &l.w_dkv,
+                                    &l.dkv_norm, &l.w_uk, &l.w_uv, &l.w_gate_up, &l.router, &l.router_b})
         if (!valid(*t)) return WR_CUDA_ERR_INVAL;
     if (!has(l.norm1)) return WR_CUDA_ERR_INVAL;
     if (l.mixer == WR_CUDA_MIXER_ATTENTION) {
@@ -200,11 +257,28 @@ int check_layer(const wr_cuda_mixed_layer &l)
         if (!has(l.w_in) || !has(l.conv) || !has(l.w_x) || !has(l.w_dt) || !has(l.a_log) || !has(l.d) || !has(l.w_out))
             return WR_CUDA_ERR_INVAL;
         if (l.state > 512) return WR_CUDA_ERR_LIMIT;
+    } else if (l.mixer == WR_CUDA_MIXER_LATENT) {
+        if (!l.n_q_heads || !l.k_dim || !l.v_dim || !l.rot_dim || l.rot_dim % 2 || !l.q_rank || !l.kv_rank || !(l.rope_base > 0))
+            return WR_CUDA_ERR_INVAL;
+        if (!has(l.w_dq) || !has(l.dq_norm) || !has(l.w_uq) || !has(l.w_uk) || !has(l.w_uv) || !has(l.wo)) return WR_CUDA_ERR_INVAL;
+        if (!l.kv_from && (!has(l.w_dkv) || !has(l.dkv_norm))) return WR_CUDA_ERR_INVAL;
+        if (l.kv_rank > 512 || l.rot_dim > 256 || l.k_dim > WR_CUDA_HEAD_DIM_MAX || l.v_dim > WR_CUDA_HEAD_DIM_MAX)
+            return WR_CUDA_ERR_LIMIT;
     } else {
         return WR_CUDA_ERR_UNSUPPORTED;
     }
-    if (l.ffn == WR_CUDA_FFN_POLYNORM) {
-        if (!l.ffn_dim || !has(l.norm2) || !has(l.w_up) || !has(l.w_down) || !has(l.act)) return WR_CUDA_ERR_INVAL;
+    if (l.ffn != WR_CUDA_FFN_NONE && !l.parallel && !has(l.norm2)) return WR_CUDA_ERR_INVAL;
+    if (l.parallel && l.mixer != WR_CUDA_MIXER_LATENT && has(l.shift)) return WR_CUDA_ERR_UNSUPPORTED;
+    if (l.ffn == WR_CUDA_FFN_SWIGLU) {
+        if (!l.ffn_dim || !has(l.w_gate_up) || !has(l.w_up) || !has(l.w_down)) return WR_CUDA_ERR_INVAL;
+    } else if (l.ffn == WR_CUDA_FFN_MOE) {
+        if (!l.ffn_dim || !l.n_experts || !l.top_k || l.top_k > l.n_experts || !has(l.router) || !has(l.router_b) || !l.experts)
+            return WR_CUDA_ERR_INVAL;
+        if (l.n_experts > 2048) return WR_CUDA_ERR_LIMIT;
+        for (uint32_t i = 0; i < 3 * l.n_experts; ++i)
+            if (!has(l.experts[i]) || !valid(l.experts[i])) return WR_CUDA_ERR_INVAL;
+    } else if (l.ffn == WR_CUDA_FFN_POLYNORM) {
+        if (!l.ffn_dim || !has(l.w_up) || !has(l.w_down) || !has(l.act)) return WR_CUDA_ERR_INVAL;
     } else if (l.ffn != WR_CUDA_FFN_NONE) {
         return WR_CUDA_ERR_UNSUPPORTED;
     }
@@ -223,13 +297,23 @@ template <typename P> void set_off(P *&p, size_t off) { p = reinterpret_cast<P *
 
 void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t width, int type)
 {
-    auto mat = [&](Mat &m, std::initializer_list<Part> parts, uint32_t n, uint32_t k) {
+    auto mat = [&](Mat &m, const Parts &parts, uint32_t n, uint32_t k) {
         m.n = n;
         m.k = k;
         set_off(m.w, pk.mat(parts, n, k, type));
     };
+    const bool bf = type == WR_CUDA_BF16;
     o.mixer = l.mixer;
     o.ffn = l.ffn;
+    o.parallel = l.parallel != 0;
+    o.fused = o.parallel && l.mixer == WR_CUDA_MIXER_LATENT && l.ffn == WR_CUDA_FFN_SWIGLU;
+    o.ff = l.ffn == WR_CUDA_FFN_NONE ? 0 : l.ffn_dim;
+    // gate and up rows from row `at` of a weight on, eight of one and eight of the other
+    auto pairs = [&](Parts &p, const wr_cuda_tensor &gate, const wr_cuda_tensor &up, uint32_t at) {
+        p.push_back(Part{&gate, 0, l.ffn_dim, at}.in_groups(8, 16));
+        p.push_back(Part{&up, 0, l.ffn_dim, at + 8}.in_groups(8, 16));
+    };
+    const uint32_t pair_rows = 2 * wr_ld(l.ffn_dim);
     set_off(o.norm1, pk.vec(l.norm1, width));
     if (has(l.shift)) {
         set_off(o.shift, pk.vec(l.shift, width));
@@ -267,6 +351,60 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
         o.diff_eps = l.diff_eps;
         if (g.maps == 2)
             o.lambda = (float)(dot_exp(l.lq1, l.lk1, g.kd) - dot_exp(l.lq2, l.lk2, g.kd) + (double)l.diff_init);
+    } else if (l.mixer == WR_CUDA_MIXER_LATENT) {
+        wr_latent_geom &g = o.lat;
+        g = {l.n_q_heads, l.k_dim, l.rot_dim, l.v_dim, l.q_rank, l.kv_rank};
+        o.kv_from = l.kv_from;
+        o.latent_eps = l.latent_eps;
+        o.scale = l.attn_scale;
+        o.g.n_q = g.heads; o.g.n_kv = 1; o.g.maps = 1; o.g.kd = g.row(); o.g.vd = g.kv_rank; o.g.shared = true;
+        o.g.kv = {1, g.row(), 0, bf ? (uint32_t)WR_CUDA_F16 : (uint32_t)WR_CUDA_F32};
+        if (!l.kv_from) { o.cache.n_kv_heads = 1; o.cache.k_dim = g.row(); o.cache.elem = o.g.kv.elem; }
+        const bool moe = o.parallel && l.ffn == WR_CUDA_FFN_MOE;
+        Parts p = {{&l.w_dq, 0, g.q_rank, 0}};
+        uint32_t n = wr_ld(g.q_rank);
+        if (!l.kv_from) {
+            o.k_off = n;
+            o.rot_off = o.k_off + wr_ld(g.kv_rank);
+            n = o.rot_off + wr_ld(g.rot);
+            p.push_back({&l.w_dkv, 0, g.kv_rank, o.k_off});
+            p.push_back({&l.w_dkv, g.kv_rank, g.rot, o.rot_off});
+        }
+        if (moe) {
+            o.logit_off = n;
+            n += wr_ld(l.n_experts);
+            p.push_back({&l.router, 0, l.n_experts, o.logit_off});
+        }
+        o.proj_ld = n;
+        if (o.fused && bf) {
+            o.first.pair.from = n = (n + 15u) & ~15u;
+            pairs(p, l.w_gate_up, l.w_up, n);
+            n += pair_rows;
+        }
+        mat(o.first, p, n, width);
+        mat(o.uq, {Part{&l.w_uq, 0, g.heads * (g.dim + g.rot), 0}.in_groups(g.dim + g.rot, g.q_head(), g.dim, g.dim_pad())},
+            g.heads * g.q_head(), g.q_rank);
+        const int half = bf ? WR_CUDA_F16 : WR_CUDA_F32;
+        set_off(o.uk, pk.mat({Part{&l.w_uk, 0, g.heads * g.dim, 0}.in_groups(g.dim, g.dim_pad())}, g.heads * g.dim_pad(), g.kv_rank, half));
+        set_off(o.uv, pk.mat({Part{&l.w_uv, 0, g.heads * g.vdim, 0}.in_groups(g.vdim, g.vdim_pad())}, g.heads * g.vdim_pad(), g.kv_rank,
+                             half));
+        const uint32_t nv = g.heads * g.vdim;
+        if (o.fused) {
+            o.ff_at = wr_ld(nv);
+            Part a{&l.wo, 0, width, 0}, b{&l.w_down, 0, width, 0};
+            a.k = nv;
+            b.k = l.ffn_dim;
+            b.col = o.ff_at;
+            mat(o.o, {a, b}, width, o.ff_at + l.ffn_dim);
+        } else {
+            mat(o.o, {{&l.wo, 0, width, 0}}, width, nv);
+        }
+        set_off(o.q_norm, pk.vec(l.dq_norm, g.q_rank));
+        if (!l.kv_from) set_off(o.c_norm, pk.vec(l.dkv_norm, g.kv_rank));
+        const size_t t = pk.place((size_t)g.rot / 2 * 8);
+        for (uint32_t i = 0; i < g.rot / 2; ++i)
+            reinterpret_cast<double *>(pk.buf.data() + t)[i] = pow(l.rope_base, -2.0 * i / g.rot) / 6.283185307179586476925;
+        set_off(o.turns, t);
     } else {
         o.inner = l.inner; o.state = l.state; o.rank = l.dt_rank; o.taps = l.taps;
         const uint32_t ldi = wr_ld(l.inner), lds = wr_ld(l.state);
@@ -300,13 +438,51 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
         o.scan_off = o.conv_off + up256((size_t)(l.taps - 1) * ldi * 4);
         o.cache.state_bytes = o.scan_off + up256((size_t)l.inner * l.state * 4);
     }
+    if (l.ffn == WR_CUDA_FFN_NONE) return;
+    if (!o.parallel) set_off(o.norm2, pk.vec(l.norm2, width));
     if (l.ffn == WR_CUDA_FFN_POLYNORM) {
-        o.ff = l.ffn_dim;
         o.ffn_eps = l.ffn_eps;
-        set_off(o.norm2, pk.vec(l.norm2, width));
         mat(o.up, {{&l.w_up, 0, l.ffn_dim, 0}}, l.ffn_dim, width);
         mat(o.down, {{&l.w_down, 0, width, 0}}, width, l.ffn_dim);
         for (int i = 0; i < 4; ++i) o.act[i] = elem(l.act, i);
+    } else if (l.ffn == WR_CUDA_FFN_SWIGLU) {
+        if (!bf) {
+            mat(o.gate, {{&l.w_gate_up, 0, l.ffn_dim, 0}}, l.ffn_dim, width);
+            mat(o.up, {{&l.w_up, 0, l.ffn_dim, 0}}, l.ffn_dim, width);
+        } else if (!o.fused) {
+            Parts p;
+            pairs(p, l.w_gate_up, l.w_up, 0);
+            o.gate.pair.from = 0;
+            mat(o.gate, p, pair_rows, width);
+        }
+        if (!o.fused) mat(o.down, {{&l.w_down, 0, width, 0}}, width, l.ffn_dim);
+    } else {
+        o.experts = l.n_experts; o.top = l.top_k; o.alpha = l.moe_alpha; o.limit = l.moe_limit;
+        set_off(o.router_b, pk.vec(l.router_b, l.n_experts));
+        if (!(o.parallel && l.mixer == WR_CUDA_MIXER_LATENT)) mat(o.router, {{&l.router, 0, l.n_experts, 0}}, l.n_experts, width);
+        // expert after expert: every one takes a multiple of 256 bytes, so they lie one stride apart
+        for (uint32_t e = 0; e < l.n_experts; ++e) {
+            Parts p;
+            if (bf) pairs(p, l.experts[3 * e], l.experts[3 * e + 1], 0);
+            else p = {{&l.experts[3 * e], 0, l.ffn_dim, 0}, {&l.experts[3 * e + 1], 0, l.ffn_dim, l.ffn_dim}};
+            const size_t at = pk.mat(p, bf ? pair_rows : 2 * l.ffn_dim, width, type);
+            if (e == 0) set_off(o.e_up.w, at);
+            if (e == 1) o.up_stride = at - (reinterpret_cast<size_t>(o.e_up.w) - 1);
+        }
+        for (uint32_t e = 0; e < l.n_experts; ++e) {
+            const size_t at = pk.mat({{&l.experts[3 * e + 2], 0, width, 0}}, width, l.ffn_dim, type);
+            if (e == 0) set_off(o.e_down.w, at);
+            if (e == 1) o.down_stride = at - (reinterpret_cast<size_t>(o.e_down.w) - 1);
+        }
+        o.e_up.n = bf ? pair_rows : l.ffn_dim;
+        o.e_up.k = width;
+        o.up_at = (size_t)l.ffn_dim * wr_ld(width);
+        o.e_up.pair.from = 0;
+        o.e_up.pair.act = WR_PAIR_LIMITED;
+        o.e_up.pair.alpha = l.moe_alpha;
+        o.e_up.pair.limit = l.moe_limit;
+        o.e_down.n = width;
+        o.e_down.k = l.ffn_dim;
     }
 }
 
@@ -315,13 +491,14 @@ template <typename P> void fix(P *&p, const char *base)
     if (p) p = reinterpret_cast<P *>(const_cast<char *>(base) + (reinterpret_cast<size_t>(p) - 1));
 }
 
-int fix_mat(Mat &m, const wr_mixed &x, const void *input, uint32_t input_rows, uint32_t input_ld)
+int fix_mat(Mat &m, const wr_mixed &x, const void *input, uint32_t input_rows, uint32_t input_ld, const void *few_input = nullptr,
+            uint32_t groups = 1)
 {
     if (!m.w) return WR_CUDA_OK;
     fix(m.w, x.weights);
     if (x.compute != WR_CUDA_BF16) return WR_CUDA_OK;
     int rc = wr_gemm_map_rows(&m.x_map, input, input_rows, m.k, input_ld);
-    if (rc == WR_CUDA_OK) rc = wr_skinny_map_rows(&m.xs_map, input, m.k, input_ld);
+    if (rc == WR_CUDA_OK) rc = wr_skinny_map_rows(&m.xs_map, few_input ? few_input : input, m.k, input_ld, groups);
     return rc;
 }
 
@@ -346,6 +523,7 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
         return WR_CUDA_ERR_INVAL;
     if (d->compute != WR_CUDA_F32 && d->compute != WR_CUDA_BF16) return WR_CUDA_ERR_INVAL;
     if (d->width % d->norm_groups) return WR_CUDA_ERR_INVAL;
+    if (d->norm != WR_CUDA_NORM_RMS && d->norm != WR_CUDA_NORM_LAYER) return WR_CUDA_ERR_UNSUPPORTED;
     if (d->position != WR_CUDA_POS_NONE && d->position != WR_CUDA_POS_SINUSOIDAL) return WR_CUDA_ERR_UNSUPPORTED;
     if (d->n_runs > WR_CUDA_MAX_LAYER_RUNS) return WR_CUDA_ERR_LIMIT;
     for (uint32_t i = 0; i < d->n_runs; ++i)
@@ -353,6 +531,21 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
     for (uint32_t L = 0; L < d->n_layers; ++L) {
         const int rc = check_layer(d->layers[L]);
         if (rc != WR_CUDA_OK) return rc;
+    }
+    // a run that borrows reads the latest earlier run of the named layer, whose rows must be laid out like its own
+    std::vector<uint32_t> rows_of(d->n_runs);
+    for (uint32_t i = 0; i < d->n_runs; ++i) {
+        const wr_cuda_mixed_layer &l = d->layers[d->runs[i]];
+        rows_of[i] = i;
+        if (l.mixer != WR_CUDA_MIXER_LATENT || !l.kv_from) continue;
+        uint32_t r = i;
+        while (r > 0 && d->runs[r - 1] != l.kv_from - 1) --r;
+        if (r == 0) return WR_CUDA_ERR_INVAL;
+        const wr_cuda_mixed_layer &from = d->layers[l.kv_from - 1];
+        if (from.mixer != WR_CUDA_MIXER_LATENT || from.kv_from || from.kv_rank != l.kv_rank || from.rot_dim != l.rot_dim ||
+            from.rope_base != l.rope_base)
+            return WR_CUDA_ERR_INVAL;
+        rows_of[i] = r - 1;
     }
     std::lock_guard<std::mutex> g(ctx->lock);
     WR_CUDA_TRY(cudaSetDevice(ctx->device));
@@ -376,6 +569,10 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
     x->max_rows = d->max_rows;
     x->groups = d->norm_groups;
     x->eps = d->norm_eps;
+    x->centre = d->norm == WR_CUDA_NORM_LAYER;
+    x->embed_scale = d->embed_scale;
+    x->residual_mult = d->residual_mult;
+    x->rows_of = rows_of;
     x->runs.assign(d->runs, d->runs + d->n_runs);
 
     Packer pk;
@@ -405,6 +602,7 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
     // row scratch: what a step of few rows keeps in F32, a BF16 model's long step keeps in 16 bits
     const size_t R = std::max<uint32_t>(d->max_rows, WR_CUDA_BATCH_MAX), few = WR_CUDA_BATCH_MAX;
     size_t proj = 0, mid = x->ldw, q = 0, q_few = 0, att = 0, dbc = 0, scan = 0;
+    size_t lat = 0, cq = 0, qa = 0, olat = 0, e_top = 0, e_list = 0, e_rows = 0, e_in = 0, e_act = 0, e_out = 0;
     for (const Layer &l : x->layers) {
         if (l.mixer == WR_CUDA_MIXER_ATTENTION) {
             proj = std::max<size_t>(proj, l.proj_ld);
@@ -413,13 +611,33 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
             q_few = std::max(q_few, ql);
             q = std::max(q, l.g.hd128 ? ql * 2 : ql * 4);
             att = std::max<size_t>(att, (size_t)l.g.vq() * l.g.o_stride());
+        } else if (l.mixer == WR_CUDA_MIXER_LATENT) {
+            const wr_latent_geom &g = l.lat;
+            lat = std::max<size_t>(lat, l.proj_ld);
+            cq = std::max<size_t>(cq, wr_ld(g.q_rank));
+            q_few = std::max<size_t>(q_few, g.heads * g.q_head());
+            q = std::max<size_t>(q, (size_t)g.heads * g.q_head() * 4);
+            mid = std::max<size_t>(mid, wr_ld(l.o.k));
+            qa = std::max<size_t>(qa, (size_t)g.heads * g.row());
+            olat = std::max<size_t>(olat, (size_t)g.heads * g.kv_rank);
         } else {
             proj = std::max<size_t>(proj, 2 * wr_ld(l.inner));
             mid = std::max<size_t>(mid, wr_ld(l.inner));
             dbc = std::max<size_t>(dbc, l.dbc_ld);
             scan = std::max<size_t>(scan, wr_ld(l.inner));
         }
-        if (l.ff) {
+        if (l.experts) {
+            const uint32_t tile = bf ? kMoeTile : kMoeTileF32, tiles = wr_route_tiles((uint32_t)R, l.experts, l.top, tile);
+            const size_t places = (size_t)tiles * tile, groups = wr_route_tiles((uint32_t)few, l.experts, l.top, 0);
+            const size_t es = bf ? 2 : 4, lf = wr_ld(l.ff);
+            lat = std::max<size_t>(lat, wr_ld(l.experts));
+            e_top = std::max<size_t>(e_top, l.top);
+            e_list = std::max<size_t>(e_list, std::max<size_t>(tiles, groups));
+            e_rows = std::max<size_t>(e_rows, places);
+            if (bf) e_in = std::max<size_t>(e_in, places * x->ldw * 2);
+            e_act = std::max<size_t>(e_act, std::max(places * lf * es, bf ? groups * 2 * few * lf * 2 : 0));
+            e_out = std::max<size_t>(e_out, std::max(places * x->ldw * es, bf ? groups * few * x->ldw * 4 : 0));
+        } else if (l.ff) {
             proj = std::max<size_t>(proj, wr_ld(l.ff));
             mid = std::max<size_t>(mid, wr_ld(l.ff));
         }
@@ -430,6 +648,10 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
         {(void **)&x->resid, R * x->ldw * 4}, {&x->xin, act(x->ldw)}, {&x->proj, act(proj)},
         {&x->mid, act(mid)}, {&x->scan_out, act(scan)}, {&x->q, std::max(R * q, few * q_few * 4)}, {(void **)&x->attn, R * att * 4},
         {(void **)&x->dbc, R * dbc * 4}, {&x->dbc16, bf ? std::max(R, 2 * few) * dbc * 2 : 0},
+        {(void **)&x->lat, R * lat * 4}, {&x->cq, act(cq)}, {(void **)&x->qa, R * qa * 4}, {(void **)&x->olat, R * olat * 4},
+        {(void **)&x->e_weight, R * e_top * 4}, {(void **)&x->e_expert, R * e_top * 4}, {(void **)&x->e_place, R * e_top * 4},
+        {(void **)&x->e_row_of, e_rows * 4}, {(void **)&x->e_list, e_list * 4}, {(void **)&x->e_count, 4},
+        {&x->e_in, e_in}, {&x->e_act, e_act}, {&x->e_out, e_out},
         {(void **)&x->conv_f32, bf ? few * scan * 4 : 0}, {(void **)&x->dt, R * scan * 4},
         {&x->head_in, (size_t)kHeadRows * x->ldw * 4}, {(void **)&x->normed, (size_t)kHeadRows * x->ldw * 4},
         {(void **)&x->logits, (size_t)kHeadRows * ldv * 4}, {(void **)&x->tokens, R * 4}, {(void **)&x->gather, R * 4},
@@ -472,6 +694,19 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
         fix(l.norm1, x->weights); fix(l.norm2, x->weights); fix(l.shift, x->weights);
         fix(l.qkv_bias, x->weights); fix(l.conv, x->weights); fix(l.conv_b, x->weights); fix(l.dt_b, x->weights);
         fix(l.a2, x->weights); fix(l.d, x->weights);
+        fix(l.uk, x->weights); fix(l.uv, x->weights); fix(l.q_norm, x->weights); fix(l.c_norm, x->weights);
+        fix(l.turns, x->weights); fix(l.router_b, x->weights);
+        if (rc == WR_CUDA_OK) rc = fix_mat(l.first, *x, x->xin, rows, x->ldw);
+        if (rc == WR_CUDA_OK) rc = fix_mat(l.uq, *x, x->cq, rows, wr_ld(l.uq.k));
+        if (rc == WR_CUDA_OK) rc = fix_mat(l.gate, *x, x->xin, rows, x->ldw);
+        if (rc == WR_CUDA_OK) rc = fix_mat(l.router, *x, x->xin, rows, x->ldw);
+        if (rc == WR_CUDA_OK && l.experts) {
+            const uint32_t places = wr_route_tiles(rows, l.experts, l.top, kMoeTile) * kMoeTile;
+            rc = fix_mat(l.e_up, *x, x->e_in, places, x->ldw, x->xin);
+            if (rc == WR_CUDA_OK)
+                rc = fix_mat(l.e_down, *x, x->e_act, places, wr_ld(l.ff), x->e_act,
+                             wr_route_tiles((uint32_t)few, l.experts, l.top, 0));
+        }
         if (rc == WR_CUDA_OK) rc = fix_mat(l.qkvg, *x, x->xin, rows, x->ldw);
         if (rc == WR_CUDA_OK) rc = fix_mat(l.o, *x, x->mid, rows, wr_ld(l.o.k));
         if (rc == WR_CUDA_OK) rc = fix_mat(l.in, *x, x->xin, rows, x->ldw);
@@ -525,10 +760,16 @@ struct Step {
     int act() const { return wide ? WR_ACT_BF16 : WR_ACT_F32; }                              // a product's output rows
     int in_act() const { return split() ? (int)WR_ACT_SPLIT : act(); }                       // a product's input rows
 
-    // out = act(mat . in + bias) + add; `in` is the buffer the matrix's row maps were made for
+    // out = act(mat . in + bias) mul + add; `in` is the buffer the matrix's row maps were made for.  Gate / up rows of
+    // the matrix (BF16 models) go to pair_out.
     int product(const Mat &mat, const void *in, uint32_t in_ld, void *out, uint32_t out_ld, int out_type,
-                const float *bias = nullptr, bool softplus = false, const float *add = nullptr, void *copy16 = nullptr)
+                const float *bias = nullptr, bool softplus = false, const float *add = nullptr, void *copy16 = nullptr,
+                void *pair_out = nullptr, uint32_t pair_ld = 0)
     {
+        const float mul = add ? x->residual_mult : 1.f;
+        wr_pair_args pair = mat.pair;
+        pair.out = pair_out;
+        pair.ld = pair_ld;
         if (wide) {
             wr_gemm_args a{};
             a.m = rw.n_rows;
@@ -538,6 +779,8 @@ struct Step {
             a.bias = bias;
             a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
             a.add = add; a.add_ld = add ? out_ld : 0;
+            a.mul = mul;
+            a.pair = pair;
             ++m->launches;
             return wr_gemm_launch(ctx, mat.x_map, {mat.w, mat.n, mat.k}, a);
         }
@@ -550,6 +793,8 @@ struct Step {
             a.bias = bias;
             a.act = softplus ? WR_GEMM_ACT_SOFTPLUS : WR_GEMM_ACT_NONE;
             a.add = add; a.add_ld = out_ld;
+            a.mul = mul;
+            a.pair = pair;
             return wr_skinny_launch(ctx, mat.xs_map, {mat.w, mat.n, mat.k}, a);
         }
         GemvParams p{};
@@ -562,6 +807,7 @@ struct Step {
         p.add = add; p.add_stride = out_ld;
         p.bias = bias;
         p.act = softplus ? WR_GEMV_ACT_SOFTPLUS : WR_GEMV_ACT_NONE;
+        p.mul = mul;
         ctx->launches++;
         return wr_gemv_launch(ctx, p, mat.n);
     }
@@ -570,7 +816,7 @@ struct Step {
     {
         wr_norm_args a{};
         a.x = x->resid; a.w = w; a.shift = shift; a.state_off = state_off;
-        a.width = x->width; a.groups = x->groups; a.eps = x->eps;
+        a.width = x->width; a.groups = x->groups; a.eps = x->eps; a.centre = x->centre;
         a.out = x->xin; a.out_type = in_act();
         ++m->launches;
         return wr_group_norm_launch(ctx, rw, a);
@@ -641,16 +887,136 @@ struct Step {
         return product(l.out, x->scan_out, ldi, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
     }
 
+    int latent(const Layer &l, uint32_t run)
+    {
+        const wr_latent_geom &g = l.lat;
+        wr_attn_geom ag = l.g;
+        ag.layer = x->rows_of[run];
+        const bool own = x->rows_of[run] == run, bf = x->compute == WR_CUDA_BF16;
+        const uint32_t ld_o = wr_ld(l.o.k), es = wide || split() ? 2 : 4;
+        void *ff = l.fused ? static_cast<char *>(x->mid) + (size_t)l.ff_at * es : nullptr;
+        TRY(product(l.first, x->xin, x->ldw, x->lat, l.proj_ld, WR_ACT_F32, nullptr, false, nullptr, nullptr, ff, ld_o));
+        if (l.fused && !bf) TRY(gate_up_f32(l, static_cast<float *>(ff), ld_o));
+        wr_latent_prep_args p{};
+        p.g = g; p.in = x->lat; p.ld = l.proj_ld; p.c_off = l.k_off; p.r_off = l.rot_off;
+        p.q_norm = l.q_norm; p.c_norm = l.c_norm; p.eps = l.latent_eps; p.turns = l.turns;
+        p.cq = x->cq; p.cq_type = in_act(); p.own = own; p.layer = run; p.kv = l.g.kv;
+        TRY(wr_latent_prep_launch(ctx, rw, p));
+        TRY(product(l.uq, x->cq, wr_ld(g.q_rank), x->q, g.heads * g.q_head(), WR_ACT_F32));
+        wr_latent_query_args q{};
+        q.g = g; q.q = static_cast<const float *>(x->q); q.w_uk = l.uk; q.w_type = bf ? WR_ACT_F16 : WR_ACT_F32;
+        q.turns = l.turns; q.scale = l.scale; q.out = x->qa;
+        TRY(wr_latent_query_launch(ctx, rw, q));
+        TRY(wr_attn_any_launch(ctx, rw, ag, x->qa, x->olat, max_len));
+        wr_latent_value_args v{};
+        v.g = g; v.o = x->olat; v.w_uv = l.uv; v.w_type = q.w_type;
+        v.out = x->mid; v.out_type = in_act(); v.out_ld = ld_o;
+        TRY(wr_latent_value_launch(ctx, rw, v));
+        m->launches += 4;
+        return product(l.o, x->mid, ld_o, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
+    }
+
+    // F32 models: silu(gate h) * (up h)
+    int gate_up_f32(const Layer &l, float *out, uint32_t out_ld)
+    {
+        GemvParams p{};
+        p.seg[0] = {static_cast<const float *>(l.gate.w), out, l.ff, out_ld};
+        p.seg[1] = {static_cast<const float *>(l.up.w), nullptr, l.ff, out_ld};
+        p.n_seg = 2;
+        p.swiglu = 1;
+        p.x = static_cast<const float *>(x->xin);
+        p.x_stride = x->ldw;
+        p.k = x->ldw;
+        p.rows = rw.n_rows;
+        ctx->launches++;
+        ++m->launches;
+        return wr_gemv_launch(ctx, p, l.ff);
+    }
+
     int feed_forward(const Layer &l)
     {
-        TRY(norm(l.norm2, nullptr, 0));
-        TRY(product(l.up, x->xin, x->ldw, x->proj, wr_ld(l.ff), act()));
-        wr_polynorm_args p{};
-        p.z = x->proj; p.z_type = act(); p.out = x->mid; p.out_type = in_act(); p.ff = l.ff;
-        p.a = l.act[0]; p.b = l.act[1]; p.c = l.act[2]; p.e = l.act[3]; p.eps = l.ffn_eps;
-        ++m->launches;
-        TRY(wr_polynorm_launch(ctx, rw, p));
-        return product(l.down, x->mid, wr_ld(l.ff), x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
+        if (!l.parallel) TRY(norm(l.norm2, nullptr, 0));
+        if (l.ffn == WR_CUDA_FFN_MOE) return experts(l);
+        const uint32_t ld = wr_ld(l.ff);
+        if (l.ffn == WR_CUDA_FFN_SWIGLU) {
+            if (x->compute != WR_CUDA_BF16) TRY(gate_up_f32(l, static_cast<float *>(x->mid), ld));
+            else TRY(product(l.gate, x->xin, x->ldw, nullptr, 8, WR_ACT_F32, nullptr, false, nullptr, nullptr, x->mid, ld));
+        } else {
+            TRY(product(l.up, x->xin, x->ldw, x->proj, ld, act()));
+            wr_polynorm_args p{};
+            p.z = x->proj; p.z_type = act(); p.out = x->mid; p.out_type = in_act(); p.ff = l.ff;
+            p.a = l.act[0]; p.b = l.act[1]; p.c = l.act[2]; p.e = l.act[3]; p.eps = l.ffn_eps;
+            ++m->launches;
+            TRY(wr_polynorm_launch(ctx, rw, p));
+        }
+        return product(l.down, x->mid, ld, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
+    }
+
+    int experts(const Layer &l)
+    {
+        uint32_t ld = l.proj_ld, off = l.logit_off;
+        if (l.router.w) {
+            ld = wr_ld(l.experts);
+            off = 0;
+            TRY(product(l.router, x->xin, x->ldw, x->lat, ld, WR_ACT_F32));
+        }
+        const bool bf = x->compute == WR_CUDA_BF16;
+        wr_route_args r{};
+        r.logits = x->lat + off; r.ld = ld; r.bias = l.router_b; r.experts = l.experts; r.top = l.top;
+        r.tile = split() ? 0 : bf ? kMoeTile : kMoeTileF32;
+        r.weight = x->e_weight; r.expert = x->e_expert; r.place = x->e_place; r.row_of = x->e_row_of;
+        r.list = x->e_list; r.count = x->e_count;
+        TRY(wr_route_launch(ctx, rw, r));
+        const uint32_t groups = wr_route_tiles(rw.n_rows, l.experts, l.top, r.tile), lf = wr_ld(l.ff);
+        wr_group_args gr;
+        gr.list = x->e_list; gr.count = x->e_count; gr.max = groups;
+        wr_combine_args c{};
+        if (split()) {
+            wr_skinny_args a{};
+            a.rows = rw.n_rows;
+            a.pair = l.e_up.pair; a.pair.out = x->e_act; a.pair.ld = lf;
+            a.group = gr; a.group.stride = l.up_stride;
+            TRY(wr_skinny_launch(ctx, l.e_up.xs_map, {l.e_up.w, l.e_up.n, l.e_up.k}, a));
+            wr_skinny_args b{};
+            b.rows = rw.n_rows;
+            b.out = static_cast<float *>(x->e_out); b.out_ld = x->ldw;
+            b.group = gr; b.group.stride = l.down_stride; b.group.x_rows = 2 * WR_CUDA_BATCH_MAX;
+            TRY(wr_skinny_launch(ctx, l.e_down.xs_map, {l.e_down.w, l.e_down.n, l.e_down.k}, b));
+            c.type = WR_ACT_F32;
+            c.few = true;
+        } else if (bf) {
+            TRY(wr_moe_gather_launch(ctx, x->xin, x->e_in, x->ldw, x->e_row_of, x->e_count, groups, kMoeTile));
+            wr_gemm_args a{};
+            a.m = groups * kMoeTile;
+            a.pair = l.e_up.pair; a.pair.out = x->e_act; a.pair.ld = lf;
+            a.group = gr; a.group.stride = l.up_stride;
+            TRY(wr_gemm_launch(ctx, l.e_up.x_map, {l.e_up.w, l.e_up.n, l.e_up.k}, a));
+            wr_gemm_args b{};
+            b.m = groups * kMoeTile;
+            b.out = x->e_out; b.out_ld = x->ldw; b.out_type = WR_GEMM_OUT_BF16;
+            b.group = gr; b.group.stride = l.down_stride;
+            TRY(wr_gemm_launch(ctx, l.e_down.x_map, {l.e_down.w, l.e_down.n, l.e_down.k}, b));
+            c.type = WR_ACT_BF16;
+            ++m->launches;
+        } else {
+            wr_moe_f32_args a{};
+            a.x = static_cast<const float *>(x->xin); a.x_ld = x->ldw; a.n = l.ff; a.k = x->width;
+            a.gate = static_cast<const float *>(l.e_up.w); a.up = a.gate + l.up_at; a.stride = l.up_stride / 4;
+            a.row_of = x->e_row_of; a.list = x->e_list; a.count = x->e_count; a.max_tiles = groups;
+            a.alpha = l.alpha; a.limit = l.limit;
+            a.out = static_cast<float *>(x->e_act); a.out_ld = lf;
+            TRY(wr_moe_f32_launch(ctx, a));
+            wr_moe_f32_args b = a;
+            b.x = a.out; b.x_ld = lf; b.n = x->width; b.k = l.ff; b.row_of = nullptr;
+            b.gate = static_cast<const float *>(l.e_down.w); b.up = nullptr; b.stride = l.down_stride / 4;
+            b.out = static_cast<float *>(x->e_out); b.out_ld = x->ldw;
+            TRY(wr_moe_f32_launch(ctx, b));
+            c.type = WR_ACT_F32;
+        }
+        c.y = x->e_out; c.ld = x->ldw; c.width = x->width; c.top = l.top; c.weight = x->e_weight; c.place = x->e_place;
+        c.mul = x->residual_mult; c.resid = x->resid;
+        m->launches += 4;
+        return wr_moe_combine_launch(ctx, rw, c);
     }
 };
 
@@ -682,8 +1048,9 @@ int wr_mixed_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t n_ro
         for (uint32_t t = 0; t < s; ++t)
             if (kv[t] == kv[s]) return WR_CUDA_ERR_INVAL;
         for (uint32_t i = 0; i < kv[s]->n_layers; ++i) {
-            const wr_kv_geom &a = kv[s]->layers[i].geom, &b = x->layers[x->runs[i]].g.kv;
-            if (a.n_kv != b.n_kv || (a.n_kv && (a.k_dim != b.k_dim || a.v_dim != b.v_dim || a.elem != b.elem)))
+            const wr_kv_geom &a = kv[s]->layers[i].geom;
+            const wr_cuda_cache_layer &b = x->cache[i];
+            if (a.n_kv != b.n_kv_heads || (a.n_kv && (a.k_dim != b.k_dim || a.v_dim != b.v_dim || a.elem != b.elem)))
                 return WR_CUDA_ERR_INVAL;
         }
         if ((uint64_t)positions[s] + per_seq > kv[s]->max_ctx) return WR_CUDA_ERR_CTX_FULL;
@@ -720,15 +1087,16 @@ int wr_mixed_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t n_ro
     step.rw = {x->seqs, n_rows, n_seq, decode ? 1u : 0u};
     step.wide = bf && n_rows > WR_CUDA_BATCH_MAX;
     step.lock = &lock;
-    TRY(wr_embed_launch(ctx, step.rw, x->tokens, x->embed, bf ? WR_ACT_BF16 : WR_ACT_F32, x->turns, x->resid, x->width));
+    TRY(wr_embed_launch(ctx, step.rw, x->tokens, x->embed, bf ? WR_ACT_BF16 : WR_ACT_F32, x->turns, x->resid, x->width, x->embed_scale));
     ++m->launches;
     const size_t row_bytes = (size_t)x->width * 4, ld_bytes = (size_t)x->ldw * 4;
     for (uint32_t i = 0; i < x->runs.size(); ++i) {
         const Layer &l = x->layers[x->runs[i]];
         TRY(step.norm(l.norm1, l.shift, x->state_off[i]));
         if (l.mixer == WR_CUDA_MIXER_ATTENTION) TRY(step.attention(l, i));
+        else if (l.mixer == WR_CUDA_MIXER_LATENT) TRY(step.latent(l, i));
         else TRY(step.mamba1(l, x->state_off[i]));
-        if (l.ffn != WR_CUDA_FFN_NONE) TRY(step.feed_forward(l));
+        if (l.ffn != WR_CUDA_FFN_NONE && !l.fused) TRY(step.feed_forward(l));
         if (x->hidden_tap)
             WR_CUDA_TRY(cudaMemcpy2DAsync(x->hidden_tap + (size_t)i * n_rows * x->width, row_bytes, x->resid, ld_bytes,
                                           row_bytes, n_rows, cudaMemcpyDeviceToHost, st));
@@ -749,7 +1117,7 @@ int wr_mixed_forward(wr_cuda_ctx *ctx, wr_cuda_model *m, int mode, uint32_t n_ro
             head.wide = bf && head.rw.n_rows > WR_CUDA_BATCH_MAX;
             wr_norm_args a{};
             a.x = x->resid; a.gather = x->gather + done; a.w = x->final_norm;
-            a.width = x->width; a.groups = x->groups; a.eps = x->eps;
+            a.width = x->width; a.groups = x->groups; a.eps = x->eps; a.centre = x->centre;
             a.out = x->head_in; a.out_type = head.in_act();
             if (logits_out || argmax_out) {
                 TRY(wr_group_norm_launch(ctx, head.rw, a));

@@ -49,7 +49,8 @@ __host__ __device__ inline uint32_t wr_elem_off(uint32_t tok, uint32_t d, uint32
 }
 // Geometry of one layer's pages.  Usually K and V rows are F16 and equally long (the layout above); a
 // layer may also keep K and V rows of different lengths, or F32 rows: its pages are then
-// [kv_head][64 tok][pad8(k_dim)] K rows followed by [64 tok][pad8(v_dim)] V rows, never swizzled.
+// [kv_head][64 tok][pad8(k_dim)] K rows followed by [64 tok][pad8(v_dim)] V rows, never swizzled.  A layer
+// whose rows are key and value in one (v_dim 0) keeps F16 rows in the tiled blocks of the layout above.
 struct wr_kv_geom {
     uint32_t n_kv, k_dim, v_dim, elem;                   // elem: WR_CUDA_F32 / WR_CUDA_F16
 };
@@ -70,7 +71,7 @@ __host__ __device__ inline uint64_t wr_geom_off(const wr_kv_geom &g, uint32_t he
     const uint32_t es = wr_geom_esize(g), dim = which ? g.v_dim : g.k_dim;
     uint64_t off = head * wr_geom_head_bytes(g);
     if (which) off += (uint64_t)kPageTokens * wr_hd_pad(g.k_dim) * es;
-    if (wr_geom_uniform(g)) return off + wr_elem_off(tok, d, dim);
+    if (wr_geom_uniform(g) || (g.elem == WR_CUDA_F16 && g.v_dim == 0)) return off + wr_elem_off(tok, d, dim);
     return off + ((uint64_t)tok * wr_hd_pad(dim) + d) * es;
 }
 // Byte offset of the (head, which) block inside a page; which: 0 = K, 1 = V.

@@ -163,3 +163,81 @@ def tumadra(ctx, c, w, dtype, max_rows):
     return B.MixedModel(ctx, layers, layer_runs(len(layers), c.get("loop")), tensor, compute=DTYPES[dtype], width=width,
                         vocab=vocab, norm_groups=c["norm"]["groups"], norm_eps=eps, position=B.POS_SINUSOIDAL,
                         position_base=SINUSOIDAL_BASE, max_rows=max_rows)
+
+
+# ---- Nurosun on the mixed layer stack
+
+EXPERT_ALPHA = 1.702
+_LATENT = {
+    "w_dq": ("mix.dq", lambda s, d: (s["q_rank"], d)), "dq_norm": ("mix.dq.norm", lambda s, d: (s["q_rank"],)),
+    "w_uq": ("mix.uq", lambda s, d: (s["n_q_heads"] * (s["k_dim"] + s["rot_dim"]), s["q_rank"])),
+    "w_uk": ("mix.uk", lambda s, d: (s["n_q_heads"] * s["k_dim"], s["kv_rank"])),
+    "w_uv": ("mix.uv", lambda s, d: (s["n_q_heads"] * s["v_dim"], s["kv_rank"])),
+    "wo": ("mix.o", lambda s, d: (d, s["n_q_heads"] * s["v_dim"])),
+}
+_LATENT_ROWS = {
+    "w_dkv": ("mix.dkv", lambda s, d: (s["kv_rank"] + s["rot_dim"], d)), "dkv_norm": ("mix.dkv.norm", lambda s, d: (s["kv_rank"],)),
+}
+_SWIGLU = {
+    "w_gate_up": ("mlp.gate", lambda s, d: (s["ffn_dim"], d)), "w_up": ("mlp.up", lambda s, d: (s["ffn_dim"], d)),
+    "w_down": ("mlp.down", lambda s, d: (d, s["ffn_dim"])),
+}
+_MOE = {
+    "router": ("mlp.router", lambda s, d: (s["n_experts"], d)), "router_b": ("mlp.router.b", lambda s, d: (s["n_experts"],)),
+}
+
+
+@register("Nurosun")
+def nurosun(ctx, c, w, dtype, max_rows):
+    """Layer-norm decoder with parallel sublayers: latent attention with rotary positions, whose rows a later layer
+    may borrow, beside a SwiGLU feed-forward, a mixture of limited experts, or nothing."""
+    width, vocab = c["width"], c["vocab"]
+    eps = float(c["norm"]["eps"])
+    layers, fields = [], []
+    for i, lay in enumerate(c["layers"]):
+        mx, f = lay["mixer"], {"norm1": ("norm1", lambda s, d: (d,)), **_LATENT}
+        if lay["type"] != "latent_attention":
+            raise CheckpointError(f"layer {i} has an unknown mixer {lay['type']!r}")
+        if mx["rot"]["dims"] != mx["rot_dim"]:
+            raise CheckpointError(f"layer {i} rotates {mx['rot']['dims']} of {mx['rot_dim']} dimensions")
+        s = dict(mixer=B.MIXER_LATENT, parallel=1, n_q_heads=mx["heads"], k_dim=mx["dim"], v_dim=mx["vdim"], rot_dim=mx["rot_dim"],
+                 q_rank=mx["q_rank"], kv_rank=mx["kv_rank"], rope_base=mx["rot"]["base"], attn_scale=mx["scale"], latent_eps=eps)
+        source = mx.get("kv_from")
+        if source is None:
+            f.update(_LATENT_ROWS)
+        else:
+            if not 0 <= source < i or c["layers"][source]["mixer"].get("kv_from") is not None:
+                raise CheckpointError(f"layer {i} takes its rows from layer {source}, which has none of its own before it")
+            theirs = c["layers"][source]["mixer"]
+            if any(theirs[k] != mx[k] for k in ("kv_rank", "rot_dim", "rot")):
+                raise CheckpointError(f"the rows of layers {i} and {source} differ")
+            s["kv_from"] = source + 1
+        mlp = lay.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            s.update(ffn=B.FFN_SWIGLU, ffn_dim=mlp["ff"])
+            f.update(_SWIGLU)
+        elif mlp and mlp["kind"] == "moe":
+            s.update(ffn=B.FFN_MOE, ffn_dim=mlp["expert"]["ff"], n_experts=mlp["router"]["experts"], top_k=mlp["router"]["top"],
+                     moe_alpha=EXPERT_ALPHA, moe_limit=mlp["expert"]["limit"])
+            f.update(_MOE)
+        elif mlp:
+            raise CheckpointError(f"layer {i} has an unknown feed-forward {mlp['kind']!r}")
+        layers.append(s)
+        fields.append(f)
+    top = {"embed": ("embed", (vocab, width)), "head": ("head", (vocab, width)), "final_norm": ("final.norm", (width,))}
+
+    def tensor(i, field):
+        if i is None:
+            return w.get(*top[field])
+        if field == "experts":
+            ff = layers[i]["ffn_dim"]
+            return [w.get(f"l{i}.mlp.e{e}.{n}", shape) for e in range(layers[i]["n_experts"])
+                    for n, shape in (("gate", (ff, width)), ("up", (ff, width)), ("down", (width, ff)))]
+        if field not in fields[i]:
+            return None
+        name, shape = fields[i][field]
+        return w.get(f"l{i}.{name}", shape(layers[i], width))
+
+    return B.MixedModel(ctx, layers, list(range(len(layers))), tensor, compute=DTYPES[dtype], width=width, vocab=vocab,
+                        norm_groups=1, norm_eps=eps, norm=B.NORM_LAYER, embed_scale=c["embedding"]["scale"],
+                        residual_mult=c["residual_mult"], max_rows=max_rows)
