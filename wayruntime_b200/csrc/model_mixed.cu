@@ -375,9 +375,10 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
             n += wr_ld(l.n_experts);
             p.push_back({&l.router, 0, l.n_experts, o.logit_off});
         }
-        o.proj_ld = n;
+        if (o.fused && bf) n = (n + 15u) & ~15u;
+        o.proj_ld = n;                                   // (the plain rows' outputs, zeros up to the first pair included)
         if (o.fused && bf) {
-            o.first.pair.from = n = (n + 15u) & ~15u;
+            o.first.pair.from = n;
             pairs(p, l.w_gate_up, l.w_up, n);
             n += pair_rows;
         }
