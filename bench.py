@@ -648,7 +648,7 @@ def measure_whole_model():
     return out
 
 
-# ---- models whose layers differ (Tumadra), beside the dense stack at the same width, depth and widths of the parts
+# ---- models whose layers differ (Tumadra, Nurosun), beside the dense stack at the same width, depth and widths of the parts
 
 MIXED_SIZES = {
     # name: width, layers, ff, query heads, kv heads, inner, dt_rank, vocab
@@ -691,6 +691,19 @@ def mixed_config(size):
             "layers": [attn if i % 2 else scan for i in range(n)]}
 
 
+def latent_config(size):
+    """Nurosun: pairs of a layer with rows of its own and a dense feed-forward, and one that borrows them and has
+    experts, of which a token uses as much as the dense layer is wide."""
+    width, n, ff, heads, _kv, _inner, _rank, vocab = MIXED_SIZES[size]
+    mixer = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": width // 2, "kv_rank": 512, "scale": 192 ** -0.5,
+             "rot": {"base": 10000.0, "dims": 64}}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": 32, "top": 4}}
+    layers = [{"type": "latent_attention", "mixer": dict(mixer, kv_from=i - 1), "mlp": moe} if i % 2 else
+              {"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}} for i in range(n)]
+    return {"architecture": "Nurosun", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "residual_mult": 0.5, "layers": layers}
+
+
 def dense_config(size):
     width, n, ff, heads, kv, _inner, _rank, vocab = MIXED_SIZES[size]
     return {"architectures": ["Qwen3ForCausalLM"], "hidden_size": width, "intermediate_size": ff, "num_hidden_layers": n,
@@ -699,7 +712,7 @@ def dense_config(size):
 
 
 def measure_mixed(args):
-    """Prefill and decode throughput of a mixed model (BF16) and of the dense F32 stack at equal size, each through
+    """Prefill and decode throughput of mixed models (BF16) and of the dense F32 stack at equal size, each through
     its forward call: prefill of MIXED_PREFILL tokens, decode of 1 and 16 sessions at MIXED_CTX tokens, arg-max on the
     device, CUDA events on the context's stream around the calls (host enqueueing included)."""
     import torch
@@ -710,7 +723,8 @@ def measure_mixed(args):
     rng = np.random.default_rng(SEED)
     for size in (args.mixed_size.split(",") if args.mixed_size else MIXED_SIZES):
         row = out["sizes"][size] = {}
-        for kind, cfg, dtype, rows in (("tumadra_bf16", mixed_config(size), "bfloat16", MIXED_PREFILL),
+        for kind, cfg, dtype, rows in (("nurosun_bf16", latent_config(size), "bfloat16", MIXED_PREFILL),
+                                       ("tumadra_bf16", mixed_config(size), "bfloat16", MIXED_PREFILL),
                                        ("dense_f32", dense_config(size), "float32", 256)):
             if args.mixed_kind and kind != args.mixed_kind:
                 continue
@@ -757,9 +771,9 @@ def measure_mixed(args):
                     pos[0] += 1
                 timed(decode, 5)
                 l0 = m.launches
-                ms = timed(decode, 50)
+                ms = timed(decode, args.mixed_reps)
                 res[f"decode_{n}"] = {"ms": r4(ms), "tok_s": r4(n / ms * 1e3), "enqueue_ms": r4(m.last_enqueue_ms),
-                                      "launches": (m.launches - l0) // 50}
+                                      "launches": (m.launches - l0) // args.mixed_reps}
                 for kv in kvs:
                     kv.close()
             m.close()
@@ -1135,10 +1149,11 @@ def main():
     ap.add_argument("--no-whole-model", action="store_true",
                     help="skip the config-1 whole-model section (about a minute of host time)")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "mixed"],
-                    help="'prefill' / 'decode': run only that kernel's measurement (for profiling); 'mixed': Tumadra "
+                    help="'prefill' / 'decode': run only that kernel's measurement (for profiling); 'mixed': Nurosun and Tumadra "
                          "models beside the dense stack at equal size, nothing else")
     ap.add_argument("--mixed-size", default="", help="with --only mixed: sizes, with commas between them")
-    ap.add_argument("--mixed-kind", default="", choices=["", "tumadra_bf16", "dense_f32"], help="with --only mixed: one model only")
+    ap.add_argument("--mixed-reps", type=int, default=50, help="with --only mixed: timed decode steps")
+    ap.add_argument("--mixed-kind", default="", choices=["", "nurosun_bf16", "tumadra_bf16", "dense_f32"], help="with --only mixed: one model only")
     args = ap.parse_args()
     if args.impl == "reference":
         if args.steps > 20:

@@ -39,12 +39,19 @@
 //     normalised, and sent out in pieces of 32 rows x 16 values through two swizzled
 //     shared-memory buffers as TMA tensor stores (a store instruction whose lanes each write a
 //     row of their own touches 32 cache lines for 512 bytes).
+// The kernel exists twice.  With LATENT = false it is what is described above, over a cache of head_dim 128.  With
+// LATENT = true it serves layers whose heads share one cached latent row (wr_latent_flash_launch): every head has K
+// and V of its own, which a matrix product has written out for the step (rows of one buffer, loaded through a tensor
+// map), the key's rotated part is shared and comes from the cache's pages; sizes are arguments (query and key
+// [unrotated | rotated] in 64-wide boxes, values up to 128 wide), and the rows leave as BF16.
 // Every wait has a time limit; on expiry the kernel records an error, still
 // frees its TMEM and returns.
 #include <cuda.h>
+#include <cuda_bf16.h>
 
 #include <algorithm>
 
+#include "mixers.cuh"
 #include "wr_internal.cuh"
 
 namespace {
@@ -112,6 +119,15 @@ struct prefill_params {
     float scale_log2;           // score scale * log2(e)
     long long wait_limit;       // SM clock cycles a device-side wait may last
     uint32_t early;             // the kernel before this one only reads what this one reads
+    // LATENT only
+    uint32_t q_boxes, nope_boxes, v_boxes;       // 64-wide boxes of a query / key, unrotated ones of them; of a value
+    uint32_t nope_steps, steps;                  // 16-wide steps of the scores, unrotated ones first
+    uint32_t q_head, q_rot;                      // columns per head of the query rows; where the rotated ones start
+    uint32_t k_head, v_at, v_head;               // columns per head of the K / V rows; where V starts
+    uint32_t rot_block;                          // 64-wide block of a page where the rotated key part starts
+    uint32_t k_stages, v_stages;
+    uint32_t vdim, v_cols, out_ld;               // value size, rounded up to 16; row length of the output
+    __nv_bfloat16 *out;
 };
 
 // A published work tile: up to two blocks over the same KV head.
@@ -120,11 +136,10 @@ struct tile_info {
     uint32_t head[2], qt[2];
 };
 
-struct smem_layout {
-    alignas(1024) uint8_t q[2][kQBytes];                 // per block: [64-dim half][128 rows][128 B]
-    alignas(1024) uint8_t k[kStages][kKVTile];           // [64-dim half][128 keys][128 B]
-    alignas(1024) uint8_t v[kStages][kKVTile];           // [page][64-dim half][64 keys][128 B]
-    alignas(8) uint64_t q_full[2];                       // per block
+// Shared memory: Q of both blocks ([64-dim box][128 rows][128 B] each), the K stages ([64-dim box][128 keys][128 B]),
+// the V stages ([page][64-dim half][64 keys][128 B]; LATENT: as K), output staging, then this.
+struct smem_bars {
+    uint64_t q_full[2];                                  // per block
     uint64_t q_free[2];                                  // per block: its last scores of the tile have completed
     uint64_t k_full[kStages], k_free[kStages];
     uint64_t v_full[kStages], v_free[kStages];
@@ -135,11 +150,13 @@ struct smem_layout {
     uint64_t tile_ready[kTileSlots];
     tile_info tile[kTileSlots];
     uint32_t tmem_base;
-    // per softmax warp: two buffers of 32 rows x 16 output values on their way out (16-byte pieces
-    // swizzled by row pair: the 64-byte swizzle of the output tensor map)
-    alignas(1024) uint8_t out_stage[8][2][32 * 64];
 };
-static_assert(sizeof(smem_layout) <= 232448, "the CTA's shared memory is 227 KB at most");
+// per softmax warp: two buffers of 32 rows x 16 output values on their way out (16-byte pieces swizzled by row pair:
+// the 64-byte swizzle of the output tensor map); LATENT: one of 32 rows x 32 BF16 values
+constexpr uint32_t kOutPiece = 32 * 64;
+constexpr uint32_t kOutBytes = 8 * 2 * kOutPiece, kOutBytesLatent = 8 * kOutPiece;
+constexpr uint32_t kSmemBytes = 2 * kQBytes + 2 * kStages * kKVTile + kOutBytes + sizeof(smem_bars);
+static_assert(kSmemBytes <= 232448, "the CTA's shared memory is 227 KB at most");
 
 // ---- tcgen05 / TMA wrappers ------------------------------------------------
 
@@ -391,12 +408,19 @@ __device__ __forceinline__ block_range range_of(const prefill_params &p, uint32_
 
 // ---- the kernel ------------------------------------------------------------
 
+// (kv_map: LATENT's K and V rows; o_map: the other's output rows)
+template <bool LATENT>
 __global__ void __launch_bounds__(kThreads, 1)
-attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap o_map,
-                          const prefill_params p)
+attn_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
+                    const __grid_constant__ CUtensorMap o_map, const prefill_params p)
 {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
-    smem_layout &sm = *reinterpret_cast<smem_layout *>(smem_raw);
+    const uint32_t q_bytes = LATENT ? p.q_boxes * kQHalfBytes : kQBytes;
+    const uint32_t k_bytes = LATENT ? p.q_boxes * kQHalfBytes : kKVTile, v_bytes = LATENT ? p.v_boxes * kQHalfBytes : kKVTile;
+    const uint32_t k_stages = LATENT ? p.k_stages : (uint32_t)kStages, v_stages = LATENT ? p.v_stages : (uint32_t)kStages;
+    uint8_t *const sm_q = smem_raw, *const sm_k = sm_q + 2 * q_bytes, *const sm_v = sm_k + k_stages * k_bytes;
+    uint8_t *const sm_out = sm_v + v_stages * v_bytes;
+    smem_bars &sm = *reinterpret_cast<smem_bars *>(sm_out + (LATENT ? kOutBytesLatent : kOutBytes));
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 #ifdef WR_PREFILL_TIMELINE
     if (tid == 0 && p.tl && blockIdx.x < kTlCtas) p.tl[kTlRoles * kTlEvents + blockIdx.x * 4] = tl_ns();
@@ -407,6 +431,59 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
     // with p.early (the kernel before is a prefill launch too: a reader) the first tile's loads
     // and arithmetic do not wait, only the counter and the output stores do.
     pdl_trigger();
+    const uint32_t n_pages_total = (p.p0 + p.n + 63u) / 64u;     // pages that hold rows of this prompt
+    auto page_ptr = [&](uint32_t t) -> const char * {
+        return p.page_base ? p.page_base + (uint64_t)t * p.page_bytes : (const char *)p.pages[t];
+    };
+    // Requests (the caller has waited for the buffer): Q of a block, a K tile, a V tile.
+    auto request_q = [&](uint32_t b, uint32_t head, uint32_t qt) {
+        uint8_t *dst = sm_q + b * q_bytes;
+        mbar_expect_tx(&sm.q_full[b], q_bytes);
+        if constexpr (LATENT) {
+            for (uint32_t i = 0; i < p.q_boxes; ++i)
+                tma_load_2d(dst + i * kQHalfBytes, &q_map,
+                            (int)(head * p.q_head + (i < p.nope_boxes ? 64 * i : p.q_rot + 64 * (i - p.nope_boxes))),
+                            (int)(qt * kBM), &sm.q_full[b]);
+        } else {
+            tma_load_2d(dst, &q_map, (int)(head * kHd), (int)(qt * kBM), &sm.q_full[b]);
+            tma_load_2d(dst + kQHalfBytes, &q_map, (int)(head * kHd + 64), (int)(qt * kBM), &sm.q_full[b]);
+        }
+    };
+    auto request_k = [&](uint32_t st, uint32_t j, uint32_t kvh) {
+        // [64-dim box][128 keys][128 B]: each page contributes 64 keys to a box
+        const uint32_t n_pg = (2 * j + 1 < n_pages_total) ? 2u : 1u;
+        uint8_t *dst = sm_k + st * k_bytes;
+        if constexpr (LATENT) {
+            const uint32_t rot_boxes = p.q_boxes - p.nope_boxes;
+            mbar_expect_tx(&sm.k_full[st], p.nope_boxes * kQHalfBytes + rot_boxes * n_pg * 8192);
+            for (uint32_t i = 0; i < p.nope_boxes; ++i)
+                tma_load_2d(dst + i * kQHalfBytes, &kv_map, (int)(kvh * p.k_head + 64 * i), (int)(j * kBN), &sm.k_full[st]);
+            for (uint32_t pg = 0; pg < n_pg; ++pg)
+                for (uint32_t i = 0; i < rot_boxes; ++i)
+                    bulk_g2s(dst + (p.nope_boxes + i) * kQHalfBytes + pg * 8192, page_ptr(2 * j + pg) + (p.rot_block + i) * 8192,
+                             8192, &sm.k_full[st]);
+        } else {
+            mbar_expect_tx(&sm.k_full[st], n_pg * kPageBlock);
+            for (uint32_t pg = 0; pg < n_pg; ++pg) {
+                const char *src = page_ptr(2 * j + pg) + wr_block_off(kvh, 0, kHd);
+                bulk_g2s(dst + pg * 8192, src, 8192, &sm.k_full[st]);
+                bulk_g2s(dst + kQHalfBytes + pg * 8192, src + 8192, 8192, &sm.k_full[st]);
+            }
+        }
+    };
+    auto request_v = [&](uint32_t st, uint32_t j, uint32_t kvh) {
+        uint8_t *dst = sm_v + st * v_bytes;
+        if constexpr (LATENT) {
+            mbar_expect_tx(&sm.v_full[st], v_bytes);
+            for (uint32_t i = 0; i < p.v_boxes; ++i)
+                tma_load_2d(dst + i * kQHalfBytes, &kv_map, (int)(p.v_at + kvh * p.v_head + 64 * i), (int)(j * kBN), &sm.v_full[st]);
+        } else {
+            const uint32_t n_pg = (2 * j + 1 < n_pages_total) ? 2u : 1u;
+            mbar_expect_tx(&sm.v_full[st], n_pg * kPageBlock);
+            for (uint32_t pg = 0; pg < n_pg; ++pg)
+                bulk_g2s(dst + pg * kPageBlock, page_ptr(2 * j + pg) + wr_block_off(kvh, 1, kHd), kPageBlock, &sm.v_full[st]);
+        }
+    };
 
     if (warp == 8 && lane == 0) {
         mbar_init(&sm.q_full[0], 1);
@@ -433,22 +510,9 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
         const tile_info ti = decode_tile(p, blockIdx.x);
         const block_range r0 = range_of(p, ti.qt[0]), r1 = range_of(p, ti.qt[ti.nblk - 1]);
         const uint32_t lo = min(r0.lo, r1.lo);
-        const uint32_t n_pages_all = (p.p0 + p.n + 63u) / 64u;
-        for (uint32_t b = 0; b < ti.nblk; ++b) {
-            mbar_expect_tx(&sm.q_full[b], kQBytes);
-            tma_load_2d(sm.q[b], &q_map, (int)(ti.head[b] * kHd), (int)(ti.qt[b] * kBM), &sm.q_full[b]);
-            tma_load_2d(sm.q[b] + kQHalfBytes, &q_map, (int)(ti.head[b] * kHd + 64), (int)(ti.qt[b] * kBM), &sm.q_full[b]);
-            if (b == 0) {
-                const uint32_t n_pg = (2 * lo + 1 < n_pages_all) ? 2u : 1u;
-                mbar_expect_tx(&sm.k_full[0], n_pg * kPageBlock);
-                for (uint32_t pg = 0; pg < n_pg; ++pg) {
-                    const char *src = (p.page_base ? p.page_base + (uint64_t)(2 * lo + pg) * p.page_bytes
-                                                   : (const char *)p.pages[2 * lo + pg]) + wr_block_off(ti.kvh, 0, kHd);
-                    bulk_g2s(sm.k[0] + pg * 8192, src, 8192, &sm.k_full[0]);
-                    bulk_g2s(sm.k[0] + kQHalfBytes + pg * 8192, src + 8192, 8192, &sm.k_full[0]);
-                }
-            }
-        }
+        request_q(0, ti.head[0], ti.qt[0]);
+        request_k(0, lo, ti.kvh);
+        if (ti.nblk > 1) request_q(1, ti.head[1], ti.qt[1]);
     }
     if (warp == 0) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;"
@@ -460,11 +524,6 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
     tc_fence_after();
     const uint32_t tmem = sm.tmem_base;
     const long long limit = p.wait_limit;
-    const uint32_t n_pages_total = (p.p0 + p.n + 63u) / 64u;     // pages that hold rows of this prompt
-
-    auto page_ptr = [&](uint32_t t) -> const char * {
-        return p.page_base ? p.page_base + (uint64_t)t * p.page_bytes : (const char *)p.pages[t];
-    };
     // Work tile number `it` of this CTA: the first one is the CTA's own number (every
     // role works it out for itself, nobody waits), later ones are published by the producer.
     auto tile_of = [&](uint32_t it, bool &ok) -> tile_info {
@@ -492,22 +551,13 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                 auto load_q = [&](uint32_t b, uint32_t head, uint32_t qt) -> bool {
                     if (q_loads[b] > 0 && !mbar_wait(&sm.q_free[b], (q_loads[b] - 1) & 1, limit)) return false;
                     ++q_loads[b];
-                    mbar_expect_tx(&sm.q_full[b], kQBytes);
-                    tma_load_2d(sm.q[b], &q_map, (int)(head * kHd), (int)(qt * kBM), &sm.q_full[b]);
-                    tma_load_2d(sm.q[b] + kQHalfBytes, &q_map, (int)(head * kHd + 64), (int)(qt * kBM), &sm.q_full[b]);
+                    request_q(b, head, qt);
                     return true;
                 };
                 auto load_k = [&](uint32_t j) -> bool {
-                    const uint32_t st = kcount % kStages;
-                    if (kcount >= kStages && !mbar_wait(&sm.k_free[st], ((kcount / kStages) - 1) & 1, limit)) return false;
-                    // [64-dim half][128 keys][128 B]: each page contributes 64 keys to each half
-                    const uint32_t n_pg = (2 * j + 1 < n_pages_total) ? 2u : 1u;
-                    mbar_expect_tx(&sm.k_full[st], n_pg * kPageBlock);
-                    for (uint32_t pg = 0; pg < n_pg; ++pg) {
-                        const char *src = page_ptr(2 * j + pg) + wr_block_off(ti.kvh, 0, kHd);
-                        bulk_g2s(sm.k[st] + pg * 8192, src, 8192, &sm.k_full[st]);
-                        bulk_g2s(sm.k[st] + kQHalfBytes + pg * 8192, src + 8192, 8192, &sm.k_full[st]);
-                    }
+                    const uint32_t st = kcount % k_stages;
+                    if (kcount >= k_stages && !mbar_wait(&sm.k_free[st], ((kcount / k_stages) - 1) & 1, limit)) return false;
+                    request_k(st, j, ti.kvh);
                     ++kcount;
                     return true;
                 };
@@ -560,16 +610,12 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                 const block_range r0 = range_of(p, ti.qt[0]), r1 = range_of(p, ti.qt[ti.nblk - 1]);
                 const uint32_t lo = min(r0.lo, r1.lo), hi = max(r0.hi, r1.hi);
                 for (uint32_t j = lo; j < hi && ok; ++j, ++vcount) {
-                    const uint32_t st = vcount % kStages;
-                    if (vcount >= kStages) {
-                        ok = mbar_wait(&sm.v_free[st], ((vcount / kStages) - 1) & 1, limit);
+                    const uint32_t st = vcount % v_stages;
+                    if (vcount >= v_stages) {
+                        ok = mbar_wait(&sm.v_free[st], ((vcount / v_stages) - 1) & 1, limit);
                         if (!ok) break;
                     }
-                    const uint32_t n_pg = (2 * j + 1 < n_pages_total) ? 2u : 1u;
-                    mbar_expect_tx(&sm.v_full[st], n_pg * kPageBlock);
-                    for (uint32_t pg = 0; pg < n_pg; ++pg)
-                        bulk_g2s(sm.v[st] + pg * kPageBlock, page_ptr(2 * j + pg) + wr_block_off(ti.kvh, 1, kHd),
-                                 kPageBlock, &sm.v_full[st]);
+                    request_v(st, j, ti.kvh);
                 }
             }
             if (!ok) atomicCAS(p.err, 0, 14);
@@ -585,15 +631,15 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
         // against 64 this way.)
         const bool lead = elect_one();
         const uint32_t idesc_s = umma_idesc(kBM, kBN, false);
-        const uint32_t idesc_o = umma_idesc(kBM, kHd, true);
+        const uint32_t idesc_o = umma_idesc(kBM, LATENT ? p.v_cols : kHd, true);
         // descriptor words: the high word is fixed per operand kind, an operand is
         // selected by adding its byte offset (>>4) to the address field of the low word
-        const uint64_t kmaj0 = umma_desc(0, 16, 1024), mnmaj0 = umma_desc(0, 8192, 1024);
+        const uint64_t kmaj0 = umma_desc(0, 16, 1024), mnmaj0 = umma_desc(0, LATENT ? kQHalfBytes : 8192, 1024);
         const uint32_t kmaj_hi = (uint32_t)(kmaj0 >> 32), kmaj_lo = (uint32_t)kmaj0;
         const uint32_t mnmaj_hi = (uint32_t)(mnmaj0 >> 32), mnmaj_lo = (uint32_t)mnmaj0;
-        const uint32_t q_lo0 = kmaj_lo | ((smem_u32(sm.q[0]) & 0x3FFFFu) >> 4);
-        const uint32_t k_lo0 = kmaj_lo | ((smem_u32(sm.k[0]) & 0x3FFFFu) >> 4);
-        const uint32_t v_lo0 = mnmaj_lo | ((smem_u32(sm.v[0]) & 0x3FFFFu) >> 4);
+        const uint32_t q_lo0 = kmaj_lo | ((smem_u32(sm_q) & 0x3FFFFu) >> 4);
+        const uint32_t k_lo0 = kmaj_lo | ((smem_u32(sm_k) & 0x3FFFFu) >> 4);
+        const uint32_t v_lo0 = mnmaj_lo | ((smem_u32(sm_v) & 0x3FFFFu) >> 4);
         // ring positions advance by one per step; parity flips when a ring wraps
         uint32_t k_st = 0, k_par = 0;            // K stage / parity of the next step to score
         uint32_t v_st = 0, v_par = 0;            // V stage / parity of the next step to multiply
@@ -604,29 +650,40 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
         TL_DECL;
         // S_b = Q_b . K^T for the K tile in stage st
         auto issue_s = [&](uint32_t b, uint32_t st) {
-            const uint32_t q_lo = q_lo0 + b * (kQBytes >> 4), k_lo = k_lo0 + st * (kKVTile >> 4);
+            const uint32_t q_lo = q_lo0 + b * (q_bytes >> 4), k_lo = k_lo0 + st * (k_bytes >> 4);
             const uint32_t d = tmem + kTmemS + 128 * b;
+            if constexpr (LATENT) {
+#pragma unroll 4
+                for (uint32_t kk = 0; kk < p.steps; ++kk) {
+                    const uint32_t at = kk < p.nope_steps ? kk : 4 * p.nope_boxes + kk - p.nope_steps;
+                    const uint32_t off = ((at >> 2) * kQHalfBytes + (at & 3) * 32) >> 4;
+                    if (lead) umma_ss(d, q_lo + off, kmaj_hi, k_lo + off, kmaj_hi, idesc_s, kk > 0);
+                }
+            } else {
 #pragma unroll
-            for (int kk = 0; kk < kHd / 16; ++kk) {
-                const uint32_t off = ((kk >> 2) * kQHalfBytes + (kk & 3) * 32) >> 4;
-                if (lead) umma_ss(d, q_lo + off, kmaj_hi, k_lo + off, kmaj_hi, idesc_s, kk > 0);
+                for (int kk = 0; kk < kHd / 16; ++kk) {
+                    const uint32_t off = ((kk >> 2) * kQHalfBytes + (kk & 3) * 32) >> 4;
+                    if (lead) umma_ss(d, q_lo + off, kmaj_hi, k_lo + off, kmaj_hi, idesc_s, kk > 0);
+                }
             }
             if (lead) umma_commit(&sm.s_full[b]);
         };
         // O_b (+)= P_b . V for the V tile in stage st, n_kk steps of 16 keys
         auto issue_pv = [&](uint32_t b, uint32_t st, uint32_t n_kk, bool accumulate) {
-            const uint32_t v_lo = v_lo0 + st * (kKVTile >> 4);
+            const uint32_t v_lo = v_lo0 + st * (v_bytes >> 4);
+            // 16 keys further down the tile
+            auto step16 = [](uint32_t kk) { return LATENT ? kk * 128u : ((kk >> 2) * kPageBlock + (kk & 3) * 2048) >> 4; };
             const uint32_t d = tmem + kTmemO + 128 * b, a = tmem + kTmemS + 128 * b;
             if (n_kk == kBN / 16) {
 #pragma unroll
                 for (int kk = 0; kk < kBN / 16; ++kk)
                     if (lead)
-                        umma_ts(d, a + 8 * kk, v_lo + (((kk >> 2) * kPageBlock + (kk & 3) * 2048) >> 4), mnmaj_hi, idesc_o,
+                        umma_ts(d, a + 8 * kk, v_lo + step16(kk), mnmaj_hi, idesc_o,
                                 accumulate || kk > 0);
             } else {
                 for (uint32_t kk = 0; kk < n_kk; ++kk)
                     if (lead)
-                        umma_ts(d, a + 8 * kk, v_lo + (((kk >> 2) * kPageBlock + (kk & 3) * 2048) >> 4), mnmaj_hi, idesc_o,
+                        umma_ts(d, a + 8 * kk, v_lo + step16(kk), mnmaj_hi, idesc_o,
                                 accumulate || kk > 0);
             }
         };
@@ -654,7 +711,7 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                 if (lead && hi1 == lo + 1) umma_commit(&sm.q_free[1]);
             }
             if (lead) umma_commit(&sm.k_free[k_st]);
-            if (++k_st == kStages) { k_st = 0; k_par ^= 1; }
+            if (++k_st == k_stages) { k_st = 0; k_par ^= 1; }
             if (lane == 0) TLT(4, 2);                            // first scores issued
             for (uint32_t j = lo; j < hi && ok; ++j) {
                 const bool more = j + 1 < hi;
@@ -697,8 +754,8 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                     umma_commit(&sm.v_free[v_st]);
                     if (more) umma_commit(&sm.k_free[k_st]);
                 }
-                if (++v_st == kStages) { v_st = 0; v_par ^= 1; }
-                if (more && ++k_st == kStages) { k_st = 0; k_par ^= 1; }
+                if (++v_st == v_stages) { v_st = 0; v_par ^= 1; }
+                if (more && ++k_st == k_stages) { k_st = 0; k_par ^= 1; }
             }
             if (lane == 0) TLT(4, 3);                            // last P.V issued
         }
@@ -790,7 +847,7 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                 if (__any_sync(0xffffffffu, grow)) {
                     const float a = grow ? ex2_approx(m_ref - tm2) : 1.0f;
 #pragma unroll 1
-                    for (int c = 0; c < kHd; c += 32) {
+                    for (int c = 0; c < (LATENT ? (int)p.v_cols : kHd); c += 32) {
                         float o[32];
                         tmem_ld32_nowait(o_addr + c, o);
                         tmem_wait_ld();
@@ -839,17 +896,17 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
                     l += (pa + pb) + (pc + pd);
                 }
                 TLS();                                           // 2: P stores issued
-                if (key0 + kBN > p.p0 + p.n) {
+                if (!LATENT && key0 + kBN > p.p0 + p.n) {       // (a tensor map fills such rows with zeros)
                     // Cache rows past the prompt's last key were never written for it
                     // (or belong to a rolled-back step): clear them in the staged V
                     // tile so that 0 * garbage cannot make a NaN (both groups do it
                     // before releasing their own P.V; the writes are equal).
-                    const uint32_t vn = vc + (j - lo), vst = vn % kStages;
-                    ok = mbar_wait(&sm.v_full[vst], (vn / kStages) & 1, limit);
+                    const uint32_t vn = vc + (j - lo), vst = vn % v_stages;
+                    ok = mbar_wait(&sm.v_full[vst], (vn / v_stages) & 1, limit);
                     if (!ok) break;
                     const uint32_t first_bad = p.p0 + p.n - key0;
                     if (row >= first_bad) {
-                        uint8_t *vrow = sm.v[vst] + (row >> 6) * kPageBlock + (row & 63u) * 128;
+                        uint8_t *vrow = sm_v + vst * v_bytes + (row >> 6) * kPageBlock + (row & 63u) * 128;
 #pragma unroll
                         for (int c = 0; c < 8; ++c) {
                             *reinterpret_cast<uint4 *>(vrow + c * 16) = make_uint4(0, 0, 0, 0);
@@ -889,12 +946,51 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
             // out as whole sectors (rows past the prompt are outside the tensor and dropped).  Two
             // buffers take turns: a piece is waited for only when its buffer is needed again.
             pdl_wait();                                      // output rows: after the earlier kernels have ended
-            {
+            if constexpr (LATENT) {
+                const float inv = (l > 0.f) ? 1.0f / l : 0.f;
+                uint8_t *stage = sm_out + warp * kOutPiece;
+#pragma unroll
+                for (int c = 0; c < kHd / 32; ++c) {             // pieces of 32 values
+                    if (32u * c >= p.vdim) break;
+                    __syncwarp();
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const __nv_bfloat162 h = __floats2bfloat162_rn(o[32 * c + 8 * k + 2 * e] * inv,
+                                                                          o[32 * c + 8 * k + 2 * e + 1] * inv);
+                            w[e] = *reinterpret_cast<const uint32_t *>(&h);
+                        }
+                        *reinterpret_cast<uint4 *>(stage + lane * 64 + ((k ^ ((lane >> 1) & 3u)) << 4)) =
+                            make_uint4(w[0], w[1], w[2], w[3]);
+                    }
+                    __syncwarp();
+                    // four lanes write a row's 64 bytes
+                    const uint32_t col = 32u * c + 8u * (lane & 3u);
+#pragma unroll
+                    for (uint32_t i = 0; i < 4; ++i) {
+                        const uint32_t r = 8 * i + (lane >> 2), tr = wq * 32u + r;
+                        if (tr >= me.rows || col >= p.vdim) continue;
+                        const uint4 w = *reinterpret_cast<const uint4 *>(stage + r * 64 + (((lane & 3u) ^ ((r >> 1) & 3u)) << 4));
+                        __nv_bfloat16 *dst = p.out + (size_t)(me.tok0 + tr) * p.out_ld + head * p.vdim + col;
+                        if (p.vdim % 8 == 0) {
+                            *reinterpret_cast<uint4 *>(dst) = w;
+                        } else {
+                            const uint32_t part[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+                            for (uint32_t e = 0; e < 8; ++e)
+                                if (col + e < p.vdim)
+                                    reinterpret_cast<uint16_t *>(dst)[e] = (uint16_t)(part[e >> 1] >> (16 * (e & 1)));
+                        }
+                    }
+                }
+            } else {
                 const float inv = (l > 0.f) ? 1.0f / l : 0.f;
                 const bool send = (lane == 0) && (wq * 32u < me.rows);   // (a piece wholly past the prompt is not sent)
 #pragma unroll
                 for (int c = 0; c < kHd / 16; ++c) {
-                    uint8_t *stage = sm.out_stage[warp][c & 1];
+                    uint8_t *stage = sm_out + (2 * warp + (c & 1)) * kOutPiece;
                     if (lane == 0) tma_store_wait_read<1>();     // the piece before the last has left this buffer
                     __syncwarp();
 #pragma unroll
@@ -910,7 +1006,7 @@ attn_prefill_hd128_kernel(const __grid_constant__ CUtensorMap q_map, const __gri
             TLST(5);                                             // output rows issued
         }
         if (!ok) atomicCAS(p.err, 0, 13);
-        if (lane == 0) tma_store_wait_read<0>();                 // shared memory stays valid until the last piece is read
+        if (!LATENT && lane == 0) tma_store_wait_read<0>();                 // shared memory stays valid until the last piece is read
     }
 
     tc_fence_before();
@@ -1042,7 +1138,7 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
         return WR_CUDA_ERR_INTERNAL;
 
-    prefill_params p;
+    prefill_params p{};
     p.pages = kv->d_pages + (size_t)layer * kv->n_pages;
     p.page_base = kv->contig[layer] ? (const char *)kv->pages[(size_t)layer * kv->n_pages] : nullptr;
     p.page_bytes = wr_page_bytes(kv->n_kv_at(layer), kHd);
@@ -1067,8 +1163,8 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
     const float scale = (scale_override > 0.0f) ? scale_override : 1.0f / sqrtf((float)kHd);   // kernels.c:1457-1459
     p.scale_log2 = scale * kLog2e;
     if (!(ctx->attr_flags & 2u)) {
-        WR_CUDA_TRY(cudaFuncSetAttribute(attn_prefill_hd128_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)sizeof(smem_layout)));
+        WR_CUDA_TRY(cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)kSmemBytes));
         ctx->attr_flags |= 2u;
     }
     const uint32_t grid = std::min<uint32_t>(p.n_tiles, (uint32_t)ctx->sm_count);
@@ -1078,7 +1174,7 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
     const bool full = grid == (uint32_t)ctx->sm_count;
     p.early = (!convert && !host && full && ctx->pdl_index == ctx->launches &&
                ctx->pdl_kind == WR_PDL_PREFILL_FULL) ? 1u : 0u;
-    WR_CUDA_TRY(wr_launch_pdl(attn_prefill_hd128_kernel, dim3(grid), dim3(kThreads), sizeof(smem_layout), ctx->stream,
+    WR_CUDA_TRY(wr_launch_pdl(attn_prefill_kernel<false>, dim3(grid), dim3(kThreads), kSmemBytes, ctx->stream, q_map,
                               q_map, o_map, p));
     ctx->launches++;
     ctx->pdl_kind = full ? WR_PDL_PREFILL_FULL : WR_PDL_NONE;
@@ -1088,6 +1184,96 @@ extern "C" int wr_cuda_attn_prefill(wr_cuda_ctx *ctx, wr_cuda_kv *kv, uint32_t l
         WR_CUDA_TRY(cudaMemcpyAsync(out, dout, out_bytes, cudaMemcpyDeviceToHost, ctx->stream));
         return wr_ctx_sync_checked(ctx);
     }
+    return WR_CUDA_OK;
+}
+
+namespace {
+
+// 64-wide boxes of rows of F16 values, 128 rows at a time
+bool box_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, uint32_t ld)
+{
+    encode_tiled_fn encode = get_encode_tiled();
+    const cuuint64_t dims[2] = {cols, rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {64, kBM};
+    const cuuint32_t estr[2] = {1, 1};
+    return encode && encode(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
+                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+// shared memory of the LATENT kernel with the most stages that fit; 0: it does not fit
+uint32_t latent_smem(const wr_latent_geom &g, uint32_t &k_stages, uint32_t &v_stages)
+{
+    const uint32_t q = (g.dim_pad() + 63) / 64 + (g.rot_pad() + 63) / 64, v = (g.vdim_pad() + 63) / 64;
+    const uint32_t try_k[3] = {2, 1, 1}, try_v[3] = {2, 2, 1};
+    for (int i = 0; i < 3; ++i) {
+        const uint64_t bytes = (uint64_t)(2 * q + try_k[i] * q + try_v[i] * v) * kQHalfBytes + kOutBytesLatent + sizeof(smem_bars);
+        if (bytes > 232448) continue;
+        k_stages = try_k[i];
+        v_stages = try_v[i];
+        return (uint32_t)bytes;
+    }
+    return 0;
+}
+
+}  // namespace
+
+bool wr_latent_flash_covers(const wr_latent_geom &g, float scale)
+{
+    uint32_t ks, vs;
+    return g.vdim <= (uint32_t)kHd && scale > 0.f && latent_smem(g, ks, vs) != 0;
+}
+
+int wr_latent_flash_launch(wr_cuda_ctx *ctx, const wr_latent_flash_args &a)
+{
+    const wr_latent_geom &g = a.g;
+    prefill_params p{};
+    const uint32_t smem = latent_smem(g, p.k_stages, p.v_stages);
+    if (!smem || a.n == 0) return WR_CUDA_ERR_LIMIT;
+    if (!ctx->prefill_sched) {
+        WR_CUDA_TRY(cudaMalloc((void **)&ctx->prefill_sched, 2 * sizeof(int)));
+        WR_CUDA_TRY(cudaMemsetAsync(ctx->prefill_sched, 0, 2 * sizeof(int), ctx->stream));
+    }
+    CUtensorMap q_map, kv_map;
+    const uint32_t q_cols = g.heads * g.q_head(), kv_cols = g.heads * (g.dim_pad() + g.vdim_pad());
+    if (!box_map(&q_map, a.q, q_cols, a.n, q_cols) || !box_map(&kv_map, a.kv, kv_cols, a.p0 + a.n, kv_cols))
+        return WR_CUDA_ERR_INTERNAL;
+    p.pages = a.pages;
+    p.page_bytes = (uint64_t)kPageTokens * g.row() * 2;
+    p.err = ctx->dev_err;
+    p.sched = ctx->prefill_sched;
+    p.wait_limit = ctx->wait_limit;
+    p.n = a.n;
+    p.p0 = a.p0;
+    p.n_q = p.n_kv = g.heads;
+    p.group = 1;
+    p.n_qtiles = (a.n + kBM - 1) / kBM;
+    p.n_tiles = prefill_tile_count(p.n_qtiles, p.n_kv, p.group);
+    p.scale_log2 = a.scale * kLog2e;
+    p.nope_boxes = (g.dim_pad() + 63) / 64;
+    p.q_boxes = p.nope_boxes + (g.rot_pad() + 63) / 64;
+    p.v_boxes = (g.vdim_pad() + 63) / 64;
+    p.nope_steps = g.dim_pad() / 16;
+    p.steps = p.nope_steps + g.rot_pad() / 16;
+    p.q_head = g.q_head();
+    p.q_rot = g.dim_pad();
+    p.k_head = g.dim_pad();
+    p.v_at = g.heads * g.dim_pad();
+    p.v_head = g.vdim_pad();
+    p.rot_block = g.rank_pad() / 64;
+    p.vdim = g.vdim;
+    p.v_cols = g.vdim_pad();
+    p.out_ld = a.out_ld;
+    p.out = static_cast<__nv_bfloat16 *>(a.out);
+    WR_CUDA_TRY(cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const uint32_t grid = std::min<uint32_t>(p.n_tiles, (uint32_t)ctx->sm_count);
+    WR_CUDA_TRY(wr_launch_pdl(attn_prefill_kernel<true>, dim3(grid), dim3(kThreads), (size_t)smem, ctx->stream, q_map, kv_map,
+                              q_map, p));
+    ctx->launches++;
+    WR_CUDA_TRY(cudaGetLastError());
+    const uint32_t n_out = g.heads * g.vdim, pad = wr_ld(n_out) - n_out;
+    if (pad) WR_CUDA_TRY(cudaMemset2DAsync(p.out + n_out, (size_t)a.out_ld * 2, 0, pad * 2, a.n, ctx->stream));
     return WR_CUDA_OK;
 }
 

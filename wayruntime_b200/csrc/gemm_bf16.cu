@@ -6,7 +6,7 @@
 // of blocks stored in the operand's layout; what lies beyond K arrives as zeros), warp 1 issues tcgen05.mma into one of two TMEM accumulators, warps 2-5 read the other one
 // back and write the finished rows (bias, softplus, residual; F32, BF16 or saturated F16), so that a
 // tile's output overlaps the next tile's products.  Columns may be gate / up pairs, of which the activation leaves
-// (wr_pair_args), and row tiles may have weights of their own (wr_group_args).  Every wait is bounded by the context's wait
+// (wr_pair_args), row tiles may have weights of their own (wr_group_args), and activations may come from a cache's pages.  Every wait is bounded by the context's wait
 // limit; a warp that gives up records an error word and all of them leave.
 #include <cuda_bf16.h>
 
@@ -96,8 +96,16 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
                     }
                     uint8_t *a = stages + st * (kABytes + T::kBBytes), *b = a + kABytes;
                     const uint32_t nb0 = n0 / kWBlock, nb = min(BN / kWBlock, wr_weight_blocks(p.w.n) - nb0);
-                    mbar_expect_tx(&full[st], kABytes + nb * kWBlockBytes);
-                    tc5::tma_load_2d(a, &x_map, (int)(kb * kBK), (int)m0, &full[st]);
+                    if (p.a.pages) {
+                        const uint32_t np = m0 + kPageTokens < p.a.m ? 2u : 1u;
+                        mbar_expect_tx(&full[st], np * kABytes / 2 + nb * kWBlockBytes);
+                        for (uint32_t i = 0; i < np; ++i)
+                            bulk_g2s(a + i * kABytes / 2, reinterpret_cast<const char *>(p.a.pages[m0 / kPageTokens + i]) + kb * kABytes / 2,
+                                     kABytes / 2, &full[st]);
+                    } else {
+                        mbar_expect_tx(&full[st], kABytes + nb * kWBlockBytes);
+                        tc5::tma_load_2d(a, &x_map, (int)(kb * kBK), (int)m0, &full[st]);
+                    }
                     const char *w = blocks + ((size_t)nb0 * p.k_blocks + kb) * kWBlockBytes;
                     for (uint32_t i = 0; i < nb; ++i)
                         bulk_g2s(b + i * kWBlockBytes, w + (size_t)i * p.k_blocks * kWBlockBytes, kWBlockBytes, &full[st]);
@@ -112,7 +120,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap x_map, const GemmParams p)
         }
     } else if (warp == 1) {
         const bool lead = tc5::elect_one();
-        constexpr uint32_t idesc = tc5::idesc_bf16(kBM, BN);
+        const uint32_t idesc = p.a.pages ? tc5::idesc_f16(kBM, BN) : tc5::idesc_bf16(kBM, BN);
         uint32_t it = 0, n_tile = 0;
         bool ok = true;
         for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++n_tile) {

@@ -25,6 +25,7 @@ struct wr_group_args {
     const uint32_t *list = nullptr;      // device memory, as is:
     const uint32_t *count = nullptr;     // how many entries the list has
     uint32_t max = 0;                    // at most this many
+    uint32_t usual = 1;                  // few rows: how many a single row has
     uint32_t x_rows = 0;
     size_t stride = 0;
 };
@@ -42,6 +43,9 @@ struct wr_gemm_args {
     float mul = 1.f;       // on the result before the residual
     wr_pair_args pair;
     wr_group_args group;   // m: rows the buffers hold
+    // Activations out of a cache instead: row r is row r % 64 of page r / 64 (F16 blocks of 64 rows x 64 values, one after
+    // the other from the page's start on), and the weight holds F16 values.
+    const uint64_t *pages = nullptr;
 };
 
 // A BF16 weight [n][k] as the tensor core reads it: blocks of 64 rows x 64 K-values, each the 8 KB image of a

@@ -240,9 +240,11 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w,
     p.err = ctx->dev_err;
     if (a.pair.from != ~0u && (a.pair.from & 15u)) return WR_CUDA_ERR_INVAL;
     const uint32_t tiles = (w.n + kM - 1) / kM, groups = a.group.list ? a.group.max : 1u;
-    // two CTAs per SM where a slice still has a few blocks of K
+    // two CTAs per SM where a slice still has a few blocks of K (with groups: `usual` of them at a time; the split has
+    // to be the same whatever the step holds)
+    const uint32_t usual = tiles * (a.group.list ? a.group.usual : 1u);
     p.split = 1;
-    while (p.split < kMaxSplit && tiles * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
+    while (p.split < kMaxSplit && usual * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
     constexpr size_t smem = kStages * kStageBytes + 1024;
     if (!(ctx->attr_flags & 128u)) {
         WR_CUDA_TRY(cudaFuncSetAttribute(gemm_skinny_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

@@ -56,6 +56,37 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const wr_rows
     }
 }
 
+// One block per row: the row's angles once, then every head's pairs.
+__global__ void __launch_bounds__(256) latent_rotate_kernel(const wr_rows rw, const wr_latent_geom g, const double *turns, __half *q)
+{
+    __shared__ float2 turn[128];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t row = blockIdx.x, half = g.rot / 2, hs = g.q_head();
+    const uint32_t pos = rw.seqs[seq_of(rw, row)].pos + tok_of(rw, row);
+    for (uint32_t i = threadIdx.x; i < half; i += 256) angle(turns[i], pos, turn[i].y, turn[i].x);
+    __syncthreads();
+    __half *base = q + (size_t)row * g.heads * hs + g.dim_pad();
+    if (half % 2 == 0) {
+        for (uint32_t i = threadIdx.x; i < g.heads * half / 2; i += 256) {
+            const uint32_t h = i / (half / 2), e = 2 * (i % (half / 2));
+            __half2 *pu = reinterpret_cast<__half2 *>(base + h * hs + e);
+            __half2 *pv = reinterpret_cast<__half2 *>(base + h * hs + half + e);
+            const float2 u = __half22float2(*pu), v = __half22float2(*pv), a = turn[e], b = turn[e + 1];
+            *pu = __halves2half2(from_f32<__half>(u.x * a.x - v.x * a.y), from_f32<__half>(u.y * b.x - v.y * b.y));
+            *pv = __halves2half2(from_f32<__half>(v.x * a.x + u.x * a.y), from_f32<__half>(v.y * b.x + u.y * b.y));
+        }
+        return;
+    }
+    for (uint32_t i = threadIdx.x; i < g.heads * half; i += 256) {
+        const uint32_t h = i / half, e = i % half;
+        __half *p = base + h * hs + e;
+        const float u = __half2float(p[0]), v = __half2float(p[half]);
+        p[0] = from_f32<__half>(u * turn[e].x - v * turn[e].y);
+        p[half] = from_f32<__half>(v * turn[e].x + u * turn[e].y);
+    }
+}
+
 // element pairs / quads of a weight row in either layout
 __device__ __forceinline__ float2 weight2(const float *w, uint32_t k, uint32_t r, uint32_t i)
 {
@@ -117,7 +148,7 @@ __global__ void __launch_bounds__(128) latent_query_kernel(const wr_rows rw, con
     for (int r = 0; r < RT; ++r) acc[r][0] = acc[r][1] = 0.f;
 #pragma unroll 8
     for (uint32_t d = lo; d < hi; ++d) {
-        const float2 w = weight2(static_cast<const TW *>(a.w_uk), g.kv_rank, head * g.dim_pad() + d, c0 + 2 * lane);
+        const float2 w = weight2(static_cast<const TW *>(a.w_ukv), g.kv_rank, head * g.dim_pad() + d, c0 + 2 * lane);
 #pragma unroll
         for (int r = 0; r < RT; ++r) {
             acc[r][0] = fmaf(Q[r * g.dim + d], w.x, acc[r][0]);
@@ -162,7 +193,8 @@ __global__ void __launch_bounds__(128) latent_value_kernel(const wr_rows rw, con
         for (int r = 0; r < RT; ++r) acc[r] = 0.f;
 #pragma unroll 4
         for (uint32_t c = 4 * lane; c < ld; c += 128) {
-            const float4 w = weight4(static_cast<const TW *>(a.w_uv), g.kv_rank, head * g.vdim_pad() + v, c);
+            const float4 w = weight4(static_cast<const TW *>(a.w_ukv), g.kv_rank,
+                                       g.heads * g.dim_pad() + head * g.vdim_pad() + v, c);
 #pragma unroll
             for (int r = 0; r < RT; ++r) {
                 const float4 o = load4(sm_lat + r * ld + c);
@@ -218,6 +250,12 @@ int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_p
     if (a.cq_type == WR_ACT_BF16) WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, ctx->stream, rw, a));
     else if (a.cq_type == WR_ACT_SPLIT) WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<Split>, grid, block, 0, ctx->stream, rw, a));
     else WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<float>, grid, block, 0, ctx->stream, rw, a));
+    return finish_launch(ctx);
+}
+
+int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, const double *turns, void *q)
+{
+    WR_CUDA_TRY(wr_launch_pdl(latent_rotate_kernel, dim3(rw.n_rows), dim3(256), 0, ctx->stream, rw, g, turns, static_cast<__half *>(q)));
     return finish_launch(ctx);
 }
 

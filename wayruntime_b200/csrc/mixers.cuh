@@ -137,27 +137,45 @@ struct wr_latent_prep_args {
 };
 int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_prep_args &a);
 
-// Queries moved into the latent: out[row][head] = scale [w_uk^T q | rotated q], padded as the cached row.  w_uk: rows of
-// dim_pad() per head, F32 rows wr_ld(kv_rank) apart or F16 in blocks (wr_weight).
+// Queries moved into the latent: out[row][head] = scale [w_uk^T q | rotated q], padded as the cached row.  w_ukv:
+// dim_pad() key rows per head, then vdim_pad() value rows per head; F32 rows wr_ld(kv_rank) apart or F16 in blocks
+// (wr_weight).
 struct wr_latent_query_args {
     wr_latent_geom g;
     const float *q;                  // [rows][heads][q_head()]
-    const void *w_uk; int w_type;    // WR_ACT_F32 / WR_ACT_F16
+    const void *w_ukv; int w_type;   // WR_ACT_F32 / WR_ACT_F16
     const double *turns;
     float scale;
     float *out;                      // [rows][heads][row()]
 };
 int wr_latent_query_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_query_args &a);
 
-// Latent attention rows back into values: out[row][head * vdim + v] = w_uv o; w_uv as w_uk, vdim_pad() rows per head.
+// Latent attention rows back into values: out[row][head * vdim + v] = w_uv o.
 struct wr_latent_value_args {
     wr_latent_geom g;
     const float *o;                  // [rows][heads][kv_rank]
-    const void *w_uv; int w_type;
+    const void *w_ukv; int w_type;
     void *out; int out_type;         // [rows][out_ld]; the columns up to wr_ld(heads * vdim) are written
     uint32_t out_ld;
 };
 int wr_latent_value_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_value_args &a);
+
+// Causal attention of a prompt's rows on the tensor cores (attn_prefill.cu), with keys and values written out per head.
+struct wr_latent_flash_args {
+    wr_latent_geom g;
+    uint32_t n, p0;                  // rows, and where they start in the session
+    const void *q;                   // F16 [n][heads][q_head()], rotated
+    const void *kv;                  // F16 [p0 + n][heads * dim_pad() keys, then heads * vdim_pad() values]
+    const uint64_t *pages;           // device page table of the rows (their rotated key part)
+    float scale;
+    void *out;                       // BF16 [n][out_ld]; the columns up to wr_ld(heads * vdim) are written
+    uint32_t out_ld;
+};
+bool wr_latent_flash_covers(const wr_latent_geom &g, float scale);
+int wr_latent_flash_launch(wr_cuda_ctx *ctx, const wr_latent_flash_args &a);
+
+// q's rotated parts turned in place (F16 rows as above)
+int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, const double *turns, void *q);
 
 // ---- mixture of experts (moe.cu)
 

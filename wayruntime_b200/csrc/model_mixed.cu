@@ -66,7 +66,8 @@ struct Layer {
     // attention over a latent: `first` = [query latent | latent | rotated key part | router | gate and up]
     wr_latent_geom lat{};
     Mat first, uq;
-    const void *uk = nullptr, *uv = nullptr;
+    Mat ukv;                             // key rows of all heads, then value rows (BF16 models: F16 values)
+    bool flash = false;                  // prompts on the tensor cores
     const float *q_norm = nullptr, *c_norm = nullptr;
     const double *turns = nullptr;
     uint32_t rot_off = 0, logit_off = 0, kv_from = 0;
@@ -386,9 +387,12 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
         mat(o.uq, {Part{&l.w_uq, 0, g.heads * (g.dim + g.rot), 0}.in_groups(g.dim + g.rot, g.q_head(), g.dim, g.dim_pad())},
             g.heads * g.q_head(), g.q_rank);
         const int half = bf ? WR_CUDA_F16 : WR_CUDA_F32;
-        set_off(o.uk, pk.mat({Part{&l.w_uk, 0, g.heads * g.dim, 0}.in_groups(g.dim, g.dim_pad())}, g.heads * g.dim_pad(), g.kv_rank, half));
-        set_off(o.uv, pk.mat({Part{&l.w_uv, 0, g.heads * g.vdim, 0}.in_groups(g.vdim, g.vdim_pad())}, g.heads * g.vdim_pad(), g.kv_rank,
-                             half));
+        o.ukv.n = g.heads * (g.dim_pad() + g.vdim_pad());
+        o.ukv.k = g.kv_rank;
+        set_off(o.ukv.w, pk.mat({Part{&l.w_uk, 0, g.heads * g.dim, 0}.in_groups(g.dim, g.dim_pad()),
+                                 Part{&l.w_uv, 0, g.heads * g.vdim, g.heads * g.dim_pad()}.in_groups(g.vdim, g.vdim_pad())},
+                                o.ukv.n, g.kv_rank, half));
+        o.flash = bf && wr_latent_flash_covers(g, l.attn_scale);
         const uint32_t nv = g.heads * g.vdim;
         if (o.fused) {
             o.ff_at = wr_ld(nv);
@@ -619,8 +623,9 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
             q_few = std::max<size_t>(q_few, g.heads * g.q_head());
             q = std::max<size_t>(q, (size_t)g.heads * g.q_head() * 4);
             mid = std::max<size_t>(mid, wr_ld(l.o.k));
-            qa = std::max<size_t>(qa, (size_t)g.heads * g.row());
-            olat = std::max<size_t>(olat, (size_t)g.heads * g.kv_rank);
+            const size_t n = l.flash ? few : R;          // rows that attend in the latent
+            qa = std::max<size_t>(qa, n * g.heads * g.row());
+            olat = std::max<size_t>(olat, n * g.heads * g.kv_rank);
         } else {
             proj = std::max<size_t>(proj, 2 * wr_ld(l.inner));
             mid = std::max<size_t>(mid, wr_ld(l.inner));
@@ -649,7 +654,7 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
         {(void **)&x->resid, R * x->ldw * 4}, {&x->xin, act(x->ldw)}, {&x->proj, act(proj)},
         {&x->mid, act(mid)}, {&x->scan_out, act(scan)}, {&x->q, std::max(R * q, few * q_few * 4)}, {(void **)&x->attn, R * att * 4},
         {(void **)&x->dbc, R * dbc * 4}, {&x->dbc16, bf ? std::max(R, 2 * few) * dbc * 2 : 0},
-        {(void **)&x->lat, R * lat * 4}, {&x->cq, act(cq)}, {(void **)&x->qa, R * qa * 4}, {(void **)&x->olat, R * olat * 4},
+        {(void **)&x->lat, R * lat * 4}, {&x->cq, act(cq)}, {(void **)&x->qa, qa * 4}, {(void **)&x->olat, olat * 4},
         {(void **)&x->e_weight, R * e_top * 4}, {(void **)&x->e_expert, R * e_top * 4}, {(void **)&x->e_place, R * e_top * 4},
         {(void **)&x->e_row_of, e_rows * 4}, {(void **)&x->e_list, e_list * 4}, {(void **)&x->e_count, 4},
         {&x->e_in, e_in}, {&x->e_act, e_act}, {&x->e_out, e_out},
@@ -695,7 +700,7 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
         fix(l.norm1, x->weights); fix(l.norm2, x->weights); fix(l.shift, x->weights);
         fix(l.qkv_bias, x->weights); fix(l.conv, x->weights); fix(l.conv_b, x->weights); fix(l.dt_b, x->weights);
         fix(l.a2, x->weights); fix(l.d, x->weights);
-        fix(l.uk, x->weights); fix(l.uv, x->weights); fix(l.q_norm, x->weights); fix(l.c_norm, x->weights);
+        fix(l.ukv.w, x->weights); fix(l.q_norm, x->weights); fix(l.c_norm, x->weights);
         fix(l.turns, x->weights); fix(l.router_b, x->weights);
         if (rc == WR_CUDA_OK) rc = fix_mat(l.first, *x, x->xin, rows, x->ldw);
         if (rc == WR_CUDA_OK) rc = fix_mat(l.uq, *x, x->cq, rows, wr_ld(l.uq.k));
@@ -903,18 +908,42 @@ struct Step {
         p.q_norm = l.q_norm; p.c_norm = l.c_norm; p.eps = l.latent_eps; p.turns = l.turns;
         p.cq = x->cq; p.cq_type = in_act(); p.own = own; p.layer = run; p.kv = l.g.kv;
         TRY(wr_latent_prep_launch(ctx, rw, p));
+        if (wide && l.flash) {
+            TRY(product(l.uq, x->cq, wr_ld(g.q_rank), x->q, g.heads * g.q_head(), WR_ACT_F16));
+            TRY(latent_prompt(l, ag, ld_o));
+            return product(l.o, x->mid, ld_o, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
+        }
         TRY(product(l.uq, x->cq, wr_ld(g.q_rank), x->q, g.heads * g.q_head(), WR_ACT_F32));
         wr_latent_query_args q{};
-        q.g = g; q.q = static_cast<const float *>(x->q); q.w_uk = l.uk; q.w_type = bf ? WR_ACT_F16 : WR_ACT_F32;
+        q.g = g; q.q = static_cast<const float *>(x->q); q.w_ukv = l.ukv.w; q.w_type = bf ? WR_ACT_F16 : WR_ACT_F32;
         q.turns = l.turns; q.scale = l.scale; q.out = x->qa;
         TRY(wr_latent_query_launch(ctx, rw, q));
         TRY(wr_attn_any_launch(ctx, rw, ag, x->qa, x->olat, max_len));
         wr_latent_value_args v{};
-        v.g = g; v.o = x->olat; v.w_uv = l.uv; v.w_type = q.w_type;
+        v.g = g; v.o = x->olat; v.w_ukv = l.ukv.w; v.w_type = q.w_type;
         v.out = x->mid; v.out_type = in_act(); v.out_ld = ld_o;
         TRY(wr_latent_value_launch(ctx, rw, v));
         m->launches += 4;
         return product(l.o, x->mid, ld_o, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
+    }
+
+    // Keys and values of every head written out for the whole context (one product on the cached rows), then attention.
+    int latent_prompt(const Layer &l, const wr_attn_geom &ag, uint32_t ld_o)
+    {
+        const wr_latent_geom &g = l.lat;
+        const uint64_t *pages = kv[0]->d_pages + (size_t)ag.layer * kv[0]->n_pages;
+        TRY(wr_latent_rotate_launch(ctx, rw, g, l.turns, x->q));
+        TRY(wr_ctx_reserve_ws(ctx, (size_t)max_len * l.ukv.n * 2, 0));
+        wr_gemm_args a{};
+        a.m = max_len;
+        a.out = ctx->ws; a.out_ld = l.ukv.n; a.out_type = WR_GEMM_OUT_F16;
+        a.pages = pages;
+        TRY(wr_gemm_launch(ctx, l.o.x_map, {l.ukv.w, l.ukv.n, l.ukv.k}, a));     // (the map is not read)
+        wr_latent_flash_args f{};
+        f.g = g; f.n = rw.n_rows; f.p0 = positions[0]; f.q = x->q; f.kv = ctx->ws; f.pages = pages; f.scale = l.scale;
+        f.out = x->mid; f.out_ld = ld_o;
+        m->launches += 3;
+        return wr_latent_flash_launch(ctx, f);
     }
 
     // F32 models: silu(gate h) * (up h)
@@ -970,7 +999,7 @@ struct Step {
         TRY(wr_route_launch(ctx, rw, r));
         const uint32_t groups = wr_route_tiles(rw.n_rows, l.experts, l.top, r.tile), lf = wr_ld(l.ff);
         wr_group_args gr;
-        gr.list = x->e_list; gr.count = x->e_count; gr.max = groups;
+        gr.list = x->e_list; gr.count = x->e_count; gr.max = groups; gr.usual = l.top;
         wr_combine_args c{};
         if (split()) {
             wr_skinny_args a{};

@@ -20,6 +20,8 @@ __host__ __device__ constexpr uint32_t idesc_bf16(uint32_t m, uint32_t n)
 {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((m >> 4) << 24);
 }
+// ... and for F16 x F16 -> F32
+__host__ __device__ constexpr uint32_t idesc_f16(uint32_t m, uint32_t n) { return (1u << 4) | ((n >> 3) << 17) | ((m >> 4) << 24); }
 __device__ __forceinline__ bool elect_one()
 {
     uint32_t pred;
