@@ -17,7 +17,7 @@ STAMP_PATH = LIB_PATH + ".sources"          # digest of what the library was bui
 INCLUDE = os.path.join(os.path.dirname(PKG), "include")
 
 SOURCES = ["kv_cache.cu", "attn_decode.cu", "attn_decode_static.cu", "attn_prefill.cu", "attn_exchange.cu",
-           "model_glue.cu", "attn_step_small.cu", "gemv.cu", "gemm_bf16.cu", "gemm_skinny.cu", "mixers.cu", "latent.cu",
+           "model_glue.cu", "attn_step_small.cu", "gemv.cu", "gemm_bf16.cu", "gemm_skinny.cu", "mixers.cu", "latent.cu", "attn_latent.cu",
            "moe.cu", "model_mixed.cu"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -174,6 +174,12 @@ struct wr_latent_flash_args {
 bool wr_latent_flash_covers(const wr_latent_geom &g, float scale);
 int wr_latent_flash_launch(wr_cuda_ctx *ctx, const wr_latent_flash_args &a);
 
+// Attention of at most WR_CUDA_BATCH_MAX rows over the cached F16 rows (attn_latent.cu): q as wr_latent_query_launch leaves
+// it, out [rows][heads][kv_rank], lens: how many keys each row sees (host).
+bool wr_latent_decode_covers(const wr_latent_geom &g);
+int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, uint32_t layer, const float *q, float *out,
+                            const uint32_t *lens);
+
 // q's rotated parts turned in place (F16 rows as above)
 int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, const double *turns, void *q);
 

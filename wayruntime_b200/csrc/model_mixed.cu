@@ -67,7 +67,7 @@ struct Layer {
     wr_latent_geom lat{};
     Mat first, uq;
     Mat ukv;                             // key rows of all heads, then value rows (BF16 models: F16 values)
-    bool flash = false;                  // prompts on the tensor cores
+    bool flash = false, tensor_decode = false;                   // prompts / few rows on the tensor cores
     const float *q_norm = nullptr, *c_norm = nullptr;
     const double *turns = nullptr;
     uint32_t rot_off = 0, logit_off = 0, kv_from = 0;
@@ -393,6 +393,7 @@ void pack_layer(Packer &pk, const wr_cuda_mixed_layer &l, Layer &o, uint32_t wid
                                  Part{&l.w_uv, 0, g.heads * g.vdim, g.heads * g.dim_pad()}.in_groups(g.vdim, g.vdim_pad())},
                                 o.ukv.n, g.kv_rank, half));
         o.flash = bf && wr_latent_flash_covers(g, l.attn_scale);
+        o.tensor_decode = bf && wr_latent_decode_covers(g);
         const uint32_t nv = g.heads * g.vdim;
         if (o.fused) {
             o.ff_at = wr_ld(nv);
@@ -918,7 +919,14 @@ struct Step {
         q.g = g; q.q = static_cast<const float *>(x->q); q.w_ukv = l.ukv.w; q.w_type = bf ? WR_ACT_F16 : WR_ACT_F32;
         q.turns = l.turns; q.scale = l.scale; q.out = x->qa;
         TRY(wr_latent_query_launch(ctx, rw, q));
-        TRY(wr_attn_any_launch(ctx, rw, ag, x->qa, x->olat, max_len));
+        if (l.tensor_decode && split()) {
+            uint32_t lens[WR_CUDA_BATCH_MAX];
+            for (uint32_t r = 0; r < rw.n_rows; ++r) lens[r] = rw.decode ? positions[r] + 1 : positions[0] + r + 1;
+            TRY(wr_latent_decode_launch(ctx, rw, g, ag.layer, x->qa, x->olat, lens));
+            ++m->launches;
+        } else {
+            TRY(wr_attn_any_launch(ctx, rw, ag, x->qa, x->olat, max_len));
+        }
         wr_latent_value_args v{};
         v.g = g; v.o = x->olat; v.w_ukv = l.ukv.w; v.w_type = q.w_type;
         v.out = x->mid; v.out_type = in_act(); v.out_ld = ld_o;

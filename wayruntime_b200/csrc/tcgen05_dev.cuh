@@ -15,6 +15,15 @@ __device__ __forceinline__ uint64_t desc_kmajor(uint32_t smem_addr)
     const uint64_t hi = (uint64_t)(1024u >> 4) | (1ull << 14) | (2ull << 29);
     return lo | (hi << 32);
 }
+// The same swizzle for an operand whose M (or N) values are contiguous: 64 of them to a 128-byte row, the next 64 `lbo`
+// bytes on, eight K values to 1024 bytes.
+__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t smem_addr, uint32_t lbo)
+{
+    const uint64_t lo = (uint64_t)((smem_addr & 0x3FFFFu) >> 4) | ((uint64_t)(lbo >> 4) << 16);
+    const uint64_t hi = (uint64_t)(1024u >> 4) | (1ull << 14) | (2ull << 29);
+    return lo | (hi << 32);
+}
+constexpr uint32_t kIdescAMnMajor = 1u << 15;            // A is laid out that way
 // kind::f16 instruction descriptor for BF16 x BF16 -> F32, both operands K-major.
 __host__ __device__ constexpr uint32_t idesc_bf16(uint32_t m, uint32_t n)
 {
@@ -69,6 +78,21 @@ __device__ __forceinline__ void ld32(uint32_t taddr, float *v)
           "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]),
           "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
         : "r"(taddr));
+}
+__device__ __forceinline__ void wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// ... and back (no wait)
+__device__ __forceinline__ void st32(uint32_t taddr, const float *v)
+{
+    const uint32_t *r = reinterpret_cast<const uint32_t *>(v);
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+        "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,"
+        "%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
+        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+          "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
+          "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
+          "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+        : "memory");
 }
 // Tiled 2-D tensor copy global -> shared (no multicast); x in elements, x * element size a multiple of 16.
 __device__ __forceinline__ void tma_load_2d(void *dst_smem, const CUtensorMap *map, int x, int y, uint64_t *bar)
