@@ -12,11 +12,12 @@
 //     products see about 22 bits of them;
 //   * warps 2-5, a thread per key: column maxima across the tile, exponentials, P^T to shared memory.  O^T stays in
 //     TMEM and is rescaled only when a maximum has grown by more than 2^8.
-// A chunk leaves (maximum, sum, O) in F32; latent_merge_kernel adds the chunks up in order.  How a session is cut into
+// The queries come as that operand already (wr_latent_query_launch).  A chunk leaves (maximum, sum) and O in F32; the
+// value kernel, or latent_merge_kernel where there are many, adds the chunks up in order.  How a session is cut into
 // chunks depends on its own length alone.  Every wait is bounded by the context's wait limit.
 #include <algorithm>
 
-#include "rows_dev.cuh"
+#include "latent_dev.cuh"
 #include "tcgen05_dev.cuh"
 
 namespace {
@@ -24,14 +25,14 @@ namespace {
 constexpr uint32_t kTile = 128, kThreads = 192, kBox = kTile * 128, kUnit = 2 * kBox, kBlock = 8192;
 constexpr uint32_t kMaxUnits = 16, kMaxRot = 8;
 constexpr uint32_t kSmemMax = 232448;
-constexpr float kLn2 = 0.6931471805599453f, kLog2 = 1.4426950408889634f;
+constexpr float kLn2 = 0.6931471805599453f;
 constexpr float kGrow = 8.0f;
 
 // tiles per chunk, by the session's length
 __host__ __device__ inline uint32_t chunk_tiles(uint32_t len)
 {
     const uint32_t tiles = (len + kTile - 1) / kTile, c = (tiles + 63) / 64;
-    return tiles > 8 && c < 2 ? 2u : c;
+    return tiles > 16 && c < 2 ? 2u : c;
 }
 __host__ __device__ inline uint32_t chunk_count(uint32_t len)
 {
@@ -41,12 +42,15 @@ __host__ __device__ inline uint32_t chunk_count(uint32_t len)
 
 struct LatentParams {
     wr_rows rw;
-    uint32_t heads, rank, row, layer;            // row: values of a cached row
+    uint32_t heads, layer;
     uint32_t units, rot_boxes, boxes;            // per tile: pairs of latent boxes, rotated boxes; boxes of a query
     uint32_t ring, rot_ring, tmem_cols;
-    uint32_t chunks;                             // of the longest row: the stride of ws
-    const float *q;                              // [rows][heads][row]
-    float *ws;                                   // [rows][heads][chunks][rank + 2]
+    uint32_t chunks;                             // of the longest row: the stride of ml and o
+    wr_latent_lens lens;
+    const char *q;                               // [rows][head groups][boxes][2 NH][128 B]
+    size_t q_row;
+    float *ml, *o;                               // [rows][heads][chunks][2], [rows][heads][chunks][rank_pad]
+    uint32_t rank_pad;
     long long wait_limit;
     int *err;
 };
@@ -104,10 +108,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t chunk = blockIdx.x, head0 = blockIdx.y * NH, row = blockIdx.z;
     pdl_trigger();
-    pdl_wait();
-    const wr_seq_dev s = p.rw.seqs[seq_of(p.rw, row)];
-    const uint32_t len = s.pos + tok_of(p.rw, row) + 1, per = chunk_tiles(len);
-    if (chunk >= chunk_count(len)) return;
+    const uint32_t len = p.lens.len[row], per = chunk_tiles(len);
+    if (chunk >= p.lens.count[row]) {
+        pdl_wait();
+        return;
+    }
     const uint32_t tile0 = chunk * per, tiles = min(per, (len + kTile - 1) / kTile - tile0);
     if (threadIdx.x == 0) {
         for (uint32_t i = 0; i < p.ring; ++i) {
@@ -118,7 +123,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
             mbar_init(&sm.rot_full[i], 1);
             mbar_init(&sm.rot_empty[i], 1);
         }
-        mbar_init(&sm.q_full, 4);
+        mbar_init(&sm.q_full, 1);
         mbar_init(&sm.s_full, 1);
         mbar_init(&sm.p_full, 4);
         mbar_init(&sm.o_full, 1);
@@ -128,10 +133,14 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     tc5::fence_before();
     __syncthreads();
     tc5::fence_after();
+    pdl_wait();
     const uint32_t tmem_s = sm.tmem, tmem_o = tmem_s + 32;       // (S: 32 columns whatever N is)
 
     if (warp == 0) {
         if (lane == 0) {
+            mbar_expect_tx(&sm.q_full, p.boxes * N * 128);
+            bulk_g2s(qs, p.q + row * p.q_row + (size_t)blockIdx.y * p.boxes * N * 128, p.boxes * N * 128, &sm.q_full);
+            const wr_seq_dev s = p.rw.seqs[seq_of(p.rw, row)];
             const uint64_t *table = s.pages + (size_t)p.layer * s.n_pages;
             const uint32_t last_page = (len - 1) / kPageTokens, rank_boxes = p.boxes - p.rot_boxes;
             uint32_t n_unit = 0, n_rot = 0;              // requested so far
@@ -166,6 +175,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
             }
             if (!ok) atomicCAS(p.err, 0, 61);
             // nothing in flight when the CTA leaves
+            (void)mbar_wait(&sm.q_full, 0, p.wait_limit);
             for (uint32_t i = n_unit - min(n_unit, p.ring); i < n_unit; ++i)
                 (void)mbar_wait(&sm.full[i % p.ring], (i / p.ring) & 1, p.wait_limit);
             for (uint32_t i = n_rot - min(n_rot, p.rot_ring); i < n_rot; ++i)
@@ -228,22 +238,6 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     } else {
         const uint32_t quarter = warp & 3, key = quarter * 32 + lane, tid = threadIdx.x - 64, lanes = (quarter * 32) << 16;
         const uint32_t nh = min((uint32_t)NH, p.heads - head0);
-        // the group's queries, split, in the log2 domain
-        const float *q = p.q + ((size_t)row * p.heads + head0) * p.row;
-        for (uint32_t i = tid; i < NH * (p.row / 2); i += 128) {
-            const uint32_t h = i / (p.row / 2), c = 2 * (i % (p.row / 2));
-            float2 v = make_float2(0.f, 0.f);
-            if (h < nh) v = *reinterpret_cast<const float2 *>(q + (size_t)h * p.row + c);
-            v.x = fminf(fmaxf(v.x * kLog2, -65504.f), 65504.f);
-            v.y = fminf(fmaxf(v.y * kLog2, -65504.f), 65504.f);
-            uint32_t hi, lo;
-            split_half2(v.x, v.y, hi, lo);
-            *reinterpret_cast<uint32_t *>(qs + swizzled(N, h, c)) = hi;
-            *reinterpret_cast<uint32_t *>(qs + swizzled(N, NH + h, c)) = lo;
-        }
-        fence_proxy_async();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&sm.q_full);
         float m[NH], l[NH];
 #pragma unroll
         for (int h = 0; h < NH; ++h) {
@@ -310,56 +304,54 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
         if (ok) ok = mbar_wait(&sm.o_full, 0, p.wait_limit);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok && lane == 0) atomicCAS(p.err, 0, 63);
-        {
-            tc5::fence_after();
-            const size_t stride = (size_t)p.chunks * (p.rank + 2);
-            float *ws = p.ws + (((size_t)row * p.heads + head0) * p.chunks + chunk) * (p.rank + 2);
+        tc5::fence_after();
+        const size_t at = ((size_t)row * p.heads + head0) * p.chunks + chunk, stride = (size_t)p.chunks * p.rank_pad;
+        float *out = p.o + at * p.rank_pad;
 #pragma unroll 1
-            for (uint32_t c = 0; c < p.units * N; c += 32) {
-                float v[32];
-                tc5::ld32(tmem_o + lanes + c, v);
-                tc5::wait_ld();
+        for (uint32_t c = 0; c < p.units * N; c += 32) {
+            float v[32];
+            tc5::ld32(tmem_o + lanes + c, v);
+            tc5::wait_ld();
 #pragma unroll
-                for (uint32_t j = 0; j < 32 / N; ++j) {
-                    const uint32_t d = (c / N + j) * 128 + key;
+            for (uint32_t j = 0; j < 32 / N; ++j) {
+                const uint32_t d = (c / N + j) * 128 + key;
 #pragma unroll
-                    for (uint32_t h = 0; h < NH; ++h)
-                        if (h < nh && d < p.rank) ws[h * stride + 2 + d] = v[j * N + h] + v[j * N + NH + h];
-                }
+                for (uint32_t h = 0; h < NH; ++h)
+                    if (h < nh && d < p.rank_pad) out[h * stride + d] = v[j * N + h] + v[j * N + NH + h];
             }
-            // the sums: across the warp's keys, then the four warps in order
-            const uint32_t b = tiles & 1;
-            uint32_t idx = 0;
-            {
-                uint32_t width = NH;
-#pragma unroll
-                for (uint32_t o = 16; o >= 1; o >>= 1) {
-                    if (width > 1) {
-                        const uint32_t half = width / 2;
-                        const bool upper = (lane & o) != 0;
-#pragma unroll
-                        for (uint32_t i = 0; i < NH / 2; ++i)
-                            if (i < half) {
-                                const float send = upper ? l[i] : l[i + half], keep = upper ? l[i + half] : l[i];
-                                l[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                            }
-                        if (upper) idx += half;
-                        width = half;
-                    } else {
-                        l[0] += __shfl_xor_sync(0xffffffffu, l[0], o);
-                    }
-                }
-            }
-            sm.red[b][idx][quarter] = l[0];
-            group_sync();
-#pragma unroll
-            for (uint32_t h = 0; h < NH; ++h)
-                if (tid == h && h < nh) {
-                    const float4 w = *reinterpret_cast<const float4 *>(sm.red[b][h]);
-                    ws[h * stride] = m[h] * kLn2;
-                    ws[h * stride + 1] = ((w.x + w.y) + w.z) + w.w;
-                }
         }
+        // the sums: across the warp's keys, then the four warps in order
+        const uint32_t b = tiles & 1;
+        uint32_t idx = 0;
+        {
+            uint32_t width = NH;
+#pragma unroll
+            for (uint32_t o = 16; o >= 1; o >>= 1) {
+                if (width > 1) {
+                    const uint32_t half = width / 2;
+                    const bool upper = (lane & o) != 0;
+#pragma unroll
+                    for (uint32_t i = 0; i < NH / 2; ++i)
+                        if (i < half) {
+                            const float send = upper ? l[i] : l[i + half], keep = upper ? l[i + half] : l[i];
+                            l[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                    if (upper) idx += half;
+                    width = half;
+                } else {
+                    l[0] += __shfl_xor_sync(0xffffffffu, l[0], o);
+                }
+            }
+        }
+        sm.red[b][idx][quarter] = l[0];
+        group_sync();
+#pragma unroll
+        for (uint32_t h = 0; h < NH; ++h)
+            if (tid == h && h < nh) {
+                const float4 w = *reinterpret_cast<const float4 *>(sm.red[b][h]);
+                *reinterpret_cast<float2 *>(p.ml + 2 * (at + (size_t)h * p.chunks)) =
+                    make_float2(m[h] * kLn2, ((w.x + w.y) + w.z) + w.w);
+            }
     }
     tc5::fence_before();
     __syncthreads();
@@ -368,36 +360,17 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
 }
 
 // Chunks of a row and head added up, in order.
-__global__ void __launch_bounds__(128) latent_merge_kernel(const wr_rows rw, const float *ws, float *out, uint32_t heads,
-                                                           uint32_t rank, uint32_t chunks)
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p, float *out)
 {
     __shared__ float w[64];
     pdl_trigger();
     pdl_wait();
-    const uint32_t head = blockIdx.x, row = blockIdx.y;
-    const uint32_t n = chunk_count(rw.seqs[seq_of(rw, row)].pos + tok_of(rw, row) + 1), stride = rank + 2;
-    const float *in = ws + ((size_t)row * heads + head) * chunks * stride;
-    if (threadIdx.x < 32) {
-        float m = -INFINITY, l = 0.f;
-        for (uint32_t i = threadIdx.x; i < n; i += 32) m = fmaxf(m, in[(size_t)i * stride]);
-#pragma unroll
-        for (int o = 16; o >= 1; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-        for (uint32_t i = threadIdx.x; i < n; i += 32) {
-            const float e = expf(in[(size_t)i * stride] - m);
-            w[i] = e;
-            l = fmaf(e, in[(size_t)i * stride + 1], l);
-        }
-        l = warp_sum(l);
-        __syncwarp();
-        for (uint32_t i = threadIdx.x; i < n; i += 32) w[i] /= l;
-    }
+    const uint32_t head = blockIdx.x, row = blockIdx.y, n = p.lens.count[row];
+    const size_t at = ((size_t)row * p.heads + head) * p.chunks;
+    if (threadIdx.x < 32) latent_chunk_weights(p.ml + 2 * at, n, w, threadIdx.x);
     __syncthreads();
-    for (uint32_t c = threadIdx.x; c < rank; c += 128) {
-        float o = 0.f;
-#pragma unroll 8
-        for (uint32_t i = 0; i < n; ++i) o = fmaf(w[i], in[(size_t)i * stride + 2 + c], o);
-        out[((size_t)row * heads + head) * rank + c] = o;
-    }
+    for (uint32_t c = 4 * threadIdx.x; c < p.rank_pad; c += 512)
+        store4(out + ((size_t)row * p.heads + head) * p.rank_pad + c, latent_chunk_sum(p.o + at * p.rank_pad + c, p.rank_pad, w, n));
 }
 
 // sizes of the rings; 0: it does not fit
@@ -434,30 +407,43 @@ template <int NH> int launch(wr_cuda_ctx *ctx, const LatentParams &p, uint32_t s
 bool wr_latent_decode_covers(const wr_latent_geom &g)
 {
     LatentParams p{};
-    return plan(g, g.heads <= 8 ? 8 : 16, p) != 0;
+    return g.dim_pad() <= 512 && plan(g, wr_latent_group(g), p) != 0;
 }
 
-int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, uint32_t layer, const float *q, float *out,
-                            const uint32_t *lens)
+int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, uint32_t layer, const void *q,
+                            const uint32_t *lens, float *merged, wr_latent_value_args &out)
 {
     LatentParams p{};
-    const uint32_t nh = g.heads <= 8 ? 8 : 16, smem = plan(g, nh, p);
-    if (!smem) return WR_CUDA_ERR_LIMIT;
+    const uint32_t nh = wr_latent_group(g), smem = plan(g, nh, p);
+    if (!smem || rw.n_rows > WR_CUDA_BATCH_MAX) return WR_CUDA_ERR_LIMIT;
     p.rw = rw;
     p.heads = g.heads;
-    p.rank = g.kv_rank;
-    p.row = g.row();
+    p.rank_pad = g.rank_pad();
     p.layer = layer;
-    for (uint32_t r = 0; r < rw.n_rows; ++r) p.chunks = std::max(p.chunks, chunk_count(lens[r]));
-    int rc = wr_ctx_reserve_ws(ctx, (size_t)rw.n_rows * g.heads * p.chunks * (g.kv_rank + 2) * sizeof(float), 0);
+    for (uint32_t r = 0; r < rw.n_rows; ++r) {
+        p.lens.len[r] = lens[r];
+        p.lens.count[r] = chunk_count(lens[r]);
+        p.chunks = std::max(p.chunks, p.lens.count[r]);
+    }
+    const size_t pieces = (size_t)rw.n_rows * g.heads * p.chunks, ml = (pieces * 2 + 63) & ~(size_t)63;
+    int rc = wr_ctx_reserve_ws(ctx, (ml + pieces * p.rank_pad) * sizeof(float), 0);
     if (rc != WR_CUDA_OK) return rc;
-    p.q = q;
-    p.ws = ctx->ws;
+    p.q = static_cast<const char *>(q);
+    p.q_row = wr_latent_split_bytes(g);
+    p.ml = ctx->ws;
+    p.o = ctx->ws + ml;
     p.wait_limit = ctx->wait_limit;
     p.err = ctx->dev_err;
     rc = nh == 8 ? launch<8>(ctx, p, smem) : launch<16>(ctx, p, smem);
     if (rc != WR_CUDA_OK) return rc;
-    WR_CUDA_TRY(wr_launch_pdl(latent_merge_kernel, dim3(g.heads, rw.n_rows), dim3(128), 0, ctx->stream, rw, (const float *)ctx->ws,
-                              out, g.heads, g.kv_rank, p.chunks));
+    out.lens = p.lens;
+    out.chunks = p.chunks;
+    out.ml = p.ml;
+    out.o = p.o;
+    // (few enough: every block of the value kernel adds them up for itself; the same sums either way)
+    if (p.chunks <= kLatentMaxFused && rw.n_rows * p.chunks <= 32) return WR_CUDA_OK;
+    WR_CUDA_TRY(wr_launch_pdl(latent_merge_kernel, dim3(g.heads, rw.n_rows), dim3(128), 0, ctx->stream, p, merged));
+    out.ml = nullptr;
+    out.o = merged;
     return finish_launch(ctx);
 }

@@ -125,7 +125,7 @@ struct prefill_params {
     uint32_t q_head, q_rot;                      // columns per head of the query rows; where the rotated ones start
     uint32_t k_head, v_at, v_head;               // columns per head of the K / V rows; where V starts
     uint32_t rot_block;                          // 64-wide block of a page where the rotated key part starts
-    uint32_t k_stages, v_stages;
+    uint32_t k_stages, v_stages, single; // single: work tiles of one block each
     uint32_t vdim, v_cols, out_ld;               // value size, rounded up to 16; row length of the output
     __nv_bfloat16 *out;
 };
@@ -152,9 +152,9 @@ struct smem_bars {
     uint32_t tmem_base;
 };
 // per softmax warp: two buffers of 32 rows x 16 output values on their way out (16-byte pieces swizzled by row pair:
-// the 64-byte swizzle of the output tensor map); LATENT: one of 32 rows x 32 BF16 values
+// the 64-byte swizzle of the output tensor map); LATENT: none
 constexpr uint32_t kOutPiece = 32 * 64;
-constexpr uint32_t kOutBytes = 8 * 2 * kOutPiece, kOutBytesLatent = 8 * kOutPiece;
+constexpr uint32_t kOutBytes = 8 * 2 * kOutPiece;
 constexpr uint32_t kSmemBytes = 2 * kQBytes + 2 * kStages * kKVTile + kOutBytes + sizeof(smem_bars);
 static_assert(kSmemBytes <= 232448, "the CTA's shared memory is 227 KB at most");
 
@@ -366,6 +366,12 @@ __device__ inline tile_info decode_tile(const prefill_params &p, uint32_t idx)
     t.head[0] = t.head[1] = 0; t.qt[0] = t.qt[1] = 0;
     if (idx >= p.n_tiles) return t;
     t.valid = 1;
+    if (p.single) {
+        t.nblk = 1;
+        t.kvh = t.head[0] = idx % p.n_kv;
+        t.qt[0] = p.n_qtiles - 1 - idx / p.n_kv;
+        return t;
+    }
     const uint32_t per = tiles_per_qpair(p.n_kv, p.group), pairs = p.group / 2u, odd = p.group & 1u;
     const uint32_t k = idx / per;                    // query-tile pair, counted from the end of the prompt
     uint32_t r = idx % per;
@@ -420,7 +426,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
     const uint32_t k_stages = LATENT ? p.k_stages : (uint32_t)kStages, v_stages = LATENT ? p.v_stages : (uint32_t)kStages;
     uint8_t *const sm_q = smem_raw, *const sm_k = sm_q + 2 * q_bytes, *const sm_v = sm_k + k_stages * k_bytes;
     uint8_t *const sm_out = sm_v + v_stages * v_bytes;
-    smem_bars &sm = *reinterpret_cast<smem_bars *>(sm_out + (LATENT ? kOutBytesLatent : kOutBytes));
+    smem_bars &sm = *reinterpret_cast<smem_bars *>(sm_out + (LATENT ? 0u : kOutBytes));
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 #ifdef WR_PREFILL_TIMELINE
     if (tid == 0 && p.tl && blockIdx.x < kTlCtas) p.tl[kTlRoles * kTlEvents + blockIdx.x * 4] = tl_ns();
@@ -717,7 +723,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
                 const bool more = j + 1 < hi;
                 // this step's V tile and the next step's K tile landed long ago
                 ok = mbar_wait(&sm.v_full[v_st], v_par, limit);
-                if (ok && more) ok = mbar_wait(&sm.k_full[k_st], k_par, limit);
+                if (!LATENT && ok && more) ok = mbar_wait(&sm.k_full[k_st], k_par, limit);
                 if (!ok) break;
                 // one block: wait for its P, issue its P.V, then its next scores
                 auto step_block = [&](uint32_t b, uint32_t blo, uint32_t bhi, uint32_t key_end, uint32_t &p_uses,
@@ -741,6 +747,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
                         }
                     }
                     if (more && j + 1 >= blo && j + 1 < bhi) {
+                        if (LATENT) {                            // (its K ring may be one stage deep)
+                            if (!mbar_wait(&sm.k_full[k_st], k_par, limit)) return false;
+                            tc_fence_after();
+                        }
                         issue_s(b, k_st);                        // (P_b of step j was consumed just above)
                         if (lead && j + 2 == bhi) umma_commit(&sm.q_free[b]);       // the block's last scores
                     }
@@ -947,41 +957,50 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             // buffers take turns: a piece is waited for only when its buffer is needed again.
             pdl_wait();                                      // output rows: after the earlier kernels have ended
             if constexpr (LATENT) {
+                // Four lanes exchange 16-byte pieces of their four rows, so that they write 64 bytes of one row at a time.
                 const float inv = (l > 0.f) ? 1.0f / l : 0.f;
-                uint8_t *stage = sm_out + warp * kOutPiece;
+                const uint32_t piece = lane & 3u;
 #pragma unroll
-                for (int c = 0; c < kHd / 32; ++c) {             // pieces of 32 values
+                for (int c = 0; c < kHd / 32; ++c) {
                     if (32u * c >= p.vdim) break;
-                    __syncwarp();
+                    uint4 e[4];
 #pragma unroll
                     for (int k = 0; k < 4; ++k) {
                         uint32_t w[4];
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const __nv_bfloat162 h = __floats2bfloat162_rn(o[32 * c + 8 * k + 2 * e] * inv,
-                                                                          o[32 * c + 8 * k + 2 * e + 1] * inv);
-                            w[e] = *reinterpret_cast<const uint32_t *>(&h);
+                        for (int x = 0; x < 4; ++x) {
+                            const __nv_bfloat162 h = __floats2bfloat162_rn(o[32 * c + 8 * k + 2 * x] * inv,
+                                                                          o[32 * c + 8 * k + 2 * x + 1] * inv);
+                            w[x] = *reinterpret_cast<const uint32_t *>(&h);
                         }
-                        *reinterpret_cast<uint4 *>(stage + lane * 64 + ((k ^ ((lane >> 1) & 3u)) << 4)) =
-                            make_uint4(w[0], w[1], w[2], w[3]);
+                        e[k] = make_uint4(w[0], w[1], w[2], w[3]);
                     }
-                    __syncwarp();
-                    // four lanes write a row's 64 bytes
-                    const uint32_t col = 32u * c + 8u * (lane & 3u);
+#pragma unroll
+                    for (int step = 1; step <= 2; ++step)
+#pragma unroll
+                        for (int k = 0; k < 2; ++k) {
+                            const int lo = step == 1 ? 2 * k : k, hi = lo + step;
+                            const bool up = (lane & step) != 0;
+                            const uint4 give = up ? e[lo] : e[hi];
+                            const uint4 got = make_uint4(__shfl_xor_sync(0xffffffffu, give.x, step), __shfl_xor_sync(0xffffffffu, give.y, step),
+                                                         __shfl_xor_sync(0xffffffffu, give.z, step), __shfl_xor_sync(0xffffffffu, give.w, step));
+                            if (up) e[lo] = got;
+                            else e[hi] = got;
+                        }
+                    const uint32_t col = 32u * c + 8u * piece;
 #pragma unroll
                     for (uint32_t i = 0; i < 4; ++i) {
-                        const uint32_t r = 8 * i + (lane >> 2), tr = wq * 32u + r;
-                        if (tr >= me.rows || col >= p.vdim) continue;
-                        const uint4 w = *reinterpret_cast<const uint4 *>(stage + r * 64 + (((lane & 3u) ^ ((r >> 1) & 3u)) << 4));
-                        __nv_bfloat16 *dst = p.out + (size_t)(me.tok0 + tr) * p.out_ld + head * p.vdim + col;
+                        const uint32_t r = wq * 32u + (lane & ~3u) + i;
+                        if (r >= me.rows || col >= p.vdim) continue;
+                        __nv_bfloat16 *dst = p.out + (size_t)(me.tok0 + r) * p.out_ld + head * p.vdim + col;
                         if (p.vdim % 8 == 0) {
-                            *reinterpret_cast<uint4 *>(dst) = w;
+                            *reinterpret_cast<uint4 *>(dst) = e[i];
                         } else {
-                            const uint32_t part[4] = {w.x, w.y, w.z, w.w};
+                            const uint32_t part[4] = {e[i].x, e[i].y, e[i].z, e[i].w};
 #pragma unroll
-                            for (uint32_t e = 0; e < 8; ++e)
-                                if (col + e < p.vdim)
-                                    reinterpret_cast<uint16_t *>(dst)[e] = (uint16_t)(part[e >> 1] >> (16 * (e & 1)));
+                            for (uint32_t x = 0; x < 8; ++x)
+                                if (col + x < p.vdim)
+                                    reinterpret_cast<uint16_t *>(dst)[x] = (uint16_t)(part[x >> 1] >> (16 * (x & 1)));
                         }
                     }
                 }
@@ -1206,9 +1225,9 @@ bool box_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, u
 uint32_t latent_smem(const wr_latent_geom &g, uint32_t &k_stages, uint32_t &v_stages)
 {
     const uint32_t q = (g.dim_pad() + 63) / 64 + (g.rot_pad() + 63) / 64, v = (g.vdim_pad() + 63) / 64;
-    const uint32_t try_k[3] = {2, 1, 1}, try_v[3] = {2, 2, 1};
+    const uint32_t try_k[3] = {2, 2, 1}, try_v[3] = {2, 1, 1};
     for (int i = 0; i < 3; ++i) {
-        const uint64_t bytes = (uint64_t)(2 * q + try_k[i] * q + try_v[i] * v) * kQHalfBytes + kOutBytesLatent + sizeof(smem_bars);
+        const uint64_t bytes = (uint64_t)(2 * q + try_k[i] * q + try_v[i] * v) * kQHalfBytes + sizeof(smem_bars);
         if (bytes > 232448) continue;
         k_stages = try_k[i];
         v_stages = try_v[i];
@@ -1250,6 +1269,10 @@ int wr_latent_flash_launch(wr_cuda_ctx *ctx, const wr_latent_flash_args &a)
     p.group = 1;
     p.n_qtiles = (a.n + kBM - 1) / kBM;
     p.n_tiles = prefill_tile_count(p.n_qtiles, p.n_kv, p.group);
+    if (p.n_tiles < (uint32_t)ctx->sm_count) {                   // too few to go round: blocks by themselves
+        p.single = 1;
+        p.n_tiles = p.n_qtiles * p.n_kv;
+    }
     p.scale_log2 = a.scale * kLog2e;
     p.nope_boxes = (g.dim_pad() + 63) / 64;
     p.q_boxes = p.nope_boxes + (g.rot_pad() + 63) / 64;

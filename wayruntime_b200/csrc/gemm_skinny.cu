@@ -242,9 +242,9 @@ int wr_skinny_launch(wr_cuda_ctx *ctx, const CUtensorMap &x, const wr_weight &w,
     const uint32_t tiles = (w.n + kM - 1) / kM, groups = a.group.list ? a.group.max : 1u;
     // two CTAs per SM where a slice still has a few blocks of K (with groups: `usual` of them at a time; the split has
     // to be the same whatever the step holds)
-    const uint32_t usual = tiles * (a.group.list ? a.group.usual : 1u);
+    const uint32_t usual = tiles * (a.group.list ? a.group.usual : 1u), room = (a.group.list ? 1.3 : 2.0) * ctx->sm_count;
     p.split = 1;
-    while (p.split < kMaxSplit && usual * p.split * 2 <= 2u * (uint32_t)ctx->sm_count && p.k_blocks >= 8 * p.split) p.split *= 2;
+    while (p.split < kMaxSplit && usual * p.split * 2 <= room && p.k_blocks >= 8 * p.split) p.split *= 2;
     constexpr size_t smem = kStages * kStageBytes + 1024;
     if (!(ctx->attr_flags & 128u)) {
         WR_CUDA_TRY(cudaFuncSetAttribute(gemm_skinny_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

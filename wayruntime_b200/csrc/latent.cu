@@ -6,6 +6,7 @@
 #include <algorithm>
 
 #include "gemm_bf16.cuh"
+#include "latent_dev.cuh"
 #include "rows_dev.cuh"
 #include "warp_reduce.cuh"
 
@@ -210,6 +211,182 @@ __global__ void __launch_bounds__(128) latent_value_kernel(const wr_rows rw, con
             Out<TO>(a.out, row0 + i / (wr_ld(n) - n), a.out_ld).put(n + i % (wr_ld(n) - n), 0.f);
 }
 
+// ---- the same two steps for at most WR_CUDA_BATCH_MAX rows of a BF16 model: the rows are the M of a warp's matrix
+// instruction (all sixteen always), F32 operands go in as two F16 numbers, the weights are F16 as they are stored and are
+// requested before the dependency wait.
+
+static_assert(WR_CUDA_BATCH_MAX == 16, "one matrix instruction's rows");
+
+// A block is one head and 64 columns of the cached row, a warp 16 of them.  What leaves is the operand the attention
+// kernel takes (wr_latent_split_query).
+__global__ void __launch_bounds__(128) latent_query_mma_kernel(const wr_rows rw, const wr_latent_query_args a)
+{
+    extern __shared__ __align__(1024) uint8_t sm_mma[];
+    pdl_trigger();
+    const wr_latent_geom g = a.g;
+    const uint32_t head = blockIdx.x, c0 = blockIdx.y * 64, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t nh = wr_latent_group(g), n = 2 * nh, hl = head % nh, hs = g.q_head();
+    const size_t q_row = (size_t)g.heads * hs;
+    const float *q = a.q + (size_t)head * hs;
+    const float scale = a.scale * 1.4426950408889634f;
+    auto operand = [&](uint32_t r) {
+        return reinterpret_cast<char *>(a.out) + wr_latent_split_bytes(g) * r + (size_t)(head / nh) * (g.row() / 64) * n * 128;
+    };
+    auto put = [&](uint32_t r, uint32_t c, float x, float y) {          // columns c, c + 1 of row r
+        uint32_t hi, lo;
+        split_half2(fminf(fmaxf(x, -65504.f), 65504.f), fminf(fmaxf(y, -65504.f), 65504.f), hi, lo);
+        char *out = operand(r);
+        *reinterpret_cast<uint32_t *>(out + wr_latent_split_off(n, hl, c)) = hi;
+        *reinterpret_cast<uint32_t *>(out + wr_latent_split_off(n, nh + hl, c)) = lo;
+    };
+    if (c0 >= g.rank_pad()) {                            // the rotated part
+        pdl_wait();
+        if (c0 > g.rank_pad()) return;                   // (one block writes all of it)
+        const uint32_t half = g.rot / 2, pairs = (g.row() - c0) / 2;
+        for (uint32_t i = threadIdx.x; i < rw.n_rows * pairs; i += 128) {
+            const uint32_t r = i / pairs, p = i % pairs;
+            float y[2] = {0.f, 0.f};
+            uint32_t c[2] = {p, half + p};
+            if (p < half) {
+                float sn, cs;
+                angle(a.turns[p], rw.seqs[seq_of(rw, r)].pos + tok_of(rw, r), sn, cs);
+                const float *in = q + r * q_row + g.dim_pad();
+                const float u = in[p], v = in[half + p];
+                y[0] = scale * (u * cs - v * sn);
+                y[1] = scale * (v * cs + u * sn);
+            } else {                                     // the columns behind it are zeros
+                c[0] = 2 * p;
+                c[1] = 2 * p + 1;
+            }
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const __half hi = from_f32<__half>(y[j]);
+                char *out = operand(r);
+                *reinterpret_cast<__half *>(out + wr_latent_split_off(n, hl, c0 + c[j])) = hi;
+                *reinterpret_cast<__half *>(out + wr_latent_split_off(n, nh + hl, c0 + c[j])) = __float2half_rn(y[j] - __half2float(hi));
+            }
+        }
+        return;
+    }
+    // weights [dim_pad][64] as stored (the head's first row is a multiple of 16: the swizzle keeps its phase)
+    const uint32_t dp = g.dim_pad(), ld = dp + 8;        // (row length of the queries in shared memory)
+    uint8_t *W = sm_mma;
+    __half *Q = reinterpret_cast<__half *>(W + dp * 128);        // [hi | lo][16][ld]
+    for (uint32_t i = threadIdx.x; i < dp * 8; i += 128) {
+        const uint32_t r = i / 8, at = head * dp + r;
+        const char *src = static_cast<const char *>(a.w_ukv) +
+                          ((size_t)(at / kWBlock) * wr_weight_blocks(g.kv_rank) + blockIdx.y) * kWBlockBytes + at % kWBlock * 128;
+        *reinterpret_cast<uint4 *>(W + r * 128 + i % 8 * 16) = *reinterpret_cast<const uint4 *>(src + i % 8 * 16);
+    }
+    pdl_wait();
+    for (uint32_t i = threadIdx.x; i < 16 * (dp / 4); i += 128) {
+        const uint32_t r = i / (dp / 4), c = 4 * (i % (dp / 4));
+        const float4 v = r < rw.n_rows ? load4(q + r * q_row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        uint32_t h0, l0, h1, l1;
+        split_half2(v.x, v.y, h0, l0);
+        split_half2(v.z, v.w, h1, l1);
+        *reinterpret_cast<uint2 *>(Q + r * ld + c) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2 *>(Q + (16 + r) * ld + c) = make_uint2(l0, l1);
+    }
+    __syncthreads();
+    float acc[2][4] = {};
+    const uint32_t w_addr = smem_u32(W), q_addr = smem_u32(Q);
+    for (uint32_t k0 = 0; k0 < dp; k0 += 16) {
+        uint32_t hi[4], lo[4], b[4];
+        // rows of the fragment: lanes 0-15 rows 0-15 at k0, lanes 16-31 the same at k0 + 8
+        const uint32_t at = ((lane & 15u) * ld + k0 + (lane >> 4) * 8) * 2;
+        ldmatrix_x4(hi[0], hi[1], hi[2], hi[3], q_addr + at);
+        ldmatrix_x4(lo[0], lo[1], lo[2], lo[3], q_addr + 16 * ld * 2 + at);
+        const uint32_t kr = k0 + (lane & 15u), piece = 2 * warp + (lane >> 4);
+        ldmatrix_x4_trans(b[0], b[1], b[2], b[3], w_addr + kr * 128 + ((piece ^ (kr & 7u)) << 4));
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+            mma_16816(acc[t], hi, b[2 * t], b[2 * t + 1]);
+            mma_16816(acc[t], lo, b[2 * t], b[2 * t + 1]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t) {
+        const uint32_t c = c0 + 16 * warp + 8 * t + 2 * (lane & 3u), r = lane >> 2;
+        if (r < rw.n_rows) put(r, c, acc[t][0] * scale, acc[t][1] * scale);
+        if (r + 8 < rw.n_rows) put(r + 8, c, acc[t][2] * scale, acc[t][3] * scale);
+    }
+}
+
+constexpr uint32_t kValueCols = 32;      // values of a block, eight per warp
+constexpr uint32_t kMaxBlocks = 8;       // 64-wide blocks of a latent
+
+// A block is one head and 32 of its values.  The attended latents come as chunks still to be added up, or finished.
+__global__ void __launch_bounds__(128) latent_value_mma_kernel(const wr_rows rw, const wr_latent_value_args a)
+{
+    extern __shared__ __align__(1024) uint8_t sm_mma[];
+    __shared__ float wt[WR_CUDA_BATCH_MAX][kLatentMaxFused];
+    pdl_trigger();
+    const wr_latent_geom g = a.g;
+    const uint32_t head = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = lane & 3u, blocks = g.rank_pad() / 64;
+    const uint32_t v0 = blockIdx.y * kValueCols + 8 * warp, row = min(v0 + (lane >> 2), g.vdim_pad() - 1);
+    const uint32_t at = g.heads * g.dim_pad() + head * g.vdim_pad() + row, sw = at & 7u;
+    const char *src = static_cast<const char *>(a.w_ukv) + (size_t)(at / kWBlock) * blocks * kWBlockBytes + at % kWBlock * 128;
+    uint4 w[kMaxBlocks][2];
+#pragma unroll
+    for (uint32_t b = 0; b < kMaxBlocks; ++b)
+        if (b < blocks) {
+            w[b][0] = *reinterpret_cast<const uint4 *>(src + (size_t)b * kWBlockBytes + ((t ^ sw) << 4));
+            w[b][1] = *reinterpret_cast<const uint4 *>(src + (size_t)b * kWBlockBytes + (((t + 4) ^ sw) << 4));
+        }
+    pdl_wait();
+    const uint32_t rp = g.rank_pad(), ld = rp + 32;
+    __half *O = reinterpret_cast<__half *>(sm_mma);      // [hi | lo][16][ld]
+    const float *ml = a.ml;
+    if (ml) {
+        for (uint32_t r = warp; r < rw.n_rows; r += 4)
+            latent_chunk_weights(ml + ((size_t)r * g.heads + head) * a.chunks * 2, a.lens.count[r], wt[r], lane);
+        __syncthreads();
+    }
+    for (uint32_t i = threadIdx.x; i < 16 * (rp / 4); i += 128) {
+        const uint32_t r = i / (rp / 4), c = 4 * (i % (rp / 4));
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < rw.n_rows) {
+            const float *in = a.o + ((size_t)r * g.heads + head) * (ml ? a.chunks : 1u) * rp + c;
+            o = ml ? latent_chunk_sum(in, rp, wt[r], a.lens.count[r]) : load4(in);
+        }
+        uint32_t h0, l0, h1, l1;
+        split_half2(o.x, o.y, h0, l0);
+        split_half2(o.z, o.w, h1, l1);
+        *reinterpret_cast<uint2 *>(O + r * ld + c) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2 *>(O + (16 + r) * ld + c) = make_uint2(l0, l1);
+    }
+    __syncthreads();
+    // The order of the latent in the sum is the weights' own: a lane's 16-byte piece is two steps of its fragment.
+    float acc[4] = {}, acc_l[4] = {}, acc2[4] = {}, acc2_l[4] = {};      // (four chains of products)
+    const __half *lo_rows = O + 16 * ld;
+#pragma unroll
+    for (uint32_t b = 0; b < kMaxBlocks; ++b)
+        if (b < blocks) {
+#pragma unroll
+            for (uint32_t p = 0; p < 2; ++p) {
+                const uint32_t c = 64 * b + 8 * (t + 4 * p), r = lane >> 2;
+                const uint4 h0 = *reinterpret_cast<const uint4 *>(O + r * ld + c), h1 = *reinterpret_cast<const uint4 *>(O + (r + 8) * ld + c);
+                const uint4 l0 = *reinterpret_cast<const uint4 *>(lo_rows + r * ld + c);
+                const uint4 l1 = *reinterpret_cast<const uint4 *>(lo_rows + (r + 8) * ld + c);
+                const uint32_t ah[2][4] = {{h0.x, h1.x, h0.y, h1.y}, {h0.z, h1.z, h0.w, h1.w}};
+                const uint32_t al[2][4] = {{l0.x, l1.x, l0.y, l1.y}, {l0.z, l1.z, l0.w, l1.w}};
+                mma_16816(acc, ah[0], w[b][p].x, w[b][p].y);
+                mma_16816(acc_l, al[0], w[b][p].x, w[b][p].y);
+                mma_16816(acc2, ah[1], w[b][p].z, w[b][p].w);
+                mma_16816(acc2_l, al[1], w[b][p].z, w[b][p].w);
+            }
+        }
+#pragma unroll
+    for (uint32_t j = 0; j < 4; ++j) {
+        const uint32_t r = (lane >> 2) + 8 * (j >> 1), v = v0 + 2 * t + (j & 1u);
+        if (r < rw.n_rows && v < g.vdim) Out<Split>(a.out, r, a.out_ld).put(head * g.vdim + v, (acc[j] + acc2[j]) + (acc_l[j] + acc2_l[j]));
+    }
+    const uint32_t n = g.heads * g.vdim, pad = wr_ld(n) - n;
+    if (head + 1 == g.heads && blockIdx.y + 1 == gridDim.y)
+        for (uint32_t i = threadIdx.x; i < rw.n_rows * pad; i += 128) Out<Split>(a.out, i / pad, a.out_ld).put(n + i % pad, 0.f);
+}
+
 template <typename TW, int RT> int query_rows(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_query_args &a)
 {
     const size_t smem = (size_t)(RT * a.g.dim + 4 * RT * 64) * 4;
@@ -261,11 +438,26 @@ int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent
 
 int wr_latent_query_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_query_args &a)
 {
+    if (a.split) {
+        const size_t smem = (size_t)a.g.dim_pad() * 128 + 2 * 16 * (a.g.dim_pad() + 8) * 2;
+        const int rc = allow_smem(latent_query_mma_kernel, smem);
+        if (rc != WR_CUDA_OK) return rc;
+        WR_CUDA_TRY(wr_launch_pdl(latent_query_mma_kernel, dim3(a.g.heads, a.g.row() / 64), dim3(128), smem, ctx->stream, rw, a));
+        return finish_launch(ctx);
+    }
     return a.w_type == WR_ACT_F16 ? query_any<__half>(ctx, rw, a) : query_any<float>(ctx, rw, a);
 }
 
 int wr_latent_value_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_value_args &a)
 {
+    if (a.split) {
+        const size_t smem = (size_t)2 * 16 * (a.g.rank_pad() + 32) * 2;
+        const int rc = allow_smem(latent_value_mma_kernel, smem);
+        if (rc != WR_CUDA_OK) return rc;
+        WR_CUDA_TRY(wr_launch_pdl(latent_value_mma_kernel, dim3(a.g.heads, (a.g.vdim + kValueCols - 1) / kValueCols), dim3(128), smem,
+                                  ctx->stream, rw, a));
+        return finish_launch(ctx);
+    }
     if (a.w_type == WR_ACT_F32) return value_any<float, float>(ctx, rw, a);
     return a.out_type == WR_ACT_SPLIT ? value_any<__half, Split>(ctx, rw, a) : value_any<__half, __nv_bfloat16>(ctx, rw, a);
 }

@@ -122,6 +122,19 @@ struct wr_latent_geom {
     __host__ __device__ uint32_t row() const { return rank_pad() + ((rot + 63u) & ~63u); }
 };
 
+// Heads that share a cached row's fetch in attn_latent.cu, and the queries as its operand: per row and group of heads, boxes
+// of 64 columns, each [2 group][128 B] in the 128-byte swizzle — the heads' F16 roundings, then what is left of them.
+__host__ __device__ inline uint32_t wr_latent_group(const wr_latent_geom &g) { return g.heads <= 8 ? 8u : 16u; }
+__host__ __device__ inline size_t wr_latent_split_bytes(const wr_latent_geom &g)
+{
+    const uint32_t nh = wr_latent_group(g);
+    return (size_t)((g.heads + nh - 1) / nh) * (2 * nh) * g.row() * 2;
+}
+__host__ __device__ inline uint32_t wr_latent_split_off(uint32_t rows, uint32_t r, uint32_t c)
+{
+    return (c >> 6) * rows * 128u + r * 128u + ((((c & 63u) >> 3) ^ (r & 7u)) << 4) + (c & 7u) * 2u;
+}
+
 // The projection's rows, normed and rotated: the query latent for the next product, and (own) the session's row.
 struct wr_latent_prep_args {
     wr_latent_geom g;
@@ -146,14 +159,22 @@ struct wr_latent_query_args {
     const void *w_ukv; int w_type;   // WR_ACT_F32 / WR_ACT_F16
     const double *turns;
     float scale;
+    bool split;                      // at most WR_CUDA_BATCH_MAX rows, F16 weights: out is the split operand above, in log2 units
     float *out;                      // [rows][heads][row()]
 };
 int wr_latent_query_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_query_args &a);
 
 // Latent attention rows back into values: out[row][head * vdim + v] = w_uv o.
+struct wr_latent_lens {
+    uint32_t len[WR_CUDA_BATCH_MAX], count[WR_CUDA_BATCH_MAX];   // keys a row sees; chunks they were cut into
+};
 struct wr_latent_value_args {
     wr_latent_geom g;
-    const float *o;                  // [rows][heads][kv_rank]
+    const float *o;                  // [rows][heads][kv_rank]; split: rank_pad() values each
+    bool split;                      // at most WR_CUDA_BATCH_MAX rows, F16 weights, split rows out
+    const float *ml;                 // split: o is still in chunks, [rows][heads][chunks][rank_pad()], with these pairs; or null
+    uint32_t chunks;
+    wr_latent_lens lens;
     const void *w_ukv; int w_type;
     void *out; int out_type;         // [rows][out_ld]; the columns up to wr_ld(heads * vdim) are written
     uint32_t out_ld;
@@ -175,10 +196,11 @@ bool wr_latent_flash_covers(const wr_latent_geom &g, float scale);
 int wr_latent_flash_launch(wr_cuda_ctx *ctx, const wr_latent_flash_args &a);
 
 // Attention of at most WR_CUDA_BATCH_MAX rows over the cached F16 rows (attn_latent.cu): q as wr_latent_query_launch leaves
-// it, out [rows][heads][kv_rank], lens: how many keys each row sees (host).
+// it with `split`, lens: how many keys each row sees (host).  Fills in out's o, ml, chunks and lens; merged: room for
+// [rows][heads][rank_pad()].
 bool wr_latent_decode_covers(const wr_latent_geom &g);
-int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, uint32_t layer, const float *q, float *out,
-                            const uint32_t *lens);
+int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, uint32_t layer, const void *q,
+                            const uint32_t *lens, float *merged, wr_latent_value_args &out);
 
 // q's rotated parts turned in place (F16 rows as above)
 int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, const double *turns, void *q);

@@ -625,8 +625,8 @@ extern "C" int wr_cuda_model_create_mixed(wr_cuda_ctx *ctx, const wr_cuda_mixed_
             q = std::max<size_t>(q, (size_t)g.heads * g.q_head() * 4);
             mid = std::max<size_t>(mid, wr_ld(l.o.k));
             const size_t n = l.flash ? few : R;          // rows that attend in the latent
-            qa = std::max<size_t>(qa, n * g.heads * g.row());
-            olat = std::max<size_t>(olat, n * g.heads * g.kv_rank);
+            qa = std::max<size_t>(qa, std::max<size_t>(n * g.heads * g.row(), few * wr_latent_split_bytes(g) / 4));
+            olat = std::max<size_t>(olat, n * g.heads * g.rank_pad());
         } else {
             proj = std::max<size_t>(proj, 2 * wr_ld(l.inner));
             mid = std::max<size_t>(mid, wr_ld(l.inner));
@@ -917,19 +917,19 @@ struct Step {
         TRY(product(l.uq, x->cq, wr_ld(g.q_rank), x->q, g.heads * g.q_head(), WR_ACT_F32));
         wr_latent_query_args q{};
         q.g = g; q.q = static_cast<const float *>(x->q); q.w_ukv = l.ukv.w; q.w_type = bf ? WR_ACT_F16 : WR_ACT_F32;
-        q.turns = l.turns; q.scale = l.scale; q.out = x->qa;
+        q.turns = l.turns; q.scale = l.scale; q.split = l.tensor_decode && split(); q.out = x->qa;
         TRY(wr_latent_query_launch(ctx, rw, q));
-        if (l.tensor_decode && split()) {
+        wr_latent_value_args v{};
+        v.g = g; v.o = x->olat; v.w_ukv = l.ukv.w; v.w_type = q.w_type; v.split = q.split;
+        v.out = x->mid; v.out_type = in_act(); v.out_ld = ld_o;
+        if (q.split) {
             uint32_t lens[WR_CUDA_BATCH_MAX];
             for (uint32_t r = 0; r < rw.n_rows; ++r) lens[r] = rw.decode ? positions[r] + 1 : positions[0] + r + 1;
-            TRY(wr_latent_decode_launch(ctx, rw, g, ag.layer, x->qa, x->olat, lens));
-            ++m->launches;
+            TRY(wr_latent_decode_launch(ctx, rw, g, ag.layer, x->qa, lens, x->olat, v));
+            if (!v.ml) ++m->launches;
         } else {
             TRY(wr_attn_any_launch(ctx, rw, ag, x->qa, x->olat, max_len));
         }
-        wr_latent_value_args v{};
-        v.g = g; v.o = x->olat; v.w_ukv = l.ukv.w; v.w_type = q.w_type;
-        v.out = x->mid; v.out_type = in_act(); v.out_ld = ld_o;
         TRY(wr_latent_value_launch(ctx, rw, v));
         m->launches += 4;
         return product(l.o, x->mid, ld_o, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
