@@ -30,9 +30,9 @@ def softmax(z):
     return e / e.sum(axis=-1, keepdims=True)
 
 
-def causal(scores):
+def causal(scores, first=0):
     t, s = scores.shape[-2:]
-    return np.where(np.arange(s)[None, :] <= np.arange(t)[:, None], scores, -np.inf)
+    return np.where(np.arange(s)[None, :] <= first + np.arange(t)[:, None], scores, -np.inf)
 
 
 def sigmoid(z):
@@ -53,16 +53,17 @@ def queries(h, w, pre, cfg, eps):
     return q[..., :cfg["dim"]], rotate_half(q[..., cfg["dim"]:], np.arange(h.shape[0]), cfg["rot"]["base"])
 
 
-def latent_attention(h, w, pre, cfg, eps, latent):
+def latent_attention(h, w, pre, cfg, eps, latent, first=0):
+    """Rows from `first` on."""
     t, H, c, kr = h.shape[0], cfg["heads"], *latent
-    qn, qr = queries(h, w, pre, cfg, eps)
+    qn, qr = (q[first:] for q in queries(h, w, pre, cfg, eps))
     k = (c @ w[pre + "uk"].T).reshape(t, H, cfg["dim"])
     v = (c @ w[pre + "uv"].T).reshape(t, H, cfg["vdim"])
-    out = np.zeros((t, H, cfg["vdim"]))
+    out = np.zeros((t - first, H, cfg["vdim"]))
     for head in range(H):
         scores = (qn[:, head] @ k[:, head].T + qr[:, head] @ kr.T) * cfg["scale"]
-        out[:, head] = softmax(causal(scores)) @ v[:, head]
-    return out.reshape(t, -1) @ w[pre + "o"].T
+        out[:, head] = softmax(causal(scores, first)) @ v[:, head]
+    return out.reshape(t - first, -1) @ w[pre + "o"].T
 
 
 def swiglu(h, gate, up, down):
@@ -102,8 +103,9 @@ def feed_forward(h, w, pre, cfg):
     return mixture(h, w, pre, cfg)
 
 
-def forward(cfg, weights, tokens, layers_out=None):
-    """Logits [n, vocab] of a whole sequence; layers_out, a list, gets the residual after every layer."""
+def forward(cfg, weights, tokens, layers_out=None, last_only=False):
+    """Logits [n, vocab] of a whole sequence; layers_out, a list, gets the residual after every layer.  last_only: the
+    last layer works on the last row alone (logits [1, vocab])."""
     w = {k: np.asarray(v, np.float64) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
@@ -113,7 +115,10 @@ def forward(cfg, weights, tokens, layers_out=None):
         h = layer_norm(x, w[pre + "norm1"], eps)
         if mx.get("kv_from") is None:
             latents[i] = latent_rows(h, w, pre + "mix.", mx, eps)
-        mixed = latent_attention(h, w, pre + "mix.", mx, eps, latents[i if mx.get("kv_from") is None else mx["kv_from"]])
+        rows = latents[i if mx.get("kv_from") is None else mx["kv_from"]]
+        first = len(tokens) - 1 if last_only and i + 1 == len(cfg["layers"]) else 0
+        mixed = latent_attention(h, w, pre + "mix.", mx, eps, rows, first)
+        x, h = x[first:], h[first:]
         x = x + cfg["residual_mult"] * (mixed + feed_forward(h, w, pre + "mlp.", lay.get("mlp")))
         if layers_out is not None:
             layers_out.append(x.copy())

@@ -260,6 +260,36 @@ def test_one_key_among_hundreds(ctx, dtype, dims):
     m.close()
 
 
+@pytest.mark.parametrize("dims", [(2, 20, 8, 24, 40), (18, 16, 64, 32, 256)])
+def test_one_key_among_thousands(ctx, dims):
+    """Long sessions, where a decoding row's keys come in chunks of several tiles: a far-out score in the first or second
+    tile of a chunk, at a chunk's first and last key, or in the last chunk."""
+    heads, dim, rot, vdim, rank = dims
+    cfg = config([latent(heads=heads, dim=dim, rot=rot, vdim=vdim, q_rank=24, kv_rank=rank, scale=0.5)], width=48, scale=1.0)
+    w = weights(cfg, 41)
+    a, b, n = 7, 8, 2700
+    planted(dims, w, a, b)
+    base = [t if t not in (a, b) else 20 for t in tokens(cfg, n, 43)]
+    models_ = {d: build(ctx, cfg, w, d, max_rows=1024) for d in DTYPES}
+    for key in (0, 127, 128, 255, 256, 1500, 2303, 2304, 2500, 2559, 2560, n - 2):
+        toks = list(base)
+        toks[key], toks[-1] = b, a
+        want = plain.forward(cfg, w, toks, last_only=True)
+        without = plain.forward(cfg, w, toks[:key] + [20] + toks[key + 1:], last_only=True)
+        assert rel(without, want) > 10 * TOL["bfloat16"], "the planted key must matter"
+        for dtype, m in models_.items():
+            for cuts in ([1000, 1000, 699, 1], [1024, 1024, 652 - 9, 9]):
+                kv, pos = m.kv_create(n), 0
+                for c in cuts:
+                    mode = m.FWD_DECODE if c == 1 else m.FWD_PREFILL
+                    got = m.forward(mode, [kv], [pos], toks[pos:pos + c], out_from=c - 1, logits=True)["logits"]
+                    pos += c
+                kv.close()
+                assert pos == n and rel(got, want) <= TOL[dtype], (key, dtype, cuts)
+    for m in models_.values():
+        m.close()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_rotation_far_out(ctx, dtype):
     """Only the rotated part decides, on positions up to 1500: a frequency or a position that is off turns the scores."""

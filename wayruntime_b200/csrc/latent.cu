@@ -7,6 +7,7 @@
 
 #include "gemm_bf16.cuh"
 #include "latent_dev.cuh"
+#include "moe_dev.cuh"
 #include "rows_dev.cuh"
 #include "warp_reduce.cuh"
 
@@ -20,14 +21,23 @@ __device__ __forceinline__ void angle(double turns, uint32_t pos, float &sn, flo
     sincospif(2.0f * (float)(a - rint(a)), &sn, &cs);
 }
 
-// grid.y 0: the query latent; 1: the session's row
+// grid.y 0: the query latent; 1 (own): the session's row; the last (routed): the row's experts, of few rows all at once
 template <typename TO>
-__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const wr_rows rw, const wr_latent_prep_args a)
+__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const wr_rows rw, const wr_latent_prep_args a, const wr_route_args route)
 {
+    extern __shared__ float sm_prep[];
     __shared__ float part[kPrepThreads / 32];
     pdl_trigger();
     pdl_wait();
     const uint32_t row = blockIdx.x, n = blockIdx.y ? a.g.kv_rank : a.g.q_rank;
+    if (blockIdx.y == (a.own ? 2u : 1u)) {
+        if (route.tile == 0) {
+            if (row == 0) route_few(sm_prep, route, rw.n_rows);
+        } else if (threadIdx.x < 32) {
+            choose(sm_prep, route, row);
+        }
+        return;
+    }
     const float *in = a.in + (size_t)row * a.ld, *x = in + (blockIdx.y ? a.c_off : 0u);
     const float *w = blockIdx.y ? a.c_norm : a.q_norm;
     float ss = 0.f;
@@ -423,11 +433,18 @@ template <typename TW, typename TO> int value_any(wr_cuda_ctx *ctx, const wr_row
 
 int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_prep_args &a)
 {
-    const dim3 grid(rw.n_rows, a.own ? 2 : 1), block(kPrepThreads);
-    if (a.cq_type == WR_ACT_BF16) WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, ctx->stream, rw, a));
-    else if (a.cq_type == WR_ACT_SPLIT) WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<Split>, grid, block, 0, ctx->stream, rw, a));
-    else WR_CUDA_TRY(wr_launch_pdl(latent_prep_kernel<float>, grid, block, 0, ctx->stream, rw, a));
-    return finish_launch(ctx);
+    const dim3 grid(rw.n_rows, (a.own ? 2 : 1) + (a.route ? 1 : 0)), block(kPrepThreads);
+    const wr_route_args route = a.route ? *a.route : wr_route_args{};
+    const size_t smem = !a.route ? 0 : route.tile ? (size_t)route.experts * 4 : route_few_smem(route);
+    auto launch = [&](auto kernel) {
+        const int rc = allow_smem(kernel, smem);
+        if (rc != WR_CUDA_OK) return rc;
+        WR_CUDA_TRY(wr_launch_pdl(kernel, grid, block, smem, ctx->stream, rw, a, route));
+        return finish_launch(ctx);
+    };
+    if (a.cq_type == WR_ACT_BF16) return launch(latent_prep_kernel<__nv_bfloat16>);
+    if (a.cq_type == WR_ACT_SPLIT) return launch(latent_prep_kernel<Split>);
+    return launch(latent_prep_kernel<float>);
 }
 
 int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_geom &g, const double *turns, void *q)

@@ -108,6 +108,27 @@ struct wr_attn_finish_args {
 };
 int wr_attn_finish_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_attn_finish_args &a);
 
+// ---- mixture of experts (moe.cu): routing
+
+// The chosen experts of every row and their weights, and the rows grouped by expert.  Many rows: expert e's (row, slot)
+// pairs take consecutive places from a multiple of `tile` on; list names the expert of each tile of places.  Few
+// rows: list names the experts somebody chose, and a pair's place is its expert's number in the list.
+struct wr_route_args {
+    const float *logits;             // [rows][ld]
+    uint32_t ld;
+    const float *bias;               // [experts]
+    uint32_t experts, top, tile;     // tile 0: few rows
+    float *weight;                   // [rows][top]
+    uint32_t *expert, *place;        // [rows][top]
+    uint32_t *row_of;                // [places]: the row at a place, ~0 where there is none (many rows)
+    uint32_t *list, *count;
+    bool chosen;                     // another kernel has done so already (many rows: their places are still to be found)
+};
+inline uint32_t wr_route_tiles(uint32_t rows, uint32_t experts, uint32_t top, uint32_t tile)
+{
+    const uint32_t pairs = rows * top, used = experts < pairs ? experts : pairs;
+    return tile ? pairs / tile + used : used;
+}
 // ---- attention over a latent (latent.cu)
 
 // Where the parts of a latent layer's rows lie: the cached row is [latent, padded to 64 | rotated key part, padded to
@@ -147,6 +168,7 @@ struct wr_latent_prep_args {
     bool own;
     uint32_t layer;                  // page-table layer
     wr_kv_geom kv;
+    const wr_route_args *route;      // the rows' experts chosen on the way, or null
 };
 int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_prep_args &a);
 
@@ -207,24 +229,6 @@ int wr_latent_rotate_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent
 
 // ---- mixture of experts (moe.cu)
 
-// The chosen experts of every row and their weights, and the rows grouped by expert.  Many rows: expert e's (row, slot)
-// pairs take consecutive places from a multiple of `tile` on; list names the expert of each tile of places.  Few
-// rows: list names the experts somebody chose, and a pair's place is its expert's number in the list.
-struct wr_route_args {
-    const float *logits;             // [rows][ld]
-    uint32_t ld;
-    const float *bias;               // [experts]
-    uint32_t experts, top, tile;     // tile 0: few rows
-    float *weight;                   // [rows][top]
-    uint32_t *expert, *place;        // [rows][top]
-    uint32_t *row_of;                // [places]: the row at a place, ~0 where there is none (many rows)
-    uint32_t *list, *count;
-};
-inline uint32_t wr_route_tiles(uint32_t rows, uint32_t experts, uint32_t top, uint32_t tile)
-{
-    const uint32_t pairs = rows * top, used = experts < pairs ? experts : pairs;
-    return tile ? pairs / tile + used : used;
-}
 int wr_route_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_route_args &a);
 
 // out[place] = x[row_of[place]] (BF16 rows of ld values)

@@ -908,6 +908,11 @@ struct Step {
         p.g = g; p.in = x->lat; p.ld = l.proj_ld; p.c_off = l.k_off; p.r_off = l.rot_off;
         p.q_norm = l.q_norm; p.c_norm = l.c_norm; p.eps = l.latent_eps; p.turns = l.turns;
         p.cq = x->cq; p.cq_type = in_act(); p.own = own; p.layer = run; p.kv = l.g.kv;
+        wr_route_args r{};
+        if (l.experts && !l.router.w) {                  // (the logits came with the first product)
+            r = route_of(l, l.logit_off, l.proj_ld);
+            p.route = &r;
+        }
         TRY(wr_latent_prep_launch(ctx, rw, p));
         if (wide && l.flash) {
             TRY(product(l.uq, x->cq, wr_ld(g.q_rank), x->q, g.heads * g.q_head(), WR_ACT_F16));
@@ -990,20 +995,27 @@ struct Step {
         return product(l.down, x->mid, ld, x->resid, x->ldw, WR_ACT_F32, nullptr, false, x->resid);
     }
 
-    int experts(const Layer &l)
+    // Router logits in columns off .. of lat.
+    wr_route_args route_of(const Layer &l, uint32_t off, uint32_t ld) const
     {
-        uint32_t ld = l.proj_ld, off = l.logit_off;
-        if (l.router.w) {
-            ld = wr_ld(l.experts);
-            off = 0;
-            TRY(product(l.router, x->xin, x->ldw, x->lat, ld, WR_ACT_F32));
-        }
-        const bool bf = x->compute == WR_CUDA_BF16;
         wr_route_args r{};
         r.logits = x->lat + off; r.ld = ld; r.bias = l.router_b; r.experts = l.experts; r.top = l.top;
-        r.tile = split() ? 0 : bf ? kMoeTile : kMoeTileF32;
+        r.tile = split() ? 0 : x->compute == WR_CUDA_BF16 ? kMoeTile : kMoeTileF32;
         r.weight = x->e_weight; r.expert = x->e_expert; r.place = x->e_place; r.row_of = x->e_row_of;
         r.list = x->e_list; r.count = x->e_count;
+        return r;
+    }
+
+    int experts(const Layer &l)
+    {
+        const bool bf = x->compute == WR_CUDA_BF16;
+        wr_route_args r = route_of(l, l.logit_off, l.proj_ld);
+        if (l.router.w) {
+            r = route_of(l, 0, wr_ld(l.experts));
+            TRY(product(l.router, x->xin, x->ldw, x->lat, r.ld, WR_ACT_F32));
+        } else {
+            r.chosen = true;                             // (by wr_latent_prep_launch)
+        }
         TRY(wr_route_launch(ctx, rw, r));
         const uint32_t groups = wr_route_tiles(rw.n_rows, l.experts, l.top, r.tile), lf = wr_ld(l.ff);
         wr_group_args gr;

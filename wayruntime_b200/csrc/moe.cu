@@ -5,49 +5,11 @@
 #include <algorithm>
 
 #include "gemm_bf16.cuh"
-#include "rows_dev.cuh"
+#include "moe_dev.cuh"
 
 namespace {
 
 constexpr uint32_t kSortThreads = 1024;
-
-// One warp's row: z (shared memory, experts values) loses the chosen logits.
-__device__ __forceinline__ void choose(float *z, const wr_route_args &a, uint32_t row)
-{
-    const uint32_t lane = threadIdx.x & 31;
-    const float *in = a.logits + (size_t)row * a.ld;
-    for (uint32_t e = lane; e < a.experts; e += 32) z[e] = in[e] + a.bias[e];
-    __syncwarp();
-    float first = 0.f, sum = 0.f;
-    for (uint32_t s = 0; s < a.top; ++s) {
-        float best = -INFINITY;
-        uint32_t at = ~0u;
-        for (uint32_t e = lane; e < a.experts; e += 32)
-            if (z[e] > best || at == ~0u) {
-                best = z[e];
-                at = e;
-            }
-#pragma unroll
-        for (int o = 16; o >= 1; o >>= 1) {
-            const float b = __shfl_xor_sync(0xffffffffu, best, o);
-            const uint32_t t = __shfl_xor_sync(0xffffffffu, at, o);
-            if (t != ~0u && (at == ~0u || b > best || (b == best && t < at))) {
-                best = b;
-                at = t;
-            }
-        }
-        if (s == 0) first = best;
-        const float w = expf(best - first);
-        sum += w;
-        if (lane == 0) {
-            a.expert[(size_t)row * a.top + s] = at;
-            a.weight[(size_t)row * a.top + s] = w;
-            z[at] = -INFINITY;
-        }
-        __syncwarp();
-    }
-    for (uint32_t s = lane; s < a.top; s += 32) a.weight[(size_t)row * a.top + s] /= sum;
-}
 
 constexpr uint32_t kRouteWarps = 8;
 
@@ -60,36 +22,12 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_choose_kernel(const wr_r
     if (row < rw.n_rows) choose(sm_moe + (threadIdx.x >> 5) * a.experts, a, row);
 }
 
-// Few rows: one block, a warp per row, then the list of the experts in use, in ascending order.
 __global__ void __launch_bounds__(WR_CUDA_BATCH_MAX * 32) moe_route_few_kernel(const wr_rows rw, const wr_route_args a)
 {
     extern __shared__ float sm_moe[];
     pdl_trigger();
     pdl_wait();
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    if (warp < rw.n_rows) choose(sm_moe + warp * a.experts, a, warp);
-    uint32_t *number = reinterpret_cast<uint32_t *>(sm_moe + WR_CUDA_BATCH_MAX * a.experts);
-    for (uint32_t e = threadIdx.x; e < a.experts; e += blockDim.x) number[e] = 0;
-    __syncthreads();
-    const uint32_t pairs = rw.n_rows * a.top;
-    for (uint32_t i = threadIdx.x; i < pairs; i += blockDim.x) number[a.expert[i]] = 1;
-    __syncthreads();
-    if (warp == 0) {
-        uint32_t used = 0;
-        for (uint32_t e0 = 0; e0 < a.experts; e0 += 32) {
-            const uint32_t e = e0 + lane;
-            const bool in = e < a.experts && number[e];
-            const uint32_t votes = __ballot_sync(0xffffffffu, in), at = used + __popc(votes & ((1u << lane) - 1u));
-            if (in) {
-                number[e] = at;
-                a.list[at] = e;
-            }
-            used += __popc(votes);
-        }
-        if (lane == 0) *a.count = used;
-    }
-    __syncthreads();
-    for (uint32_t i = threadIdx.x; i < pairs; i += blockDim.x) a.place[i] = number[a.expert[i]];
+    route_few(sm_moe, a, rw.n_rows);
 }
 
 // Many rows: places by expert, every expert's from a multiple of the tile on.
@@ -216,7 +154,8 @@ template <bool PAIR> __global__ void __launch_bounds__(256) moe_f32_kernel(const
 int wr_route_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_route_args &a)
 {
     if (!a.tile) {
-        const size_t smem = (size_t)(WR_CUDA_BATCH_MAX + 1) * a.experts * 4;
+        if (a.chosen) return WR_CUDA_OK;
+        const size_t smem = route_few_smem(a);
         const int rc = allow_smem(moe_route_few_kernel, smem);
         if (rc != WR_CUDA_OK) return rc;
         WR_CUDA_TRY(wr_launch_pdl(moe_route_few_kernel, dim3(1), dim3(WR_CUDA_BATCH_MAX * 32), smem, ctx->stream, rw, a));
@@ -225,10 +164,12 @@ int wr_route_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_route_args &a)
     size_t smem = (size_t)kRouteWarps * a.experts * 4;
     int rc = allow_smem(moe_choose_kernel, smem);
     if (rc != WR_CUDA_OK) return rc;
-    WR_CUDA_TRY(wr_launch_pdl(moe_choose_kernel, dim3((rw.n_rows + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem,
-                              ctx->stream, rw, a));
-    rc = finish_launch(ctx);
-    if (rc != WR_CUDA_OK) return rc;
+    if (!a.chosen) {
+        WR_CUDA_TRY(wr_launch_pdl(moe_choose_kernel, dim3((rw.n_rows + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32),
+                                  smem, ctx->stream, rw, a));
+        rc = finish_launch(ctx);
+        if (rc != WR_CUDA_OK) return rc;
+    }
     smem = (size_t)2 * a.experts * 4;
     rc = allow_smem(moe_sort_kernel, smem);
     if (rc != WR_CUDA_OK) return rc;
