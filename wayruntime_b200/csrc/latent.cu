@@ -13,7 +13,7 @@
 
 namespace {
 
-constexpr uint32_t kPrepThreads = 256, kTileRows = 16;
+constexpr uint32_t kPrepThreads = 256, kTileRows = 16;           // (prompts: half as many)
 
 __device__ __forceinline__ void angle(double turns, uint32_t pos, float &sn, float &cs)
 {
@@ -40,30 +40,48 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const wr_rows
     }
     const float *in = a.in + (size_t)row * a.ld, *x = in + (blockIdx.y ? a.c_off : 0u);
     const float *w = blockIdx.y ? a.c_norm : a.q_norm;
-    float ss = 0.f;
-    for (uint32_t i = threadIdx.x; i < n; i += kPrepThreads) ss = fmaf(x[i], x[i], ss);
-    const float inv = 1.0f / sqrtf(block_sum<kPrepThreads / 32>(ss, part) / (float)n + a.eps);
+    // pieces of eight; the pad columns of the projection and of the weights are zeros
+    float ss = 0.f, v[8], u[8];
+    for (uint32_t i = 8 * threadIdx.x; i < n; i += 8 * blockDim.x) {
+        load8v(x + i, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, part) / (float)n + a.eps);
+    auto scaled = [&](uint32_t i) {
+        load8v(x + i, v);
+        load8v(w + i, u);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= inv * u[e];
+    };
     if (blockIdx.y == 0) {
         const Out<TO> out(a.cq, row, wr_ld(n));
-        for (uint32_t i = threadIdx.x; i < wr_ld(n); i += kPrepThreads) out.put(i, i < n ? x[i] * inv * w[i] : 0.f);
+        for (uint32_t i = 8 * threadIdx.x; i < n; i += 8 * blockDim.x) {
+            scaled(i);
+            out.put8(i, v);
+        }
         return;
     }
     const wr_seq_dev s = rw.seqs[seq_of(rw, row)];
     const uint32_t pos = s.pos + tok_of(rw, row), tok = pos % kPageTokens, half = a.g.rot / 2;
     char *page = reinterpret_cast<char *>(s.pages[(size_t)a.layer * s.n_pages + pos / kPageTokens]);
-    auto put = [&](uint32_t d, float v) {
+    for (uint32_t i = 8 * threadIdx.x; i < n; i += 8 * blockDim.x) {
+        scaled(i);
+        char *p = page + wr_geom_off(a.kv, 0, 0, tok, i);
+        if (a.kv.elem == WR_CUDA_F32) store8v(reinterpret_cast<float *>(p), v);
+        else store8v(reinterpret_cast<__half *>(p), v);
+    }
+    auto put = [&](uint32_t d, float y) {
         char *p = page + wr_geom_off(a.kv, 0, 0, tok, d);
-        if (a.kv.elem == WR_CUDA_F32) *reinterpret_cast<float *>(p) = v;
-        else *reinterpret_cast<__half *>(p) = from_f32<__half>(v);
+        if (a.kv.elem == WR_CUDA_F32) *reinterpret_cast<float *>(p) = y;
+        else *reinterpret_cast<__half *>(p) = from_f32<__half>(y);
     };
-    for (uint32_t i = threadIdx.x; i < n; i += kPrepThreads) put(i, x[i] * inv * w[i]);
     const float *r = in + a.r_off;
-    for (uint32_t i = threadIdx.x; i < half; i += kPrepThreads) {
+    for (uint32_t i = blockDim.x - 1 - threadIdx.x; i < half; i += blockDim.x) {         // (by threads without a piece first)
         float sn, cs;
         angle(a.turns[i], pos, sn, cs);
-        const float u = r[i], v = r[i + half];
-        put(a.g.rank_pad() + i, u * cs - v * sn);
-        put(a.g.rank_pad() + half + i, v * cs + u * sn);
+        put(a.g.rank_pad() + i, r[i] * cs - r[i + half] * sn);
+        put(a.g.rank_pad() + half + i, r[i + half] * cs + r[i] * sn);
     }
 }
 
@@ -433,7 +451,8 @@ template <typename TW, typename TO> int value_any(wr_cuda_ctx *ctx, const wr_row
 
 int wr_latent_prep_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent_prep_args &a)
 {
-    const dim3 grid(rw.n_rows, (a.own ? 2 : 1) + (a.route ? 1 : 0)), block(kPrepThreads);
+    const dim3 grid(rw.n_rows, (a.own ? 2 : 1) + (a.route ? 1 : 0));
+    const dim3 block(rw.n_rows <= WR_CUDA_BATCH_MAX ? kPrepThreads : kPrepThreads / 2);
     const wr_route_args route = a.route ? *a.route : wr_route_args{};
     const size_t smem = !a.route ? 0 : route.tile ? (size_t)route.experts * 4 : route_few_smem(route);
     auto launch = [&](auto kernel) {

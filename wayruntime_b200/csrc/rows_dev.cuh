@@ -152,16 +152,14 @@ __device__ __forceinline__ float warp_sum(float v)
     return v;
 }
 
-template <int N> __device__ __forceinline__ float block_sum(float v, float *part)
+// the whole block's sum, warps in order; part: a float per warp
+__device__ __forceinline__ float block_sum(float v, float *part)
 {
-    // N warps; part: N floats, free again after the next barrier of the caller
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     v = warp_sum(v);
-    if (lane == 0) part[warp] = v;
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
     __syncthreads();
     float t = 0.f;
-#pragma unroll
-    for (int i = 0; i < N; ++i) t += part[i];
+    for (uint32_t i = 0; i < blockDim.x >> 5; ++i) t += part[i];
     return t;
 }
 
