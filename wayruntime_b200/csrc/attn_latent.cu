@@ -3,7 +3,8 @@
 // All heads of a layer read the same cached row, once as key and (its first part) once as value, so a page is fetched
 // once for up to 16 heads and serves both products.  Operands are swapped: keys are the tensor core's M.
 //
-// A CTA is one row, one group of NH heads and one chunk of keys; per tile of 128 keys (two pages):
+// A work item is one row, one group of NH heads and one chunk of keys.  CTAs are persistent (one per SM at most): the next
+// item's pages are on their way while this one's last tile is being worked off.  Per tile of 128 keys (two pages):
 //   * warp 0 brings the pages' blocks of 64 keys x 64 values in with linear bulk copies (they are stored in the
 //     operand's layout): the latent in units of 128 values, which stay until the second product has read them, the
 //     rotated part in a ring of its own, free again after the first;
@@ -19,6 +20,7 @@
 
 #include "latent_dev.cuh"
 #include "tcgen05_dev.cuh"
+#include "warp_reduce.cuh"
 
 namespace {
 
@@ -46,6 +48,7 @@ struct LatentParams {
     uint32_t units, rot_boxes, boxes;            // per tile: pairs of latent boxes, rotated boxes; boxes of a query
     uint32_t ring, rot_ring, tmem_cols;
     uint32_t chunks;                             // of the longest row: the stride of ml and o
+    uint32_t items, groups;                      // work items; groups of heads
     wr_latent_lens lens;
     const char *q;                               // [rows][head groups][boxes][2 NH][128 B]
     size_t q_row;
@@ -57,7 +60,7 @@ struct LatentParams {
 
 struct LatentBars {
     uint64_t full[kMaxUnits], empty[kMaxUnits], rot_full[kMaxRot], rot_empty[kMaxRot];
-    uint64_t q_full, s_full, p_full, o_full;
+    uint64_t q_full, q_empty, s_full, p_full, o_full, o_free;
     uint32_t tmem;
     alignas(16) float red[2][16][4];             // per head: the four warps' maxima (or sums)
 };
@@ -91,10 +94,22 @@ __device__ __forceinline__ float ex2(float x)
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
-// element (r, c) of a K-major operand of F16 values: boxes of 64 columns, `rows` rows each
-__device__ __forceinline__ uint32_t swizzled(uint32_t rows, uint32_t r, uint32_t c)
+struct Item {
+    uint32_t row, group, chunk, len, tile0, tiles;
+};
+__device__ __forceinline__ Item item_of(const LatentParams &p, uint32_t i)
 {
-    return (c >> 6) * rows * 128u + r * 128u + ((((c & 63u) >> 3) ^ (r & 7u)) << 4) + (c & 7u) * 2u;
+    Item it;
+    it.group = i % p.groups;
+    i /= p.groups;
+    it.row = 0;
+    while (i >= p.lens.count[it.row]) i -= p.lens.count[it.row++];
+    it.chunk = i;
+    it.len = p.lens.len[it.row];
+    const uint32_t per = chunk_tiles(it.len);
+    it.tile0 = i * per;
+    it.tiles = min(per, (it.len + kTile - 1) / kTile - it.tile0);
+    return it;
 }
 
 template <int NH>
@@ -106,14 +121,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     uint8_t *const ps = qs + p.boxes * N * 128;          // [2 key boxes][N][128 B]
     LatentBars &sm = *reinterpret_cast<LatentBars *>(ps + 2 * N * 128);
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t chunk = blockIdx.x, head0 = blockIdx.y * NH, row = blockIdx.z;
     pdl_trigger();
-    const uint32_t len = p.lens.len[row], per = chunk_tiles(len);
-    if (chunk >= p.lens.count[row]) {
-        pdl_wait();
-        return;
-    }
-    const uint32_t tile0 = chunk * per, tiles = min(per, (len + kTile - 1) / kTile - tile0);
     if (threadIdx.x == 0) {
         for (uint32_t i = 0; i < p.ring; ++i) {
             mbar_init(&sm.full[i], 1);
@@ -124,9 +132,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
             mbar_init(&sm.rot_empty[i], 1);
         }
         mbar_init(&sm.q_full, 1);
+        mbar_init(&sm.q_empty, 1);
         mbar_init(&sm.s_full, 1);
         mbar_init(&sm.p_full, 4);
         mbar_init(&sm.o_full, 1);
+        mbar_init(&sm.o_free, 4);
         fence_barrier_init();
     }
     if (warp == 1) tc5::alloc(&sm.tmem, p.tmem_cols);
@@ -137,221 +147,230 @@ __global__ void __launch_bounds__(kThreads, 1) latent_decode_kernel(const Latent
     const uint32_t tmem_s = sm.tmem, tmem_o = tmem_s + 32;       // (S: 32 columns whatever N is)
 
     if (warp == 0) {
-        if (lane == 0) {
-            mbar_expect_tx(&sm.q_full, p.boxes * N * 128);
-            bulk_g2s(qs, p.q + row * p.q_row + (size_t)blockIdx.y * p.boxes * N * 128, p.boxes * N * 128, &sm.q_full);
-            const wr_seq_dev s = p.rw.seqs[seq_of(p.rw, row)];
-            const uint64_t *table = s.pages + (size_t)p.layer * s.n_pages;
-            const uint32_t last_page = (len - 1) / kPageTokens, rank_boxes = p.boxes - p.rot_boxes;
+        if (lane == 0) {                                 // the pages
+            const uint32_t rank_boxes = p.boxes - p.rot_boxes;
             uint32_t n_unit = 0, n_rot = 0;              // requested so far
             bool ok = true;
-            for (uint32_t t = 0; t < tiles && ok; ++t) {
-                // (a tile's second page may lie behind the last one: the first comes twice, its weights are zeros)
-                const uint32_t pg = (tile0 + t) * 2;
-                const char *src[2] = {reinterpret_cast<const char *>(table[pg]),
-                                      reinterpret_cast<const char *>(table[min(pg + 1, last_page)])};
-                for (uint32_t u = 0; u < p.units && ok; ++u, ++n_unit) {
-                    const uint32_t st = n_unit % p.ring;
-                    if (n_unit >= p.ring && !mbar_wait(&sm.empty[st], (n_unit / p.ring - 1) & 1, p.wait_limit)) {
-                        ok = false;
-                        break;
+            for (uint32_t i = blockIdx.x; i < p.items && ok; i += gridDim.x) {
+                const Item it = item_of(p, i);
+                const wr_seq_dev s = p.rw.seqs[seq_of(p.rw, it.row)];
+                const uint64_t *table = s.pages + (size_t)p.layer * s.n_pages;
+                const uint32_t last_page = (it.len - 1) / kPageTokens;
+                for (uint32_t t = 0; t < it.tiles && ok; ++t) {
+                    // (a tile's second page may lie behind the last one: the first comes twice, its weights are zeros)
+                    const uint32_t pg = (it.tile0 + t) * 2;
+                    const char *src[2] = {reinterpret_cast<const char *>(table[pg]),
+                                          reinterpret_cast<const char *>(table[min(pg + 1, last_page)])};
+                    for (uint32_t u = 0; u < p.units && ok; ++u, ++n_unit) {
+                        const uint32_t st = n_unit % p.ring;
+                        if (n_unit >= p.ring && !mbar_wait(&sm.empty[st], (n_unit / p.ring - 1) & 1, p.wait_limit)) {
+                            ok = false;
+                            break;
+                        }
+                        const uint32_t nb = min(2u, rank_boxes - 2 * u);
+                        mbar_expect_tx(&sm.full[st], nb * kBox);
+                        for (uint32_t b = 0; b < nb; ++b)
+                            for (uint32_t h = 0; h < 2; ++h)
+                                bulk_g2s(units + st * kUnit + b * kBox + h * kBlock, src[h] + (2 * u + b) * kBlock, kBlock,
+                                         &sm.full[st]);
                     }
-                    const uint32_t nb = min(2u, rank_boxes - 2 * u);
-                    mbar_expect_tx(&sm.full[st], nb * kBox);
-                    for (uint32_t b = 0; b < nb; ++b)
+                    for (uint32_t r = 0; r < p.rot_boxes && ok; ++r, ++n_rot) {
+                        const uint32_t st = n_rot % p.rot_ring;
+                        if (n_rot >= p.rot_ring && !mbar_wait(&sm.rot_empty[st], (n_rot / p.rot_ring - 1) & 1, p.wait_limit)) {
+                            ok = false;
+                            break;
+                        }
+                        mbar_expect_tx(&sm.rot_full[st], kBox);
                         for (uint32_t h = 0; h < 2; ++h)
-                            bulk_g2s(units + st * kUnit + b * kBox + h * kBlock, src[h] + (2 * u + b) * kBlock, kBlock, &sm.full[st]);
-                }
-                for (uint32_t r = 0; r < p.rot_boxes && ok; ++r, ++n_rot) {
-                    const uint32_t st = n_rot % p.rot_ring;
-                    if (n_rot >= p.rot_ring && !mbar_wait(&sm.rot_empty[st], (n_rot / p.rot_ring - 1) & 1, p.wait_limit)) {
-                        ok = false;
-                        break;
+                            bulk_g2s(rots + st * kBox + h * kBlock, src[h] + (rank_boxes + r) * kBlock, kBlock, &sm.rot_full[st]);
                     }
-                    mbar_expect_tx(&sm.rot_full[st], kBox);
-                    for (uint32_t h = 0; h < 2; ++h)
-                        bulk_g2s(rots + st * kBox + h * kBlock, src[h] + (rank_boxes + r) * kBlock, kBlock, &sm.rot_full[st]);
                 }
             }
             if (!ok) atomicCAS(p.err, 0, 61);
             // nothing in flight when the CTA leaves
-            (void)mbar_wait(&sm.q_full, 0, p.wait_limit);
             for (uint32_t i = n_unit - min(n_unit, p.ring); i < n_unit; ++i)
                 (void)mbar_wait(&sm.full[i % p.ring], (i / p.ring) & 1, p.wait_limit);
             for (uint32_t i = n_rot - min(n_rot, p.rot_ring); i < n_rot; ++i)
                 (void)mbar_wait(&sm.rot_full[i % p.rot_ring], (i / p.rot_ring) & 1, p.wait_limit);
+        } else if (lane == 1) {                          // the queries
+            uint32_t n = 0;
+            bool ok = true;
+            for (uint32_t i = blockIdx.x; i < p.items; i += gridDim.x, ++n) {
+                if (n > 0) ok = mbar_wait(&sm.q_empty, (n - 1) & 1, p.wait_limit);
+                if (!ok) break;
+                const Item it = item_of(p, i);
+                mbar_expect_tx(&sm.q_full, p.boxes * N * 128);
+                bulk_g2s(qs, p.q + it.row * p.q_row + (size_t)it.group * p.boxes * N * 128, p.boxes * N * 128, &sm.q_full);
+            }
+            if (!ok) atomicCAS(p.err, 0, 64);
+            if (n > 0) (void)mbar_wait(&sm.q_full, (n - 1) & 1, p.wait_limit);
         }
         __syncwarp();
     } else if (warp == 1) {
         const bool lead = tc5::elect_one();
         constexpr uint32_t idesc_s = tc5::idesc_f16(kTile, N), idesc_o = idesc_s | tc5::kIdescAMnMajor;
         const uint32_t q_addr = smem_u32(qs), p_addr = smem_u32(ps);
-        uint32_t n_unit = 0, n_rot = 0;
-        bool ok = mbar_wait(&sm.q_full, 0, p.wait_limit);
-        tc5::fence_after();
-        for (uint32_t t = 0; t < tiles && ok; ++t) {
-            // S^T, box by box as they arrive
-            uint32_t box = 0;
-            auto score = [&](uint32_t rows) {
-                const uint64_t a = tc5::desc_kmajor(rows), b = tc5::desc_kmajor(q_addr + box * N * 128);
+        uint32_t n_unit = 0, n_rot = 0, n_tile = 0, n_item = 0;
+        bool ok = true;
+        for (uint32_t i = blockIdx.x; i < p.items && ok; i += gridDim.x, ++n_item) {
+            const Item it = item_of(p, i);
+            ok = mbar_wait(&sm.q_full, n_item & 1, p.wait_limit);
+            if (!ok) break;
+            for (uint32_t t = 0; t < it.tiles && ok; ++t, ++n_tile) {
+                // S^T, box by box as they arrive
+                uint32_t box = 0;
+                auto score = [&](uint32_t rows) {
+                    const uint64_t a = tc5::desc_kmajor(rows), b = tc5::desc_kmajor(q_addr + box * N * 128);
 #pragma unroll
-                for (uint32_t kk = 0; kk < 4; ++kk)
-                    if (lead) tc5::mma_ss(tmem_s, a + 2 * kk, b + 2 * kk, idesc_s, (box | kk) != 0);
-                ++box;
-            };
-            for (uint32_t u = 0; u < p.units && ok; ++u) {
-                const uint32_t i = n_unit + u, st = i % p.ring;
-                ok = mbar_wait(&sm.full[st], (i / p.ring) & 1, p.wait_limit);
+                    for (uint32_t kk = 0; kk < 4; ++kk)
+                        if (lead) tc5::mma_ss(tmem_s, a + 2 * kk, b + 2 * kk, idesc_s, (box | kk) != 0);
+                    ++box;
+                };
+                for (uint32_t u = 0; u < p.units && ok; ++u) {
+                    const uint32_t j = n_unit + u, st = j % p.ring;
+                    ok = mbar_wait(&sm.full[st], (j / p.ring) & 1, p.wait_limit);
+                    if (!ok) break;
+                    tc5::fence_after();
+                    score(smem_u32(units + st * kUnit));
+                    if (2 * u + 1 < p.boxes - p.rot_boxes) score(smem_u32(units + st * kUnit + kBox));
+                }
+                for (uint32_t r = 0; r < p.rot_boxes && ok; ++r, ++n_rot) {
+                    const uint32_t st = n_rot % p.rot_ring;
+                    ok = mbar_wait(&sm.rot_full[st], (n_rot / p.rot_ring) & 1, p.wait_limit);
+                    if (!ok) break;
+                    tc5::fence_after();
+                    score(smem_u32(rots + st * kBox));
+                    if (lead) tc5::commit(&sm.rot_empty[st]);
+                }
+                if (!ok) break;
+                if (lead) {
+                    if (t + 1 == it.tiles) tc5::commit(&sm.q_empty);
+                    tc5::commit(&sm.s_full);
+                }
+                ok = mbar_wait(&sm.p_full, n_tile & 1, p.wait_limit);
+                // the item's first product overwrites O: the one before must have left TMEM
+                if (ok && t == 0 && n_item > 0) ok = mbar_wait(&sm.o_free, (n_item - 1) & 1, p.wait_limit);
                 if (!ok) break;
                 tc5::fence_after();
-                score(smem_u32(units + st * kUnit));
-                if (2 * u + 1 < p.boxes - p.rot_boxes) score(smem_u32(units + st * kUnit + kBox));
-            }
-            for (uint32_t r = 0; r < p.rot_boxes && ok; ++r, ++n_rot) {
-                const uint32_t st = n_rot % p.rot_ring;
-                ok = mbar_wait(&sm.rot_full[st], (n_rot / p.rot_ring) & 1, p.wait_limit);
-                if (!ok) break;
-                tc5::fence_after();
-                score(smem_u32(rots + st * kBox));
-                if (lead) tc5::commit(&sm.rot_empty[st]);
-            }
-            if (!ok) break;
-            if (lead) tc5::commit(&sm.s_full);
-            ok = mbar_wait(&sm.p_full, t & 1, p.wait_limit);
-            if (!ok) break;
-            tc5::fence_after();
-            // O^T: 128 latents of a unit at a time, 16 keys a step
-            for (uint32_t u = 0; u < p.units; ++u, ++n_unit) {
-                const uint32_t st = n_unit % p.ring;
-                const uint64_t a = tc5::desc_mnmajor(smem_u32(units + st * kUnit), kBox), b = tc5::desc_kmajor(p_addr);
+                // O^T: 128 latents of a unit at a time, 16 keys a step
+                for (uint32_t u = 0; u < p.units; ++u, ++n_unit) {
+                    const uint32_t st = n_unit % p.ring;
+                    const uint64_t a = tc5::desc_mnmajor(smem_u32(units + st * kUnit), kBox), b = tc5::desc_kmajor(p_addr);
 #pragma unroll
-                for (uint32_t kk = 0; kk < kTile / 16; ++kk)
-                    if (lead)
-                        tc5::mma_ss(tmem_o + u * N, a + kk * (2048 >> 4), b + (kk >> 2) * (N * 128 >> 4) + (kk & 3) * 2, idesc_o,
-                                    (t | kk) != 0);
-                if (lead) tc5::commit(&sm.empty[st]);
+                    for (uint32_t kk = 0; kk < kTile / 16; ++kk)
+                        if (lead)
+                            tc5::mma_ss(tmem_o + u * N, a + kk * (2048 >> 4), b + (kk >> 2) * (N * 128 >> 4) + (kk & 3) * 2,
+                                        idesc_o, (t | kk) != 0);
+                    if (lead) tc5::commit(&sm.empty[st]);
+                }
             }
+            if (ok && lead) tc5::commit(&sm.o_full);
         }
-        if (ok && lead) tc5::commit(&sm.o_full);
         if (!ok && lane == 0) atomicCAS(p.err, 0, 62);
         __syncwarp();
     } else {
         const uint32_t quarter = warp & 3, key = quarter * 32 + lane, tid = threadIdx.x - 64, lanes = (quarter * 32) << 16;
-        const uint32_t nh = min((uint32_t)NH, p.heads - head0);
-        float m[NH], l[NH];
-#pragma unroll
-        for (int h = 0; h < NH; ++h) {
-            m[h] = WR_NEG_SENTINEL;
-            l[h] = 0.f;
-        }
+        uint32_t n_tile = 0, n_item = 0, n_red = 0;
         bool ok = true;
         // (a warp whose wait ran out goes through the motions: the group's barriers count on all four)
-        for (uint32_t t = 0; t < tiles; ++t) {
-            if (ok) ok = mbar_wait(&sm.s_full, t & 1, p.wait_limit);     // (the tile before has been multiplied: P and O are quiet)
+        for (uint32_t i = blockIdx.x; i < p.items; i += gridDim.x, ++n_item) {
+            const Item it = item_of(p, i);
+            const uint32_t head0 = it.group * NH, nh = min((uint32_t)NH, p.heads - head0);
+            float m[NH], l[NH];
+#pragma unroll
+            for (int h = 0; h < NH; ++h) {
+                m[h] = WR_NEG_SENTINEL;
+                l[h] = 0.f;
+            }
+            for (uint32_t t = 0; t < it.tiles; ++t, ++n_tile, ++n_red) {
+                if (ok) ok = mbar_wait(&sm.s_full, n_tile & 1, p.wait_limit);    // (the tile before has been multiplied: P is quiet)
+                ok = __all_sync(0xffffffffu, ok);
+                tc5::fence_after();
+                float v[32];
+                tc5::ld32(tmem_s + lanes, v);
+                tc5::wait_ld();
+                const bool seen = (it.tile0 + t) * kTile + key < it.len;
+                float sc[NH], mx[NH];
+#pragma unroll
+                for (int h = 0; h < NH; ++h) mx[h] = sc[h] = seen ? v[h] + v[NH + h] : WR_NEG_SENTINEL;
+                const uint32_t idx = warp_max_many<NH>(mx, lane), b = n_red & 1;
+                sm.red[b][idx][quarter] = mx[0];                 // (lanes that share an index hold one value)
+                group_sync();
+                bool grow = false;
+                float a[NH];
+#pragma unroll
+                for (int h = 0; h < NH; ++h) {
+                    const float4 w = *reinterpret_cast<const float4 *>(sm.red[b][h]);
+                    const float top = fmaxf(fmaxf(w.x, w.y), fmaxf(w.z, w.w));
+                    a[h] = 1.0f;
+                    if (t == 0) {
+                        m[h] = top;
+                    } else if (top > m[h] + kGrow) {
+                        a[h] = ex2(m[h] - top);
+                        m[h] = top;
+                        grow = true;
+                    }
+                }
+                if (grow) {                                      // (the same in all threads)
+#pragma unroll
+                    for (int h = 0; h < NH; ++h) l[h] *= a[h];
+#pragma unroll 1
+                    for (uint32_t c = 0; c < p.units * N; c += 32) {
+                        tc5::ld32(tmem_o + lanes + c, v);
+                        tc5::wait_ld();
+#pragma unroll
+                        for (int e = 0; e < 32; ++e) v[e] *= a[e % NH];
+                        tc5::st32(tmem_o + lanes + c, v);
+                    }
+                    tc5::wait_st();
+                }
+#pragma unroll
+                for (int h = 0; h < NH; ++h) {
+                    const float w = ex2(sc[h] - m[h]);
+                    l[h] += w;
+                    const __half hi = __float2half_rn(w);
+                    *reinterpret_cast<__half *>(ps + wr_latent_split_off(N, h, key)) = hi;
+                    *reinterpret_cast<__half *>(ps + wr_latent_split_off(N, NH + h, key)) = __float2half_rn(w - __half2float(hi));
+                }
+                fence_proxy_async();
+                tc5::fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&sm.p_full);
+            }
+            if (ok) ok = mbar_wait(&sm.o_full, n_item & 1, p.wait_limit);
             ok = __all_sync(0xffffffffu, ok);
             tc5::fence_after();
-            float v[32];
-            tc5::ld32(tmem_s + lanes, v);
-            tc5::wait_ld();
-            const bool seen = (tile0 + t) * kTile + key < len;
-            float sc[NH], mx[NH];
-#pragma unroll
-            for (int h = 0; h < NH; ++h) mx[h] = sc[h] = seen ? v[h] + v[NH + h] : WR_NEG_SENTINEL;
-            const uint32_t idx = warp_max_many<NH>(mx, lane);
-            sm.red[t & 1][idx][quarter] = mx[0];                 // (lanes that share an index hold one value)
-            group_sync();
-            bool grow = false;
-            float a[NH];
-#pragma unroll
-            for (int h = 0; h < NH; ++h) {
-                const float4 w = *reinterpret_cast<const float4 *>(sm.red[t & 1][h]);
-                const float top = fmaxf(fmaxf(w.x, w.y), fmaxf(w.z, w.w));
-                a[h] = 1.0f;
-                if (t == 0) {
-                    m[h] = top;
-                } else if (top > m[h] + kGrow) {
-                    a[h] = ex2(m[h] - top);
-                    m[h] = top;
-                    grow = true;
-                }
-            }
-            if (grow) {                                          // (the same in all threads)
-#pragma unroll
-                for (int h = 0; h < NH; ++h) l[h] *= a[h];
+            const size_t at = ((size_t)it.row * p.heads + head0) * p.chunks + it.chunk, stride = (size_t)p.chunks * p.rank_pad;
+            float *out = p.o + at * p.rank_pad;
 #pragma unroll 1
-                for (uint32_t c = 0; c < p.units * N; c += 32) {
-                    tc5::ld32(tmem_o + lanes + c, v);
-                    tc5::wait_ld();
+            for (uint32_t c = 0; c < p.units * N; c += 32) {
+                float v[32];
+                tc5::ld32(tmem_o + lanes + c, v);
+                tc5::wait_ld();
 #pragma unroll
-                    for (int e = 0; e < 32; ++e) v[e] *= a[e % NH];
-                    tc5::st32(tmem_o + lanes + c, v);
+                for (uint32_t j = 0; j < 32 / N; ++j) {
+                    const uint32_t d = (c / N + j) * 128 + key;
+#pragma unroll
+                    for (uint32_t h = 0; h < NH; ++h)
+                        if (h < nh && d < p.rank_pad) out[h * stride + d] = v[j * N + h] + v[j * N + NH + h];
                 }
-                tc5::wait_st();
             }
-#pragma unroll
-            for (int h = 0; h < NH; ++h) {
-                const float w = ex2(sc[h] - m[h]);
-                l[h] += w;
-                const __half hi = __float2half_rn(w);
-                *reinterpret_cast<__half *>(ps + swizzled(N, h, key)) = hi;
-                *reinterpret_cast<__half *>(ps + swizzled(N, NH + h, key)) = __float2half_rn(w - __half2float(hi));
-            }
-            fence_proxy_async();
             tc5::fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(&sm.p_full);
-        }
-        if (ok) ok = mbar_wait(&sm.o_full, 0, p.wait_limit);
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok && lane == 0) atomicCAS(p.err, 0, 63);
-        tc5::fence_after();
-        const size_t at = ((size_t)row * p.heads + head0) * p.chunks + chunk, stride = (size_t)p.chunks * p.rank_pad;
-        float *out = p.o + at * p.rank_pad;
-#pragma unroll 1
-        for (uint32_t c = 0; c < p.units * N; c += 32) {
-            float v[32];
-            tc5::ld32(tmem_o + lanes + c, v);
-            tc5::wait_ld();
+            if (lane == 0) mbar_arrive(&sm.o_free);
+            // the sums: across the warp's keys, then the four warps in order
+            const uint32_t idx = warp_reduce_many<NH>(l, lane), b = n_red++ & 1;
+            sm.red[b][idx][quarter] = l[0];
+            group_sync();
 #pragma unroll
-            for (uint32_t j = 0; j < 32 / N; ++j) {
-                const uint32_t d = (c / N + j) * 128 + key;
-#pragma unroll
-                for (uint32_t h = 0; h < NH; ++h)
-                    if (h < nh && d < p.rank_pad) out[h * stride + d] = v[j * N + h] + v[j * N + NH + h];
-            }
-        }
-        // the sums: across the warp's keys, then the four warps in order
-        const uint32_t b = tiles & 1;
-        uint32_t idx = 0;
-        {
-            uint32_t width = NH;
-#pragma unroll
-            for (uint32_t o = 16; o >= 1; o >>= 1) {
-                if (width > 1) {
-                    const uint32_t half = width / 2;
-                    const bool upper = (lane & o) != 0;
-#pragma unroll
-                    for (uint32_t i = 0; i < NH / 2; ++i)
-                        if (i < half) {
-                            const float send = upper ? l[i] : l[i + half], keep = upper ? l[i + half] : l[i];
-                            l[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                        }
-                    if (upper) idx += half;
-                    width = half;
-                } else {
-                    l[0] += __shfl_xor_sync(0xffffffffu, l[0], o);
+            for (uint32_t h = 0; h < NH; ++h)
+                if (tid == h && h < nh) {
+                    const float4 w = *reinterpret_cast<const float4 *>(sm.red[b][h]);
+                    *reinterpret_cast<float2 *>(p.ml + 2 * (at + (size_t)h * p.chunks)) =
+                        make_float2(m[h] * kLn2, ((w.x + w.y) + w.z) + w.w);
                 }
-            }
         }
-        sm.red[b][idx][quarter] = l[0];
-        group_sync();
-#pragma unroll
-        for (uint32_t h = 0; h < NH; ++h)
-            if (tid == h && h < nh) {
-                const float4 w = *reinterpret_cast<const float4 *>(sm.red[b][h]);
-                *reinterpret_cast<float2 *>(p.ml + 2 * (at + (size_t)h * p.chunks)) =
-                    make_float2(m[h] * kLn2, ((w.x + w.y) + w.z) + w.w);
-            }
+        if (!ok && lane == 0) atomicCAS(p.err, 0, 63);
     }
     tc5::fence_before();
     __syncthreads();
@@ -397,7 +416,7 @@ uint32_t plan(const wr_latent_geom &g, uint32_t nh, LatentParams &p)
 template <int NH> int launch(wr_cuda_ctx *ctx, const LatentParams &p, uint32_t smem)
 {
     WR_CUDA_TRY(cudaFuncSetAttribute(latent_decode_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    WR_CUDA_TRY(wr_launch_pdl(latent_decode_kernel<NH>, dim3(p.chunks, (p.heads + NH - 1) / NH, p.rw.n_rows), dim3(kThreads),
+    WR_CUDA_TRY(wr_launch_pdl(latent_decode_kernel<NH>, dim3(std::min<uint32_t>(p.items, ctx->sm_count)), dim3(kThreads),
                               (size_t)smem, ctx->stream, p));
     return finish_launch(ctx);
 }
@@ -424,7 +443,10 @@ int wr_latent_decode_launch(wr_cuda_ctx *ctx, const wr_rows &rw, const wr_latent
         p.lens.len[r] = lens[r];
         p.lens.count[r] = chunk_count(lens[r]);
         p.chunks = std::max(p.chunks, p.lens.count[r]);
+        p.items += p.lens.count[r];
     }
+    p.groups = (g.heads + nh - 1) / nh;
+    p.items *= p.groups;
     const size_t pieces = (size_t)rw.n_rows * g.heads * p.chunks, ml = (pieces * 2 + 63) & ~(size_t)63;
     int rc = wr_ctx_reserve_ws(ctx, (ml + pieces * p.rank_pad) * sizeof(float), 0);
     if (rc != WR_CUDA_OK) return rc;
