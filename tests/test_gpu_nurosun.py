@@ -175,6 +175,58 @@ def test_embedding_norm_and_residual_factors(ctx, dtype, width, scale, mult, eps
     m.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("mlp", [dense(56), moe(6, 2, 24)], ids=["dense", "experts"])
+def test_sublayers_one_after_the_other(ctx, dtype, mlp):
+    """The same mechanisms in a stack of another make: root-mean-square norms, the feed-forward with a norm of its own
+    behind the attention's residual, layers run twice (a borrowing run reads the latest rows)."""
+    from wayruntime_b200 import binding as B
+    from wayruntime_b200.models import DTYPES as TYPES
+    cfg = config([latent(mlp=mlp), latent(heads=2, source=0, mlp=mlp)], width=48)
+    w, runs, eps = weights(cfg, 51), [0, 1, 0, 1], cfg["norm"]["eps"]
+    w.update({f"l{i}.norm2": w[f"l{1 - i}.norm1"] for i in (0, 1)})
+    toks = tokens(cfg, 70, 52)
+
+    x, want, rows = w["embed"][toks].astype(np.float64) * 1.5, [], None
+    d = {k: v.astype(np.float64) for k, v in w.items()}
+    for i in runs:
+        pre, mx = f"l{i}.", cfg["layers"][i]["mixer"]
+        h = plain.rms_norm(x, d[pre + "norm1"], eps)
+        rows = plain.latent_rows(h, d, pre + "mix.", mx, eps) if i == 0 else rows
+        x = x + 0.8 * plain.latent_attention(h, d, pre + "mix.", mx, eps, rows)
+        x = x + 0.8 * plain.feed_forward(plain.rms_norm(x, d[pre + "norm2"], eps), d, pre + "mlp.", mlp)
+        want.append(x)
+
+    layers = []
+    for lay in cfg["layers"]:
+        mx = lay["mixer"]
+        s = dict(mixer=B.MIXER_LATENT, n_q_heads=mx["heads"], k_dim=mx["dim"], v_dim=mx["vdim"], rot_dim=mx["rot_dim"], q_rank=mx["q_rank"],
+                 kv_rank=mx["kv_rank"], rope_base=mx["rot"]["base"], attn_scale=mx["scale"], latent_eps=eps, kv_from=int("kv_from" in mx))
+        if mlp["kind"] == "dense":
+            s.update(ffn=B.FFN_SWIGLU, ffn_dim=mlp["ff"])
+        else:
+            s.update(ffn=B.FFN_MOE, ffn_dim=mlp["expert"]["ff"], n_experts=6, top_k=2, moe_alpha=1.702, moe_limit=mlp["expert"]["limit"])
+        layers.append(s)
+    names = {"w_dq": "mix.dq", "dq_norm": "mix.dq.norm", "w_uq": "mix.uq", "w_dkv": "mix.dkv", "dkv_norm": "mix.dkv.norm",
+             "w_uk": "mix.uk", "w_uv": "mix.uv", "wo": "mix.o", "w_gate_up": "mlp.gate", "w_up": "mlp.up", "w_down": "mlp.down",
+             "router": "mlp.router", "router_b": "mlp.router.b", "norm1": "norm1", "norm2": "norm2"}
+
+    def tensor(i, field):
+        if i is None:
+            return w[field.replace("_", ".")]
+        if field == "experts":
+            return [w[f"l{i}.mlp.e{e}.{n}"] for e in range(6) for n in ("gate", "up", "down")]
+        return w.get(f"l{i}.{names[field]}") if field in names else None
+
+    m = B.MixedModel(ctx, layers, runs, tensor, compute=TYPES[dtype], width=48, vocab=cfg["vocab"], norm_groups=1, norm_eps=eps,
+                     embed_scale=1.5, residual_mult=0.8, max_rows=128)
+    for cuts in ([70], cuts_of(70, 8), [40] + [1] * 30):
+        got = residuals(m, cfg, toks, cuts, len(runs))
+        for k in range(len(runs)):
+            assert rel(got[k], want[k]) <= TOL[dtype], (k, cuts[:3])
+    m.close()
+
+
 # ----------------------------------------------------------------- whole models
 
 MODELS = {
